@@ -163,6 +163,14 @@ int pg_gdn_recurrent(const void* q, const void* k, long long ld_qk, const void* 
 int pg_kda_recurrent(const void* q, const void* k, const void* v, long long ld, const void* f, long long ldf, const void* b, long long ldb,
                      const void* a_log, const void* dt_bias, float lower, void* state, void* out, const void* q_indptr, const void* slots,
                      int num_seqs, int heads, int dk, int dv, int max_q_len, cudaStream_t stream);
+// Further rules of the same kernel, bf16 or f32 rows, key width up to 256.  channel_delta: decay exp(-exp(A_log) *
+// softplus(f + dt_bias)) with f in f32, query / key heads shared by heads / kv_heads value heads.  decay_recurrent: linear
+// attention with a fixed decay per head, SiLU on q, k, v inside.  skip_len > 0 leaves sequences of at least that many rows out.
+int pg_channel_delta(const void* q, const void* k, const void* v, long long ld, const void* f, long long ldf, const void* b, long long ldb, const void* a_log, const void* dt_bias,
+                     void* state, void* out, const void* q_indptr, const void* slots, int num_seqs, int heads, int kv_heads, int dk, int dv, int max_q_len, int skip_len, int is_f32,
+                     cudaStream_t stream);
+int pg_decay_recurrent(const void* q, const void* k, const void* v, long long ld, const void* decay, void* state, void* out, const void* q_indptr, const void* slots, int num_seqs,
+                       int heads, int dk, int dv, int max_q_len, int skip_len, int is_f32, cudaStream_t stream);
 // Softmax mix of the first nb snapshot rows of each token (snaps [T, cap, hidden], ld_tok = cap * hidden) and its current row.
 int pg_attnres_mix(const void* cur, long long ld_cur, const void* snaps, long long ld_tok, const void* score_w, void* out, long long ld_out,
                    int tokens, int nb, int hidden, float eps, cudaStream_t stream);
@@ -177,6 +185,29 @@ void pg_attn_set_decode_stages(int stages);  // 2 (three CTAs per SM) or 3 (two 
 int pg_paged_attention(const void* q, const void* kv, void* out, const void* q_indptr, const void* kv_lens, const void* table, int table_stride,
                        int num_seqs, int hq, int hkv, int dim, int page_size, long long num_pages, float scale, int mode, int splits,
                        void* part_o, void* part_lse, int q_tiles, int window, void* status, cudaStream_t stream);
+
+int pg_attention_capped(const void* q, const void* kv, void* out, const void* q_indptr, const void* kv_lens, const void* table, int table_stride, int num_seqs, int hq, int hkv, int dim,
+                        int vdim, int page_size, long long num_pages, float scale, float softcap, const void* gate, long long ld_gate, int mode, int splits, void* part_o, void* part_lse,
+                        int q_tiles, void* status, cudaStream_t stream);
+
+// ---- layers with runtime head sizes, bf16 or f32 (attention_general.cu) -----------------
+int pg_row_norm_rope_append(const void* q, const void* k, const void* v, long long ld, const void* q_w, const void* k_w, const void* cos, const void* sin, int rot, int max_pos,
+                            const void* positions, const void* slots, void* q_out, void* kv, int tokens, int hq, int hkv, int dim, int vdim, int page_size, long long num_pages, float eps,
+                            int is_f32, void* status, cudaStream_t stream);
+int pg_attention_plain(const void* q, const void* kv, void* out, const void* q_indptr, const void* kv_lens, const void* table, int table_stride, int tokens, int num_seqs, int hq, int hkv,
+                       int dim, int vdim, int page_size, long long num_pages, float scale, float softcap, const void* gate, long long ld_gate, int is_f32, cudaStream_t stream);
+
+// ---- rows around an f32 residual stream (stream32.cu) --------------------------------
+int pg_embed_rows(const void* table, int table_f32, long long ldt, const void* ids, void* x_f32, void* xt, int xt_f32, long long ldxt, int tokens, int width, long long rows, void* status,
+                  cudaStream_t stream);
+int pg_post_norm(const void* y, int y_f32, long long ldy, const void* x_in, void* x_out, float alpha, const void* w, void* xt, int xt_f32, long long ldxt, int tokens, int width, float eps,
+                 cudaStream_t stream);
+int pg_gated_row_norm(const void* x, const void* gate, long long ldg, const void* w, void* y, int tokens, int heads, int dim, float eps, int is_f32, cudaStream_t stream);
+int pg_glu_rows_f32(const void* gu, void* out, int rows, int inter, long long ldin, cudaStream_t stream);
+int pg_softcap_f32(const void* x, void* y, long long n, float cap, cudaStream_t stream);
+int pg_gemm_simt(const void* x, const void* w, int x_f32, void* y, int y_f32, int T, int M, int K, long long ldx, long long ldw, long long ldy, cudaStream_t stream);
+int pg_conv_silu(const void* x, long long ldx, const void* w, void* state, void* out, long long ldo, const void* q_indptr, const void* slots, int num_seqs, int channels, int taps,
+                 long long slot_stride, int max_q_len, int is_f32, cudaStream_t stream);
 
 // ---- sampling (sampling.cu) --------------------------------------------------------
 long long pg_argmax_scratch_bytes(int rows, int vocab);

@@ -78,7 +78,24 @@ struct AttnParams {
   long long num_pages;
   uint32_t* status;
   int window;  // decode: a row sees its last `window` keys only (0: all of them)
+  // General form (GEN kernels): key / query size dk and value size dv below the padded tile width D, groups of more than
+  // eight query heads cut into parts, a soft cap on the scores, a sigmoid gate per (token, head) on the output.
+  int dk, dv, parts;         // parts: ceil(query heads per KV head / 8), decode only
+  float cap_in, cap_out;     // cap_in > 0: score = cap_out * tanh(cap_in * dot), already times log2(e)
+  const bf16* gate;          // [T, >= hq] rows of stride ld_gate, or null
+  long long ld_gate;
 };
+
+// A score in units of log2(e): scaled, and capped when the layer has a cap.  tanh(x) = 1 - 2 / (1 + e^2x), whose absolute
+// error (1e-7 of the cap) is what a 32-bit score needs.
+template <bool GEN>
+__device__ __forceinline__ float score_of(const AttnParams& p, float dot) {
+  if (GEN && p.cap_in > 0.f) return p.cap_out - __fdividef(2.f * p.cap_out, 1.f + exp2f(dot * p.cap_in * 2.f * LOG2E));
+  return dot * p.scale_log2;
+}
+__device__ __forceinline__ float head_gate(const AttnParams& p, long long row, int hq) {
+  return 1.f / (1.f + __expf(-__bfloat162float(p.gate[row * p.ld_gate + hq])));
+}
 
 // Row address of token `tok` of sequence b, kv head h (kvsel 0 = K, 1 = V).
 template <int D>
@@ -290,11 +307,13 @@ struct DecodeUnit {
   const int* table_row;
 };
 
+template <bool GEN>
 __device__ __forceinline__ bool load_decode_unit(const AttnParams& p, int u, DecodeUnit& o) {
-  if (u >= p.num_seqs * p.hkv * p.splits) return false;
+  const int hu = GEN ? p.hkv * p.parts : p.hkv;  // GEN: h counts (KV head, part of its group)
+  if (u >= p.num_seqs * hu * p.splits) return false;
   o.split = u % p.splits;
-  o.h = (u / p.splits) % p.hkv;
-  o.b = u / (p.splits * p.hkv);
+  o.h = (u / p.splits) % hu;
+  o.b = u / (p.splits * hu);
   o.kv_len = p.kv_lens[o.b];
   o.qrow = p.q_indptr[o.b];
   o.table_row = p.table + (long long)o.b * p.table_stride;
@@ -307,7 +326,7 @@ __device__ __forceinline__ bool load_decode_unit(const AttnParams& p, int u, Dec
   return true;
 }
 
-template <int D>
+template <int D, bool GEN>
 __global__ void __launch_bounds__(128, D <= 128 ? 2 : 1) decode_attn_persistent_kernel(const AttnParams p) {
   PG_PDL_ENTRY();
   extern __shared__ __align__(128) uint8_t smem_raw[];
@@ -325,19 +344,21 @@ __global__ void __launch_bounds__(128, D <= 128 ? 2 : 1) decode_attn_persistent_
   float* mo = reinterpret_cast<float*>(smem_raw + (size_t)4 * STAGES * STAGE_ELEMS * 2);
   float* mm = mo + 4 * 8 * D;
   float* ml = mm + 4 * 8;
-  const long long row_stride = (long long)p.hkv * D;
+  const int dk = GEN ? p.dk : D, dv = GEN ? p.dv : D;
+  const long long row_stride = (long long)p.hkv * dk, v_stride = (long long)p.hkv * dv;
   const long long v_plane = (long long)p.page_size * row_stride;
+  const long long page_elems = v_plane + (long long)p.page_size * v_stride;
   const uint64_t kv_policy = l2_policy_evict_first();
 
   // issue cursor
   DecodeUnit ui;
   int iu = blockIdx.x;
-  bool vi = load_decode_unit(p, iu, ui);
+  bool vi = load_decode_unit<GEN>(p, iu, ui);
   int ti = vi ? ui.t_begin + warp : 0;
   auto issue_next = [&](int stage) {
     while (vi && ti >= ui.t_end) {
       iu += gridDim.x;
-      vi = load_decode_unit(p, iu, ui);
+      vi = load_decode_unit<GEN>(p, iu, ui);
       ti = vi ? ui.t_begin + warp : 0;
     }
     if (vi) {
@@ -345,15 +366,17 @@ __global__ void __launch_bounds__(128, D <= 128 ? 2 : 1) decode_attn_persistent_
       bf16* vs_ = ks_ + TILE * D;
       const int tok0 = ti * TILE;
       const int page = ui.table_row[tok0 / p.page_size];
-      const bf16* kbase = p.kv + ((long long)page * 2 * p.page_size + (tok0 % p.page_size)) * row_stride + (long long)ui.h * D;
+      const int kvh = GEN ? ui.h / p.parts : ui.h;
+      const bf16* kbase = p.kv + page * page_elems + (tok0 % p.page_size) * row_stride + (long long)kvh * dk;
+      const bf16* vbase = p.kv + page * page_elems + v_plane + (tok0 % p.page_size) * v_stride + (long long)kvh * dv;
 #pragma unroll
       for (int i = 0; i < (TILE * CH) / 32; ++i) {
         const int c = lane + 32 * i;
         const int r = c / CH, ch = c % CH;
         const bool valid = tok0 + r < ui.kv_len;
-        const bf16* src = kbase + (valid ? r : 0) * row_stride + ch * 8;
-        cp_async16_stream(ks_ + swz<D>(r, ch), src, valid, kv_policy);
-        cp_async16_stream(vs_ + swz<D>(r, ch), src + v_plane, valid, kv_policy);
+        const bool kin = !GEN || ch * 8 < dk, vin = !GEN || ch * 8 < dv;  // chunks past the head are filled with zeros
+        cp_async16_stream(ks_ + swz<D>(r, ch), kbase + (valid && kin ? r * row_stride + ch * 8 : 0), valid && kin, kv_policy);
+        cp_async16_stream(vs_ + swz<D>(r, ch), vbase + (valid && vin ? r * v_stride + ch * 8 : 0), valid && vin, kv_policy);
       }
       ti += 4;
     }
@@ -365,15 +388,21 @@ __global__ void __launch_bounds__(128, D <= 128 ? 2 : 1) decode_attn_persistent_
   // compute cursor
   DecodeUnit uc;
   int cu = blockIdx.x;
-  bool vc = load_decode_unit(p, cu, uc);
+  bool vc = load_decode_unit<GEN>(p, cu, uc);
   int it = 0;
   while (vc) {
+    int head0, Gu;  // first query head of the unit, and how many
     uint32_t qf[KS][2];
     {
-      const bf16* qh = p.q + ((long long)uc.qrow * p.hq + (long long)uc.h * G + g) * D;
+      head0 = GEN ? (uc.h / p.parts) * G + (uc.h % p.parts) * 8 : uc.h * G;
+      Gu = GEN ? min(8, G - (uc.h % p.parts) * 8) : G;
+      const bf16* qh = p.q + ((long long)uc.qrow * p.hq + head0 + g) * dk;
 #pragma unroll
       for (int ks = 0; ks < KS; ++ks) {
-        if (g < G) {
+        if (GEN) {
+          qf[ks][0] = g < Gu && ks * 16 < dk ? *reinterpret_cast<const uint32_t*>(qh + ks * 16 + 2 * t4) : 0u;
+          qf[ks][1] = g < Gu && ks * 16 + 8 < dk ? *reinterpret_cast<const uint32_t*>(qh + ks * 16 + 8 + 2 * t4) : 0u;
+        } else if (g < G) {
           qf[ks][0] = *reinterpret_cast<const uint32_t*>(qh + ks * 16 + 2 * t4);
           qf[ks][1] = *reinterpret_cast<const uint32_t*>(qh + ks * 16 + 8 + 2 * t4);
         } else {
@@ -408,10 +437,10 @@ __global__ void __launch_bounds__(128, D <= 128 ? 2 : 1) decode_attn_persistent_
       }
       float sv[4];
       const int tok0 = tile * TILE + 2 * t4;
-      sv[0] = (tok0 < uc.kv_len && tok0 >= uc.kv_lo) ? s_acc[0][0] * p.scale_log2 : NEG_BIG;
-      sv[1] = (tok0 + 1 < uc.kv_len && tok0 + 1 >= uc.kv_lo) ? s_acc[0][1] * p.scale_log2 : NEG_BIG;
-      sv[2] = (tok0 + 8 < uc.kv_len && tok0 + 8 >= uc.kv_lo) ? s_acc[1][0] * p.scale_log2 : NEG_BIG;
-      sv[3] = (tok0 + 9 < uc.kv_len && tok0 + 9 >= uc.kv_lo) ? s_acc[1][1] * p.scale_log2 : NEG_BIG;
+      sv[0] = (tok0 < uc.kv_len && tok0 >= uc.kv_lo) ? score_of<GEN>(p, s_acc[0][0]) : NEG_BIG;
+      sv[1] = (tok0 + 1 < uc.kv_len && tok0 + 1 >= uc.kv_lo) ? score_of<GEN>(p, s_acc[0][1]) : NEG_BIG;
+      sv[2] = (tok0 + 8 < uc.kv_len && tok0 + 8 >= uc.kv_lo) ? score_of<GEN>(p, s_acc[1][0]) : NEG_BIG;
+      sv[3] = (tok0 + 9 < uc.kv_len && tok0 + 9 >= uc.kv_lo) ? score_of<GEN>(p, s_acc[1][1]) : NEG_BIG;
       float mx = fmaxf(fmaxf(sv[0], sv[1]), fmaxf(sv[2], sv[3]));
       mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
       mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
@@ -453,8 +482,9 @@ __global__ void __launch_bounds__(128, D <= 128 ? 2 : 1) decode_attn_persistent_
       ml[warp * 8 + g] = l_run;
     }
     __syncthreads();
-    for (int idx = threadIdx.x; idx < G * D; idx += 128) {
+    for (int idx = threadIdx.x; idx < Gu * D; idx += 128) {
       const int row = idx / D, d = idx % D;
+      if (GEN && d >= dv) continue;
       float M = NEG_BIG;
 #pragma unroll
       for (int w = 0; w < 4; ++w) M = fmaxf(M, mm[w * 8 + row]);
@@ -465,23 +495,24 @@ __global__ void __launch_bounds__(128, D <= 128 ? 2 : 1) decode_attn_persistent_
         L += f * ml[w * 8 + row];
         O += f * mo[(w * 8 + row) * D + d];
       }
-      const int hq = uc.h * G + row;
-      const float val = L > 0.f ? O / L : 0.f;
+      const int hq = head0 + row;
+      float val = L > 0.f ? O / L : 0.f;
       if (p.splits == 1) {
-        p.out[((long long)uc.qrow * p.hq + hq) * D + d] = __float2bfloat16(val);
+        if (GEN && p.gate) val *= head_gate(p, uc.qrow, hq);
+        p.out[((long long)uc.qrow * p.hq + hq) * dv + d] = __float2bfloat16(val);
       } else {
-        p.part_o[(((long long)uc.b * p.hq + hq) * p.splits + uc.split) * D + d] = val;
+        p.part_o[(((long long)uc.b * p.hq + hq) * p.splits + uc.split) * dv + d] = val;
         if (d == 0) p.part_lse[((long long)uc.b * p.hq + hq) * p.splits + uc.split] = L > 0.f ? M + log2f(L) : NEG_BIG;
       }
     }
     __syncthreads();  // the scratch is free again
     cu += gridDim.x;
-    vc = load_decode_unit(p, cu, uc);
+    vc = load_decode_unit<GEN>(p, cu, uc);
   }
   cp_async_wait<0>();
 }
 
-template <int D>
+template <int D, bool GEN>
 __global__ void __launch_bounds__(128) decode_merge_kernel(const AttnParams p) {
   PG_PDL_ENTRY();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -495,26 +526,33 @@ __global__ void __launch_bounds__(128) decode_merge_kernel(const AttnParams p) {
 #pragma unroll
   for (int i = 0; i < D / 32; ++i) acc[i] = 0.f;
   float W = 0.f;
+  const int dv = GEN ? p.dv : D;
   for (int s = 0; s < p.splits; ++s) {
     const float l = lse[s];
     if (l <= NEG_BIG) continue;
     const float f = exp2f(l - M);
     W += f;
-    const float* po = p.part_o + (unit * p.splits + s) * D;
+    const float* po = p.part_o + (unit * p.splits + s) * dv;
 #pragma unroll
-    for (int i = 0; i < D / 32; ++i) acc[i] += f * po[lane + 32 * i];
+    for (int i = 0; i < D / 32; ++i)
+      if (!GEN || lane + 32 * i < dv) acc[i] += f * po[lane + 32 * i];
   }
   const int qrow = p.q_indptr[b];
-  bf16* out = p.out + ((long long)qrow * p.hq + hq) * D;
+  bf16* out = p.out + ((long long)qrow * p.hq + hq) * dv;
+  const float gate = GEN && p.gate ? head_gate(p, qrow, hq) : 1.f;
 #pragma unroll
-  for (int i = 0; i < D / 32; ++i) out[lane + 32 * i] = __float2bfloat16(W > 0.f ? acc[i] / W : 0.f);
+  for (int i = 0; i < D / 32; ++i) {
+    float v = W > 0.f ? acc[i] / W : 0.f;
+    if (GEN) v *= gate;
+    if (!GEN || lane + 32 * i < dv) out[lane + 32 * i] = __float2bfloat16(v);
+  }
 }
 
 // -----------------------------------------------------------------------------------
 // prefill / mixed
 // -----------------------------------------------------------------------------------
 // MINB: CTAs per SM the register allocation aims for (3 costs a few spilled words at D = 128).
-template <int D, int MINB>
+template <int D, int MINB, bool GEN>
 __global__ void __launch_bounds__(128, MINB) prefill_attn_kernel(const AttnParams p, int window) {
   PG_PDL_ENTRY();
   extern __shared__ __align__(128) uint8_t smem_raw[];
@@ -527,6 +565,7 @@ __global__ void __launch_bounds__(128, MINB) prefill_attn_kernel(const AttnParam
   const int hq = blockIdx.y;
   const int G = p.hq / p.hkv;
   const int h = hq / G;
+  const int dk = GEN ? p.dk : D, dv = GEN ? p.dv : D;
 
   // locate (sequence, q tile) for this CTA
   int b = 0, tile_in_seq = 0;
@@ -551,16 +590,16 @@ __global__ void __launch_bounds__(128, MINB) prefill_attn_kernel(const AttnParam
   const int rows_here = min(BQ, q_len - row_base);
   const int pos_base = kv_len - q_len + row_base;  // absolute position of that row
   if (kv_len == 0) {
-    for (int idx = threadIdx.x; idx < rows_here * D; idx += 128)
-      p.out[((long long)(q0 + row_base + idx / D) * p.hq + hq) * D + idx % D] = __float2bfloat16(0.f);
+    for (int idx = threadIdx.x; idx < rows_here * dv; idx += 128)
+      p.out[((long long)(q0 + row_base + idx / dv) * p.hq + hq) * dv + idx % dv] = __float2bfloat16(0.f);
     return;
   }
 
   // stage Q tile [64][D] into shared memory (swizzled), then into A fragments
   for (int c = threadIdx.x; c < BQ * CH; c += 128) {
     const int r = c / CH, ch = c % CH;
-    const bool valid = r < rows_here;
-    const bf16* src = p.q + ((long long)(q0 + row_base + (valid ? r : 0)) * p.hq + hq) * D + ch * 8;
+    const bool valid = r < rows_here && (!GEN || ch * 8 < dk);
+    const bf16* src = p.q + ((long long)(q0 + row_base + (valid ? r : 0)) * p.hq + hq) * dk + (valid ? ch * 8 : 0);
     cp_async16(sm + swz<D>(r, ch), src, valid);
   }
   cp_async_commit();
@@ -593,10 +632,13 @@ __global__ void __launch_bounds__(128, MINB) prefill_attn_kernel(const AttnParam
   // a division per chunk made address generation the larger part of this kernel's instructions).
   constexpr int RPT = BKV * CH / 128, RSTEP = 128 / CH;
   const int ps_shift = __ffs(p.page_size) - 1;
-  const long long row_stride = (long long)p.hkv * D;
+  const long long row_stride = (long long)p.hkv * dk, v_stride = (long long)p.hkv * dv;
   const long long v_plane = (long long)p.page_size * row_stride;
+  const long long page_elems = v_plane + (long long)p.page_size * v_stride;
   const int my_ch = threadIdx.x % CH, my_r0 = threadIdx.x / CH;
-  const bf16* kv_head = p.kv + (long long)h * D + my_ch * 8;
+  const bool kin = !GEN || my_ch * 8 < dk, vin = !GEN || my_ch * 8 < dv;  // chunks past the head are filled with zeros
+  const bf16* k_head = p.kv + (long long)h * dk + (kin ? my_ch * 8 : 0);
+  const bf16* v_head = p.kv + v_plane + (long long)h * dv + (vin ? my_ch * 8 : 0);
   auto issue = [&](int kt, int stage) {
     bf16* ks_ = sm + stage * 2 * TILE_ELEMS;
     bf16* vs_ = ks_ + TILE_ELEMS;
@@ -613,9 +655,9 @@ __global__ void __launch_bounds__(128, MINB) prefill_attn_kernel(const AttnParam
         const int rr = valid ? r : 0;
         const int j = rr >> ps_shift;
         const int page = j == 0 ? pg[0] : j == 1 ? pg[1] : j == 2 ? pg[2] : pg[3];
-        const bf16* src = kv_head + ((long long)page * 2 * p.page_size + (rr & (p.page_size - 1))) * row_stride;
-        cp_async16(ks_ + swz<D>(r, my_ch), src, valid);
-        cp_async16(vs_ + swz<D>(r, my_ch), src + v_plane, valid);
+        const int off = rr & (p.page_size - 1);
+        cp_async16(ks_ + swz<D>(r, my_ch), k_head + page * page_elems + off * row_stride, valid && kin);
+        cp_async16(vs_ + swz<D>(r, my_ch), v_head + page * page_elems + off * v_stride, valid && vin);
       }
     }
     cp_async_commit();
@@ -656,7 +698,7 @@ __global__ void __launch_bounds__(128, MINB) prefill_attn_kernel(const AttnParam
       for (int n = 0; n < BKV / 8; ++n) {
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-          const float v = s_acc[n][e] * p.scale_log2;
+          const float v = score_of<GEN>(p, s_acc[n][e]);
           s_acc[n][e] = v;
           mx[e >> 1] = fmaxf(mx[e >> 1], v);
         }
@@ -670,7 +712,7 @@ __global__ void __launch_bounds__(128, MINB) prefill_attn_kernel(const AttnParam
           const int qp = qpos0 + (e >> 1) * 8;
           bool ok = tok <= qp && tok < kv_end;
           if (window > 0) ok = ok && tok > qp - window;
-          const float v = ok ? s_acc[n][e] * p.scale_log2 : NEG_BIG;
+          const float v = ok ? score_of<GEN>(p, s_acc[n][e]) : NEG_BIG;
           s_acc[n][e] = v;
           mx[e >> 1] = fmaxf(mx[e >> 1], v);
         }
@@ -732,11 +774,12 @@ __global__ void __launch_bounds__(128, MINB) prefill_attn_kernel(const AttnParam
   for (int rr = 0; rr < 2; ++rr) {
     const int r = warp * 16 + g + rr * 8;
     if (r < rows_here) {
-      const float inv = l_run[rr] > 0.f ? 1.f / l_run[rr] : 0.f;
-      bf16* dst = p.out + ((long long)(q0 + row_base + r) * p.hq + hq) * D;
+      float inv = l_run[rr] > 0.f ? 1.f / l_run[rr] : 0.f;
+      if (GEN && p.gate) inv *= head_gate(p, q0 + row_base + r, hq);
+      bf16* dst = p.out + ((long long)(q0 + row_base + r) * p.hq + hq) * dv;
 #pragma unroll
       for (int n = 0; n < NT; ++n) {
-        *reinterpret_cast<uint32_t*>(dst + n * 8 + 2 * t4) = pack_bf16(o[n][rr * 2] * inv, o[n][rr * 2 + 1] * inv);
+        if (!GEN || n * 8 < dv) *reinterpret_cast<uint32_t*>(dst + n * 8 + 2 * t4) = pack_bf16(o[n][rr * 2] * inv, o[n][rr * 2 + 1] * inv);
       }
     }
   }
@@ -757,7 +800,7 @@ int launch_decode_s(const AttnParams& p, cudaStream_t stream) {
   PG_CUDA(launch_pdl(decode_attn_kernel<D, STAGES>, dim3(p.num_seqs * p.hkv * p.splits), dim3(128), (size_t)(smem), stream, p));
   PG_LAUNCH_CHECK();
   if (p.splits > 1) {
-    PG_CUDA(launch_pdl(decode_merge_kernel<D>, dim3((p.num_seqs * p.hq + 3) / 4), dim3(128), (size_t)(0), stream, p));
+    PG_CUDA(launch_pdl(decode_merge_kernel<D, false>, dim3((p.num_seqs * p.hq + 3) / 4), dim3(128), (size_t)(0), stream, p));
     PG_LAUNCH_CHECK();
   }
   return PG_OK;
@@ -765,7 +808,7 @@ int launch_decode_s(const AttnParams& p, cudaStream_t stream) {
 
 int g_decode_persistent = -1;  // PEGAINFER_ATTN_PERSISTENT=0 selects the one-unit-per-CTA kernel
 
-template <int D>
+template <int D, bool GEN = false>
 int launch_decode_persistent(const AttnParams& p, cudaStream_t stream) {
   const size_t pipe = (size_t)4 * 3 * 2 * 16 * D * 2;
   const size_t merge = (size_t)(4 * 8 * D + 64) * 4;
@@ -775,14 +818,14 @@ int launch_decode_persistent(const AttnParams& p, cudaStream_t stream) {
     int dev = 0;
     PG_CUDA(cudaGetDevice(&dev));
     PG_CUDA(cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev));
-    PG_CUDA(cudaFuncSetAttribute(decode_attn_persistent_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    PG_CUDA(cudaFuncSetAttribute(decode_attn_persistent_kernel<D, GEN>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
   }
-  const int units = p.num_seqs * p.hkv * p.splits;
+  const int units = p.num_seqs * p.hkv * (GEN ? p.parts : 1) * p.splits;
   const int slots = sms * (D <= 128 ? 2 : 1);
-  PG_CUDA(launch_pdl(decode_attn_persistent_kernel<D>, dim3(units < slots ? units : slots), dim3(128), smem, stream, p));
+  PG_CUDA(launch_pdl(decode_attn_persistent_kernel<D, GEN>, dim3(units < slots ? units : slots), dim3(128), smem, stream, p));
   PG_LAUNCH_CHECK();
   if (p.splits > 1) {
-    PG_CUDA(launch_pdl(decode_merge_kernel<D>, dim3((p.num_seqs * p.hq + 3) / 4), dim3(128), (size_t)(0), stream, p));
+    PG_CUDA(launch_pdl(decode_merge_kernel<D, GEN>, dim3((p.num_seqs * p.hq + 3) / 4), dim3(128), (size_t)(0), stream, p));
     PG_LAUNCH_CHECK();
   }
   return PG_OK;
@@ -801,16 +844,16 @@ int launch_decode(const AttnParams& p, cudaStream_t stream) {
 
 int g_prefill_ctas = 0;  // PEGAINFER_PREFILL_CTAS=2|3: register budget of the prefill kernel (CTAs per SM)
 
-template <int D, int MINB>
+template <int D, int MINB, bool GEN = false>
 int launch_prefill_b(const AttnParams& p, int q_tiles, int window, cudaStream_t stream) {
   const size_t smem = (size_t)2 * 2 * 64 * D * 2;
   static bool set = false;
   if (!set) {
-    PG_CUDA(cudaFuncSetAttribute(prefill_attn_kernel<D, MINB>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    PG_CUDA(cudaFuncSetAttribute(prefill_attn_kernel<D, MINB, GEN>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     set = true;
   }
   dim3 grid(q_tiles, p.hq);
-  PG_CUDA(launch_pdl(prefill_attn_kernel<D, MINB>, dim3(grid), dim3(128), (size_t)(smem), stream, p, window));
+  PG_CUDA(launch_pdl(prefill_attn_kernel<D, MINB, GEN>, dim3(grid), dim3(128), (size_t)(smem), stream, p, window));
   PG_LAUNCH_CHECK();
   return PG_OK;
 }
@@ -866,6 +909,7 @@ extern "C" int pg_paged_attention(const void* q, const void* kv, void* out, cons
   PG_REQUIRE(page_size == 16 || page_size == 32 || page_size == 64, "paged_attention: page size %d not supported", page_size);
   if (num_seqs == 0) return PG_OK;
   AttnParams p;
+  memset(&p, 0, sizeof(p));
   p.q = (const bf16*)q;
   p.kv = (const bf16*)kv;
   p.out = (bf16*)out;
@@ -894,4 +938,55 @@ extern "C" int pg_paged_attention(const void* q, const void* kv, void* out, cons
   if (dim == 64) return launch_prefill<64>(p, q_tiles, window, stream);
   if (dim == 128) return launch_prefill<128>(p, q_tiles, window, stream);
   return launch_prefill<256>(p, q_tiles, window, stream);
+}
+
+// The general form: key / query size `dim` and value size `vdim` (multiples of 8, up to 256), any group, softcap > 0 caps
+// the scores, `gate` (bf16 rows [T, >= hq] of stride ld_gate, or null) multiplies a head's output by its sigmoid.
+// KV page: [page_size, hkv, dim] keys, then [page_size, hkv, vdim] values.  Modes as above.
+extern "C" int pg_attention_capped(const void* q, const void* kv, void* out, const void* q_indptr, const void* kv_lens, const void* table, int table_stride, int num_seqs, int hq, int hkv, int dim,
+                                   int vdim, int page_size, long long num_pages, float scale, float softcap, const void* gate, long long ld_gate, int mode, int splits, void* part_o, void* part_lse,
+                                   int q_tiles, void* status, cudaStream_t stream) {
+  PG_REQUIRE(dim % 8 == 0 && vdim % 8 == 0 && dim >= 8 && vdim >= 8 && dim <= 256 && vdim <= 256, "attention_capped: head sizes %d / %d not supported (multiples of 8 up to 256)", dim, vdim);
+  PG_REQUIRE(hq % hkv == 0, "attention_capped: %d query heads over %d KV heads", hq, hkv);
+  PG_REQUIRE(page_size == 16 || page_size == 32 || page_size == 64, "attention_capped: page size %d not supported", page_size);
+  PG_REQUIRE((((uintptr_t)q | (uintptr_t)kv | (uintptr_t)out) & 15) == 0, "attention_capped: operands must be 16-byte aligned");
+  if (num_seqs == 0) return PG_OK;
+  AttnParams p;
+  memset(&p, 0, sizeof(p));
+  p.q = (const bf16*)q;
+  p.kv = (const bf16*)kv;
+  p.out = (bf16*)out;
+  p.q_indptr = (const int*)q_indptr;
+  p.kv_lens = (const int*)kv_lens;
+  p.table = (const int*)table;
+  p.table_stride = table_stride;
+  p.num_seqs = num_seqs;
+  p.hq = hq;
+  p.hkv = hkv;
+  p.page_size = page_size;
+  p.scale_log2 = scale * LOG2E;
+  p.splits = splits < 1 ? 1 : splits;
+  p.part_o = (float*)part_o;
+  p.part_lse = (float*)part_lse;
+  p.num_pages = num_pages;
+  p.status = (uint32_t*)status;
+  p.dk = dim;
+  p.dv = vdim;
+  p.parts = (hq / hkv + 7) / 8;
+  p.cap_in = softcap > 0.f ? scale / softcap : 0.f;
+  p.cap_out = softcap * LOG2E;
+  p.gate = (const bf16*)gate;
+  p.ld_gate = ld_gate;
+  const int wide = dim > vdim ? dim : vdim;
+  if (mode == 0) {
+    PG_REQUIRE(p.splits == 1 || (part_o && part_lse), "attention_capped: split-KV decode needs partial buffers");
+    if (wide <= 64) return launch_decode_persistent<64, true>(p, stream);
+    if (wide <= 128) return launch_decode_persistent<128, true>(p, stream);
+    return launch_decode_persistent<256, true>(p, stream);
+  }
+  if (q_tiles == 0) return PG_OK;
+  PG_REQUIRE(hq <= 65535, "attention_capped: %d heads", hq);
+  if (wide <= 64) return launch_prefill_b<64, 2, true>(p, q_tiles, 0, stream);
+  if (wide <= 128) return launch_prefill_b<128, 2, true>(p, q_tiles, 0, stream);
+  return launch_prefill_b<256, 1, true>(p, q_tiles, 0, stream);
 }

@@ -9,6 +9,9 @@
 //    rule in gdn.cu: a CTA takes 32 columns of one (sequence, head), four lanes share a column and each keeps a
 //    quarter of its Dk elements in registers; a stage of 8 tokens is normalised into shared memory, then
 //    walked in order.  A decode step is one pass over the state (read + write).
+//    The same kernel runs two more rules (RULE below): the decay in its softplus form, exp(-exp(A_log) softplus(f + dt_bias)),
+//    with query / key heads shared by several value heads, and plain linear attention with one fixed decay per head
+//    (S = decay S + k (x) v, out = S^T q, SiLU on q, k and v).  Those take bf16 or f32 rows and any key width up to 256.
 //  * attnres_mix: the attention-residual mix.  Every token keeps up to `cap` snapshot rows of its own residual
 //    stream; a mix scores each of the first nb snapshots and the current row with
 //    dot(x / rms(x), score_w) and returns the softmax-weighted sum of the un-normalised rows.
@@ -17,110 +20,163 @@
 // :304-410 (kda_core) and pegainfer-kernels/csrc/k3/k3_flash_kda.cu (chunked prefill of the same rule).
 #include "api.h"
 #include "common.cuh"
+#include "types.cuh"
 
 namespace {
 
 constexpr int KDA_STAGE = 8;
 constexpr int KDA_COLS = 32;
 
+// What a token does to the state.  BOUNDED and SOFTPLUS are the delta rule with a decay per key channel and two forms of
+// the decay; DECAY is linear attention with a fixed decay per head (no correction term).
+enum { RULE_BOUNDED = 0, RULE_SOFTPLUS = 1, RULE_DECAY = 2 };
+
+template <typename T>
+struct RecArgs {
+  const T *q, *k, *v;  // token rows of stride ld; q and k [kv_heads * dk], v [heads * dv]
+  long long ld;
+  const void* f;  // raw decay projection [heads * dk]: T (BOUNDED) or f32 (SOFTPLUS)
+  long long ldf;
+  const T* b;  // raw step-size projection [heads]
+  long long ldb;
+  const float *a_log, *dt_bias, *decay;  // decay [heads]: DECAY only
+  float lower;
+  float* state;
+  T* out;
+  const int *q_indptr, *slots;
+  int heads, kv_heads, dk, dv, col_groups;
+  int skip_len;  // > 0: sequences of at least that many tokens belong to another kernel
+};
+
 // XW = false: four adjacent lanes share a state column and reduce with shuffles (prompt chunks: no barrier per token).
 // XW = true: a warp owns one quarter of Dk for all 32 columns, so every state load and store of a warp is one 128-byte row
 // and the shared-memory reads of k, q and the decays are broadcasts; the four quarters meet through shared memory with two
 // barriers per token (decode rows and other steps of a few tokens).
-template <int DK, bool XW>
-__global__ void __launch_bounds__(128) kda_recurrent_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k, const bf16* __restrict__ v, long long ld,
-                                                             const bf16* __restrict__ f, long long ldf, const bf16* __restrict__ b, long long ldb,
-                                                             const float* __restrict__ a_log, const float* __restrict__ dt_bias, float lower,
-                                                             float* __restrict__ state, bf16* __restrict__ out, const int* __restrict__ q_indptr,
-                                                             const int* __restrict__ slots, int heads, int dv, int col_groups) {
+// DK is the key width rounded up to an instantiated size; entries past p.dk are zero (PAD).
+template <typename T, int DK, bool XW, int RULE, bool PAD>
+__global__ void __launch_bounds__(128) kda_recurrent_kernel(const RecArgs<T> p) {
+  PG_PDL_ENTRY();
   constexpr int QK = DK / 4;   // state elements per thread
   constexpr int QS = QK + 4;   // padded quarter stride: the four quarters land in different banks
   constexpr int QL = DK / 32;  // elements per lane when a warp holds one token
-  __shared__ __align__(16) float sq[KDA_STAGE][4 * QS], sk[KDA_STAGE][4 * QS], sd[KDA_STAGE][4 * QS];
+  constexpr bool DELTA = RULE != RULE_DECAY;
+  __shared__ __align__(16) float sq[KDA_STAGE][4 * QS], sk[KDA_STAGE][4 * QS], sd[DELTA ? KDA_STAGE : 1][4 * QS];
   __shared__ float sv[KDA_STAGE][KDA_COLS], sb[KDA_STAGE];
-  __shared__ float red_kv[4][KDA_COLS], red_o[4][KDA_COLS];
-  const int h = blockIdx.x / col_groups, cg = blockIdx.x % col_groups, seq = blockIdx.y;
-  const int slot = slots[seq];
-  const int q0 = q_indptr[seq], q1 = q_indptr[seq + 1];
+  __shared__ float red_kv[4][KDA_COLS], red_o[2][4][KDA_COLS];
+  const int dk = PAD ? p.dk : DK, dv = p.dv, heads = p.heads;
+  const int h = blockIdx.x / p.col_groups, cg = blockIdx.x % p.col_groups, seq = blockIdx.y;
+  const int slot = p.slots[seq];
+  const int q0 = p.q_indptr[seq], q1 = p.q_indptr[seq + 1];
   if (q1 == q0 || slot < 0) return;
+  if (p.skip_len > 0 && q1 - q0 >= p.skip_len) return;
+  const int kh = h / (heads / p.kv_heads);
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int qtr = XW ? warp : (tid & 3), lc = XW ? lane : (tid >> 2), col = cg * KDA_COLS + lc;
   const bool owner = col < dv;
-  float* S = state + (((long long)slot * heads + h) * DK) * dv;  // [DK][dv], v contiguous
+  float* S = p.state + (((long long)slot * heads + h) * dk) * dv;  // [dk][dv], v contiguous
   // Shuffle mapping: a thread's own elements sit DK / 4 rows apart, so a warp reads 32-byte pieces of four rows.  Staging
   // the CTA's slice through shared memory instead was measured slower (200 us against 111 us for 32 decode rows of 96
   // heads: the extra 17 KB per CTA costs resident CTAs); the XW mapping reads whole rows without it (86 us).
   float s_col[QK];
 #pragma unroll
-  for (int i = 0; i < QK; ++i) s_col[i] = owner ? S[(long long)(qtr * QK + i) * dv + col] : 0.f;
-  const float q_scale = rsqrtf((float)DK);
-  const float a = __expf(a_log[h]);
+  for (int i = 0; i < QK; ++i) s_col[i] = owner && (!PAD || qtr * QK + i < dk) ? S[(long long)(qtr * QK + i) * dv + col] : 0.f;
+  const float q_scale = DELTA ? rsqrtf((float)dk) : 1.f;
+  const float a = DELTA ? __expf(p.a_log[h]) : 0.f;
+  const float fixed = DELTA ? 0.f : p.decay[h];
 
   for (int t0 = q0; t0 < q1; t0 += KDA_STAGE) {
     const int nt = min(KDA_STAGE, q1 - t0);
-    // stage: each warp normalises two tokens' q and k and turns the gate row into decays
+    // stage: each warp prepares two tokens' q and k (unit rows, or SiLU of the projections) and their decays
     for (int j = warp; j < nt; j += 4) {
       const long long row = (long long)(t0 + j);
-      const bf16* qp = q + row * ld + (long long)h * DK;
-      const bf16* kp = k + row * ld + (long long)h * DK;
-      const bf16* fp = f + row * ldf + (long long)h * DK;
+      const T* qp = p.q + row * p.ld + (long long)kh * dk;
+      const T* kp = p.k + row * p.ld + (long long)kh * dk;
       float rq[QL], rk[QL], qs = 0.f, ks = 0.f;
 #pragma unroll
       for (int i = 0; i < QL; ++i) {
-        rq[i] = __bfloat162float(qp[lane + 32 * i]);
-        rk[i] = __bfloat162float(kp[lane + 32 * i]);
-        qs += rq[i] * rq[i];
-        ks += rk[i] * rk[i];
+        const bool in = !PAD || lane + 32 * i < dk;
+        rq[i] = in ? to_f32(qp[lane + 32 * i]) : 0.f;
+        rk[i] = in ? to_f32(kp[lane + 32 * i]) : 0.f;
+        if (DELTA) {
+          qs += rq[i] * rq[i];
+          ks += rk[i] * rk[i];
+        } else {  // the activation's result is what the layer works with, in the activation type
+          rq[i] = to_f32(from_f32<T>(rq[i] / (1.f + __expf(-rq[i]))));
+          rk[i] = to_f32(from_f32<T>(rk[i] / (1.f + __expf(-rk[i]))));
+        }
       }
-      qs = warp_sum(qs);
-      ks = warp_sum(ks);
-      const float qn = rsqrtf(qs + 1e-6f) * q_scale, kn = rsqrtf(ks + 1e-6f);
+      float qn = 1.f, kn = 1.f;
+      if (DELTA) {
+        qs = warp_sum(qs);
+        ks = warp_sum(ks);
+        qn = rsqrtf(qs + 1e-6f) * q_scale, kn = rsqrtf(ks + 1e-6f);
+      }
 #pragma unroll
       for (int i = 0; i < QL; ++i) {
         const int e = lane + 32 * i, at = (e / QK) * QS + (e % QK);
-        const float raw = __bfloat162float(fp[e]) + dt_bias[h * DK + e];
         sq[j][at] = rq[i] * qn;
         sk[j][at] = rk[i] * kn;
-        sd[j][at] = __expf(lower / (1.f + __expf(-a * raw)));
+        if (RULE == RULE_BOUNDED) {
+          const float raw = to_f32(((const T*)p.f)[row * p.ldf + (long long)h * dk + e]) + p.dt_bias[h * dk + e];
+          sd[j][at] = __expf(p.lower / (1.f + __expf(-a * raw)));
+        } else if (RULE == RULE_SOFTPLUS) {
+          float dec = 1.f;
+          if (!PAD || e < dk) {
+            const float raw = ((const float*)p.f)[row * p.ldf + (long long)h * dk + e] + p.dt_bias[h * dk + e];
+            dec = __expf(-a * (raw > 20.f ? raw : log1pf(__expf(raw))));
+          }
+          sd[j][at] = dec;
+        }
       }
     }
     for (int idx = tid; idx < nt * KDA_COLS; idx += 128) {
       const int j = idx / KDA_COLS, d = cg * KDA_COLS + idx % KDA_COLS;
-      sv[j][idx % KDA_COLS] = d < dv ? __bfloat162float(v[(long long)(t0 + j) * ld + (long long)h * dv + d]) : 0.f;
+      float x = d < dv ? to_f32(p.v[(long long)(t0 + j) * p.ld + (long long)h * dv + d]) : 0.f;
+      if (!DELTA) x = to_f32(from_f32<T>(x / (1.f + __expf(-x))));
+      sv[j][idx % KDA_COLS] = x;
     }
-    if (tid < nt) sb[tid] = 1.f / (1.f + __expf(-__bfloat162float(b[(long long)(t0 + tid) * ldb + h])));
+    if (DELTA && tid < nt) sb[tid] = 1.f / (1.f + __expf(-to_f32(p.b[(long long)(t0 + tid) * p.ldb + h])));
     __syncthreads();
     for (int j = 0; j < nt; ++j) {
       const float4* kq = reinterpret_cast<const float4*>(&sk[j][qtr * QS]);
       const float4* qq = reinterpret_cast<const float4*>(&sq[j][qtr * QS]);
-      const float4* dq = reinterpret_cast<const float4*>(&sd[j][qtr * QS]);
-      float4 kv4 = make_float4(0.f, 0.f, 0.f, 0.f);
+      float delta = sv[j][lc];
+      if (DELTA) {
+        const float4* dq = reinterpret_cast<const float4*>(&sd[DELTA ? j : 0][qtr * QS]);
+        float4 kv4 = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
-      for (int i = 0; i < QK / 4; ++i) {
-        const float4 kk = kq[i], dd = dq[i];
-        s_col[4 * i + 0] *= dd.x;
-        s_col[4 * i + 1] *= dd.y;
-        s_col[4 * i + 2] *= dd.z;
-        s_col[4 * i + 3] *= dd.w;
-        kv4.x += s_col[4 * i + 0] * kk.x;
-        kv4.y += s_col[4 * i + 1] * kk.y;
-        kv4.z += s_col[4 * i + 2] * kk.z;
-        kv4.w += s_col[4 * i + 3] * kk.w;
+        for (int i = 0; i < QK / 4; ++i) {
+          const float4 kk = kq[i], dd = dq[i];
+          s_col[4 * i + 0] *= dd.x;
+          s_col[4 * i + 1] *= dd.y;
+          s_col[4 * i + 2] *= dd.z;
+          s_col[4 * i + 3] *= dd.w;
+          kv4.x += s_col[4 * i + 0] * kk.x;
+          kv4.y += s_col[4 * i + 1] * kk.y;
+          kv4.z += s_col[4 * i + 2] * kk.z;
+          kv4.w += s_col[4 * i + 3] * kk.w;
+        }
+        float kv = (kv4.x + kv4.y) + (kv4.z + kv4.w);
+        if (XW) {
+          red_kv[qtr][lc] = kv;
+          __syncthreads();
+          kv = (red_kv[0][lc] + red_kv[1][lc]) + (red_kv[2][lc] + red_kv[3][lc]);
+        } else {
+          kv += __shfl_xor_sync(0xffffffffu, kv, 1);
+          kv += __shfl_xor_sync(0xffffffffu, kv, 2);
+        }
+        delta = (delta - kv) * sb[j];
       }
-      float kv = (kv4.x + kv4.y) + (kv4.z + kv4.w);
-      if (XW) {
-        red_kv[qtr][lc] = kv;
-        __syncthreads();
-        kv = (red_kv[0][lc] + red_kv[1][lc]) + (red_kv[2][lc] + red_kv[3][lc]);
-      } else {
-        kv += __shfl_xor_sync(0xffffffffu, kv, 1);
-        kv += __shfl_xor_sync(0xffffffffu, kv, 2);
-      }
-      const float delta = (sv[j][lc] - kv) * sb[j];
       float4 o4 = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
       for (int i = 0; i < QK / 4; ++i) {
         const float4 kk = kq[i], qv = qq[i];
+        if (!DELTA) {
+          s_col[4 * i + 0] *= fixed;
+          s_col[4 * i + 1] *= fixed;
+          s_col[4 * i + 2] *= fixed;
+          s_col[4 * i + 3] *= fixed;
+        }
         s_col[4 * i + 0] += kk.x * delta;
         s_col[4 * i + 1] += kk.y * delta;
         s_col[4 * i + 2] += kk.z * delta;
@@ -132,21 +188,50 @@ __global__ void __launch_bounds__(128) kda_recurrent_kernel(const bf16* __restri
       }
       float o = (o4.x + o4.y) + (o4.z + o4.w);
       if (XW) {
-        red_o[qtr][lc] = o;
+        // two buffers: with the delta rule the barrier in front of it orders a token's reads before the next token's
+        // writes, without it the next token writes the other buffer and the one after that comes behind its barrier
+        red_o[j & 1][qtr][lc] = o;
         __syncthreads();  // also orders this token's reads of red_kv before the next token's writes
-        o = (red_o[0][lc] + red_o[1][lc]) + (red_o[2][lc] + red_o[3][lc]);
+        o = (red_o[j & 1][0][lc] + red_o[j & 1][1][lc]) + (red_o[j & 1][2][lc] + red_o[j & 1][3][lc]);
       } else {
         o += __shfl_xor_sync(0xffffffffu, o, 1);
         o += __shfl_xor_sync(0xffffffffu, o, 2);
       }
-      if (owner && qtr == 0) out[((long long)(t0 + j) * heads + h) * dv + col] = __float2bfloat16(o);
+      if (owner && qtr == 0) p.out[((long long)(t0 + j) * heads + h) * dv + col] = from_f32<T>(o);
     }
     __syncthreads();
   }
   if (owner) {
 #pragma unroll
-    for (int i = 0; i < QK; ++i) S[(long long)(qtr * QK + i) * dv + col] = s_col[i];
+    for (int i = 0; i < QK; ++i)
+      if (!PAD || qtr * QK + i < dk) S[(long long)(qtr * QK + i) * dv + col] = s_col[i];
   }
+}
+
+template <typename T, int DK, int RULE, bool PAD>
+cudaError_t launch_rule(const RecArgs<T>& p, dim3 grid, bool few, cudaStream_t stream) {
+  return few ? launch_pdl(kda_recurrent_kernel<T, DK, true, RULE, PAD>, grid, dim3(128), (size_t)0, stream, p)
+             : launch_pdl(kda_recurrent_kernel<T, DK, false, RULE, PAD>, grid, dim3(128), (size_t)0, stream, p);
+}
+// any key width up to 256, on the next larger instantiated size
+template <typename T, int RULE>
+cudaError_t launch_padded(const RecArgs<T>& p, dim3 grid, bool few, cudaStream_t stream) {
+  if (p.dk == 128) return launch_rule<T, 128, RULE, false>(p, grid, few, stream);
+  if (p.dk == 64) return launch_rule<T, 64, RULE, false>(p, grid, few, stream);
+  if (p.dk <= 32) return launch_rule<T, 32, RULE, true>(p, grid, few, stream);
+  if (p.dk <= 64) return launch_rule<T, 64, RULE, true>(p, grid, few, stream);
+  if (p.dk <= 128) return launch_rule<T, 128, RULE, true>(p, grid, few, stream);
+  return launch_rule<T, 256, RULE, true>(p, grid, few, stream);
+}
+
+template <typename T>
+int run_rule(int rule, RecArgs<T> p, int num_seqs, int max_q_len, cudaStream_t stream) {
+  p.col_groups = (p.dv + KDA_COLS - 1) / KDA_COLS;
+  const dim3 grid(p.heads * p.col_groups, num_seqs);
+  const bool few = max_q_len <= 4;  // decode rows and verify steps: the row-coalesced mapping
+  PG_CUDA(rule == RULE_SOFTPLUS ? (launch_padded<T, RULE_SOFTPLUS>(p, grid, few, stream)) : (launch_padded<T, RULE_DECAY>(p, grid, few, stream)));
+  PG_LAUNCH_CHECK();
+  return PG_OK;
 }
 
 constexpr int ATTNRES_MAX = 16;  // candidates of one mix (snapshots + the current row)
@@ -211,33 +296,56 @@ extern "C" int pg_kda_recurrent(const void* q, const void* k, const void* v, lon
                                 int num_seqs, int heads, int dk, int dv, int max_q_len, cudaStream_t stream) {
   PG_REQUIRE(dv <= 128 && lower < 0.f, "kda_recurrent: dv=%d must be <= 128 and the decay lower bound %f negative", dv, (double)lower);
   if (num_seqs == 0) return PG_OK;
-  const int col_groups = (dv + KDA_COLS - 1) / KDA_COLS;
-  dim3 grid(heads * col_groups, num_seqs);
-  const bool few = max_q_len <= 4;  // decode rows and verify steps: the row-coalesced mapping
-#define PG_KDA_ARGS                                                                                                                              \
-  (const bf16*)q, (const bf16*)k, (const bf16*)v, ld, (const bf16*)f, ldf, (const bf16*)b, ldb, (const float*)a_log, (const float*)dt_bias, lower, \
-      (float*)state, (bf16*)out, (const int*)q_indptr, (const int*)slots, heads, dv, col_groups
-#define PG_KDA_LAUNCH(DKV)                                                     \
-  do {                                                                         \
-    if (few)                                                                   \
-      kda_recurrent_kernel<DKV, true><<<grid, 128, 0, stream>>>(PG_KDA_ARGS);  \
-    else                                                                       \
-      kda_recurrent_kernel<DKV, false><<<grid, 128, 0, stream>>>(PG_KDA_ARGS); \
-  } while (0)
+  RecArgs<bf16> p = {(const bf16*)q, (const bf16*)k, (const bf16*)v, ld, f, ldf, (const bf16*)b, ldb, (const float*)a_log, (const float*)dt_bias, nullptr, lower,
+                     (float*)state, (bf16*)out, (const int*)q_indptr, (const int*)slots, heads, heads, dk, dv, (dv + KDA_COLS - 1) / KDA_COLS, 0};
+  const dim3 grid(heads * p.col_groups, num_seqs);
+  const bool few = max_q_len <= 4;
   if (dk == 128)
-    PG_KDA_LAUNCH(128);
+    PG_CUDA((launch_rule<bf16, 128, RULE_BOUNDED, false>(p, grid, few, stream)));
   else if (dk == 64)
-    PG_KDA_LAUNCH(64);
+    PG_CUDA((launch_rule<bf16, 64, RULE_BOUNDED, false>(p, grid, few, stream)));
   else if (dk == 32)
-    PG_KDA_LAUNCH(32);
+    PG_CUDA((launch_rule<bf16, 32, RULE_BOUNDED, false>(p, grid, few, stream)));
   else {
     pg_set_error("kda_recurrent: dk=%d not supported (32, 64, 128)", dk);
     return PG_ERR_UNSUPPORTED;
   }
-#undef PG_KDA_LAUNCH
-#undef PG_KDA_ARGS
   PG_LAUNCH_CHECK();
   return PG_OK;
+}
+
+// The delta rule with the decay exp(-exp(A_log) * softplus(f + dt_bias)), f in f32, and query / key heads that several
+// value heads may share.
+extern "C" int pg_channel_delta(const void* q, const void* k, const void* v, long long ld, const void* f, long long ldf, const void* b, long long ldb, const void* a_log, const void* dt_bias,
+                                void* state, void* out, const void* q_indptr, const void* slots, int num_seqs, int heads, int kv_heads, int dk, int dv, int max_q_len, int skip_len, int is_f32,
+                                cudaStream_t stream) {
+  PG_REQUIRE(dk >= 1 && dk <= 256 && dv >= 1 && heads % kv_heads == 0, "channel_delta: heads %d / %d, key width %d (at most 256), value width %d", heads, kv_heads, dk, dv);
+  PG_REQUIRE(num_seqs <= 65535, "channel_delta: %d sequences", num_seqs);
+  if (num_seqs == 0) return PG_OK;
+  if (is_f32) {
+    RecArgs<float> p = {(const float*)q, (const float*)k, (const float*)v, ld, f, ldf, (const float*)b, ldb, (const float*)a_log, (const float*)dt_bias, nullptr, 0.f,
+                        (float*)state, (float*)out, (const int*)q_indptr, (const int*)slots, heads, kv_heads, dk, dv, 0, skip_len};
+    return run_rule<float>(RULE_SOFTPLUS, p, num_seqs, max_q_len, stream);
+  }
+  RecArgs<bf16> p = {(const bf16*)q, (const bf16*)k, (const bf16*)v, ld, f, ldf, (const bf16*)b, ldb, (const float*)a_log, (const float*)dt_bias, nullptr, 0.f,
+                     (float*)state, (bf16*)out, (const int*)q_indptr, (const int*)slots, heads, kv_heads, dk, dv, 0, skip_len};
+  return run_rule<bf16>(RULE_SOFTPLUS, p, num_seqs, max_q_len, stream);
+}
+
+// Linear attention with a fixed decay per head: S <- decay S + k v^T, o = S^T q, with SiLU on q, k and v inside.
+extern "C" int pg_decay_recurrent(const void* q, const void* k, const void* v, long long ld, const void* decay, void* state, void* out, const void* q_indptr, const void* slots, int num_seqs,
+                                  int heads, int dk, int dv, int max_q_len, int skip_len, int is_f32, cudaStream_t stream) {
+  PG_REQUIRE(dk >= 1 && dk <= 256 && dv >= 1, "decay_recurrent: key width %d (at most 256), value width %d", dk, dv);
+  PG_REQUIRE(num_seqs <= 65535, "decay_recurrent: %d sequences", num_seqs);
+  if (num_seqs == 0) return PG_OK;
+  if (is_f32) {
+    RecArgs<float> p = {(const float*)q, (const float*)k, (const float*)v, ld, nullptr, 0, nullptr, 0, nullptr, nullptr, (const float*)decay, 0.f,
+                        (float*)state, (float*)out, (const int*)q_indptr, (const int*)slots, heads, heads, dk, dv, 0, skip_len};
+    return run_rule<float>(RULE_DECAY, p, num_seqs, max_q_len, stream);
+  }
+  RecArgs<bf16> p = {(const bf16*)q, (const bf16*)k, (const bf16*)v, ld, nullptr, 0, nullptr, 0, nullptr, nullptr, (const float*)decay, 0.f,
+                     (float*)state, (bf16*)out, (const int*)q_indptr, (const int*)slots, heads, heads, dk, dv, 0, skip_len};
+  return run_rule<bf16>(RULE_DECAY, p, num_seqs, max_q_len, stream);
 }
 
 extern "C" int pg_attnres_mix(const void* cur, long long ld_cur, const void* snaps, long long ld_tok, const void* score_w, void* out, long long ld_out,

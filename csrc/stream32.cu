@@ -1,0 +1,354 @@
+// Row kernels around a residual stream that is kept in 32 bits, for bf16 and f32 activations.
+//
+//  * embed_rows: table row -> f32 stream row (+ a copy in the activation type for the next projection).
+//  * post_norm: the norm after the sum.  s = alpha * x + y; x = s / sqrt(mean(s^2) + eps) * w.  The stream x is read and
+//    written in f32, y is a projection's output (f32 or bf16), and the activation-type copy that the next projection
+//    reads is written in the same pass.  Without y and with alpha = 1 it is a plain RMS norm of the stream.
+//  * gated_row_norm: RMS norm over a row (one head, or all heads of a token at once), times a weight, times the sigmoid
+//    of a gate row that may lie inside a wider projection output.
+//  * glu_rows: silu(gate) * up on f32 rows; softcap_f32: cap * tanh(x / cap) on f32 values.
+//  * gemm_simt: y = x w^T on the CUDA cores with f32 accumulation, for f32 operands (the 32-bit mode) and for bf16
+//    problems whose rows the TMA kernels cannot address (an inner size that is not a multiple of 8).
+//  * conv_silu: causal depthwise convolution of any length + SiLU over ragged sequences with carried inputs.
+#include "api.h"
+#include "common.cuh"
+#include "types.cuh"
+
+namespace {
+
+template <typename TI, typename TO>
+__global__ void __launch_bounds__(256) embed_rows_kernel(const TI* __restrict__ table, long long ldt, const int* __restrict__ ids, float* __restrict__ x, TO* __restrict__ xt, long long ldxt,
+                                                         int width, long long rows, uint32_t* status) {
+  PG_PDL_ENTRY();
+  const int t = blockIdx.x;
+  long long id = ids[t];
+  if (id < 0 || id >= rows) {
+    if (threadIdx.x == 0) atomicCAS(status, PG_ST_OK, PG_ST_BOUNDS | (50u << 8));
+    id = 0;
+  }
+  for (int i = threadIdx.x; i < width; i += blockDim.x) {
+    const float v = to_f32(table[id * ldt + i]);
+    if (x) x[(long long)t * width + i] = v;
+    if (xt) xt[(long long)t * ldxt + i] = from_f32<TO>(v);
+  }
+}
+
+// One CTA per row; V consecutive elements per access (4 when every row allows it, else 1).
+template <typename TY, typename TO, int V>
+__global__ void __launch_bounds__(256) post_norm_kernel(const TY* __restrict__ y, long long ldy, const float* __restrict__ xin, float* __restrict__ x, float alpha, const float* __restrict__ w, TO* __restrict__ xt,
+                                                        long long ldxt, int width, float eps) {
+  PG_PDL_ENTRY();
+  __shared__ float red[32];
+  constexpr int KEEP = 8;
+  const long long row = blockIdx.x;
+  const int nv = width / V;
+  const float* xi = xin + row * width;
+  const TY* yr = y ? y + row * ldy : nullptr;
+  float s[KEEP][V];
+  float ss = 0.f;
+  auto sum_at = [&](int i, float* o) {
+    load_vec<V>(xi + i * V, o);
+#pragma unroll
+    for (int j = 0; j < V; ++j) o[j] *= alpha;
+    if (yr) {
+      float f[V];
+      load_vec<V>(yr + i * V, f);
+#pragma unroll
+      for (int j = 0; j < V; ++j) o[j] += f[j];
+    }
+  };
+#pragma unroll
+  for (int k = 0; k < KEEP; ++k) {
+    const int i = threadIdx.x + k * 256;
+    if (i < nv) {
+      sum_at(i, s[k]);
+#pragma unroll
+      for (int j = 0; j < V; ++j) ss += s[k][j] * s[k][j];
+    }
+  }
+  for (int i = threadIdx.x + KEEP * 256; i < nv; i += 256) {  // wider rows: summed again below
+    float o[V];
+    sum_at(i, o);
+#pragma unroll
+    for (int j = 0; j < V; ++j) ss += o[j] * o[j];
+  }
+  ss = block_sum(ss, red);
+  const float inv = rsqrtf(ss / (float)width + eps);
+  auto put = [&](int i, float* o) {
+    float wf[V];
+    load_vec<V>(w + i * V, wf);
+#pragma unroll
+    for (int j = 0; j < V; ++j) o[j] = o[j] * inv * wf[j];
+    if (x) store_vec<V>(x + row * width + i * V, o);
+    if (xt) store_vec<V>(xt + row * ldxt + i * V, o);
+  };
+#pragma unroll
+  for (int k = 0; k < KEEP; ++k) {
+    const int i = threadIdx.x + k * 256;
+    if (i < nv) put(i, s[k]);
+  }
+  for (int i = threadIdx.x + KEEP * 256; i < nv; i += 256) {
+    float o[V];
+    sum_at(i, o);
+    put(i, o);
+  }
+}
+
+// TPR threads per row (32 or 256); row r = token * heads + head; the gate row of (token, head) is gate + token * ldg + head * dim.
+template <typename T, int V, int TPR>
+__global__ void __launch_bounds__(256) gated_row_norm_kernel(const T* __restrict__ x, const T* __restrict__ gate, long long ldg, const float* __restrict__ w, T* __restrict__ y, long long rows, int heads, int dim,
+                                                             float eps) {
+  PG_PDL_ENTRY();
+  __shared__ float red[32];
+  const long long row = TPR == 256 ? (long long)blockIdx.x : (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
+  const int me = TPR == 256 ? threadIdx.x : (threadIdx.x & 31);
+  if (row >= rows) return;  // whole warps leave together; with TPR == 256 the grid has no spare blocks
+  const T* xr = x + row * dim;
+  const T* gr = gate + (row / heads) * ldg + (row % heads) * dim;
+  constexpr int KEEP = 4;
+  const int nv = dim / V;
+  float f[KEEP][V], ss = 0.f;
+#pragma unroll
+  for (int k = 0; k < KEEP; ++k) {
+    const int i = me + k * TPR;
+    if (i < nv) {
+      load_vec<V>(xr + i * V, f[k]);
+#pragma unroll
+      for (int j = 0; j < V; ++j) ss += f[k][j] * f[k][j];
+    }
+  }
+  for (int i = me + KEEP * TPR; i < nv; i += TPR) {
+    float o[V];
+    load_vec<V>(xr + i * V, o);
+#pragma unroll
+    for (int j = 0; j < V; ++j) ss += o[j] * o[j];
+  }
+  ss = TPR == 256 ? block_sum(ss, red) : warp_sum(ss);
+  const float inv = rsqrtf(ss / (float)dim + eps);
+  auto put = [&](int i, const float* o) {
+    float g[V], wf[V], r[V];
+    load_vec<V>(gr + i * V, g);
+    load_vec<V>(w + i * V, wf);
+#pragma unroll
+    for (int j = 0; j < V; ++j) r[j] = o[j] * inv * wf[j] / (1.f + __expf(-g[j]));
+    store_vec<V>(y + row * dim + i * V, r);
+  };
+#pragma unroll
+  for (int k = 0; k < KEEP; ++k) {
+    const int i = me + k * TPR;
+    if (i < nv) put(i, f[k]);
+  }
+  for (int i = me + KEEP * TPR; i < nv; i += TPR) {
+    float o[V];
+    load_vec<V>(xr + i * V, o);
+    put(i, o);
+  }
+}
+
+__global__ void glu_rows_kernel(const float* __restrict__ gu, float* __restrict__ out, int rows, int inter, long long ldin) {
+  PG_PDL_ENTRY();
+  const long long total = (long long)rows * inter;
+  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (long long)gridDim.x * blockDim.x) {
+    const long long r = i / inter, c = i % inter;
+    const float g = gu[r * ldin + c], u = gu[r * ldin + inter + c];
+    out[i] = g / (1.f + __expf(-g)) * u;
+  }
+}
+
+__global__ void softcap_f32_kernel(const float* __restrict__ x, float* __restrict__ y, long long n, float cap) {
+  PG_PDL_ENTRY();
+  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x) y[i] = cap * tanh_full(x[i] / cap);
+}
+
+// 64 x 64 output tile, 256 threads of 4 x 4 outputs, 16-deep k steps.
+template <typename TX, typename TY>
+__global__ void __launch_bounds__(256) gemm_simt_kernel(const TX* __restrict__ x, const TX* __restrict__ w, TY* __restrict__ y, int T, int M, int K, long long ldx, long long ldw, long long ldy) {
+  PG_PDL_ENTRY();
+  __shared__ float xs[16][68], ws[16][68];
+  const int m0 = blockIdx.x * 64, t0 = blockIdx.y * 64;
+  const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+  float acc[4][4] = {};
+  for (int k0 = 0; k0 < K; k0 += 16) {
+    for (int i = threadIdx.x; i < 64 * 16; i += 256) {
+      const int r = i >> 4, k = i & 15;
+      const bool kin = k0 + k < K;
+      xs[k][r] = (kin && t0 + r < T) ? to_f32(x[(long long)(t0 + r) * ldx + k0 + k]) : 0.f;
+      ws[k][r] = (kin && m0 + r < M) ? to_f32(w[(long long)(m0 + r) * ldw + k0 + k]) : 0.f;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < 16; ++k) {
+      const float4 a = *reinterpret_cast<const float4*>(&xs[k][ty * 4]), b = *reinterpret_cast<const float4*>(&ws[k][tx * 4]);
+      const float av[4] = {a.x, a.y, a.z, a.w}, bv[4] = {b.x, b.y, b.z, b.w};
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(av[i], bv[j], acc[i][j]);
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int t = t0 + ty * 4 + i, m = m0 + tx * 4 + j;
+      if (t < T && m < M) y[(long long)t * ldy + m] = from_f32<TY>(acc[i][j]);
+    }
+}
+
+constexpr int CONV_MAX = 16;   // taps
+constexpr int CONV_TILE = 32;  // tokens per CTA; at least CONV_MAX, so a sequence of more than one tile fills the carried inputs from its own rows
+
+// A thread owns one channel for CONV_TILE tokens.  The CTA of a sequence's first tile reads the carried inputs and is also
+// the one that replaces them (from the sequence's last rows), so no other CTA touches the state.
+template <typename T>
+__global__ void __launch_bounds__(128) conv_silu_kernel(const T* __restrict__ x, long long ldx, const float* __restrict__ w, T* __restrict__ state, T* __restrict__ out, long long ldo, const int* __restrict__ q_indptr,
+                                                        const int* __restrict__ slots, int channels, int taps, long long slot_stride) {
+  PG_PDL_ENTRY();
+  const int b = blockIdx.z, c = blockIdx.x * 128 + threadIdx.x;
+  const int q0 = q_indptr[b], n = q_indptr[b + 1] - q0;
+  const int s0 = blockIdx.y * CONV_TILE;
+  const int slot = slots[b];
+  if (c >= channels || s0 >= n || slot < 0) return;
+  T* st = state + slot * slot_stride + (long long)c * (taps - 1);
+  const int back = taps - 1;
+  // history: inputs s0 - back .. s0 - 1 of the sequence (from the state where they lie before this step)
+  float win[CONV_MAX], wt[CONV_MAX];
+#pragma unroll
+  for (int j = 0; j < CONV_MAX; ++j) wt[j] = j < taps ? w[(long long)c * taps + j] : 0.f;
+#pragma unroll
+  for (int j = 0; j < CONV_MAX - 1; ++j) {
+    const int at = s0 - back + j;
+    win[j] = j < back ? (at < 0 ? to_f32(st[back + at]) : to_f32(x[(long long)(q0 + at) * ldx + c])) : 0.f;
+  }
+  T keep[CONV_MAX];
+  if (s0 == 0) {
+#pragma unroll
+    for (int j = 0; j < CONV_MAX - 1; ++j) {
+      const int at = n - back + j;
+      if (j < back) keep[j] = at < 0 ? st[back + at] : x[(long long)(q0 + at) * ldx + c];
+    }
+  }
+  const int end = min(s0 + CONV_TILE, n);
+  for (int s = s0; s < end; ++s) {
+    const float cur = to_f32(x[(long long)(q0 + s) * ldx + c]);
+    float a = 0.f;
+#pragma unroll
+    for (int j = 0; j < CONV_MAX; ++j) {
+      if (j < back) a = fmaf(win[j], wt[j], a);
+      if (j == back) a = fmaf(cur, wt[j], a);
+    }
+    out[(long long)(q0 + s) * ldo + c] = from_f32<T>(a / (1.f + __expf(-a)));
+#pragma unroll
+    for (int j = 0; j < CONV_MAX - 1; ++j) {
+      if (j + 1 < back) win[j] = win[j + 1];
+      if (j + 1 == back) win[j] = cur;
+    }
+  }
+  if (s0 == 0) {
+#pragma unroll
+    for (int j = 0; j < CONV_MAX - 1; ++j)
+      if (j < back) st[j] = keep[j];
+  }
+}
+
+inline bool al(const void* p, int bytes) { return ((uintptr_t)p % bytes) == 0; }
+
+}  // namespace
+
+// Element types of the calls below: 0 bf16, 1 f32.
+extern "C" int pg_embed_rows(const void* table, int table_f32, long long ldt, const void* ids, void* x_f32, void* xt, int xt_f32, long long ldxt, int tokens, int width, long long rows, void* status, cudaStream_t stream) {
+  if (tokens == 0) return PG_OK;
+#define PG_EMBED(TI, TO) launch_pdl(embed_rows_kernel<TI, TO>, dim3(tokens), dim3(256), (size_t)0, stream, (const TI*)table, ldt, (const int*)ids, (float*)x_f32, (TO*)xt, ldxt, width, rows, (uint32_t*)status)
+  if (table_f32)
+    PG_CUDA(xt_f32 ? PG_EMBED(float, float) : PG_EMBED(float, bf16));
+  else
+    PG_CUDA(xt_f32 ? PG_EMBED(bf16, float) : PG_EMBED(bf16, bf16));
+#undef PG_EMBED
+  PG_LAUNCH_CHECK();
+  return PG_OK;
+}
+
+extern "C" int pg_post_norm(const void* y, int y_f32, long long ldy, const void* x_in, void* x_out, float alpha, const void* w, void* xt, int xt_f32, long long ldxt, int tokens, int width, float eps, cudaStream_t stream) {
+  PG_REQUIRE(x_in != nullptr && w != nullptr && (x_out || xt), "post_norm: the stream, its norm weight and a destination are required");
+  if (tokens == 0) return PG_OK;
+  const int yb = y_f32 ? 4 : 2, tb = xt_f32 ? 4 : 2;
+  const bool v4 = width % 4 == 0 && al(x_in, 16) && al(w, 16) && (!x_out || al(x_out, 16)) && (!y || (ldy % 4 == 0 && al(y, 4 * yb))) && (!xt || (ldxt % 4 == 0 && al(xt, 4 * tb)));
+#define PG_PN(TY, TO, V) launch_pdl(post_norm_kernel<TY, TO, V>, dim3(tokens), dim3(256), (size_t)0, stream, (const TY*)y, ldy, (const float*)x_in, (float*)x_out, alpha, (const float*)w, (TO*)xt, ldxt, width, eps)
+#define PG_PN2(TY, TO) (v4 ? PG_PN(TY, TO, 4) : PG_PN(TY, TO, 1))
+  if (y_f32)
+    PG_CUDA(xt_f32 ? PG_PN2(float, float) : PG_PN2(float, bf16));
+  else
+    PG_CUDA(xt_f32 ? PG_PN2(bf16, float) : PG_PN2(bf16, bf16));
+#undef PG_PN2
+#undef PG_PN
+  PG_LAUNCH_CHECK();
+  return PG_OK;
+}
+
+extern "C" int pg_gated_row_norm(const void* x, const void* gate, long long ldg, const void* w, void* y, int tokens, int heads, int dim, float eps, int is_f32, cudaStream_t stream) {
+  if (tokens == 0) return PG_OK;
+  const long long rows = (long long)tokens * heads;
+  const bool wide = dim > 512;
+  const dim3 grid((unsigned)(wide ? rows : (rows + 7) / 8));
+#define PG_GRN(T, V, TPR) launch_pdl(gated_row_norm_kernel<T, V, TPR>, grid, dim3(256), (size_t)0, stream, (const T*)x, (const T*)gate, ldg, (const float*)w, (T*)y, rows, heads, dim, eps)
+  if (is_f32) {
+    PG_CUDA(wide ? PG_GRN(float, 1, 256) : PG_GRN(float, 1, 32));
+  } else {
+    const bool v8 = dim % 8 == 0 && ldg % 8 == 0 && al(x, 16) && al(gate, 16) && al(w, 16) && al(y, 16);
+    if (v8)
+      PG_CUDA(wide ? PG_GRN(bf16, 8, 256) : PG_GRN(bf16, 8, 32));
+    else
+      PG_CUDA(wide ? PG_GRN(bf16, 1, 256) : PG_GRN(bf16, 1, 32));
+  }
+#undef PG_GRN
+  PG_LAUNCH_CHECK();
+  return PG_OK;
+}
+
+extern "C" int pg_glu_rows_f32(const void* gu, void* out, int rows, int inter, long long ldin, cudaStream_t stream) {
+  if (rows == 0 || inter == 0) return PG_OK;
+  long long blocks = ((long long)rows * inter + 255) / 256;
+  if (blocks > 148 * 16) blocks = 148 * 16;
+  PG_CUDA(launch_pdl(glu_rows_kernel, dim3((unsigned)blocks), dim3(256), (size_t)0, stream, (const float*)gu, (float*)out, rows, inter, ldin));
+  PG_LAUNCH_CHECK();
+  return PG_OK;
+}
+
+extern "C" int pg_softcap_f32(const void* x, void* y, long long n, float cap, cudaStream_t stream) {
+  PG_REQUIRE(cap > 0.f, "softcap: the cap must be positive");
+  if (n == 0) return PG_OK;
+  long long blocks = (n + 255) / 256;
+  if (blocks > 148 * 16) blocks = 148 * 16;
+  PG_CUDA(launch_pdl(softcap_f32_kernel, dim3((unsigned)blocks), dim3(256), (size_t)0, stream, (const float*)x, (float*)y, n, cap));
+  PG_LAUNCH_CHECK();
+  return PG_OK;
+}
+
+extern "C" int pg_gemm_simt(const void* x, const void* w, int x_f32, void* y, int y_f32, int T, int M, int K, long long ldx, long long ldw, long long ldy, cudaStream_t stream) {
+  PG_REQUIRE(T > 0 && M > 0 && K > 0, "gemm_simt: empty problem %dx%dx%d", T, M, K);
+  const dim3 grid((M + 63) / 64, (T + 63) / 64);
+  PG_REQUIRE(grid.y <= 65535u, "gemm_simt: %d rows", T);
+#define PG_SG(TX, TY) launch_pdl(gemm_simt_kernel<TX, TY>, grid, dim3(256), (size_t)0, stream, (const TX*)x, (const TX*)w, (TY*)y, T, M, K, ldx, ldw, ldy)
+  if (x_f32)
+    PG_CUDA(y_f32 ? PG_SG(float, float) : PG_SG(float, bf16));
+  else
+    PG_CUDA(y_f32 ? PG_SG(bf16, float) : PG_SG(bf16, bf16));
+#undef PG_SG
+  PG_LAUNCH_CHECK();
+  return PG_OK;
+}
+
+extern "C" int pg_conv_silu(const void* x, long long ldx, const void* w, void* state, void* out, long long ldo, const void* q_indptr, const void* slots, int num_seqs, int channels, int taps, long long slot_stride,
+                            int max_q_len, int is_f32, cudaStream_t stream) {
+  PG_REQUIRE(taps >= 1 && taps <= CONV_MAX, "conv_silu: %d taps (1..%d)", taps, CONV_MAX);
+  if (num_seqs == 0) return PG_OK;
+  const dim3 grid((channels + 127) / 128, (max_q_len + CONV_TILE - 1) / CONV_TILE, num_seqs);
+  PG_REQUIRE(grid.y <= 65535u && grid.z <= 65535u, "conv_silu: %d sequences of %d rows", num_seqs, max_q_len);
+  if (is_f32)
+    PG_CUDA(launch_pdl(conv_silu_kernel<float>, grid, dim3(128), (size_t)0, stream, (const float*)x, ldx, (const float*)w, (float*)state, (float*)out, ldo, (const int*)q_indptr, (const int*)slots, channels, taps, slot_stride));
+  else
+    PG_CUDA(launch_pdl(conv_silu_kernel<bf16>, grid, dim3(128), (size_t)0, stream, (const bf16*)x, ldx, (const float*)w, (bf16*)state, (bf16*)out, ldo, (const int*)q_indptr, (const int*)slots, channels, taps, slot_stride));
+  PG_LAUNCH_CHECK();
+  return PG_OK;
+}

@@ -24,13 +24,26 @@ ARCH_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a"]
 COMMON_FLAGS = ["-O3", "-std=c++17", "-lineinfo", "--use_fast_math", "-Xcompiler", "-fPIC", "-Xcompiler", "-O3", "--expt-relaxed-constexpr"]
 
 _lib = None
+_units = None  # names of the translation units the library is made of (None: all)
+
+
+def use_units(names) -> None:
+    """Build and load a library of these translation units only (``csrc/<name>.cu``), unless the full library is up to
+    date.  For programs that serve one model from a fresh checkout; call it before the first kernel."""
+    global _units, LIB_PATH, STAMP
+    if names is None or _lib is not None or is_current():
+        return
+    _units = tuple(sorted(names))
+    tag = hashlib.sha256(" ".join(_units).encode()).hexdigest()[:8]
+    LIB_PATH = os.path.join(LIB_DIR, f"libpegainfer_b200_{tag}.so")
+    STAMP = os.path.join(LIB_DIR, f"build_{tag}.stamp")
 
 
 def _sources():
     out = []
     for dp, _, fns in os.walk(CSRC):
         for fn in sorted(fns):
-            if fn.endswith((".cu", ".cpp")):
+            if fn.endswith((".cu", ".cpp")) and (_units is None or os.path.splitext(fn)[0] in _units):
                 out.append(os.path.join(dp, fn))
     return sorted(out)
 

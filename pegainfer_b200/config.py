@@ -18,9 +18,37 @@ from dataclasses import dataclass, field, replace
 from typing import Optional
 
 
+@dataclass(frozen=True)
+class MixerSpec:
+    """Token mixer of one layer, for families whose layers are listed one by one.  ``kind``: ``"attention"`` (all fields but
+    the recurrent ones), ``"lightning"`` (fixed decay per head) or ``"channel_delta"`` (gated delta rule with a decay per key
+    channel; ``conv`` taps, low-rank decay and output-gate projections of the given ranks)."""
+
+    kind: str
+    heads: int
+    dim: int  # query / key size of a head
+    vdim: int
+    kv_heads: int = 0  # attention: KV heads; channel_delta: query / key heads
+    scale: float = 1.0
+    softcap: float = 0.0  # 0: no cap
+    rot_dims: int = 0
+    rot_base: float = 10000.0
+    kv_from: int = -1  # attention: layer whose cache this layer reads (-1: its own)
+    decay: tuple = ()
+    conv: int = 0
+    decay_rank: int = 0
+    gate_rank: int = 0
+
+
+@dataclass(frozen=True)
+class LayerSpec:
+    mixer: MixerSpec
+    ff: int = 0  # width of the SwiGLU feed-forward (0: the layer has none)
+
+
 @dataclass
 class ModelConfig:
-    family: str = "qwen3"  # qwen3 | qwen35 | deepseek_v2 | kimi_k2 | glm_dsa | gemma4 | kimi_k3
+    family: str = "qwen3"  # qwen3 | qwen35 | deepseek_v2 | kimi_k2 | glm_dsa | gemma4 | kimi_k3 | nemipel
     vocab_size: int = 1024
     hidden_size: int = 256
     num_layers: int = 2
@@ -88,6 +116,10 @@ class ModelConfig:
     attn_res_block: int = 0
     kda_gate_rank: int = 0
     kda_gate_lower_bound: float = -5.0
+    # families whose layers are listed one by one (Nemipel line): the mixer and feed-forward of every layer, the factor on
+    # the stream in the norm after the sum; final_logit_softcapping caps the logits
+    layer_specs: tuple = ()
+    postln_alpha: float = 1.0
 
     # -- derived ---------------------------------------------------------------
     @property
@@ -221,6 +253,27 @@ PRESETS["kimi-k3"] = replace(PRESETS["small-k3"], vocab_size=163840, hidden_size
 # a one-GPU slice of the released shape for benchmarks (not a released configuration): full-width layers (6 KDA + 2 MLA, one dense
 # and seven latent-MoE layers), 32 routed experts instead of 896, top 8
 PRESETS["k3-8layer-shape"] = replace(PRESETS["kimi-k3"], num_layers=8, layer_types=_k3_pattern(8), n_routed_experts=32, num_experts_per_tok=8, attn_res_block=4, max_position=131072)
+def _nemipel(width: int, vocab: int, ff: int, heads: int, kv_heads: int, dim: int, lin_heads: int, lin_dim: int, rank: int, periods: int, **kw) -> ModelConfig:
+    """A Nemipel stack of ``periods`` x (lightning, attention, channel-delta); every second attention layer reads the cache
+    of the one before it, the attention layers have the feed-forwards."""
+    layers = []
+    for n in range(periods):
+        own = 3 * n + 1 if n % 2 == 0 else 3 * (n - 1) + 1
+        layers.append(LayerSpec(MixerSpec("lightning", lin_heads, lin_dim, lin_dim, decay=tuple(float(f"{1 - 2.0 ** (-1 - 7 * h / max(lin_heads - 1, 1)):.6f}") for h in range(lin_heads)))))
+        layers.append(LayerSpec(MixerSpec("attention", heads, dim, dim, kv_heads=kv_heads, scale=dim ** -0.5, softcap=30.0, rot_dims=dim // 2, rot_base=1e4,
+                                          kv_from=-1 if own == 3 * n + 1 else own), ff))
+        layers.append(LayerSpec(MixerSpec("channel_delta", lin_heads, lin_dim, lin_dim, kv_heads=lin_heads // 2, conv=4, decay_rank=rank, gate_rank=rank), ff))
+    base = dict(family="nemipel", vocab_size=vocab, hidden_size=width, num_layers=len(layers), num_q_heads=heads, num_kv_heads=kv_heads, head_dim=dim, intermediate_size=ff, qk_norm=False,
+                layer_specs=tuple(layers), postln_alpha=2.0, final_logit_softcapping=20.0, max_position=131072)
+    base.update(kw)
+    return ModelConfig(**base)
+
+
+PRESETS["tiny-nemipel"] = _nemipel(96, 256, 160, 4, 2, 32, 4, 16, 12, 2, max_position=4096)
+PRESETS["small-nemipel"] = _nemipel(1024, 4096, 2048, 8, 2, 128, 8, 128, 64, 2, max_position=8192)
+# layers as wide as those of an 8 B-parameter model, for benchmarks (not a released configuration): 12 lightning, 12
+# attention (6 of them with a cache of their own) and 12 channel-delta layers
+PRESETS["nemipel-8b-shape"] = _nemipel(4096, 151936, 12288, 32, 8, 128, 32, 128, 128, 12)
 PRESETS["small-glm-fp8"] = replace(PRESETS["small-glm"], expert_quant="fp8_block128", dense_quant="fp8_block128")
 for _name in ("tiny-dsv2", "small-dsv2", "dsv2-lite"):
     if _name in PRESETS:
@@ -235,6 +288,8 @@ def preset(name: str, **overrides) -> ModelConfig:
 
 def detect_family(cfg: dict) -> str:
     """Map a ``config.json`` to a model line (exactly one line must claim it)."""
+    if cfg.get("architecture") == "Nemipel":
+        return "nemipel"
     mt = cfg.get("model_type", "")
     archs = " ".join(cfg.get("architectures", []))
     if mt in ("qwen3",) or "Qwen3ForCausalLM" in archs:
@@ -294,9 +349,67 @@ def _k3_from_hf(cfg: dict, top: dict, model_dir: Optional[str]) -> ModelConfig:
                        eos_token_ids=_eos_ids(model_dir, top))
 
 
+def _nemipel_from_json(cfg: dict, model_dir: Optional[str]) -> ModelConfig:
+    """``config.json`` of the Nemipel line: sizes and constants per layer."""
+    layers = []
+    for i, entry in enumerate(cfg["layers"]):
+        m, kind = entry["mixer"], entry["type"]
+        common = dict(kind=kind, heads=m["heads"], dim=m["dim"], vdim=m["vdim"])
+        if kind == "attention":
+            rot = m.get("rot") or {}
+            src = m.get("kv_from")
+            spec = MixerSpec(kv_heads=m["kv_heads"], scale=float(m["scale"]), softcap=float(m.get("softcap") or 0.0), rot_dims=rot.get("dims", 0), rot_base=float(rot.get("base", 1e4)),
+                             kv_from=-1 if src is None else src, **common)
+            if src is not None:
+                own = layers[src].mixer if 0 <= src < i else None
+                if own is None or own.kind != "attention" or own.kv_from >= 0 or (own.kv_heads, own.dim, own.vdim) != (spec.kv_heads, spec.dim, spec.vdim):
+                    raise ValueError(f"layer {i}: kv_from={src} is not an earlier attention layer with a cache of the same shape")
+        elif kind == "lightning":
+            spec = MixerSpec(decay=tuple(float(d) for d in m["decay"]), **common)
+        elif kind == "channel_delta":
+            spec = MixerSpec(kv_heads=m["kv_heads"], conv=m["conv"], **common)
+        else:
+            raise ValueError(f"layer {i}: no mixer of type {kind!r}")
+        mlp = entry.get("mlp")
+        if mlp is not None and mlp.get("kind", "dense") != "dense":
+            raise ValueError(f"layer {i}: no feed-forward of kind {mlp['kind']!r}")
+        layers.append(LayerSpec(spec, mlp["ff"] if mlp else 0))
+    attn = [l.mixer for l in layers if l.mixer.kind == "attention"] or [layers[0].mixer]
+    return ModelConfig(family="nemipel", vocab_size=cfg["vocab"], hidden_size=cfg["width"], num_layers=len(layers), num_q_heads=attn[0].heads, num_kv_heads=max(attn[0].kv_heads, 1),
+                       head_dim=attn[0].dim, intermediate_size=max(l.ff for l in layers), rms_eps=cfg["norm"]["eps"], qk_norm=False, layer_specs=tuple(layers),
+                       postln_alpha=float(cfg["postln_alpha"]), final_logit_softcapping=float(cfg.get("logit_softcap") or 0.0), max_position=131072, eos_token_ids=_eos_ids(model_dir, cfg))
+
+
+def nemipel_to_json(cfg: ModelConfig) -> dict:
+    """The ``config.json`` that ``_nemipel_from_json`` reads back."""
+    layers = []
+    for l in cfg.layer_specs:
+        m = l.mixer
+        mix = dict(heads=m.heads, dim=m.dim, vdim=m.vdim)
+        if m.kind == "attention":
+            mix.update(kv_heads=m.kv_heads, scale=m.scale, rot=dict(dims=m.rot_dims, base=m.rot_base))
+            if m.softcap:
+                mix["softcap"] = m.softcap
+            if m.kv_from >= 0:
+                mix["kv_from"] = m.kv_from
+        elif m.kind == "lightning":
+            mix["decay"] = list(m.decay)
+        else:
+            mix.update(kv_heads=m.kv_heads, conv=m.conv)
+        layers.append(dict(type=m.kind, mixer=mix, mlp=dict(kind="dense", ff=l.ff) if l.ff else None))
+    out = dict(architecture="Nemipel", vocab=cfg.vocab_size, width=cfg.hidden_size, norm=dict(eps=cfg.rms_eps), postln_alpha=cfg.postln_alpha, layers=layers)
+    if cfg.final_logit_softcapping:
+        out["logit_softcap"] = cfg.final_logit_softcapping
+    if cfg.eos_token_ids:
+        out["eos_token_id"] = list(cfg.eos_token_ids)
+    return out
+
+
 def from_hf(cfg: dict, model_dir: Optional[str] = None) -> ModelConfig:
     family = detect_family(cfg)
     top = cfg
+    if family == "nemipel":
+        return _nemipel_from_json(cfg, model_dir)
     if family == "qwen35" and "text_config" in cfg:
         cfg = cfg["text_config"]
     if family == "kimi_k2" and "text_config" in cfg:
@@ -449,7 +562,8 @@ class EngineConfig:
     comm: str = "fused"  # fused | nccl
     gemm: str = "sm100"  # sm100 | cublas
     seed: int = 0
-    dtype: str = "bfloat16"
+    dtype: str = "bfloat16"  # activations and cache on the GPU; "float32" on the lines that have 32-bit kernels
+    state_slots: Optional[int] = None  # lines with recurrent state: requests that hold state at a time (default: from the decode batch)
 
     def validate(self) -> None:
         if self.kv_page_size not in (16, 32, 64):
@@ -462,6 +576,10 @@ class EngineConfig:
             raise ValueError("--comm must be fused or nccl")
         if self.gemm not in ("sm100", "cublas"):
             raise ValueError("--gemm must be sm100 or cublas")
+        if self.dtype not in ("bfloat16", "float32"):
+            raise ValueError("--dtype must be bfloat16 or float32")
+        if self.state_slots is not None and self.state_slots < 1:
+            raise ValueError("--state-slots must be positive")
         for n in ("tp_size", "dp_size", "ep_size"):
             if getattr(self, n) < 1:
                 raise ValueError(f"--{n.replace('_', '-')} must be >= 1")

@@ -25,6 +25,9 @@ from .contract import EngineInfo, KvCapacity
 from .driver import Engine
 
 
+F32_FAMILIES = ("nemipel",)  # lines whose kernels also run in 32-bit on the GPU
+
+
 def resolve_model_config(ecfg: EngineConfig) -> ModelConfig:
     if ecfg.model_path:
         return load_model_config(ecfg.model_path)
@@ -65,6 +68,8 @@ def profile_kv_blocks(model, ecfg: EngineConfig, page_size: int) -> int:
     act = rows * (model.cfg.hidden_size * 8 + getattr(model.cfg, "intermediate_size", 0) * 6 // max(model.tp.world, 1)) * elem
     logits = ecfg.max_decode_batch * model.cfg.vocab_size * (2 + 4)
     budget = int(total * ecfg.gpu_memory_utilization) - base - act - logits - (ecfg.kv_cache_memory_margin_mib << 20)
+    if hasattr(model, "state_bytes"):  # recurrent-state slots are allocated beside the cache
+        budget -= model.state_bytes(ecfg.state_slots or ecfg.max_decode_batch)
     return max(0, budget // per_block)
 
 
@@ -75,7 +80,9 @@ def build_engine(ecfg: EngineConfig, mcfg: Optional[ModelConfig] = None, device=
         device = f"cuda:{ecfg.device_ordinal}" if torch.cuda.is_available() else "cpu"
     device = torch.device(device)
     if dtype is None:
-        dtype = torch.bfloat16 if device.type == "cuda" else torch.float32
+        dtype = getattr(torch, ecfg.dtype) if device.type == "cuda" else torch.float32
+    if device.type == "cuda" and dtype != torch.bfloat16 and model is None and mcfg.family not in F32_FAMILIES:
+        raise ValueError(f"the {mcfg.family} line has bfloat16 kernels only")
     if ecfg.gemm == "cublas" and device.type == "cuda":
         from .. import ops
 
@@ -107,12 +114,13 @@ def build_engine(ecfg: EngineConfig, mcfg: Optional[ModelConfig] = None, device=
     kv = model.make_kv(nblocks, page) if hasattr(model, "make_kv") else KvBuffer(KvLayout(page_size=page, num_pages=nblocks, dtype=dtype, **model.kv_geometry()), device)
     pool = BlockPool(nblocks, page, enable_prefix_cache=not ecfg.no_prefix_cache and getattr(model, "supports_prefix_cache", True))
     max_blocks_per_seq = (max_len + page - 1) // page
+    extra = {"state_slots": ecfg.state_slots} if ecfg.state_slots else {}
     executor = (model.make_executor if hasattr(model, "make_executor") else TorchExecutor)(
-        model, kv, page, cuda_graph=ecfg.cuda_graph, max_decode_batch=ecfg.max_decode_batch, max_blocks_per_seq=max_blocks_per_seq, seed=ecfg.seed
+        model, kv, page, cuda_graph=ecfg.cuda_graph, max_decode_batch=ecfg.max_decode_batch, max_blocks_per_seq=max_blocks_per_seq, seed=ecfg.seed, **extra
     )
     scfg = SchedulerConfig(
         max_prefill_tokens=ecfg.max_prefill_tokens,
-        max_decode_batch=ecfg.max_decode_batch,
+        max_decode_batch=min(ecfg.max_decode_batch, ecfg.state_slots or ecfg.max_decode_batch),
         max_model_len=max_len,
         eos_token_ids=tuple(mcfg.eos_token_ids),
         batch_invariant=ecfg.batch_invariant,

@@ -7,6 +7,10 @@ page's K or V with one tiled copy, and the host tier moves one logical block as
 ``layers`` strided chunks.  ``LatentKvBuffer`` is the MLA variant: one row of
 ``kv_lora_rank + rope_dim`` per token, ``[layers, pages, page_size, width]``.
 
+``MixedKvBuffer`` holds layers of different geometries (KV heads, key size, value size): one tensor
+``[pages, page_size * kv_heads * (dim + vdim)]`` per layer, a page's keys ``[page_size, kv_heads, dim]`` in front of
+its values ``[page_size, kv_heads, vdim]``; with ``dim == vdim`` a page is laid out as in ``KvBuffer``.
+
 ``PagePool``/``KvPool`` are the simple non-prefix page allocators used by model
 lines that keep per-request recurrent state next to paged attention KV.
 
@@ -72,6 +76,21 @@ class LatentKvBuffer:
 
     def block_view(self, bid: int) -> torch.Tensor:
         return self.data[:, bid]
+
+
+class MixedKvBuffer:
+    def __init__(self, geometries, num_pages: int, page_size: int, dtype=torch.bfloat16, device="cpu"):
+        """``geometries``: ``(kv_heads, dim, vdim)`` of every layer that owns a cache."""
+        self.page_size = page_size
+        self.geometries = tuple(geometries)
+        self.data = [torch.zeros((num_pages, page_size * h * (d + v)), dtype=dtype, device=device) for h, d, v in self.geometries]
+
+    @staticmethod
+    def bytes_per_block(geometries, page_size: int, dtype) -> int:
+        return sum(page_size * h * (d + v) for h, d, v in geometries) * torch.empty((), dtype=dtype).element_size()
+
+    def layer(self, i: int) -> torch.Tensor:
+        return self.data[i]
 
 
 class PagePool:

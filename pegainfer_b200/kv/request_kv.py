@@ -90,6 +90,12 @@ class RequestKv:
             out.append(parent)
         return out
 
+    def extend_prompt(self, tokens: Sequence[int]) -> None:
+        """More prompt tokens for a request that is fed in portions from outside (trace replay)."""
+        assert len(self.tokens) == self.prompt_len, "the request has sampled tokens"
+        self.tokens.extend(tokens)
+        self.prompt_len = len(self.tokens)
+
     # -- scheduling --------------------------------------------------------------
     def blocks_needed(self, new_tokens: int) -> int:
         return max(0, blocks_for(self.committed + new_tokens, self.bs) - len(self.blocks))

@@ -47,6 +47,10 @@ def default_source(cfg: ModelConfig, seed: int = 0, dtype=torch.bfloat16):
         from ..models.gemma4 import gemma4_source
 
         return gemma4_source(cfg, seed=seed, dtype=dtype)
+    if cfg.family == "nemipel":
+        from ..models.nemipel import nemipel_source
+
+        return nemipel_source(cfg, seed=seed, dtype=dtype)
     from ..models import registry
 
     shapes = registry.shapes_for(cfg)
@@ -59,6 +63,10 @@ def default_source(cfg: ModelConfig, seed: int = 0, dtype=torch.bfloat16):
 
 def to_hf_config(cfg: ModelConfig) -> dict:
     """``config.json`` contents that ``config.from_hf`` maps back to ``cfg``."""
+    if cfg.family == "nemipel":
+        from ..config import nemipel_to_json
+
+        return nemipel_to_json(cfg)
     arch = {"qwen3": ("qwen3", "Qwen3ForCausalLM"), "qwen35": ("qwen3_5", "Qwen3_5ForCausalLM"), "deepseek_v2": ("deepseek_v2", "DeepseekV2ForCausalLM"),
             "kimi_k2": ("kimi_k2", "DeepseekV3ForCausalLM")}.get(cfg.family, (cfg.family, cfg.family))
     out = {

@@ -37,7 +37,8 @@ from ..loader.sources import RandomSource, WeightSource, shard_range
 from ..ops.reference import AttnMeta
 from ..parallel.ep import LOCAL_EP, EPContext
 from ..parallel.tp import SINGLE, TPContext
-from .qwen35 import HybridExecutor, RecurrentState
+from ..kv.state import RecurrentState
+from ..sched.executor import HybridExecutor
 
 TEXT = "language_model."
 

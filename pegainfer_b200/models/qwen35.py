@@ -23,10 +23,11 @@ import torch
 from .. import ops
 from ..config import ModelConfig
 from ..kv.buffer import KvBuffer, KvLayout
+from ..kv.state import RecurrentState
 from ..loader.sources import RandomSource, WeightSource, shard_range
 from ..ops.reference import AttnMeta, rope_tables
 from ..parallel.tp import SINGLE, TPContext
-from ..sched.executor import TorchExecutor
+from ..sched.executor import HybridExecutor
 
 
 def qwen35_shapes(cfg: ModelConfig, wp: str = "model.language_model") -> dict:
@@ -103,34 +104,6 @@ class HybridLayer:
     down: torch.Tensor
     full: Optional[FullLayer] = None
     linear: Optional[LinearLayer] = None
-
-
-class RecurrentState:
-    """Slot pool of per-request conv and delta-rule state (slot 0 is the padding slot)."""
-
-    def __init__(self, num_slots: int, n_linear: int, channels: int, conv_k: int, hv: int, dk: int, dv: int, dtype, device):
-        self.conv = torch.zeros((n_linear, num_slots, channels, conv_k - 1), dtype=dtype, device=device)
-        self.ssm = torch.zeros((n_linear, num_slots, hv, dk, dv), dtype=torch.float32, device=device)
-        self._free = list(range(num_slots - 1, 0, -1))
-        self.by_rid: dict = {}
-
-    def slot_for(self, rid: int, fresh: bool) -> int:
-        s = self.by_rid.get(rid)
-        if s is None:
-            if not self._free:
-                raise RuntimeError("recurrent-state slot pool exhausted")
-            s = self._free.pop()
-            self.by_rid[rid] = s
-            fresh = True
-        if fresh:
-            self.conv[:, s].zero_()
-            self.ssm[:, s].zero_()
-        return s
-
-    def release(self, rid: int) -> None:
-        s = self.by_rid.pop(rid, None)
-        if s is not None:
-            self._free.append(s)
 
 
 class Qwen35Model:
@@ -270,21 +243,3 @@ class Qwen35Model:
 
     def forward(self, token_ids, meta, kv, logits_rows=None):
         return self.logits(self.forward_hidden(token_ids, meta, kv), logits_rows)
-
-
-class HybridExecutor(TorchExecutor):
-    """Adds recurrent-state slot management to the generic executor."""
-
-    def __init__(self, model, kv, page_size, **kw):
-        slots = kw.get("max_decode_batch", 64) + 8
-        model.make_state(slots)
-        super().__init__(model, kv, page_size, **kw)
-
-    def prepare_meta(self, seqs, meta: AttnMeta) -> None:
-        slots = [self.model.rec.slot_for(s.rid, s.fresh_state and s.start_pos == 0) for s in seqs]
-        slots += [0] * (meta.num_seqs - len(slots))
-        meta.h_state_slots = slots
-        meta.state_slots = torch.tensor(slots, dtype=torch.int32, device=self.device)
-
-    def release_request(self, rid: int) -> None:
-        self.model.rec.release(rid)

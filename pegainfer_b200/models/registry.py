@@ -47,7 +47,25 @@ def _k3(cfg, **kw):
     return K3Model(cfg, **kw)
 
 
-BUILDERS = {"kimi_k3": _k3, "gemma4": _gemma4, "glm_dsa": _glm_dsa, "qwen3": _qwen3, "qwen35": _qwen35, "deepseek_v2": _mla_moe, "kimi_k2": _mla_moe}
+def _nemipel(cfg, **kw):
+    from .nemipel import NemipelModel
+
+    kw.pop("ep", None)
+    return NemipelModel(cfg, **kw)
+
+
+BUILDERS = {"nemipel": _nemipel, "kimi_k3": _k3, "gemma4": _gemma4, "glm_dsa": _glm_dsa, "qwen3": _qwen3, "qwen35": _qwen35, "deepseek_v2": _mla_moe, "kimi_k2": _mla_moe}
+
+
+# Translation units (csrc/<name>.cu) that a family's kernels come from, for programs that build only what one model needs
+KERNEL_UNITS = {
+    "nemipel": ("runtime", "gemm_sm100", "gemm2sm_sm100", "elementwise", "stream32", "attention", "attention_general", "kda", "sampling"),
+}
+
+
+def kernel_units(family: str):
+    """The units of a family, or ``None`` for all of them."""
+    return KERNEL_UNITS.get(family)
 
 
 def build(cfg: ModelConfig, **kw):
@@ -70,6 +88,10 @@ def shapes_for(cfg: ModelConfig) -> dict:
         from .k3 import k3_shapes
 
         return k3_shapes(cfg)
+    if cfg.family == "nemipel":
+        from .nemipel import nemipel_shapes
+
+        return nemipel_shapes(cfg)
     raise ValueError(f"no tensor-shape table for family {cfg.family!r}")
 
 

@@ -137,11 +137,18 @@ def embedding(ids, table):
 
 
 def gather_rows(x, idx):
-    _bf16(x)
     x2 = x.reshape(-1, x.shape[-1])
     if not x2.is_contiguous():
         x2 = x2.contiguous()
     idx = idx.to(torch.int32).contiguous()
+    if x.dtype == torch.float32 or x2.shape[1] % 8:
+        f32 = _is_f32(x2)
+        out = torch.empty((idx.numel(), x2.shape[1]), dtype=x.dtype, device=x.device)
+        c = ctx(x.device)
+        _check(lib().pg_embed_rows(_ptr(x2), _ci(f32), _ll(x2.stride(0)), _ptr(idx), _vp(0), _ptr(out), _ci(f32), _ll(out.stride(0)), _ci(idx.numel()), _ci(x2.shape[1]), _ll(x2.shape[0]),
+                                   _ptr(c.status), _stream()), c)
+        return out
+    _bf16(x)
     out = torch.empty((idx.numel(), x2.shape[1]), dtype=x.dtype, device=x.device)
     c = ctx(x.device)
     _check(lib().pg_gather_rows(_ptr(x2), _ptr(idx), _ptr(out), _ci(idx.numel()), _ci(x2.shape[1]), _ll(x2.shape[0]), _ptr(c.status), _stream()), c)
@@ -841,6 +848,205 @@ def kda_recurrent(q, k, v, f, b, a_log, dt_bias, lower: float, state, meta: Attn
     out = torch.empty((t, h, dv), dtype=q.dtype, device=q.device)
     rc = lib().pg_kda_recurrent(_ptr(q), _ptr(k), _ptr(v), _ll(q.stride(0)), _ptr(f), _ll(f.stride(0)), _ptr(b), _ll(b.stride(0)), _ptr(a_log), _ptr(dt_bias), _cf(lower),
                                 _ptr(state), _ptr(out), _ptr(meta.q_indptr), _ptr(meta.state_slots), _ci(meta.num_seqs), _ci(h), _ci(dk), _ci(dv), _ci(int(meta.max_q_len)), _stream())
+    _check(rc, ctx(q.device))
+    return out
+
+
+# ----------------------------------------------------------------------------------
+# 32-bit residual stream, layers with runtime head sizes (bf16 or f32 activations)
+# ----------------------------------------------------------------------------------
+def _is_f32(t) -> int:
+    if t.dtype == torch.float32:
+        return 1
+    _bf16(t)
+    return 0
+
+
+def embed_stream(ids, table, act_dtype):
+    """Table rows as an f32 residual stream ``[T, W]`` and their copy in the activation dtype (the same tensor when that
+    is f32)."""
+    ids = ids.to(torch.int32).contiguous()
+    t, w = ids.numel(), table.shape[1]
+    x = torch.empty((t, w), dtype=torch.float32, device=table.device)
+    xt = x if act_dtype == torch.float32 else torch.empty((t, w), dtype=act_dtype, device=table.device)
+    c = ctx(table.device)
+    _check(lib().pg_embed_rows(_ptr(table), _ci(_is_f32(table)), _ll(table.stride(0)), _ptr(ids), _ptr(x), _vp(0) if xt is x else _ptr(xt), _ci(0), _ll(xt.stride(0)), _ci(t), _ci(w),
+                               _ll(table.shape[0]), _ptr(c.status), _stream()), c)
+    return x, xt
+
+
+def _post_norm(y, x, x_out, w, eps, alpha, act_dtype):
+    t, width = x.shape
+    assert x.dtype == torch.float32 and w.dtype == torch.float32 and x.is_contiguous() and (y is None or (y.shape == x.shape and y.stride(1) == 1))
+    f32 = act_dtype == torch.float32
+    xt = x_out if f32 and x_out is not None else torch.empty((t, width), dtype=act_dtype, device=x.device)
+    c = ctx(x.device)
+    _check(lib().pg_post_norm(_ptr(y), _ci(_is_f32(y) if y is not None else 0), _ll(y.stride(0) if y is not None else 0), _ptr(x), _ptr(x_out), _cf(alpha), _ptr(w),
+                              _vp(0) if xt is x_out else _ptr(xt), _ci(int(f32)), _ll(xt.stride(0)), _ci(t), _ci(width), _cf(eps), _stream()), c)
+    return xt
+
+
+def post_norm(y, x, w, eps: float, alpha: float, act_dtype):
+    """``x <- rms_norm(alpha * x + y) * w`` on the f32 stream, in place; returns the activation-dtype copy."""
+    return _post_norm(y, x, x, w, eps, alpha, act_dtype)
+
+
+def stream_norm(x, w, eps: float, act_dtype):
+    """RMS norm of the f32 stream in the activation dtype."""
+    return _post_norm(None, x, None, w, eps, 1.0, act_dtype)
+
+
+def gated_row_norm(x, gate, w, eps: float):
+    """``rms_norm(x) * w * sigmoid(gate)`` over the last axis of ``x`` [T, H, D]; ``gate`` [T, H * D], unit column stride."""
+    t, h, d = x.shape
+    assert x.is_contiguous() and gate.shape == (t, h * d) and gate.stride(1) == 1 and gate.dtype == x.dtype and w.dtype == torch.float32
+    y = torch.empty((t, h, d), dtype=x.dtype, device=x.device)
+    _check(lib().pg_gated_row_norm(_ptr(x), _ptr(gate), _ll(gate.stride(0)), _ptr(w), _ptr(y), _ci(t), _ci(h), _ci(d), _cf(eps), _ci(_is_f32(x)), _stream()), ctx(x.device))
+    return y
+
+
+def dense(x, w, out_dtype=None):
+    """``x @ w.T`` for any sizes.  bf16 operands whose rows TMA can address run on the tcgen05 GEMM (outputs wanted in f32
+    come back in bf16 where the two-SM kernel, which stores bf16, serves the problem); f32 operands and odd bf16 sizes
+    run on the CUDA-core GEMM.  ``x`` may be a column slice."""
+    t, k = x.shape
+    m = w.shape[0]
+    assert x.stride(1) == 1 and w.stride(1) == 1 and x.dtype == w.dtype
+    f32 = _is_f32(x)
+    out_dtype = out_dtype or x.dtype
+    if not f32 and k % 8 == 0 and x.stride(0) % 8 == 0 and x.data_ptr() % 16 == 0 and w.stride(0) % 8 == 0:
+        if out_dtype == torch.float32 and not _BATCH_INVARIANT and lib().pg_gemm2sm_eligible(_ci(t), _ci(m), _ci(k)):
+            out_dtype = torch.bfloat16
+        return linear(x, w, out_dtype)
+    y = torch.empty((t, m), dtype=out_dtype, device=x.device)
+    _check(lib().pg_gemm_simt(_ptr(x), _ptr(w), _ci(f32), _ptr(y), _ci(_is_f32(y)), _ci(t), _ci(m), _ci(k), _ll(x.stride(0)), _ll(w.stride(0)), _ll(y.stride(0)), _stream()), ctx(x.device))
+    return y
+
+
+def dense_glu(x, gate_up, interleaved: bool = False):
+    """``silu(gate) * up`` of the fused projection ``x @ gate_up.T``: in the GEMM's epilogue where a kernel has it (decode
+    steps on the on-chip split-K path, prefill-sized steps on the two-SM kernel; interleaved rows), else two launches."""
+    if _is_f32(x):
+        gu = dense(x, gate_up)
+        assert not interleaved
+        out = torch.empty((x.shape[0], gu.shape[1] // 2), dtype=torch.float32, device=x.device)
+        _check(lib().pg_glu_rows_f32(_ptr(gu), _ptr(out), _ci(gu.shape[0]), _ci(out.shape[1]), _ll(gu.stride(0)), _stream()), ctx(x.device))
+        return out
+    t, k = x.shape
+    m = gate_up.shape[0]
+    if interleaved and k % 8 == 0 and x.stride(0) % 8 == 0:
+        if m % 4 == 0 and fused_plan_ok(t, m, k):
+            return linear_fused(x, gate_up, EPI_SWIGLU)
+        act = linear_swiglu_2sm(x, gate_up)
+        if act is not None:
+            return act
+    return swiglu(dense(x, gate_up), interleaved)
+
+
+def softcap_rows(logits, cap: float):
+    """``cap * tanh(logits / cap)`` on f32 logits."""
+    assert logits.dtype == torch.float32
+    x = logits.contiguous()
+    y = torch.empty_like(x)
+    _check(lib().pg_softcap_f32(_ptr(x), _ptr(y), _ll(x.numel()), _cf(cap), _stream()), ctx(x.device))
+    return y
+
+
+def row_norm_rope_append(q, k, v, q_norm_w, k_norm_w, cos, sin, meta: AttnMeta, kv_layer, heads: int, kv_heads: int, dim: int, vdim: int, eps: float):
+    t = q.shape[0]
+    assert q.stride(1) == 1 and q.shape[1] == heads * dim and cos.dtype == sin.dtype == torch.float32 and q_norm_w.dtype == torch.float32
+    if k is not None:
+        assert k.stride(0) == v.stride(0) == q.stride(0) and k.stride(1) == v.stride(1) == 1 and k.dtype == v.dtype == q.dtype == kv_layer.dtype
+        assert kv_layer.is_contiguous() and kv_layer.shape[1] == meta.page_size * kv_heads * (dim + vdim) and k_norm_w.dtype == torch.float32
+    out = torch.empty((t, heads, dim), dtype=q.dtype, device=q.device)
+    c = ctx(q.device)
+    _check(lib().pg_row_norm_rope_append(_ptr(q), _ptr(k), _ptr(v), _ll(q.stride(0)), _ptr(q_norm_w), _ptr(k_norm_w if k is not None else None), _ptr(cos), _ptr(sin), _ci(2 * cos.shape[1]), _ci(cos.shape[0]),
+                                         _ptr(meta.positions), _ptr(meta.slot_mapping), _ptr(out), _ptr(kv_layer if k is not None else None), _ci(t), _ci(heads), _ci(kv_heads), _ci(dim), _ci(vdim),
+                                         _ci(meta.page_size), _ll(kv_layer.shape[0] if k is not None else 0), _cf(eps), _ci(_is_f32(q)), _ptr(c.status), _stream()), c)
+    return out
+
+
+def capped_attention(q, kv_layer, kv_heads: int, vdim: int, meta: AttnMeta, scale: float, softcap: float = 0.0, gate=None):
+    """Causal attention over the paged cache with its own value size, an optional soft cap on the scores and an optional
+    sigmoid gate per (token, head).  Head sizes that are multiples of 8 up to 256 run on tensor-core kernels (split-KV
+    decode, tiled prefill), others and f32 on the CUDA-core kernel."""
+    t, hq, dim = q.shape
+    f32 = _is_f32(q)
+    assert q.is_contiguous() and kv_layer.is_contiguous() and kv_layer.dtype == q.dtype and (gate is None or (gate.dtype == q.dtype and gate.stride(1) == 1))
+    out = torch.empty((t, hq * vdim), dtype=q.dtype, device=q.device)
+    c = ctx(q.device)
+    ps, pages, table = meta.page_size, kv_layer.shape[0], meta.block_table
+    assert kv_layer.shape[1] == ps * kv_heads * (dim + vdim)
+    gate_args = (_ptr(gate), _ll(gate.stride(0) if gate is not None else 0))
+    if f32 or dim % 8 or vdim % 8 or max(dim, vdim) > 256 or ps not in (16, 32, 64):
+        _check(lib().pg_attention_plain(_ptr(q), _ptr(kv_layer), _ptr(out), _ptr(meta.q_indptr), _ptr(meta.kv_lens), _ptr(table), _ci(table.stride(0)), _ci(t), _ci(meta.num_seqs), _ci(hq), _ci(kv_heads),
+                                        _ci(dim), _ci(vdim), _ci(ps), _ll(pages), _cf(scale), _cf(softcap), *gate_args, _ci(f32), _stream()), c)
+        return out
+
+    def run(first: int, n: int, mode: int, splits: int = 1, q_tiles: int = 0):
+        lse_off = n * hq * splits * vdim * 4
+        rc = lib().pg_attention_capped(_ptr(q), _ptr(kv_layer), _ptr(out), _ptr(meta.q_indptr[first:]), _ptr(meta.kv_lens[first:]), _ptr(table[first:]), _ci(table.stride(0)), _ci(n), _ci(hq),
+                                       _ci(kv_heads), _ci(dim), _ci(vdim), _ci(ps), _ll(pages), _cf(scale), _cf(softcap), *gate_args, _ci(mode), _ci(splits), _ptr(c.attn_part),
+                                       _ptr(c.attn_part[lse_off:]), _ci(q_tiles), _ptr(c.status), _stream())
+        _check(rc, c, 2 if splits > 1 else 1)
+
+    def decode_rows(first: int, n: int, plan=None):
+        splits = plan if isinstance(plan, int) else plan_decode_splits(n, kv_heads * ((hq // kv_heads + 7) // 8), meta.max_kv_len, q.device)
+        need = n * hq * splits * (vdim + 1) * 4
+        if need > c.attn_part.numel():
+            splits = max(1, c.attn_part.numel() // (n * hq * (vdim + 1) * 4))
+        run(first, n, 0, splits)
+
+    if meta.decode_only:
+        decode_rows(0, meta.num_seqs, meta.plan)
+        return out
+    qi = meta.h_q_indptr if meta.h_q_indptr is not None else meta.q_indptr.tolist()
+    n_pf = meta.num_seqs
+    while n_pf > 0 and qi[n_pf] - qi[n_pf - 1] == 1:  # trailing single-row sequences take the decode kernel (see paged_attention)
+        n_pf -= 1
+    if meta.num_seqs - n_pf < (1 if _BATCH_INVARIANT else _MIXED_DECODE_MIN):
+        n_pf = meta.num_seqs
+    if n_pf > 0:
+        run(0, n_pf, 1, 1, sum((qi[b + 1] - qi[b] + 63) // 64 for b in range(n_pf)))
+    if n_pf < meta.num_seqs:
+        decode_rows(n_pf, meta.num_seqs - n_pf)
+    return out
+
+
+def conv_silu(x, conv_w, conv_state, meta: AttnMeta):
+    """Causal depthwise convolution of up to 16 taps + SiLU with carried inputs; ``conv_w`` f32 [C, taps]."""
+    t, ch = x.shape
+    taps = conv_w.shape[1]
+    assert x.stride(1) == 1 and conv_w.is_contiguous() and conv_w.dtype == torch.float32 and conv_state.is_contiguous() and conv_state.dtype == x.dtype
+    out = torch.empty((t, ch), dtype=x.dtype, device=x.device)
+    _check(lib().pg_conv_silu(_ptr(x), _ll(x.stride(0)), _ptr(conv_w), _ptr(conv_state), _ptr(out), _ll(out.stride(0)), _ptr(meta.q_indptr), _ptr(meta.state_slots), _ci(meta.num_seqs), _ci(ch), _ci(taps),
+                              _ll(conv_state.stride(0)), _ci(max(int(meta.max_q_len), 1)), _ci(_is_f32(x)), _stream()), ctx(x.device))
+    return out
+
+
+def channel_delta(q, k, v, f, b, a_log, dt_bias, state, meta: AttnMeta):
+    """Delta rule with a softplus-form decay per key channel (``reference.channel_delta``); ``q, k, v`` share a row stride."""
+    t, hk, dk = q.shape
+    h, dv = v.shape[1], v.shape[2]
+    assert q.stride(2) == 1 and q.stride(1) == dk and k.stride(1) == dk and v.stride(1) == dv and q.stride(0) == k.stride(0) == v.stride(0)
+    assert f.dtype == torch.float32 and f.stride(1) == 1 and f.shape[1] == h * dk and b.stride(1) == 1 and b.dtype == q.dtype
+    assert state.is_contiguous() and state.dtype == a_log.dtype == dt_bias.dtype == torch.float32
+    out = torch.empty((t, h, dv), dtype=q.dtype, device=q.device)
+    rc = lib().pg_channel_delta(_ptr(q), _ptr(k), _ptr(v), _ll(q.stride(0)), _ptr(f), _ll(f.stride(0)), _ptr(b), _ll(b.stride(0)), _ptr(a_log), _ptr(dt_bias), _ptr(state), _ptr(out), _ptr(meta.q_indptr),
+                                _ptr(meta.state_slots), _ci(meta.num_seqs), _ci(h), _ci(hk), _ci(dk), _ci(dv), _ci(int(meta.max_q_len)), _ci(0), _ci(_is_f32(q)), _stream())
+    _check(rc, ctx(q.device))
+    return out
+
+
+def decay_attention(q, k, v, decay, state, meta: AttnMeta):
+    """Linear attention with a fixed decay per head (``reference.decay_attention``); ``q, k, v`` share a row stride."""
+    t, h, dk = q.shape
+    dv = v.shape[2]
+    assert q.stride(2) == 1 and q.stride(1) == dk and k.stride(1) == dk and v.stride(1) == dv and q.stride(0) == k.stride(0) == v.stride(0)
+    assert state.is_contiguous() and state.dtype == decay.dtype == torch.float32
+    out = torch.empty((t, h, dv), dtype=q.dtype, device=q.device)
+    rc = lib().pg_decay_recurrent(_ptr(q), _ptr(k), _ptr(v), _ll(q.stride(0)), _ptr(decay), _ptr(state), _ptr(out), _ptr(meta.q_indptr), _ptr(meta.state_slots), _ci(meta.num_seqs), _ci(h), _ci(dk), _ci(dv),
+                                  _ci(int(meta.max_q_len)), _ci(0), _ci(_is_f32(q)), _stream())
     _check(rc, ctx(q.device))
     return out
 

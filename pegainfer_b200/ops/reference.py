@@ -82,6 +82,49 @@ def add_rms_norm(x, residual, w, eps, offset=False, round_before_norm=True):
     return (src * inv * wf).to(x.dtype)
 
 
+def embed_stream(ids, table, act_dtype):
+    """Table rows as an f32 residual stream ``[T, W]`` and their copy in the activation dtype."""
+    x = table[ids.long()].float()
+    return x, x.to(act_dtype)
+
+
+def post_norm(y, x, w, eps: float, alpha: float, act_dtype):
+    """Norm after the sum, in f32: ``x <- rms_norm(alpha * x + y) * w`` (in place on the f32 stream ``x``); returns the
+    copy in the activation dtype.  ``y`` is a sublayer's output, f32 or the activation dtype."""
+    s = alpha * x + y.float()
+    x.copy_(s * torch.rsqrt(s.pow(2).mean(-1, keepdim=True) + eps) * w.float())
+    return x.to(act_dtype)
+
+
+def stream_norm(x, w, eps: float, act_dtype):
+    """RMS norm of the f32 stream in the activation dtype (the stream is left as it is)."""
+    return (x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps) * w.float()).to(act_dtype)
+
+
+def gated_row_norm(x, gate, w, eps: float):
+    """``rms_norm(x) * w * sigmoid(gate)`` over the last axis of ``x`` [T, H, D], rounded once; ``gate`` [T, H * D] may be a
+    column slice of a wider projection."""
+    xf = x.float()
+    n = xf * torch.rsqrt(xf.pow(2).mean(-1, keepdim=True) + eps) * w.float()
+    return (n * torch.sigmoid(gate.float().reshape(x.shape))).to(x.dtype)
+
+
+def dense(x, w, out_dtype=None):
+    """``x @ w.T`` for any sizes in f32 or bf16 (f32 accumulation)."""
+    y = x.float() @ w.float().t()
+    return y.to(out_dtype or x.dtype)
+
+
+def dense_glu(x, gate_up, interleaved: bool = False):
+    """``silu(gate) * up`` of the fused projection ``x @ gate_up.T``."""
+    return swiglu(dense(x, gate_up), interleaved)
+
+
+def softcap_rows(logits, cap: float):
+    """``cap * tanh(logits / cap)`` in f32."""
+    return torch.tanh(logits.float() / cap) * cap
+
+
 def geglu(gate_up: torch.Tensor) -> torch.Tensor:
     """``round(gelu_tanh(gate)) * up`` on a fused ``[T, 2I]`` buffer, gate half first."""
     i = gate_up.shape[-1] // 2
@@ -277,6 +320,69 @@ def qk_norm_rope_append(qkv, q_norm_w, k_norm_w, cos, sin, meta: AttnMeta, kv_la
 # ----------------------------------------------------------------------------------
 # attention
 # ----------------------------------------------------------------------------------
+def pair_rope_tables(max_pos: int, rotary_dim: int, theta: float, device="cpu"):
+    """f32 cos / sin ``[max_pos, rotary_dim / 2]``; the angles ``p * theta^(-2 i / rotary_dim)`` are formed in f64."""
+    inv = theta ** (-torch.arange(0, rotary_dim, 2, dtype=torch.float64) / max(rotary_dim, 1))
+    ang = torch.outer(torch.arange(max_pos, dtype=torch.float64), inv)
+    return ang.cos().float().to(device), ang.sin().float().to(device)
+
+
+def _pages_kv(kv_layer, kv_heads: int, dim: int, vdim: int, page_size: int):
+    """Key and value views ``[pages, page_size, kv_heads, dim / vdim]`` of a layer's flat pages."""
+    n, cut = kv_layer.shape[0], page_size * kv_heads * dim
+    return kv_layer[:, :cut].view(n, page_size, kv_heads, dim), kv_layer[:, cut:].view(n, page_size, kv_heads, vdim)
+
+
+def row_norm_rope_append(q, k, v, q_norm_w, k_norm_w, cos, sin, meta: AttnMeta, kv_layer, heads: int, kv_heads: int, dim: int, vdim: int, eps: float):
+    """RMS norm over the whole query and key projection rows, rotation of neighbouring pairs on the first
+    ``2 * cos.shape[1]`` entries of every head, append of keys and values to the paged cache.  ``k`` / ``v`` are ``None``
+    for a layer that reads another layer's cache.  Returns the queries ``[T, heads, dim]``."""
+    t, pos, rot = q.shape[0], meta.positions.long(), 2 * cos.shape[1]
+
+    def make(x, w, h):
+        xf = x.float()
+        xf = (xf * torch.rsqrt(xf.pow(2).mean(-1, keepdim=True) + eps) * w.float()).view(t, h, dim)
+        c, s = cos[pos][:, None, :], sin[pos][:, None, :]
+        u, w2 = xf[..., 0:rot:2], xf[..., 1:rot:2]
+        r = torch.stack((u * c - w2 * s, w2 * c + u * s), -1).flatten(-2)
+        return torch.cat((r, xf[..., rot:]), -1).to(x.dtype)
+
+    if k is not None:
+        kp, vp = _pages_kv(kv_layer, kv_heads, dim, vdim, meta.page_size)
+        slot = meta.slot_mapping.long()
+        page, off = slot // meta.page_size, slot % meta.page_size
+        kp[page, off] = make(k, k_norm_w, kv_heads).to(kv_layer.dtype)
+        vp[page, off] = v.reshape(t, kv_heads, vdim).to(kv_layer.dtype)
+    return make(q, q_norm_w, heads)
+
+
+def capped_attention(q, kv_layer, kv_heads: int, vdim: int, meta: AttnMeta, scale: float, softcap: float = 0.0, gate=None):
+    """Causal attention over the paged cache with different key and value sizes, an optional soft cap on the scaled scores
+    and an optional sigmoid gate per (token, head) (``gate`` [T, >= heads]).  Returns ``[T, heads * vdim]``."""
+    t, hq, dim = q.shape
+    rep = hq // kv_heads
+    kp, vp = _pages_kv(kv_layer, kv_heads, dim, vdim, meta.page_size)
+    qi = meta.h_q_indptr if meta.h_q_indptr is not None else meta.q_indptr.tolist()
+    kl = meta.h_kv_lens if meta.h_kv_lens is not None else meta.kv_lens.tolist()
+    out = torch.zeros(t, hq, vdim, dtype=torch.float32, device=q.device)
+    for b in range(meta.num_seqs):
+        q0, q1, n = qi[b], qi[b + 1], kl[b]
+        if n == 0 or q1 == q0:
+            continue
+        pages = meta.block_table[b, : (n + meta.page_size - 1) // meta.page_size].long()
+        k = kp[pages].reshape(-1, kv_heads, dim)[:n].float().repeat_interleave(rep, 1)
+        v = vp[pages].reshape(-1, kv_heads, vdim)[:n].float().repeat_interleave(rep, 1)
+        s = torch.einsum("qhd,khd->hqk", q[q0:q1].float(), k) * scale
+        if softcap:
+            s = torch.tanh(s / softcap) * softcap
+        pos = torch.arange(n - (q1 - q0), n, device=q.device)
+        s = s.masked_fill(torch.arange(n, device=q.device)[None, None, :] > pos[None, :, None], float("-inf"))
+        out[q0:q1] = torch.einsum("hqk,khd->qhd", torch.softmax(s, -1), v)
+    if gate is not None:
+        out = out * torch.sigmoid(gate[:, :hq].float())[:, :, None]
+    return out.to(q.dtype).reshape(t, hq * vdim)
+
+
 def _gather_kv(kv_layer, pages, kv_len, page_size):
     k = kv_layer[pages, 0].reshape(-1, kv_layer.shape[-2], kv_layer.shape[-1])[:kv_len]
     v = kv_layer[pages, 1].reshape(-1, kv_layer.shape[-2], kv_layer.shape[-1])[:kv_len]
@@ -822,6 +928,71 @@ def kda_recurrent(q, k, v, f, b, a_log, dt_bias, lower: float, state, meta: Attn
             kv = torch.einsum("hkv,hk->hv", S, kf[i])
             delta = (vf[i] - kv) * beta[i].view(h, 1)
             S = S + torch.einsum("hk,hv->hkv", kf[i], delta)
+            out[i] = torch.einsum("hkv,hk->hv", S, qf[i]).to(q.dtype)
+        state[slots[s]] = S
+    return out
+
+
+def conv_silu(x, conv_w, conv_state, meta: AttnMeta):
+    """Causal depthwise convolution of any length + SiLU, rounded once; ``conv_w`` f32 [C, taps], ``conv_state``
+    [slots, C, taps - 1] holds the last inputs of each sequence and is updated in place."""
+    taps = conv_w.shape[1]
+    out = torch.zeros(x.shape, dtype=x.dtype, device=x.device)
+    qi = meta.h_q_indptr if meta.h_q_indptr is not None else meta.q_indptr.tolist()
+    slots = meta.h_state_slots if meta.h_state_slots is not None else meta.state_slots.tolist()
+    for b in range(meta.num_seqs):
+        q0, q1 = qi[b], qi[b + 1]
+        if q1 == q0 or slots[b] < 0:
+            continue
+        seq = torch.cat([conv_state[slots[b]].t().to(x.dtype), x[q0:q1]], 0)
+        pre = (seq.float().unfold(0, taps, 1) * conv_w.float()).sum(-1)
+        out[q0:q1] = (pre * torch.sigmoid(pre)).to(x.dtype)
+        conv_state[slots[b]] = seq[seq.shape[0] - (taps - 1) :].t().to(conv_state.dtype)
+    return out
+
+
+def channel_delta(q, k, v, f, b, a_log, dt_bias, state, meta: AttnMeta):
+    """Delta rule with the decay ``exp(-exp(a_log) * softplus(f + dt_bias))`` per head and key channel.  ``q, k``
+    [T, Hk, Dk] and ``v`` [T, H, Dv] after the short convolution (value head h reads query / key head ``h // (H / Hk)``),
+    ``f`` f32 [T, H * Dk], ``b`` [T, H] raw, ``state`` [slots, H, Dk, Dv] f32 updated in place.  Returns [T, H, Dv]."""
+    t, hk, dk = q.shape
+    h, dv = v.shape[1], v.shape[2]
+    qf, kf, vf = q.float(), k.float(), v.float()
+    qf = (qf * torch.rsqrt(qf.pow(2).sum(-1, keepdim=True) + 1e-6) * dk ** -0.5).repeat_interleave(h // hk, 1)
+    kf = (kf * torch.rsqrt(kf.pow(2).sum(-1, keepdim=True) + 1e-6)).repeat_interleave(h // hk, 1)
+    raw = (f.float() + dt_bias.float()).view(t, h, dk)
+    dec = torch.exp(-torch.exp(a_log.float()).view(1, h, 1) * F.softplus(raw))
+    beta = torch.sigmoid(b.float())
+    out = torch.zeros(t, h, dv, dtype=q.dtype, device=q.device)
+    qi = meta.h_q_indptr if meta.h_q_indptr is not None else meta.q_indptr.tolist()
+    slots = meta.h_state_slots if meta.h_state_slots is not None else meta.state_slots.tolist()
+    for s in range(meta.num_seqs):
+        if slots[s] < 0:
+            continue
+        S = state[slots[s]]
+        for i in range(qi[s], qi[s + 1]):
+            S = S * dec[i].unsqueeze(-1)
+            delta = (vf[i] - torch.einsum("hkv,hk->hv", S, kf[i])) * beta[i].view(h, 1)
+            S = S + torch.einsum("hk,hv->hkv", kf[i], delta)
+            out[i] = torch.einsum("hkv,hk->hv", S, qf[i]).to(q.dtype)
+        state[slots[s]] = S
+    return out
+
+
+def decay_attention(q, k, v, decay, state, meta: AttnMeta):
+    """Linear attention with a fixed decay per head (lightning attention): SiLU on the projections ``q, k`` [T, H, Dk] and
+    ``v`` [T, H, Dv], then ``S <- decay_h S + k v^T``, ``o = S^T q`` over the f32 ``state`` [slots, H, Dk, Dv]."""
+    t, h, dv = v.shape
+    qf, kf, vf = (F.silu(z.float()).to(z.dtype).float() for z in (q, k, v))
+    out = torch.zeros(t, h, dv, dtype=q.dtype, device=q.device)
+    qi = meta.h_q_indptr if meta.h_q_indptr is not None else meta.q_indptr.tolist()
+    slots = meta.h_state_slots if meta.h_state_slots is not None else meta.state_slots.tolist()
+    for s in range(meta.num_seqs):
+        if slots[s] < 0:
+            continue
+        S = state[slots[s]]
+        for i in range(qi[s], qi[s + 1]):
+            S = S * decay.view(h, 1, 1) + torch.einsum("hk,hv->hkv", kf[i], vf[i])
             out[i] = torch.einsum("hkv,hk->hv", S, qf[i]).to(q.dtype)
         state[slots[s]] = S
     return out

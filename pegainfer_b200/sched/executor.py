@@ -273,6 +273,37 @@ class TorchExecutor(ModelExecutor):
                     return res
         return self._execute(batch)
 
+    def _build_meta(self, seqs):
+        token_ids, meta = build_meta(seqs, self.page_size, self.device)
+        if meta.decode_only and self.device.type == "cuda" and self.max_blocks_per_seq:
+            # the same KV-split plan a captured graph of this batch size uses (it depends on the batch
+            # size and the longest sequence the engine admits, not on the live lengths), so an eager
+            # decode step and a graph replay of the same batch are bit-identical
+            from ..ops import cuda as K
+
+            geo = self.model.kv_geometry()
+            meta.plan = K.plan_decode_splits(len(seqs), geo["kv_heads"], min(self.max_blocks_per_seq * self.page_size, 2048), self.device)
+        return token_ids, meta
+
+    def step_logits(self, batch: StepBatch, want: Sequence[Sequence[int]]) -> Optional[torch.Tensor]:
+        """One step without sampling: run ``batch`` and return the logits at the rows ``want[i]`` of sequence ``i`` (row
+        numbers within its input tokens), in order, or ``None`` when nothing is wanted.  A decode batch replays the
+        CUDA graph that ``execute`` replays for a sampled decode step."""
+        seqs = batch.seqs
+        self.steps += 1
+        if self._graphs is not None and batch.is_decode() and len(seqs) <= self.max_decode_batch and self.mtp is None and self.aux_sink is None:
+            logits = self._graphs.run(seqs, greedy=False)
+            keep = [i for i, w in enumerate(want) for _ in w]
+            return logits[torch.tensor(keep, device=self.device)] if keep else None
+        token_ids, meta = self._build_meta(seqs)
+        self.prepare_meta(seqs, meta)
+        hidden = self.model.forward_hidden(token_ids, meta, self.kv)
+        rows = [meta.h_q_indptr[i] + r for i, w in enumerate(want) for r in w]
+        if not rows:
+            return None
+        logits = self.model.logits(hidden, torch.tensor(rows, dtype=torch.int32, device=self.device))
+        return self.model.full_logits(logits) if hasattr(self.model, "full_logits") else logits
+
     def _execute(self, batch: StepBatch) -> StepResult:
         t0 = time.perf_counter()
         self.steps += 1
@@ -291,15 +322,7 @@ class TorchExecutor(ModelExecutor):
                 toks, _ = self._sample(out[: len(seqs)], seqs, [1] * len(seqs))
                 toks = toks.tolist()
             return StepResult(tokens={s.rid: [toks[i]] for i, s in enumerate(seqs)}, elapsed_s=time.perf_counter() - t0)
-        token_ids, meta = build_meta(seqs, self.page_size, self.device)
-        if meta.decode_only and self.device.type == "cuda" and self.max_blocks_per_seq:
-            # the same KV-split plan a captured graph of this batch size uses (it depends on the batch
-            # size and the longest sequence the engine admits, not on the live lengths), so an eager
-            # decode step and a graph replay of the same batch are bit-identical
-            from ..ops import cuda as K
-
-            geo = self.model.kv_geometry()
-            meta.plan = K.plan_decode_splits(len(seqs), geo["kv_heads"], min(self.max_blocks_per_seq * self.page_size, 2048), self.device)
+        token_ids, meta = self._build_meta(seqs)
         if any(s.lora_slot >= 0 for s in seqs):
             rows = []
             for s in seqs:
@@ -426,3 +449,22 @@ class TorchExecutor(ModelExecutor):
         for rid, n in owners:
             res.drafts[rid] = toks[k : k + n]
             k += n
+
+
+class HybridExecutor(TorchExecutor):
+    """Adds recurrent-state slot management to the generic executor.  ``state_slots``: requests that can hold state at a
+    time (default: the decode batch and a few more)."""
+
+    def __init__(self, model, kv, page_size, state_slots: Optional[int] = None, **kw):
+        slots = state_slots or kw.get("max_decode_batch", 64) + 8
+        model.make_state(slots)
+        super().__init__(model, kv, page_size, **kw)
+
+    def prepare_meta(self, seqs, meta: AttnMeta) -> None:
+        slots = [self.model.rec.slot_for(s.rid, s.fresh_state and s.start_pos == 0) for s in seqs]
+        slots += [0] * (meta.num_seqs - len(slots))
+        meta.h_state_slots = slots
+        meta.state_slots = torch.tensor(slots, dtype=torch.int32, device=self.device)
+
+    def release_request(self, rid: int) -> None:
+        self.model.rec.release(rid)

@@ -62,6 +62,7 @@ LINES = [
     ModelLine("glm-5", ("glm_dsa",), frozenset({"ep_backend", "spec_method"})),
     ModelLine("gemma4", ("gemma4",), frozenset()),
     ModelLine("kimi-k3", ("kimi_k3",), frozenset({"ep_backend"})),
+    ModelLine("nemipel", ("nemipel",), frozenset({"dtype", "state_slots"})),
 ]
 LINES[0].validate = _qwen3_validate  # type: ignore[method-assign]
 
@@ -115,6 +116,8 @@ def build_parser() -> argparse.ArgumentParser:
     x.add_argument("--no-run-ahead", action="store_true", help="read every decode step's tokens before launching the next step")
     x.add_argument("--no-gc-tuning", action="store_true", help="leave the interpreter's garbage collector at its defaults")
     x.add_argument("--decode-sm-pct", type=int, default=50)
+    x.add_argument("--dtype", choices=["bfloat16", "float32"], default="bfloat16", help="activations and KV cache (float32: CUDA-core kernels, for comparisons)")
+    x.add_argument("--state-slots", type=int, default=None, help="requests that hold recurrent state at a time (default: --max-decode-batch)")
     x.add_argument("--max-batch", type=int, default=64)
     x.add_argument("--ep-backend", choices=["fused", "nccl"], default=None)
     return ap
@@ -155,7 +158,7 @@ def engine_config_from(ns: argparse.Namespace) -> EngineConfig:
         kv_offload_host_gib=ns.kv_offload_host_gib, kv_offload_disk_dir=ns.kv_offload_disk_dir, kv_offload_disk_gib=ns.kv_offload_disk_gib, max_prefill_tokens=ns.max_prefill_tokens, max_decode_batch=ns.max_decode_batch,
         max_model_len=ns.max_model_len, batch_invariant=ns.batch_invariant, decode_overlap=ns.decode_overlap, run_ahead=not ns.no_run_ahead, tune_gc=not ns.no_gc_tuning, decode_sm_pct=ns.decode_sm_pct,
         enable_lora=ns.enable_lora, max_loras=ns.max_loras, max_lora_rank=ns.max_lora_rank, lora_modules=tuple(ns.lora_modules), spec_method=ns.spec_method,
-        spec_draft_len=ns.spec_draft_len, draft_model_path=ns.draft_model_path, comm=ns.ep_backend or ns.comm, gemm=ns.gemm, seed=ns.seed,
+        spec_draft_len=ns.spec_draft_len, draft_model_path=ns.draft_model_path, comm=ns.ep_backend or ns.comm, gemm=ns.gemm, seed=ns.seed, dtype=ns.dtype, state_slots=ns.state_slots,
     )
 
 
