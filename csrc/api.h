@@ -89,6 +89,9 @@ int pg_prefill_attention_tc(const void* q, const void* kv_layer, void* out, cons
                             int num_seqs, int tokens, int hq, int hkv, int dim, int page_size, long long num_pages, float scale, int q_tiles, void* status,
                             cudaStream_t stream);
 void pg_prefill_attention_tc_variant(int v);
+int pg_prefill_attention_tc_capped(const void* q, const void* kv_layer, void* out, const void* q_indptr, const void* kv_lens, const void* table, int table_stride, int num_seqs, int tokens,
+                                   int hq, int hkv, int page_size, long long num_pages, float scale, float softcap, const void* gate, long long ld_gate, int q_tiles, void* status,
+                                   cudaStream_t stream);
 
 // ---- block-scaled FP8 GEMM on tcgen05 kind::f8f6f4 (gemm_fp8_sm100.cu) --------------------
 long long pg_gemm_fp8_ws_bytes(int T, int M);
@@ -171,6 +174,9 @@ int pg_channel_delta(const void* q, const void* k, const void* v, long long ld, 
                      cudaStream_t stream);
 int pg_decay_recurrent(const void* q, const void* k, const void* v, long long ld, const void* decay, void* state, void* out, const void* q_indptr, const void* slots, int num_seqs,
                        int heads, int dk, int dv, int max_q_len, int skip_len, int is_f32, cudaStream_t stream);
+// Chunk-wise (64-token) tensor-core form of decay_recurrent for sequences of >= min_len tokens, bf16 (lightning.cu).
+int pg_lightning_chunked(const void* q, const void* k, const void* v, long long ld, const void* decay, void* state, void* out, const void* q_indptr, const void* slots, int num_seqs,
+                         int heads, int dk, int dv, int min_len, cudaStream_t stream);
 // Softmax mix of the first nb snapshot rows of each token (snaps [T, cap, hidden], ld_tok = cap * hidden) and its current row.
 int pg_attnres_mix(const void* cur, long long ld_cur, const void* snaps, long long ld_tok, const void* score_w, void* out, long long ld_out,
                    int tokens, int nb, int hidden, float eps, cudaStream_t stream);

@@ -49,6 +49,9 @@ struct TcAttnParams {
   long long num_pages;
   float scale_log2;       // softmax scale * log2(e)
   int window;             // head dim 256 only: a row sees its last `window` keys (0: all of them)
+  float cap_in;           // capped form: softmax scale / cap, and scale_log2 holds cap * log2(e); 0: no cap
+  const bf16* gate;       // capped form: [T, >= hq] rows of stride ld_gate whose sigmoid multiplies a head's output, or null
+  long long ld_gate;
   int mn_lbo_first;       // descriptor variant of the MN-major operand (1: LBO = stride between 64-column blocks)
   uint32_t* status;
 };
@@ -112,6 +115,24 @@ __device__ __forceinline__ float ex2_approx(float x) {
   return y;
 }
 
+// tanh for the soft cap of a score row.  Up to |z| = 1 (scores up to the cap) an odd polynomial of degree 13 with packed
+// f32x2 arithmetic: tanh(z) / z fitted in z^2 by interpolation at Chebyshev nodes of [0, 1], relative error 1.6e-7, so that
+// the special-function unit is left to the exponentials; beyond that 1 - 2 / (1 + e^2z).
+__device__ __forceinline__ float2 tanh2_poly(float2 z) {
+  const float2 u = __fmul2_rn(z, z);
+  auto c = [](float a) { return make_float2(a, a); };
+  float2 y = __ffma2_rn(u, c(0.0010455536f), c(-0.0062170699f));
+  y = __ffma2_rn(u, y, c(0.02030552f));
+  y = __ffma2_rn(u, y, c(-0.053465176f));
+  y = __ffma2_rn(u, y, c(0.13325398f));
+  y = __ffma2_rn(u, y, c(-0.33332857f));
+  y = __ffma2_rn(u, y, c(0.99999994f));
+  return __fmul2_rn(y, z);
+}
+__device__ __forceinline__ float tanh_ex2(float z) { return 1.f - __fdividef(2.f, 1.f + ex2_approx(z * 2.8853900817779268f)); }
+
+// CAPPED: soft cap on the scores and a sigmoid gate per (token, head) on the output.
+template <bool CAPPED>
 __global__ void __launch_bounds__(THREADS, 1) prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_kv, const TcAttnParams p) {
   extern __shared__ uint8_t smem_raw[];
   const uint32_t base = smem_u32(smem_raw);
@@ -327,6 +348,25 @@ __global__ void __launch_bounds__(THREADS, 1) prefill_attn_tc_kernel(const __gri
       tmem_ld32(s_row + 64, v + 64);
       tmem_ld32(s_row + 96, v + 96);
       tmem_ld_wait();
+      if constexpr (CAPPED) {
+        if (p.cap_in > 0.f) {
+          float big = 0.f;
+#pragma unroll
+          for (int i = 0; i < BKV; i += 2) big = max3(big, fabsf(__uint_as_float(v[i])), fabsf(__uint_as_float(v[i + 1])));
+          if (__any_sync(0xFFFFFFFFu, big * p.cap_in > 1.f)) {
+#pragma unroll
+            for (int i = 0; i < BKV; ++i) v[i] = __float_as_uint(tanh_ex2(__uint_as_float(v[i]) * p.cap_in));
+          } else {
+            const float2 ci = make_float2(p.cap_in, p.cap_in);
+#pragma unroll
+            for (int i = 0; i < BKV; i += 2) {
+              const float2 t = tanh2_poly(__fmul2_rn(make_float2(__uint_as_float(v[i]), __uint_as_float(v[i + 1])), ci));
+              v[i] = __float_as_uint(t.x);
+              v[i + 1] = __float_as_uint(t.y);
+            }
+          }
+        }
+      }
       float mx_raw;
       if constexpr (MASK) {
         mx_raw = -INFINITY;
@@ -425,7 +465,10 @@ __global__ void __launch_bounds__(THREADS, 1) prefill_attn_tc_kernel(const __gri
       ok = mbar_wait(&sh->o_full[g], (uint32_t)((my_n - 1) & 1), abort_flag);
       tc_fence_after();
     }
-    const float inv = (ok && l > 0.f) ? 1.f / l : 0.f;
+    float inv = (ok && l > 0.f) ? 1.f / l : 0.f;
+    if constexpr (CAPPED) {
+      if (p.gate && r < rows_g) inv /= 1.f + __expf(-__bfloat162float(p.gate[(long long)(q0 + row_base + g * 128 + r) * p.ld_gate + hq]));
+    }
     bf16* dst = p.out + ((long long)(q0 + row_base + g * 128 + r) * p.hq + hq) * D;
 #pragma unroll
     for (int c = 0; c < D; c += 32) {
@@ -1085,9 +1128,28 @@ extern "C" void pg_prefill_attention_tc_variant(int v) { g_mn_variant = v; }
 
 // q [T, hq, d] bf16 (contiguous), kv_layer [pages, 2, page_size, hkv, d], out [T, hq * d], d = 128 or 256.  `q_tiles` = sum
 // over the sequences of ceil(query rows / 256) for d = 128 and of ceil(query rows / 128) for d = 256.
+static int prefill_tc_impl(const void* q, const void* kv_layer, void* out, const void* q_indptr, const void* kv_lens, const void* table, int table_stride, int num_seqs, int tokens, int hq,
+                           int hkv, int dim, int page_size, long long num_pages, float scale, int q_tiles, int window, bool capped, float softcap, const void* gate, long long ld_gate,
+                           void* status, cudaStream_t stream);
+
 extern "C" int pg_prefill_attention_tc(const void* q, const void* kv_layer, void* out, const void* q_indptr, const void* kv_lens, const void* table, int table_stride,
                                        int num_seqs, int tokens, int hq, int hkv, int dim, int page_size, long long num_pages, float scale, int q_tiles, int window,
                                        void* status, cudaStream_t stream) {
+  return prefill_tc_impl(q, kv_layer, out, q_indptr, kv_lens, table, table_stride, num_seqs, tokens, hq, hkv, dim, page_size, num_pages, scale, q_tiles, window, false, 0.f, nullptr, 0, status,
+                         stream);
+}
+
+// Head dim 128 with a soft cap on the scores (softcap > 0) and a sigmoid gate per (token, head) (gate: bf16 rows or null).
+extern "C" int pg_prefill_attention_tc_capped(const void* q, const void* kv_layer, void* out, const void* q_indptr, const void* kv_lens, const void* table, int table_stride, int num_seqs,
+                                              int tokens, int hq, int hkv, int page_size, long long num_pages, float scale, float softcap, const void* gate, long long ld_gate, int q_tiles,
+                                              void* status, cudaStream_t stream) {
+  return prefill_tc_impl(q, kv_layer, out, q_indptr, kv_lens, table, table_stride, num_seqs, tokens, hq, hkv, D, page_size, num_pages, scale, q_tiles, 0, true, softcap, gate, ld_gate, status,
+                         stream);
+}
+
+static int prefill_tc_impl(const void* q, const void* kv_layer, void* out, const void* q_indptr, const void* kv_lens, const void* table, int table_stride, int num_seqs, int tokens, int hq,
+                           int hkv, int dim, int page_size, long long num_pages, float scale, int q_tiles, int window, bool capped, float softcap, const void* gate, long long ld_gate,
+                           void* status, cudaStream_t stream) {
   PG_REQUIRE(window == 0 || dim == D2, "tcgen05 prefill attention: a sliding window is built for head dim 256 only");
   PG_REQUIRE(dim == D || dim == D2, "tcgen05 prefill attention is built for head dims 128 and 256 (got %d)", dim);
   const int key_tile = dim == D ? BKV : BKV2;
@@ -1111,7 +1173,10 @@ extern "C" int pg_prefill_attention_tc(const void* q, const void* kv_layer, void
   p.hkv = hkv;
   p.page_size = page_size;
   p.num_pages = num_pages;
-  p.scale_log2 = scale * 1.4426950408889634f;
+  p.scale_log2 = (softcap > 0.f ? softcap : scale) * 1.4426950408889634f;
+  p.cap_in = softcap > 0.f ? scale / softcap : 0.f;
+  p.gate = (const bf16*)gate;
+  p.ld_gate = ld_gate;
   p.window = window;
   p.mn_lbo_first = g_mn_variant < 0 ? 1 : g_mn_variant;
   p.status = (uint32_t*)status;
@@ -1129,10 +1194,11 @@ extern "C" int pg_prefill_attention_tc(const void* q, const void* kv_layer, void
   const size_t smem = 1024 + (GROUPS + 4) * (size_t)TILE_BYTES + sizeof(TcSmem) + 64;
   static bool attr_done = false;
   if (!attr_done) {
-    PG_CUDA(cudaFuncSetAttribute(prefill_attn_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    PG_CUDA(cudaFuncSetAttribute(prefill_attn_tc_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    PG_CUDA(cudaFuncSetAttribute(prefill_attn_tc_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     attr_done = true;
   }
-  PG_CUDA(launch_pdl(prefill_attn_tc_kernel, dim3((unsigned)q_tiles * (unsigned)hq), dim3(THREADS), smem, stream, tm_q, tm_kv, p));
+  PG_CUDA(launch_pdl(capped ? prefill_attn_tc_kernel<true> : prefill_attn_tc_kernel<false>, dim3((unsigned)q_tiles * (unsigned)hq), dim3(THREADS), smem, stream, tm_q, tm_kv, p));
   PG_LAUNCH_CHECK();
   return PG_OK;
 }

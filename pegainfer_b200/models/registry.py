@@ -59,7 +59,7 @@ BUILDERS = {"nemipel": _nemipel, "kimi_k3": _k3, "gemma4": _gemma4, "glm_dsa": _
 
 # Translation units (csrc/<name>.cu) that a family's kernels come from, for programs that build only what one model needs
 KERNEL_UNITS = {
-    "nemipel": ("runtime", "gemm_sm100", "gemm2sm_sm100", "elementwise", "stream32", "attention", "attention_general", "kda", "sampling"),
+    "nemipel": ("runtime", "gemm_sm100", "gemm2sm_sm100", "elementwise", "stream32", "attention", "attention_tc", "attention_general", "kda", "lightning", "sampling"),
 }
 
 

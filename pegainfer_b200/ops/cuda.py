@@ -956,7 +956,8 @@ def row_norm_rope_append(q, k, v, q_norm_w, k_norm_w, cos, sin, meta: AttnMeta, 
     t = q.shape[0]
     assert q.stride(1) == 1 and q.shape[1] == heads * dim and cos.dtype == sin.dtype == torch.float32 and q_norm_w.dtype == torch.float32
     if k is not None:
-        assert k.stride(0) == v.stride(0) == q.stride(0) and k.stride(1) == v.stride(1) == 1 and k.dtype == v.dtype == q.dtype == kv_layer.dtype
+        _same_rows(q, k, v)
+        assert k.stride(1) == v.stride(1) == 1 and k.dtype == v.dtype == q.dtype == kv_layer.dtype
         assert kv_layer.is_contiguous() and kv_layer.shape[1] == meta.page_size * kv_heads * (dim + vdim) and k_norm_w.dtype == torch.float32
     out = torch.empty((t, heads, dim), dtype=q.dtype, device=q.device)
     c = ctx(q.device)
@@ -1006,7 +1007,14 @@ def capped_attention(q, kv_layer, kv_heads: int, vdim: int, meta: AttnMeta, scal
         n_pf -= 1
     if meta.num_seqs - n_pf < (1 if _BATCH_INVARIANT else _MIXED_DECODE_MIN):
         n_pf = meta.num_seqs
-    if n_pf > 0:
+    if (n_pf > 0 and dim == vdim == 128 and _PREFILL_TC and not _BATCH_INVARIANT and max(qi[b + 1] - qi[b] for b in range(n_pf)) >= _PREFILL_TC_MIN_ROWS
+            and (meta.h_kv_lens is None or max(meta.h_kv_lens[:n_pf]) >= _PREFILL_TC_MIN_KV)):
+        PREFILL_TC_CALLS["hd128"] += 1
+        rc = lib().pg_prefill_attention_tc_capped(_ptr(q), _ptr(kv_layer), _ptr(out), _ptr(meta.q_indptr), _ptr(meta.kv_lens), _ptr(table), _ci(table.stride(0)), _ci(n_pf), _ci(qi[n_pf]), _ci(hq),
+                                                  _ci(kv_heads), _ci(ps), _ll(pages), _cf(scale), _cf(softcap), *gate_args, _ci(sum((qi[b + 1] - qi[b] + 255) // 256 for b in range(n_pf))),
+                                                  _ptr(c.status), _stream())
+        _check(rc, c)
+    elif n_pf > 0:
         run(0, n_pf, 1, 1, sum((qi[b + 1] - qi[b] + 63) // 64 for b in range(n_pf)))
     if n_pf < meta.num_seqs:
         decode_rows(n_pf, meta.num_seqs - n_pf)
@@ -1024,30 +1032,54 @@ def conv_silu(x, conv_w, conv_state, meta: AttnMeta):
     return out
 
 
+_LINEAR_CHUNKED = os.environ.get("PEGAINFER_LINEAR_CHUNKED", "1") != "0"
+
+
+def _has_short_rows(meta: AttnMeta, limit: int) -> bool:
+    """Is there a sequence below ``limit`` rows in the step (decode rows beside prompt portions)?"""
+    qi = meta.h_q_indptr
+    return qi is None or any(qi[i + 1] - qi[i] < limit for i in range(meta.num_seqs))
+
+
+def _same_rows(*ts) -> int:
+    """The common row stride of row-major tensors (a lone row has none)."""
+    if ts[0].shape[0] <= 1:
+        return 0
+    assert all(t.stride(0) == ts[0].stride(0) for t in ts), "rows of one fused buffer are expected"
+    return ts[0].stride(0)
+
+
 def channel_delta(q, k, v, f, b, a_log, dt_bias, state, meta: AttnMeta):
     """Delta rule with a softplus-form decay per key channel (``reference.channel_delta``); ``q, k, v`` share a row stride."""
     t, hk, dk = q.shape
     h, dv = v.shape[1], v.shape[2]
-    assert q.stride(2) == 1 and q.stride(1) == dk and k.stride(1) == dk and v.stride(1) == dv and q.stride(0) == k.stride(0) == v.stride(0)
+    assert q.stride(2) == 1 and q.stride(1) == dk and k.stride(1) == dk and v.stride(1) == dv
     assert f.dtype == torch.float32 and f.stride(1) == 1 and f.shape[1] == h * dk and b.stride(1) == 1 and b.dtype == q.dtype
     assert state.is_contiguous() and state.dtype == a_log.dtype == dt_bias.dtype == torch.float32
     out = torch.empty((t, h, dv), dtype=q.dtype, device=q.device)
-    rc = lib().pg_channel_delta(_ptr(q), _ptr(k), _ptr(v), _ll(q.stride(0)), _ptr(f), _ll(f.stride(0)), _ptr(b), _ll(b.stride(0)), _ptr(a_log), _ptr(dt_bias), _ptr(state), _ptr(out), _ptr(meta.q_indptr),
+    rc = lib().pg_channel_delta(_ptr(q), _ptr(k), _ptr(v), _ll(_same_rows(q, k, v)), _ptr(f), _ll(f.stride(0)), _ptr(b), _ll(b.stride(0)), _ptr(a_log), _ptr(dt_bias), _ptr(state), _ptr(out), _ptr(meta.q_indptr),
                                 _ptr(meta.state_slots), _ci(meta.num_seqs), _ci(h), _ci(hk), _ci(dk), _ci(dv), _ci(int(meta.max_q_len)), _ci(0), _ci(_is_f32(q)), _stream())
     _check(rc, ctx(q.device))
     return out
 
 
-def decay_attention(q, k, v, decay, state, meta: AttnMeta):
-    """Linear attention with a fixed decay per head (``reference.decay_attention``); ``q, k, v`` share a row stride."""
+def decay_attention(q, k, v, decay, state, meta: AttnMeta, chunked: Optional[bool] = None):
+    """Linear attention with a fixed decay per head (``reference.decay_attention``); ``q, k, v`` share a row stride.
+    Sequences of 32 tokens or more run on the chunk-wise tensor-core kernel (bf16, sizes that are multiples of 8), shorter
+    ones on the recurrence."""
     t, h, dk = q.shape
     dv = v.shape[2]
-    assert q.stride(2) == 1 and q.stride(1) == dk and k.stride(1) == dk and v.stride(1) == dv and q.stride(0) == k.stride(0) == v.stride(0)
+    assert q.stride(2) == 1 and q.stride(1) == dk and k.stride(1) == dk and v.stride(1) == dv
     assert state.is_contiguous() and state.dtype == decay.dtype == torch.float32
     out = torch.empty((t, h, dv), dtype=q.dtype, device=q.device)
-    rc = lib().pg_decay_recurrent(_ptr(q), _ptr(k), _ptr(v), _ll(q.stride(0)), _ptr(decay), _ptr(state), _ptr(out), _ptr(meta.q_indptr), _ptr(meta.state_slots), _ci(meta.num_seqs), _ci(h), _ci(dk), _ci(dv),
-                                  _ci(int(meta.max_q_len)), _ci(0), _ci(_is_f32(q)), _stream())
-    _check(rc, ctx(q.device))
+    f32, ld, c = _is_f32(q), _same_rows(q, k, v), ctx(q.device)
+    args = (_ptr(q), _ptr(k), _ptr(v), _ll(ld), _ptr(decay), _ptr(state), _ptr(out), _ptr(meta.q_indptr), _ptr(meta.state_slots), _ci(meta.num_seqs), _ci(h), _ci(dk), _ci(dv))
+    aligned = dk % 8 == 0 and dv % 8 == 0 and dk <= 128 and ld % 8 == 0 and all(x.data_ptr() % 16 == 0 for x in (q, k, v))
+    chunked = (_LINEAR_CHUNKED if chunked is None else chunked) and int(meta.max_q_len) >= _GDN_CHUNK_MIN and not f32 and aligned
+    if chunked:
+        _check(lib().pg_lightning_chunked(*args, _ci(_GDN_CHUNK_MIN), _stream()), c)
+    if not chunked or _has_short_rows(meta, _GDN_CHUNK_MIN):
+        _check(lib().pg_decay_recurrent(*args, _ci(int(meta.max_q_len)), _ci(_GDN_CHUNK_MIN if chunked else 0), _ci(f32), _stream()), c)
     return out
 
 

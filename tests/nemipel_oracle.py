@@ -67,7 +67,8 @@ def short_conv(x, w):
     y = torch.zeros_like(x)
     for j in range(taps):
         back = taps - 1 - j
-        y[back:] += w[:, j] * x[: x.shape[0] - back]
+        if back < x.shape[0]:
+            y[back:] += w[:, j] * x[: x.shape[0] - back]
     return silu(y)
 
 
