@@ -51,6 +51,7 @@ def parse():
     ap.add_argument("--prefill-chunk", type=int, default=4096, help="token budget of one prefill step (max_prefill_tokens)")
     ap.add_argument("--profile-host", default=None, help="write a cProfile of the scheduler thread during the e2e phase to this path")
     ap.add_argument("--no-library-arm", action="store_true", help="skip the cuBLAS + NCCL arm that is timed after the main arm and reported as `library_arm`")
+    ap.add_argument("--line-speed", action="store_true", help="instead of the headline workload: prefill and decode throughput of the Nemipel line beside the Qwen3.5 line at equal layer sizes, one JSON line per size")
     return ap.parse_args()
 
 
@@ -448,6 +449,10 @@ def main():
     args = parse()
     if args.impl == "reference":
         return reference_arm(args)
+    if args.line_speed:
+        from pegainfer_b200.utils.line_speed import run
+
+        return run(steps=min(args.steps, 64), warmup=max(args.warmup, 3), sampler=ClockSampler(0))
     import torch
 
     rank, local, world = init_dist(args)

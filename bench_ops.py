@@ -6,7 +6,7 @@ distinct weight / KV buffers (larger than L2 in total, so every launch streams f
 HBM), replayed after warm-up and timed with CUDA events.  Fractions are against the
 measured peaks in MEASURED_PEAKS.json (copy bandwidth, cuBLAS bf16 throughput).
 
-    python bench_ops.py [--only gemm|attn|small|gdn|kda|moe|mla] [--iters 16] [--json out.json]
+    python bench_ops.py [--only gemm|attn|small|gdn|kda|nemipel|moe|mla] [--iters 16] [--json out.json]
     python bench_ops.py --single gemm:64x4096x4096      # one op, few launches (ncu target)
 
 Plays the role of the reference's kernel/op report binaries
@@ -172,6 +172,76 @@ def gdn_cases(iters, only=None):
         if max(q_lens) >= 64:  # the row above ran the chunk-wise scan; this one the token-by-token kernel
             ms = time_graph(lambda i: K.gdn_recurrent(q, k, v, g, beta, states[i], meta, chunked=False), 3, max(2, iters // 4))
             rows.append((f"  recurrence kernel {name}", ms, state_bytes + t * (2 * hk * dk + 2 * hv * dv) * 2, 4.0 * t * hv * dk * dv * 2))
+    return rows
+
+
+def nemipel_cases(iters):
+    """Kernels of the Nemipel line, each beside the like kernel of the closest line at the same size (indented rows):
+    32 query / 8 KV heads of 128, 32 recurrent heads with a 128 x 128 state, width 4096."""
+    from pegainfer_b200.ops import cuda as K
+    from pegainfer_b200.ops.reference import pair_rope_tables, rope_tables
+
+    rows, page, hq, hkv, d, h = [], 16, 32, 8, 128, 32
+    few = max(2, iters // 4)
+    bf = lambda *s: torch.randn(*s, device=DEV).bfloat16()
+
+    def pair(name, like, new, old, by, by_old, fl, nvar, it):
+        rows.append((name, time_graph(new, nvar, it), by, fl))
+        rows.append(("  " + like, time_graph(old, nvar, it), by_old, fl))
+
+    for bs, ctx in ((64, 1152), (64, 4096), (8, 16384), (1, 1152)):
+        meta, pages = _meta_for([1] * bs, [ctx] * bs, page)
+        kv = [bf(pages, 2, page, hkv, d) for _ in range(1 if bs * ctx > 1 << 16 else 4)]
+        q, gate = bf(bs, hq, d), bf(bs, hq)
+        by = bs * ctx * 2 * hkv * d * 2
+        pair(f"capped_attention decode {bs}x{ctx}", "paged_attention", lambda i: K.capped_attention(q, kv[i].view(pages, -1), hkv, d, meta, d ** -0.5, 30.0, gate), lambda i: K.paged_attention(q, kv[i], meta), by, by,
+             4.0 * bs * ctx * hq * d, len(kv), iters)
+    for ns, ql in ((4, 1024), (1, 4096), (1, 16384), (16, 256)):
+        meta, pages = _meta_for([ql] * ns, [ql] * ns, page)
+        kv, q, gate = bf(pages, 2, page, hkv, d), bf(ns * ql, hq, d), bf(ns * ql, hq)
+        by = ns * ql * (2 * hq + 2 * hkv) * d * 2
+        pair(f"capped_attention prefill {ns}x{ql}", "paged_attention", lambda i: K.capped_attention(q, kv.view(pages, -1), hkv, d, meta, d ** -0.5, 30.0, gate), lambda i: K.paged_attention(q, kv, meta), by, by,
+             2.0 * ns * ql * ql * hq * d, 1, few)
+    for name, lens in (("decode 64", [1] * 64), ("decode 1", [1]), ("prefill 1x4096", [4096]), ("prefill 8x1024", [1024] * 8), ("prefill 16x256", [256] * 16)):
+        meta, _ = _meta_for(lens, lens, page)
+        meta.state_slots = torch.arange(len(lens), dtype=torch.int32, device=DEV)
+        t, n = sum(lens), len(lens)
+        st = [torch.zeros(n, h, d, d, device=DEV) for _ in range(3)]
+        x = bf(t, 3 * h * d)
+        q, k, v = (x[:, j * h * d : (j + 1) * h * d].view(t, h, d) for j in range(3))
+        dec, b, a_log, dt = torch.full((h,), 0.98, device=DEV), bf(t, h), torch.zeros(h, device=DEV), torch.zeros(h * d, device=DEV)
+        f32, f16, g, beta = torch.randn(t, h * d, device=DEV), bf(t, h * d), -torch.rand(t, h, device=DEV) * 0.1, torch.rand(t, h, device=DEV)
+        sb, fl = n * h * d * d * 8, 4.0 * t * h * d * d * 2
+        pair(f"decay_attention {name}", "gdn_recurrent", lambda i: K.decay_attention(q, k, v, dec, st[i], meta), lambda i: K.gdn_recurrent(q, k, v, g, beta, st[i], meta), sb + t * 4 * h * d * 2, sb + t * 4 * h * d * 2, fl, 3, few)
+        pair(f"channel_delta {name}", "kda_recurrent", lambda i: K.channel_delta(q, k, v, f32, b, a_log, dt, st[i], meta), lambda i: K.kda_recurrent(q, k, v, f16, b, a_log, dt, -5.0, st[i], meta), sb + t * 6 * h * d * 2,
+             sb + t * 5 * h * d * 2, fl, 3, few)
+    for t in (64, 4096):
+        w = 4096
+        y16, y32, x32, r16 = [[f(t, w) for _ in range(4)] for f in (bf, lambda *s: torch.randn(*s, device=DEV), lambda *s: torch.randn(*s, device=DEV), bf)]
+        w32, w16 = torch.ones(w, device=DEV), torch.ones(w, device=DEV).bfloat16()
+        y = y32 if t == 64 else y16
+        pair(f"post_norm {t}x{w}", "add_rms_norm", lambda i: K.post_norm(y[i], x32[i], w32, 1e-6, 2.0, torch.bfloat16), lambda i: K.add_rms_norm(y16[i], r16[i], w16, 1e-6), t * w * (8 + 2 + y[0].element_size()), t * w * 8, 0, 4, iters)
+        for hh, dd in ((32, 128), (1, 4096)):
+            o, gt, nw = [bf(t, hh, dd) for _ in range(4)], [bf(t, hh * dd) for _ in range(4)], torch.ones(dd, device=DEV)
+            pair(f"gated_row_norm {t}x{hh}x{dd}", "gated_rms_norm", lambda i: K.gated_row_norm(o[i], gt[i], nw, 1e-6), lambda i: K.gated_rms_norm(o[i], gt[i].view(t, hh, dd), nw, 1e-6, "sigmoid"), t * w * 6, t * w * 6, 0, 4, iters)
+        for lens in ([1] * 64,) if t == 64 else ([1024] * 4, [4096]):
+            meta, pages = _meta_for(lens, lens, page)
+            meta.state_slots = torch.arange(len(lens), dtype=torch.int32, device=DEV)
+            ch = 8192
+            z, cw = [bf(t, ch) for _ in range(4)], torch.randn(ch, 4, device=DEV)
+            cs, cw16 = torch.zeros(len(lens), ch, 3, device=DEV).bfloat16(), cw.bfloat16()
+            pair(f"conv_silu {len(lens)}x{lens[0]} {ch} channels", "gdn_conv1d", lambda i: K.conv_silu(z[i], cw, cs, meta), lambda i: K.gdn_conv1d(z[i], cw16, cs, meta), t * ch * 4, t * ch * 4, 0, 4, iters)
+        meta, pages = _meta_for([1] * 64 if t == 64 else [t], [1] * 64 if t == 64 else [t], page)
+        z = [bf(t, (hq + 2 * hkv) * d) for _ in range(4)]
+        kv, qn, kn = bf(pages, 2, page, hkv, d), torch.ones(hq * d, device=DEV), torch.ones(hkv * d, device=DEV)
+        c32, s32 = pair_rope_tables(8192, d, 1e4, DEV)
+        c16, s16 = rope_tables(8192, d, 1e4, torch.bfloat16, DEV)
+        one = torch.ones(d, device=DEV).bfloat16()
+        cut = lambda x: (x[:, : hq * d], x[:, hq * d : (hq + hkv) * d], x[:, (hq + hkv) * d :])
+        pair(f"row_norm_rope_append {t}", "qk_norm_rope_append", lambda i: K.row_norm_rope_append(*cut(z[i]), qn, kn, c32, s32, meta, kv.view(pages, -1), hq, hkv, d, d, 1e-6),
+             lambda i: K.qk_norm_rope_append(z[i], one, one, c16, s16, meta, kv, hq, hkv, d, 1e-6), t * (hq + 2 * hkv) * d * 4, t * (hq + 2 * hkv) * d * 4, 0, 4, iters)
+    lg32, lg16 = [torch.randn(64, 151936, device=DEV) for _ in range(4)], [bf(64, 151936) for _ in range(4)]
+    pair("softcap_rows 64x151936", "softcap", lambda i: K.softcap_rows(lg32[i], 30.0), lambda i: K.softcap(lg16[i], 30.0), 64 * 151936 * 8, 64 * 151936 * 4, 0, 4, iters)
     return rows
 
 
@@ -549,6 +619,8 @@ def main():
             rows.extend(gdn_cases(args.iters))
         if args.only in (None, "kda"):
             rows.extend(kda_cases(args.iters))
+        if args.only in (None, "nemipel"):
+            rows.extend(nemipel_cases(args.iters))
         if args.only in (None, "moe"):
             rows.extend(moe_cases(args.iters))
         if args.only in (None, "mla"):

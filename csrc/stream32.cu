@@ -94,19 +94,19 @@ __global__ void __launch_bounds__(256) post_norm_kernel(const TY* __restrict__ y
   }
 }
 
-// TPR threads per row (32 or 256); row r = token * heads + head; the gate row of (token, head) is gate + token * ldg + head * dim.
+// TPR threads per row (16, 32 or 256); row r = token * heads + head; the gate row of (token, head) is gate + token * ldg + head * dim.
 template <typename T, int V, int TPR>
 __global__ void __launch_bounds__(256) gated_row_norm_kernel(const T* __restrict__ x, const T* __restrict__ gate, long long ldg, const float* __restrict__ w, T* __restrict__ y, long long rows, int heads, int dim,
                                                              float eps) {
   PG_PDL_ENTRY();
   __shared__ float red[32];
-  const long long row = TPR == 256 ? (long long)blockIdx.x : (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
-  const int me = TPR == 256 ? threadIdx.x : (threadIdx.x & 31);
-  if (row >= rows) return;  // whole warps leave together; with TPR == 256 the grid has no spare blocks
+  const long long row = TPR == 256 ? (long long)blockIdx.x : (long long)blockIdx.x * (256 / TPR) + threadIdx.x / TPR;
+  const int me = threadIdx.x % TPR;
+  const bool live = row < rows;  // with TPR == 256 the grid has no spare blocks
   const T* xr = x + row * dim;
   const T* gr = gate + (row / heads) * ldg + (row % heads) * dim;
   constexpr int KEEP = 4;
-  const int nv = dim / V;
+  const int nv = live ? dim / V : 0;
   float f[KEEP][V], ss = 0.f;
 #pragma unroll
   for (int k = 0; k < KEEP; ++k) {
@@ -123,7 +123,12 @@ __global__ void __launch_bounds__(256) gated_row_norm_kernel(const T* __restrict
 #pragma unroll
     for (int j = 0; j < V; ++j) ss += o[j] * o[j];
   }
-  ss = TPR == 256 ? block_sum(ss, red) : warp_sum(ss);
+  if (TPR == 256) {
+    ss = block_sum(ss, red);
+  } else {
+#pragma unroll
+    for (int o = TPR / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+  }
   const float inv = rsqrtf(ss / (float)dim + eps);
   auto put = [&](int i, const float* o) {
     float g[V], wf[V], r[V];
@@ -197,11 +202,12 @@ __global__ void __launch_bounds__(256) gemm_simt_kernel(const TX* __restrict__ x
 }
 
 constexpr int CONV_MAX = 16;   // taps
-constexpr int CONV_TILE = 32;  // tokens per CTA; at least CONV_MAX, so a sequence of more than one tile fills the carried inputs from its own rows
+constexpr int CONV_TILE = 16;  // tokens per CTA; at least CONV_MAX - 1, so a sequence of more than one tile fills the carried inputs from its own rows
 
 // A thread owns one channel for CONV_TILE tokens.  The CTA of a sequence's first tile reads the carried inputs and is also
 // the one that replaces them (from the sequence's last rows), so no other CTA touches the state.
-template <typename T>
+// CM: the number of taps rounded up to an instantiated size.
+template <typename T, int CM>
 __global__ void __launch_bounds__(128) conv_silu_kernel(const T* __restrict__ x, long long ldx, const float* __restrict__ w, T* __restrict__ state, T* __restrict__ out, long long ldo, const int* __restrict__ q_indptr,
                                                         const int* __restrict__ slots, int channels, int taps, long long slot_stride) {
   PG_PDL_ENTRY();
@@ -212,42 +218,41 @@ __global__ void __launch_bounds__(128) conv_silu_kernel(const T* __restrict__ x,
   if (c >= channels || s0 >= n || slot < 0) return;
   T* st = state + slot * slot_stride + (long long)c * (taps - 1);
   const int back = taps - 1;
-  // history: inputs s0 - back .. s0 - 1 of the sequence (from the state where they lie before this step)
-  float win[CONV_MAX], wt[CONV_MAX];
+  const int n_here = min(CONV_TILE, n - s0);
+  T rows[CONV_TILE];  // all loads of the tile in flight together
 #pragma unroll
-  for (int j = 0; j < CONV_MAX; ++j) wt[j] = j < taps ? w[(long long)c * taps + j] : 0.f;
+  for (int i = 0; i < CONV_TILE; ++i)
+    if (i < n_here) rows[i] = x[(long long)(q0 + s0 + i) * ldx + c];
+  // window and weights are right-aligned: entry CM - 1 belongs to the current row; inputs before this step come from the state
+  float win[CM], wt[CM];
 #pragma unroll
-  for (int j = 0; j < CONV_MAX - 1; ++j) {
-    const int at = s0 - back + j;
-    win[j] = j < back ? (at < 0 ? to_f32(st[back + at]) : to_f32(x[(long long)(q0 + at) * ldx + c])) : 0.f;
+  for (int j = 0; j < CM; ++j) {
+    const int tap = j - (CM - taps), at = s0 + j - (CM - 1);
+    wt[j] = tap >= 0 ? w[(long long)c * taps + tap] : 0.f;
+    win[j] = tap >= 0 && j < CM - 1 ? (at < 0 ? to_f32(st[back + at]) : to_f32(x[(long long)(q0 + at) * ldx + c])) : 0.f;
   }
-  T keep[CONV_MAX];
+  T keep[CM];
   if (s0 == 0) {
 #pragma unroll
-    for (int j = 0; j < CONV_MAX - 1; ++j) {
+    for (int j = 0; j < CM - 1; ++j) {
       const int at = n - back + j;
       if (j < back) keep[j] = at < 0 ? st[back + at] : x[(long long)(q0 + at) * ldx + c];
     }
   }
-  const int end = min(s0 + CONV_TILE, n);
-  for (int s = s0; s < end; ++s) {
-    const float cur = to_f32(x[(long long)(q0 + s) * ldx + c]);
+#pragma unroll
+  for (int i = 0; i < CONV_TILE; ++i) {
+    if (i >= n_here) break;
+    win[CM - 1] = to_f32(rows[i]);
     float a = 0.f;
 #pragma unroll
-    for (int j = 0; j < CONV_MAX; ++j) {
-      if (j < back) a = fmaf(win[j], wt[j], a);
-      if (j == back) a = fmaf(cur, wt[j], a);
-    }
-    out[(long long)(q0 + s) * ldo + c] = from_f32<T>(a / (1.f + __expf(-a)));
+    for (int j = 0; j < CM; ++j) a = fmaf(win[j], wt[j], a);
+    out[(long long)(q0 + s0 + i) * ldo + c] = from_f32<T>(__fdividef(a, 1.f + __expf(-a)));
 #pragma unroll
-    for (int j = 0; j < CONV_MAX - 1; ++j) {
-      if (j + 1 < back) win[j] = win[j + 1];
-      if (j + 1 == back) win[j] = cur;
-    }
+    for (int j = 0; j < CM - 1; ++j) win[j] = win[j + 1];
   }
   if (s0 == 0) {
 #pragma unroll
-    for (int j = 0; j < CONV_MAX - 1; ++j)
+    for (int j = 0; j < CM - 1; ++j)
       if (j < back) st[j] = keep[j];
   }
 }
@@ -290,14 +295,15 @@ extern "C" int pg_gated_row_norm(const void* x, const void* gate, long long ldg,
   if (tokens == 0) return PG_OK;
   const long long rows = (long long)tokens * heads;
   const bool wide = dim > 512;
-  const dim3 grid((unsigned)(wide ? rows : (rows + 7) / 8));
+  const bool v8 = !is_f32 && dim % 8 == 0 && ldg % 8 == 0 && al(x, 16) && al(gate, 16) && al(w, 16) && al(y, 16);
+  const bool half = v8 && dim <= 128;  // a half warp covers the row with one access per lane
+  const dim3 grid((unsigned)(wide ? rows : half ? (rows + 15) / 16 : (rows + 7) / 8));
 #define PG_GRN(T, V, TPR) launch_pdl(gated_row_norm_kernel<T, V, TPR>, grid, dim3(256), (size_t)0, stream, (const T*)x, (const T*)gate, ldg, (const float*)w, (T*)y, rows, heads, dim, eps)
   if (is_f32) {
     PG_CUDA(wide ? PG_GRN(float, 1, 256) : PG_GRN(float, 1, 32));
   } else {
-    const bool v8 = dim % 8 == 0 && ldg % 8 == 0 && al(x, 16) && al(gate, 16) && al(w, 16) && al(y, 16);
     if (v8)
-      PG_CUDA(wide ? PG_GRN(bf16, 8, 256) : PG_GRN(bf16, 8, 32));
+      PG_CUDA(wide ? PG_GRN(bf16, 8, 256) : half ? PG_GRN(bf16, 8, 16) : PG_GRN(bf16, 8, 32));
     else
       PG_CUDA(wide ? PG_GRN(bf16, 1, 256) : PG_GRN(bf16, 1, 32));
   }
@@ -345,10 +351,11 @@ extern "C" int pg_conv_silu(const void* x, long long ldx, const void* w, void* s
   if (num_seqs == 0) return PG_OK;
   const dim3 grid((channels + 127) / 128, (max_q_len + CONV_TILE - 1) / CONV_TILE, num_seqs);
   PG_REQUIRE(grid.y <= 65535u && grid.z <= 65535u, "conv_silu: %d sequences of %d rows", num_seqs, max_q_len);
-  if (is_f32)
-    PG_CUDA(launch_pdl(conv_silu_kernel<float>, grid, dim3(128), (size_t)0, stream, (const float*)x, ldx, (const float*)w, (float*)state, (float*)out, ldo, (const int*)q_indptr, (const int*)slots, channels, taps, slot_stride));
-  else
-    PG_CUDA(launch_pdl(conv_silu_kernel<bf16>, grid, dim3(128), (size_t)0, stream, (const bf16*)x, ldx, (const float*)w, (bf16*)state, (bf16*)out, ldo, (const int*)q_indptr, (const int*)slots, channels, taps, slot_stride));
+#define PG_CONV(T, CM) launch_pdl(conv_silu_kernel<T, CM>, grid, dim3(128), (size_t)0, stream, (const T*)x, ldx, (const float*)w, (T*)state, (T*)out, ldo, (const int*)q_indptr, (const int*)slots, channels, taps, slot_stride)
+#define PG_CONVS(T) (taps <= 2 ? PG_CONV(T, 2) : taps <= 4 ? PG_CONV(T, 4) : taps <= 8 ? PG_CONV(T, 8) : PG_CONV(T, 16))
+  PG_CUDA(is_f32 ? PG_CONVS(float) : PG_CONVS(bf16));
+#undef PG_CONVS
+#undef PG_CONV
   PG_LAUNCH_CHECK();
   return PG_OK;
 }

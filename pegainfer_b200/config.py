@@ -253,13 +253,13 @@ PRESETS["kimi-k3"] = replace(PRESETS["small-k3"], vocab_size=163840, hidden_size
 # a one-GPU slice of the released shape for benchmarks (not a released configuration): full-width layers (6 KDA + 2 MLA, one dense
 # and seven latent-MoE layers), 32 routed experts instead of 896, top 8
 PRESETS["k3-8layer-shape"] = replace(PRESETS["kimi-k3"], num_layers=8, layer_types=_k3_pattern(8), n_routed_experts=32, num_experts_per_tok=8, attn_res_block=4, max_position=131072)
-def _nemipel(width: int, vocab: int, ff: int, heads: int, kv_heads: int, dim: int, lin_heads: int, lin_dim: int, rank: int, periods: int, **kw) -> ModelConfig:
+def _nemipel(width: int, vocab: int, ff: int, heads: int, kv_heads: int, dim: int, lin_heads: int, lin_dim: int, rank: int, periods: int, lightning_ff: int = 0, **kw) -> ModelConfig:
     """A Nemipel stack of ``periods`` x (lightning, attention, channel-delta); every second attention layer reads the cache
-    of the one before it, the attention layers have the feed-forwards."""
+    of the one before it, the lightning layers have no feed-forward unless ``lightning_ff`` gives its width."""
     layers = []
     for n in range(periods):
         own = 3 * n + 1 if n % 2 == 0 else 3 * (n - 1) + 1
-        layers.append(LayerSpec(MixerSpec("lightning", lin_heads, lin_dim, lin_dim, decay=tuple(float(f"{1 - 2.0 ** (-1 - 7 * h / max(lin_heads - 1, 1)):.6f}") for h in range(lin_heads)))))
+        layers.append(LayerSpec(MixerSpec("lightning", lin_heads, lin_dim, lin_dim, decay=tuple(float(f"{1 - 2.0 ** (-1 - 7 * h / max(lin_heads - 1, 1)):.6f}") for h in range(lin_heads))), lightning_ff))
         layers.append(LayerSpec(MixerSpec("attention", heads, dim, dim, kv_heads=kv_heads, scale=dim ** -0.5, softcap=30.0, rot_dims=dim // 2, rot_base=1e4,
                                           kv_from=-1 if own == 3 * n + 1 else own), ff))
         layers.append(LayerSpec(MixerSpec("channel_delta", lin_heads, lin_dim, lin_dim, kv_heads=lin_heads // 2, conv=4, decay_rank=rank, gate_rank=rank), ff))
@@ -273,7 +273,11 @@ PRESETS["tiny-nemipel"] = _nemipel(96, 256, 160, 4, 2, 32, 4, 16, 12, 2, max_pos
 PRESETS["small-nemipel"] = _nemipel(1024, 4096, 2048, 8, 2, 128, 8, 128, 64, 2, max_position=8192)
 # layers as wide as those of an 8 B-parameter model, for benchmarks (not a released configuration): 12 lightning, 12
 # attention (6 of them with a cache of their own) and 12 channel-delta layers
-PRESETS["nemipel-8b-shape"] = _nemipel(4096, 151936, 12288, 32, 8, 128, 32, 128, 128, 12)
+PRESETS["nemipel-8b-shape"] = _nemipel(4096, 151936, 12288, 32, 8, 128, 32, 128, 128, 12, lightning_ff=12288)
+# the Qwen3.5 line at the same sizes: Gated DeltaNet layers in the place of the lightning and channel-delta layers
+PRESETS["qwen35-8b-shape"] = replace(PRESETS["small-qwen35"], vocab_size=151936, hidden_size=4096, num_layers=36, num_q_heads=32, num_kv_heads=8, head_dim=128, intermediate_size=12288,
+                                     layer_types=("linear_attention", "full_attention", "linear_attention") * 12, partial_rotary_factor=0.5, gdn_num_k_heads=16, gdn_num_v_heads=32, gdn_head_dim=128,
+                                     max_position=131072)
 PRESETS["small-glm-fp8"] = replace(PRESETS["small-glm"], expert_quant="fp8_block128", dense_quant="fp8_block128")
 for _name in ("tiny-dsv2", "small-dsv2", "dsv2-lite"):
     if _name in PRESETS:

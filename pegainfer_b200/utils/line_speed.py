@@ -1,0 +1,106 @@
+"""Throughput of the Nemipel line beside the Qwen3.5 line (the closest: linear-attention layers with recurrent state
+interleaved with paged attention) at equal sizes, random weights: ``bench.py --line-speed``.
+
+Device time (CUDA events) of whole steps of the executor: prefill steps of the given batches, and replays of the decode graph
+at a batch and context.  Weights and state are larger than L2 at every size, so no flush is needed.
+"""
+from __future__ import annotations
+
+import json
+from dataclasses import replace
+
+# (name, width, feed-forward, query heads, KV heads, recurrent heads); heads of 128, 12 layers each
+SIZES = (("2048", 2048, 6144, 16, 8, 16), ("4096", 4096, 12288, 32, 8, 32), ("5120", 5120, 17408, 40, 8, 40))
+PREFILL = ((1, 4096), (8, 1024))
+DECODE = ((64, 1024), (8, 1024), (1, 1024))
+
+
+def configs(width, ff, heads, kv_heads, lin_heads, periods=4, vocab=32768):
+    from ..config import PRESETS, _nemipel
+
+    a = _nemipel(width, vocab, ff, heads, kv_heads, 128, lin_heads, 128, 128, periods, lightning_ff=ff, max_position=16384)
+    b = replace(PRESETS["qwen35-8b-shape"], vocab_size=vocab, hidden_size=width, num_layers=3 * periods, num_q_heads=heads, num_kv_heads=kv_heads, intermediate_size=ff,
+                layer_types=("linear_attention", "full_attention", "linear_attention") * periods, gdn_num_k_heads=lin_heads // 2, gdn_num_v_heads=lin_heads, max_position=16384)
+    return {"nemipel": a, "qwen35": b}
+
+
+def _timed(fn, n, warmup):
+    import torch
+
+    for _ in range(warmup):
+        fn()
+    e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    torch.cuda.synchronize()
+    e0.record()
+    for _ in range(n):
+        fn()
+    e1.record()
+    torch.cuda.synchronize()
+    return e0.elapsed_time(e1) / n
+
+
+def measure(mcfg, steps: int, warmup: int, device="cuda:0") -> dict:
+    import torch
+
+    from ..config import EngineConfig
+    from ..engine.build import build_engine
+    from ..kv.request_kv import KvView
+    from ..sched.executor import SeqStep, build_meta
+
+    page, out = 16, {}
+    longest = max(max(n for _, n in PREFILL), max(n for _, n in DECODE) + steps)
+    blocks = 64 * ((1024 + 2 * page) // page + 1) + longest // page + 8
+    eng = build_engine(EngineConfig(num_kv_blocks=blocks, max_decode_batch=64, max_model_len=longest + page, no_prefix_cache=True), mcfg, device=device, dtype=torch.bfloat16, start=False)
+    ex = eng.executor
+    try:
+        out["weight_gb"] = round(torch.cuda.memory_allocated(device) / 1e9, 2)
+
+        def sequences(n, length, new):
+            per = (length + page - 1) // page
+            return [SeqStep(rid=i, input_tokens=[(7 * j + i) % mcfg.vocab_size for j in range(new)], start_pos=length - new, view=KvView(list(range(1 + i * per, 1 + (i + 1) * per)), length, page)) for i in range(n)]
+
+        for n, length in PREFILL:
+            seqs = sequences(n, length, length)
+            ids, meta = build_meta(seqs, page, device)
+            ex.prepare_meta(seqs, meta)
+            last = torch.tensor([meta.h_q_indptr[i + 1] - 1 for i in range(n)], dtype=torch.int32, device=device)
+            ms = _timed(lambda: ex.model.logits(ex.model.forward_hidden(ids, meta, ex.kv), last), 8, warmup)
+            out[f"prefill_{n}x{length}_tok_s"] = round(n * length / ms * 1e3)
+            for s in seqs:
+                ex.release_request(s.rid)
+        for n, ctx in DECODE:
+            seqs = sequences(n, ctx, 1)
+            ex._graphs.run(seqs)
+            b = next(x for x in ex._graphs.buckets if x >= n)
+            ms = _timed(ex._graphs.graphs[(b, True)].replay, steps, warmup)
+            out[f"decode_{n}x{ctx}_ms"], out[f"decode_{n}x{ctx}_tok_s"] = round(ms, 3), round(n / ms * 1e3)
+            for s in seqs:
+                ex.release_request(s.rid)
+        from ..ops import cuda as K
+
+        assert K.read_status(device) == 0, "device status word is set"
+    finally:
+        eng.shutdown()
+        ex._graphs.release()
+    return out
+
+
+def run(steps: int = 64, warmup: int = 8, sampler=None) -> int:
+    import gc
+
+    import torch
+
+    for name, *dims in SIZES:
+        line = {"metric": "prefill and decode tok/s, Nemipel line beside the Qwen3.5 line", "size": name, "config": dict(zip(("width", "ff", "heads", "kv_heads", "recurrent_heads"), dims), layers=12, head_dim=128), "dtype": "bf16",
+                "data": "random-init weights, synthetic tokens", "steps": steps, "warmup": warmup}
+        if sampler is not None:
+            sampler.start()
+        for fam, cfg in configs(*dims).items():
+            line[fam] = measure(cfg, steps, warmup)
+            gc.collect()
+            torch.cuda.empty_cache()
+        if sampler is not None:
+            line["clocks"] = sampler.stop()
+        line["nemipel_over_qwen35"] = {k[:-6]: round(line["nemipel"][k] / line["qwen35"][k], 3) for k in line["nemipel"] if k.endswith("_tok_s")}
+        print(json.dumps(line), flush=True)
+    return 0

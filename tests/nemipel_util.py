@@ -45,12 +45,15 @@ CONFIGS = {
     "odd": _cfg(50, 1e-3, 0.5, 0.0, [(_attn(18, 1, 18, 13, 2), 30), (_light(5, 6, 11, (0.5, 0.7, 0.8, 0.9, 0.999)), 0), (_delta(3, 1, 7, 9, 5), 21)]),
     # more than eight heads per group, heads of 256, key width past 128, no rotation
     "large": _cfg(128, 1e-6, 2.5, 12.0, [(_attn(20, 2, 256, 72, 64, softcap=50.0), 96), (_light(2, 144, 40, (0.95, 0.8)), 0), (_delta(4, 2, 136, 48, 4), 72), (_attn(2, 1, 32, 64, 0), 24)]),
+    # no cache at all; no recurrent state at all
+    "recurrent": _cfg(48, 1e-6, 2.0, 9.0, [(_light(2, 24, 8, (0.9, 0.3)), 0), (_delta(2, 1, 16, 8, 2), 32)]),
+    "attention": _cfg(40, 1e-6, 2.0, 9.0, [(_attn(2, 2, 16, 8, 4, softcap=3.0), 0), (_attn(3, 1, 40, 24, 40, softcap=8.0), 32)]),
 }
 
 
 # largest error of a position in bf16 (twice what rounding the activations of the plain path to bf16 gives; a small
 # postln_alpha lets the sublayers' rounding through)
-BF16_ERROR = {"mixed": 0.12, "wide": 0.08, "odd": 0.36, "large": 0.03}
+BF16_ERROR = {"mixed": 0.12, "wide": 0.08, "odd": 0.36, "large": 0.03, "recurrent": 0.08, "attention": 0.08}
 
 
 def weights(cfg, seed=0, dtype=torch.bfloat16):
