@@ -245,6 +245,27 @@ def nemipel_cases(iters):
     return rows
 
 
+def nemipel_single(kind, n, length, iters):
+    from pegainfer_b200.ops import cuda as K
+
+    page, hq, hkv, d, t = 16, 32, 8, 128, n * length
+    meta, pages = _meta_for([length] * n, [length] * n, page)
+    meta.state_slots = torch.arange(n, dtype=torch.int32, device=DEV)
+    bf = lambda *s: torch.randn(*s, device=DEV).bfloat16()
+    x, st = bf(t, 3 * hq * d), torch.zeros(n, hq, d, d, device=DEV)
+    q, k, v = (x[:, j * hq * d : (j + 1) * hq * d].view(t, hq, d) for j in range(3))
+    if kind == "capped":
+        kv, qq, gate = bf(pages, 2 * page * hkv * d), q.contiguous(), bf(t, hq)
+        return kind, time_graph(lambda i: K.capped_attention(qq, kv, hkv, d, meta, d ** -0.5, 30.0, gate), 1, iters), t * (2 * hq + 2 * hkv) * d * 2, 2.0 * n * length * length * hq * d
+    if kind == "lightning":
+        dec = torch.full((hq,), 0.98, device=DEV)
+        fn = lambda i: K.decay_attention(q, k, v, dec, st, meta)
+    else:
+        f, b, z = torch.randn(t, hq * d, device=DEV), bf(t, hq), torch.zeros(hq * d, device=DEV)
+        fn = lambda i: K.channel_delta(q, k, v, f, b, z[:hq], z, st, meta)
+    return kind, time_graph(fn, 1, iters), n * hq * d * d * 8 + t * 4 * hq * d * 2, 8.0 * t * hq * d * d
+
+
 def kda_cases(iters, only=None):
     """KDA recurrence (decay per key channel, gate arithmetic in the kernel) and the attention-residual mix at the Kimi-K3
     shape: 96 heads with a 128x128 f32 state, hidden 7168, 8 snapshots."""
@@ -562,6 +583,8 @@ def main():
             ms, by, fl = gemm_case(*dims, iters=args.iters, mode={"gemm": "auto", "gemm2sm": "two_sm", "gemm1cta": "one_cta"}[kind])
         elif kind == "gdn":
             name, ms, by, fl = gdn_cases(args.iters, only=[("single", [dims[1]] * dims[0])])[0]
+        elif kind in ("capped", "lightning", "chdelta"):  # sequences x tokens: one prompt step of the Nemipel line's kernel
+            name, ms, by, fl = nemipel_single(kind, dims[0], dims[1], args.iters)
         elif kind == "chain":
             ms, by, fl = chain_case(dims[0], dims[1], dims[2], dims[3], args.iters)
         elif kind == "fp8":

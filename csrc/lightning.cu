@@ -41,7 +41,6 @@ template <int DK>
 __global__ void __launch_bounds__(256, 1) lightning_chunk_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k, const bf16* __restrict__ v, long long ld, const float* __restrict__ decay,
                                                                  float* __restrict__ state, bf16* __restrict__ out, const int* __restrict__ q_indptr, const int* __restrict__ slots, int heads,
                                                                  int dk, int dv, int col_blocks, int min_len) {
-  PG_PDL_ENTRY();
   extern __shared__ __align__(16) uint8_t smem_raw[];
   LightSmem<DK>& sm = *reinterpret_cast<LightSmem<DK>*>(smem_raw);
   constexpr int LDK = LightSmem<DK>::LDK;
@@ -265,8 +264,8 @@ int launch_lightning(const void* q, const void* k, const void* v, long long ld, 
     set = true;
   }
   const int cb = (dv + DVC - 1) / DVC;
-  PG_CUDA(launch_pdl(lightning_chunk_kernel<DK>, dim3(heads * cb, num_seqs), dim3(256), sizeof(LightSmem<DK>), stream, (const bf16*)q, (const bf16*)k, (const bf16*)v, ld, (const float*)decay,
-                     (float*)state, (bf16*)out, (const int*)q_indptr, (const int*)slots, heads, dk, dv, cb, min_len));
+  lightning_chunk_kernel<DK><<<dim3(heads * cb, num_seqs), 256, sizeof(LightSmem<DK>), stream>>>((const bf16*)q, (const bf16*)k, (const bf16*)v, ld, (const float*)decay, (float*)state,
+                                                                                                 (bf16*)out, (const int*)q_indptr, (const int*)slots, heads, dk, dv, cb, min_len);
   PG_LAUNCH_CHECK();
   return PG_OK;
 }

@@ -81,8 +81,8 @@ def build_engine(ecfg: EngineConfig, mcfg: Optional[ModelConfig] = None, device=
     device = torch.device(device)
     if dtype is None:
         dtype = getattr(torch, ecfg.dtype) if device.type == "cuda" else torch.float32
-    if device.type == "cuda" and dtype != torch.bfloat16 and model is None and mcfg.family not in F32_FAMILIES:
-        raise ValueError(f"the {mcfg.family} line has bfloat16 kernels only")
+        if device.type == "cuda" and dtype != torch.bfloat16 and mcfg.family not in F32_FAMILIES:
+            raise ValueError(f"the {mcfg.family} line has bfloat16 kernels only")
     if ecfg.gemm == "cublas" and device.type == "cuda":
         from .. import ops
 
