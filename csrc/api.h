@@ -93,6 +93,13 @@ int pg_prefill_attention_tc_capped(const void* q, const void* kv_layer, void* ou
                                    int hq, int hkv, int page_size, long long num_pages, float scale, float softcap, const void* gate, long long ld_gate, int q_tiles, void* status,
                                    cudaStream_t stream);
 
+// ---- expanded-form latent prefill on tcgen05 (mla_prefill.cu) ------------------------------
+int pg_latent_gather(const void* latent_layer, int page_size, long long num_pages, int width, const void* table, int table_stride, const void* kv_indptr, const void* starts, int num_seqs, int total_kv,
+                     void* out, void* status, cudaStream_t stream);
+int pg_latent_prefill_tc(const void* q, long long q_tok, long long q_head, const void* q_pe, long long pe_tok, long long pe_head, const void* k, const void* v, long long ld_kv, const void* k_pe,
+                         long long pe_ld, const void* gate, long long ld_gate, void* out, const void* q_indptr, const void* kv_indptr, const void* kv_lens, int num_seqs, int tokens, int total_kv, int heads,
+                         int dim, int rot, int vdim, float scale, int window, int q_tiles, void* status, cudaStream_t stream);
+
 // ---- block-scaled FP8 GEMM on tcgen05 kind::f8f6f4 (gemm_fp8_sm100.cu) --------------------
 long long pg_gemm_fp8_ws_bytes(int T, int M);
 int pg_gemm_fp8_block(const void* xq, long long ldx, const void* x_scale, long long ldxs, const void* wq, long long ldw, const void* w_scale, void* y,
@@ -124,9 +131,21 @@ int pg_mla_attention(const void* q_abs, const void* q_pe, const void* latent, vo
                      const void* table, int table_stride, const void* unit_seq, int num_seqs, int tokens, int heads, int c, int rope,
                      int page_size, float scale, int splits, void* part_o, void* part_lse, void* status, cudaStream_t stream);
 
+// Absorbed latent attention with runtime sizes (latent c, shared rotated key part r, any number of heads), an optional
+// sliding window, and rotation of neighbouring query columns inside the kernel; token / head strides in elements.
+int pg_latent_attention(const void* q_abs, long long q_tok, long long q_head, const void* q_pe, long long pe_tok, long long pe_head, const void* cos, const void* sin, int max_pos, const void* latent,
+                        void* out, long long o_tok, long long o_head, const void* q_indptr, const void* kv_lens, const void* table, int table_stride, const void* unit_seq, int first_row, int num_seqs,
+                        int tokens, int heads, int c, int r, int page_size, float scale, int window, int splits, void* part_o, void* part_lse, cudaStream_t stream);
+int pg_latent_attention_plain(const void* q_abs, long long q_tok, long long q_head, const void* q_pe, long long pe_tok, long long pe_head, const void* cos, const void* sin, int max_pos, const void* latent,
+                              void* out, long long o_tok, long long o_head, const void* q_indptr, const void* kv_lens, const void* table, int table_stride, const void* unit_seq, int tokens, int heads, int c,
+                              int r, int page_size, float scale, int window, int is_f32, cudaStream_t stream);
+int pg_latent_rows(const void* zq, const void* zkv, long long ld, const void* q_w, const void* kv_w, const void* cos, const void* sin, const void* positions, const void* slots, void* cq, void* latent,
+                   int tokens, int qr, int c, int r, int max_pos, long long num_slots, float eps, int is_f32, void* status, cudaStream_t stream);
+int pg_rotate_pairs(void* x, long long tok, long long head, const void* cos, const void* sin, const void* positions, int tokens, int heads, int r, int max_pos, int is_f32, cudaStream_t stream);
+
 // ---- mixture of experts (moe_route.cu, moe_gemm.cu) --------------------------------
 int pg_router_topk(const void* logits, long long ld, const void* bias, void* ids, void* weights, int tokens, int E, int k, int sigmoid, int n_group,
-                   int topk_group, int norm, float scale, cudaStream_t stream);
+                   int topk_group, int group_top, int norm, float scale, cudaStream_t stream);
 int pg_moe_align(const void* ids, int routes, int e0, int e_local, void* offsets, void* sorted_src, void* route_pos, cudaStream_t stream);
 int pg_moe_gather(const void* x, long long ldx, const void* sorted_src, const void* offsets, int e_local, int k, void* out, int width, int max_rows,
                   cudaStream_t stream);
@@ -136,6 +155,10 @@ int pg_moe_combine(const void* y, long long ldy, const void* route_pos, const vo
 int pg_moe_grouped_gemm(const void* x, long long ldx, long long x_rows, const void* w, const void* scales, int quant, void* y, long long ldy,
                         const void* offsets, int E, int M, int K, int bn, void* status, cudaStream_t stream);
 
+int pg_moe_grouped_gemm_relu2(const void* x, long long ldx, long long x_rows, const void* w, void* y, long long ldy, const void* offsets, int E, int M, int K, int bn, void* status, cudaStream_t stream);
+// Per-head products of strided activations: y[t, h, :] = x[t, h, :] w[h]^T (times the sigmoid of a gate)
+int pg_head_gemm(const void* x, long long ldx, long long x_head, const void* w, void* y, long long ldy, long long y_head, const void* gate, long long ldg, long long g_head, int heads, int rows, int M, int K,
+                 int bn, void* status, cudaStream_t stream);
 int pg_moe_grouped_gemm_return(const void* x, long long ldx, long long x_rows, const void* w, const void* scales, int quant, long long ldy,
                                const void* offsets, int E, int M, int K, int bn, void* status, const void* scatter_src, void* const* peer_out,
                                void* const* peer_flags, int cap, int rank, int world, int site, cudaStream_t stream);
@@ -208,6 +231,12 @@ int pg_embed_rows(const void* table, int table_f32, long long ldt, const void* i
                   cudaStream_t stream);
 int pg_post_norm(const void* y, int y_f32, long long ldy, const void* x_in, void* x_out, float alpha, const void* w, void* xt, int xt_f32, long long ldxt, int tokens, int width, float eps,
                  cudaStream_t stream);
+int pg_add_layer_norm(const void* y, int y_f32, long long ldy, const void* pos, const void* weights, int k, void* x, const void* w, void* xt, int xt_f32, long long ldxt, int tokens, int width, float eps,
+                      cudaStream_t stream);
+int pg_head_gemm_simt(const void* x, long long ldx, long long x_head, const void* w, void* y, long long ldy, long long y_head, const void* gate, long long ldg, long long g_head, int heads, int rows, int M,
+                      int K, int is_f32, cudaStream_t stream);
+int pg_expert_gemm_simt(const void* x, long long ldx, const void* sorted_src, int k, const void* w, void* y, const void* offsets, int routes, int E, int M, int K, int relu2, int is_f32,
+                        cudaStream_t stream);
 int pg_gated_row_norm(const void* x, const void* gate, long long ldg, const void* w, void* y, int tokens, int heads, int dim, float eps, int is_f32, cudaStream_t stream);
 int pg_glu_rows_f32(const void* gu, void* out, int rows, int inter, long long ldin, cudaStream_t stream);
 int pg_softcap_f32(const void* x, void* y, long long n, float cap, cudaStream_t stream);

@@ -10,6 +10,11 @@
 // derived on the device from `offsets`, so the launch shape does not depend on the
 // routing and the kernel can sit inside a captured graph.
 //
+// Two further forms of the bf16 kernel: the squared ReLU on the output (experts without a gate projection), and heads in
+// the place of experts (pg_head_gemm): every head has the same number of rows, taken from a strided [rows, heads, K]
+// activation through a tensor map of its own and stored strided, so that the per-head products around latent attention
+// read and write token-major buffers; a sigmoid gate may multiply the output.
+//
 // Weight formats:
 //   bf16   W [E, M, K]: TMA straight into the swizzled A tile.
 //   int4   W packed [E, M, K/8] int32 (offset-binary nibbles, pair-interleaved inside each word:
@@ -63,6 +68,13 @@ struct MoeGemmParams {
   bf16* peer_out[8];
   uint32_t* peer_flags[8];
   int cap, rank, world, site;
+  int relu2;  // y = max(y, 0)^2
+  // heads instead of experts: `head_rows` rows each (0: rows come from `offsets`), output of head h at y + h * y_head, and
+  // an optional gate[row * ldg + h * g_head + m] whose sigmoid multiplies the output
+  int head_rows;
+  long long y_head;
+  const bf16* gate;
+  long long ldg, g_head;
 };
 
 struct Item {
@@ -86,7 +98,7 @@ __device__ __forceinline__ bool locate(const MoeGemmParams& p, const int* s_tile
   out.e = c.e;
   out.m_tile = local / n_tiles;
   const int n_tile = local - out.m_tile * n_tiles;
-  const int r0 = p.offsets[c.e], r1 = p.offsets[c.e + 1];
+  const int r0 = p.head_rows ? 0 : p.offsets[c.e], r1 = p.head_rows ? p.head_rows : p.offsets[c.e + 1];
   out.row0 = r0 + n_tile * p.bn;
   out.rows = min(p.bn, r1 - out.row0);
   return true;
@@ -141,7 +153,7 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant_
   }
   // per-expert item counts (every CTA derives the same list from the routing offsets)
   for (int e = threadIdx.x; e < p.E; e += blockDim.x) {
-    const int n = p.offsets[e + 1] - p.offsets[e];
+    const int n = p.head_rows ? p.head_rows : p.offsets[e + 1] - p.offsets[e];
     s_tiles[e] = n > 0 ? p.m_tiles * ((n + p.bn - 1) / p.bn) : 0;
   }
   if (warp == 1) {
@@ -193,7 +205,10 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant_
             mbar_expect_tx(&full[stage], (uint32_t)(A_BYTES + b_bytes));
             tma_load_3d(st, &tm_w, &full[stage], kb * BK, it.m_tile * BM, it.e, pol_w);
           }
-          tma_load_2d(st + A_BYTES, &tm_x, &full[stage], kb * BK, it.row0, pol_x);
+          if (p.head_rows)
+            tma_load_3d(st + A_BYTES, &tm_x, &full[stage], kb * BK, it.e, it.row0, pol_x);
+          else
+            tma_load_2d(st + A_BYTES, &tm_x, &full[stage], kb * BK, it.row0, pol_x);
           used[stage] = true;
           last_phase[stage] = phase;
           if (++stage == p.stages) {
@@ -268,9 +283,25 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant_
         tmem_ld_wait();
         if (m < p.M) {
           if (p.scatter_src == nullptr) {
+            if (p.relu2) {
+#pragma unroll
+              for (int j = 0; j < 16; ++j) {
+                const float f = fmaxf(__uint_as_float(v[j]), 0.f);
+                v[j] = __float_as_uint(f * f);
+              }
+            }
+            bf16* dst = p.y + (p.head_rows ? it.e * p.y_head : 0ll) + (long long)(it.row0 + c) * p.ldy + m;
+            if (p.gate != nullptr) {
+              const bf16* gp = p.gate + it.e * p.g_head + (long long)(it.row0 + c) * p.ldg + m;
+              float gv[16];
+#pragma unroll
+              for (int j = 0; j < 16; ++j) gv[j] = c + j < it.rows ? __bfloat162float(gp[j * p.ldg]) : 0.f;
+#pragma unroll
+              for (int j = 0; j < 16; ++j) v[j] = __float_as_uint(__uint_as_float(v[j]) / (1.f + __expf(-gv[j])));
+            }
 #pragma unroll
             for (int j = 0; j < 16; ++j)
-              if (c + j < it.rows) p.y[(size_t)(it.row0 + c + j) * p.ldy + m] = __float2bfloat16(__uint_as_float(v[j]));
+              if (c + j < it.rows) dst[j * p.ldy] = __float2bfloat16(__uint_as_float(v[j]));
           } else {
 #pragma unroll
             for (int j = 0; j < 16; ++j) {
@@ -451,15 +482,20 @@ std::mutex g_mu;
 
 }  // namespace
 
+struct HeadArgs {
+  long long x_head, y_head, g_head, ldg;
+  const void* gate;
+};
+
 // x [rows, K] bf16 (rows sorted by expert), offsets [E+1] device int32, y [rows, M] bf16.
 // w: bf16 [E, M, K] (quant 0); packed int32 [E, M, K/8] with scales bf16 [E, M, K/32] (quant 1);
 // fp8 e4m3 [E, M, K] with f32 scale_inv [E, ceil(M/128), ceil(K/128)] (quant 2).
 // `bn` is the token tile (multiple of 16, <= 256): pick it near the expected rows per expert.
 static int moe_gemm_impl(const void* x, long long ldx, long long x_rows, const void* w, const void* scales, int quant, void* y, long long ldy,
                          const void* offsets, int E, int M, int K, int bn, void* status, const void* scatter_src, void* const* peer_out,
-                         void* const* peer_flags, int cap, int rank, int world, int site, cudaStream_t stream) {
+                         void* const* peer_flags, int cap, int rank, int world, int site, cudaStream_t stream, int relu2 = 0, const HeadArgs* heads = nullptr) {
   PG_REQUIRE(E >= 1 && E <= MAX_EXPERTS, "moe gemm: %d experts not supported (<= %d)", E, MAX_EXPERTS);
-  PG_REQUIRE(K % 64 == 0, "moe gemm: K=%d must be a multiple of 64", K);
+  PG_REQUIRE(quant == 0 ? K % 8 == 0 : K % 64 == 0, "moe gemm: K=%d must be a multiple of %d", K, quant == 0 ? 8 : 64);
   PG_REQUIRE(bn >= 16 && bn <= 256 && bn % 16 == 0, "moe gemm: token tile %d must be a multiple of 16 in [16, 256]", bn);
   PG_REQUIRE(status != nullptr, "moe gemm: a device status word is required");
   if (x_rows == 0 && scatter_src == nullptr) return PG_OK;
@@ -487,7 +523,7 @@ static int moe_gemm_impl(const void* x, long long ldx, long long x_rows, const v
   p.K = K;
   p.E = E;
   p.bn = bn;
-  p.kblocks = K / BK;
+  p.kblocks = ceil_div(K, BK);  // the last block of an odd K is filled with zeros by TMA on both operands
   p.m_tiles = ceil_div(M, BM);
   PG_REQUIRE(quant >= 0 && quant <= 2, "moe gemm: unknown weight storage mode %d", quant);
   PG_REQUIRE(quant == 0 || scales != nullptr, "moe gemm: quantised weights need scales");
@@ -495,6 +531,14 @@ static int moe_gemm_impl(const void* x, long long ldx, long long x_rows, const v
   p.scales = scales;
   p.offsets = (const int*)offsets;
   p.status = (uint32_t*)status;
+  p.relu2 = relu2;
+  if (heads) {
+    p.head_rows = (int)x_rows;
+    p.y_head = heads->y_head;
+    p.gate = (const bf16*)heads->gate;
+    p.ldg = heads->ldg;
+    p.g_head = heads->g_head;
+  }
   p.scatter_src = (const int*)scatter_src;
   if (scatter_src) {
     for (int q = 0; q < world; ++q) {
@@ -547,8 +591,19 @@ static int moe_gemm_impl(const void* x, long long ldx, long long x_rows, const v
                      CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
     PG_REQUIRE(r == CUDA_SUCCESS, "moe gemm: weight tensor map failed (%d)", (int)r);
   }
-  int rc = pg_make_tmap_bf16_2d(&tm_x, x, x_rows, K, ldx, bn, BK);
-  if (rc) return rc;
+  if (heads) {
+    PG_REQUIRE(((uintptr_t)x & 15) == 0 && ldx % 8 == 0 && heads->x_head % 8 == 0, "head gemm: activations must start and step on 16-byte boundaries");
+    PG_REQUIRE(heads->x_head >= K && ldx >= heads->x_head * E, "head gemm: heads lie inside a row (row stride %lld, head stride %lld, %d heads of %d)", ldx, heads->x_head, E, K);
+    cuuint64_t dims[3] = {(cuuint64_t)K, (cuuint64_t)E, (cuuint64_t)x_rows};
+    cuuint64_t strides[2] = {(cuuint64_t)heads->x_head * 2, (cuuint64_t)ldx * 2};
+    cuuint32_t box[3] = {BK, 1, (cuuint32_t)bn};
+    CUresult r = enc(&tm_x, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(x), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
+                     CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+    PG_REQUIRE(r == CUDA_SUCCESS, "head gemm: activation tensor map failed (%d)", (int)r);
+  } else {
+    int rc = pg_make_tmap_bf16_2d(&tm_x, x, x_rows, K, ldx, bn, BK);
+    if (rc) return rc;
+  }
   const size_t smem = 1024 + (size_t)p.stages * stage_bytes + tail;
   moe_gemm_kernel<<<g_sms[dev & 63], quant ? 448 : 192, smem, stream>>>(tm_w, tm_x, p);
   PG_LAUNCH_CHECK();
@@ -558,6 +613,20 @@ static int moe_gemm_impl(const void* x, long long ldx, long long x_rows, const v
 extern "C" int pg_moe_grouped_gemm(const void* x, long long ldx, long long x_rows, const void* w, const void* scales, int quant, void* y,
                                    long long ldy, const void* offsets, int E, int M, int K, int bn, void* status, cudaStream_t stream) {
   return moe_gemm_impl(x, ldx, x_rows, w, scales, quant, y, ldy, offsets, E, M, K, bn, status, nullptr, nullptr, nullptr, 0, 0, 1, 0, stream);
+}
+
+// bf16 experts with the squared ReLU on the output.
+extern "C" int pg_moe_grouped_gemm_relu2(const void* x, long long ldx, long long x_rows, const void* w, void* y, long long ldy, const void* offsets, int E, int M, int K, int bn, void* status,
+                                         cudaStream_t stream) {
+  return moe_gemm_impl(x, ldx, x_rows, w, nullptr, 0, y, ldy, offsets, E, M, K, bn, status, nullptr, nullptr, nullptr, 0, 0, 1, 0, stream, 1);
+}
+
+// y[t, h, :] = x[t, h, :] w[h]^T, w [heads, M, K]; row / head strides in elements; gate (bf16, or null) strided like y.
+extern "C" int pg_head_gemm(const void* x, long long ldx, long long x_head, const void* w, void* y, long long ldy, long long y_head, const void* gate, long long ldg, long long g_head, int heads, int rows,
+                            int M, int K, int bn, void* status, cudaStream_t stream) {
+  HeadArgs a;
+  a.x_head = x_head, a.y_head = y_head, a.g_head = g_head, a.ldg = ldg, a.gate = gate;
+  return moe_gemm_impl(x, ldx, rows, w, nullptr, 0, y, ldy, nullptr, heads, M, K, bn, status, nullptr, nullptr, nullptr, 0, 0, 1, 0, stream, 0, &a);
 }
 
 // Expert-parallel W2: output rows are stored straight into their source ranks' combine

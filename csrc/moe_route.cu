@@ -2,8 +2,8 @@
 //
 //  * router_topk: one warp per token over f32 logits [T, E] (E <= 512).  softmax or
 //    sigmoid scores, optional selection bias, optional group-limited routing (keep the
-//    `topk_group` best of `n_group` groups, group score = sum of its two best biased
-//    scores), k rounds of warp arg-max (ties -> lowest expert id), weights from the
+//    `topk_group` best of `n_group` groups, group score = the sum of its two best
+//    biased scores, or the best one), k rounds of warp arg-max (ties -> lowest expert id), weights from the
 //    un-biased scores, optional renormalisation, scaling.
 //  * moe_align: stable counting sort of the routes that hit local experts ->
 //    expert offsets, source token per sorted row, sorted row per route.
@@ -28,7 +28,7 @@ struct RouterParams {
   const float* bias;
   int* ids;
   float* weights;
-  int tokens, E, k, sigmoid, n_group, topk_group, norm;
+  int tokens, E, k, sigmoid, n_group, topk_group, group_top, norm;
   float scale;
 };
 
@@ -84,7 +84,7 @@ __global__ void __launch_bounds__(128) router_topk_kernel(const RouterParams p) 
     choice[s] = e < p.E ? score[s] + (p.bias ? p.bias[e] : 0.f) : -FLT_MAX;
   }
   if (p.n_group > 1) {
-    // group g = experts [g*gs, (g+1)*gs); score = sum of its two best choices
+    // group g = experts [g*gs, (g+1)*gs); score = sum of its group_top (1 or 2) best choices
     const int gs = p.E / p.n_group;
     uint32_t keep = 0u;  // bit g set = group g survives (n_group <= 32)
     float gscore_mine = -FLT_MAX;  // lane g holds group g's score
@@ -112,7 +112,7 @@ __global__ void __launch_bounds__(128) router_topk_kernel(const RouterParams p) 
         b1 = n1;
         b2 = n2;
       }
-      const float gsc = gs >= 2 ? b1 + b2 : b1;
+      const float gsc = gs >= 2 && p.group_top == 2 ? b1 + b2 : b1;
       if (lane == g) gscore_mine = gsc;
     }
     for (int r = 0; r < p.topk_group; ++r) {
@@ -214,7 +214,9 @@ __global__ void moe_combine_kernel(const bf16* __restrict__ y, long long ldy, co
 }  // namespace
 
 extern "C" int pg_router_topk(const void* logits, long long ld, const void* bias, void* ids, void* weights, int tokens, int E, int k, int sigmoid,
-                              int n_group, int topk_group, int norm, float scale, cudaStream_t stream) {
+                              int n_group, int topk_group, int group_top, int norm, float scale, cudaStream_t stream) {
+  PG_REQUIRE(group_top == 1 || group_top == 2, "router: a group's score is its best or its two best, not %d", group_top);
+  PG_REQUIRE(n_group < 1 || topk_group < 1 || (long long)E / n_group * topk_group >= k, "router: %d groups of %d keep fewer than %d experts", topk_group, E / n_group, k);
   PG_REQUIRE(E <= 32 * MAXE_PER_LANE && k >= 1 && k <= 32 && k <= E, "router: E=%d (<= 512) / k=%d (<= 32) out of range", E, k);
   PG_REQUIRE(n_group >= 1 && n_group <= 32 && E % n_group == 0 && topk_group >= 1 && topk_group <= n_group, "router: bad group routing %d/%d", topk_group, n_group);
   if (tokens == 0) return PG_OK;
@@ -230,6 +232,7 @@ extern "C" int pg_router_topk(const void* logits, long long ld, const void* bias
   p.sigmoid = sigmoid;
   p.n_group = n_group;
   p.topk_group = topk_group;
+  p.group_top = group_top;
   p.norm = norm;
   p.scale = scale;
   router_topk_kernel<<<(tokens + 3) / 4, 128, 0, stream>>>(p);

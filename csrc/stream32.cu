@@ -4,11 +4,16 @@
 //  * post_norm: the norm after the sum.  s = alpha * x + y; x = s / sqrt(mean(s^2) + eps) * w.  The stream x is read and
 //    written in f32, y is a projection's output (f32 or bf16), and the activation-type copy that the next projection
 //    reads is written in the same pass.  Without y and with alpha = 1 it is a plain RMS norm of the stream.
+//  * add_layer_norm: the norm of a sublayer's output before the sum.  x += (y - mean(y)) / sqrt(mean((y - mean)^2) + eps) * w
+//    on the f32 stream, with the activation-type copy of the new stream written in the same pass.  y is a projection's
+//    output, or the weighted sum of a token's expert rows, which is then formed here instead of by a kernel of its own.
+//    With y = x and no sum it is the plain layer norm of the stream.
 //  * gated_row_norm: RMS norm over a row (one head, or all heads of a token at once), times a weight, times the sigmoid
 //    of a gate row that may lie inside a wider projection output.
 //  * glu_rows: silu(gate) * up on f32 rows; softcap_f32: cap * tanh(x / cap) on f32 values.
 //  * gemm_simt: y = x w^T on the CUDA cores with f32 accumulation, for f32 operands (the 32-bit mode) and for bf16
-//    problems whose rows the TMA kernels cannot address (an inner size that is not a multiple of 8).
+//    problems whose rows the TMA kernels cannot address (an inner size that is not a multiple of 8).  head_gemm_simt is the
+//    same per attention head (strided operands, sigmoid gate on the output), expert_gemm_simt per expert over sorted rows.
 //  * conv_silu: causal depthwise convolution of any length + SiLU over ragged sequences with carried inputs.
 #include "api.h"
 #include "common.cuh"
@@ -94,6 +99,100 @@ __global__ void __launch_bounds__(256) post_norm_kernel(const TY* __restrict__ y
   }
 }
 
+// A row's y: a row of one matrix, or sum_j weights[j] * rows[pos[j]] over the token's k expert rows (rows of one matrix
+// sorted by expert; pos < 0: none).
+template <typename TY>
+struct RowSource {
+  const TY* y;
+  long long ld;
+  const int* pos;
+  const float* weights;
+  int k;
+  template <int V>
+  __device__ __forceinline__ void load(long long row, int at, float* o) const {
+    if (pos == nullptr) {
+      load_vec<V>(y + row * ld + at, o);
+      return;
+    }
+#pragma unroll
+    for (int j = 0; j < V; ++j) o[j] = 0.f;
+    for (int s = 0; s < k; ++s) {
+      const int r = pos[row * k + s];
+      if (r < 0) continue;
+      const float w = weights[row * k + s];
+      float f[V];
+      load_vec<V>(y + r * ld + at, f);
+#pragma unroll
+      for (int j = 0; j < V; ++j) o[j] = fmaf(w, f[j], o[j]);
+    }
+  }
+};
+
+// One CTA per row.  x (f32 stream) is read and written; x == nullptr: only the norm goes to xt.
+template <typename TY, typename TO, int V>
+__global__ void __launch_bounds__(256) add_layer_norm_kernel(const RowSource<TY> src, float* __restrict__ x, const float* __restrict__ w, TO* __restrict__ xt, long long ldxt, int width, float eps) {
+  PG_PDL_ENTRY();
+  __shared__ float red[32];
+  constexpr int KEEP = 8;
+  const long long row = blockIdx.x;
+  const int nv = width / V;
+  float v[KEEP][V], sum = 0.f;
+#pragma unroll
+  for (int k = 0; k < KEEP; ++k) {
+    const int i = threadIdx.x + k * 256;
+    if (i < nv) {
+      src.template load<V>(row, i * V, v[k]);
+#pragma unroll
+      for (int j = 0; j < V; ++j) sum += v[k][j];
+    }
+  }
+  for (int i = threadIdx.x + KEEP * 256; i < nv; i += 256) {  // wider rows: read again below
+    float o[V];
+    src.template load<V>(row, i * V, o);
+#pragma unroll
+    for (int j = 0; j < V; ++j) sum += o[j];
+  }
+  const float mean = block_sum(sum, red) / (float)width;
+  float ss = 0.f;
+#pragma unroll
+  for (int k = 0; k < KEEP; ++k)
+    if (threadIdx.x + k * 256 < nv) {
+#pragma unroll
+      for (int j = 0; j < V; ++j) ss += (v[k][j] - mean) * (v[k][j] - mean);
+    }
+  for (int i = threadIdx.x + KEEP * 256; i < nv; i += 256) {
+    float o[V];
+    src.template load<V>(row, i * V, o);
+#pragma unroll
+    for (int j = 0; j < V; ++j) ss += (o[j] - mean) * (o[j] - mean);
+  }
+  const float inv = rsqrtf(block_sum(ss, red) / (float)width + eps);
+  auto put = [&](int i, float* o) {
+    float wf[V];
+    load_vec<V>(w + i * V, wf);
+#pragma unroll
+    for (int j = 0; j < V; ++j) o[j] = (o[j] - mean) * inv * wf[j];
+    if (x) {
+      float xf[V];
+      load_vec<V>(x + row * width + i * V, xf);
+#pragma unroll
+      for (int j = 0; j < V; ++j) o[j] += xf[j];
+      store_vec<V>(x + row * width + i * V, o);
+    }
+    if (xt) store_vec<V>(xt + row * ldxt + i * V, o);
+  };
+#pragma unroll
+  for (int k = 0; k < KEEP; ++k) {
+    const int i = threadIdx.x + k * 256;
+    if (i < nv) put(i, v[k]);
+  }
+  for (int i = threadIdx.x + KEEP * 256; i < nv; i += 256) {
+    float o[V];
+    src.template load<V>(row, i * V, o);
+    put(i, o);
+  }
+}
+
 // TPR threads per row (16, 32 or 256); row r = token * heads + head; the gate row of (token, head) is gate + token * ldg + head * dim.
 template <typename T, int V, int TPR>
 __global__ void __launch_bounds__(256) gated_row_norm_kernel(const T* __restrict__ x, const T* __restrict__ gate, long long ldg, const float* __restrict__ w, T* __restrict__ y, long long rows, int heads, int dim,
@@ -165,19 +264,17 @@ __global__ void softcap_f32_kernel(const float* __restrict__ x, float* __restric
   for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x) y[i] = cap * tanh_full(x[i] / cap);
 }
 
-// 64 x 64 output tile, 256 threads of 4 x 4 outputs, 16-deep k steps.
-template <typename TX, typename TY>
-__global__ void __launch_bounds__(256) gemm_simt_kernel(const TX* __restrict__ x, const TX* __restrict__ w, TY* __restrict__ y, int T, int M, int K, long long ldx, long long ldw, long long ldy) {
-  PG_PDL_ENTRY();
+// 64 x 64 output tile, 256 threads of 4 x 4 outputs, 16-deep k steps: acc = x rows [t0, T) times w rows [m0, M).
+// `xrow(t)` is the row of x that output row t reads.
+template <typename TX, typename XRow>
+__device__ __forceinline__ void simt_tile(const TX* __restrict__ x, const TX* __restrict__ w, int t0, int T, int m0, int M, int K, long long ldx, long long ldw, XRow xrow, float (&acc)[4][4]) {
   __shared__ float xs[16][68], ws[16][68];
-  const int m0 = blockIdx.x * 64, t0 = blockIdx.y * 64;
   const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
-  float acc[4][4] = {};
   for (int k0 = 0; k0 < K; k0 += 16) {
     for (int i = threadIdx.x; i < 64 * 16; i += 256) {
       const int r = i >> 4, k = i & 15;
       const bool kin = k0 + k < K;
-      xs[k][r] = (kin && t0 + r < T) ? to_f32(x[(long long)(t0 + r) * ldx + k0 + k]) : 0.f;
+      xs[k][r] = (kin && t0 + r < T) ? to_f32(x[(long long)xrow(t0 + r) * ldx + k0 + k]) : 0.f;
       ws[k][r] = (kin && m0 + r < M) ? to_f32(w[(long long)(m0 + r) * ldw + k0 + k]) : 0.f;
     }
     __syncthreads();
@@ -192,12 +289,80 @@ __global__ void __launch_bounds__(256) gemm_simt_kernel(const TX* __restrict__ x
     }
     __syncthreads();
   }
+}
+
+template <typename TX, typename TY>
+__global__ void __launch_bounds__(256) gemm_simt_kernel(const TX* __restrict__ x, const TX* __restrict__ w, TY* __restrict__ y, int T, int M, int K, long long ldx, long long ldw, long long ldy) {
+  PG_PDL_ENTRY();
+  const int m0 = blockIdx.x * 64, t0 = blockIdx.y * 64;
+  const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+  float acc[4][4] = {};
+  simt_tile(x, w, t0, T, m0, M, K, ldx, ldw, [](int t) { return t; }, acc);
 #pragma unroll
   for (int i = 0; i < 4; ++i)
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int t = t0 + ty * 4 + i, m = m0 + tx * 4 + j;
       if (t < T && m < M) y[(long long)t * ldy + m] = from_f32<TY>(acc[i][j]);
+    }
+}
+
+// Head h (grid z): y[t, h, :] = x[t, h, :] w[h]^T, times sigmoid(gate[t, h, :]) when a gate is given.
+template <typename T>
+__global__ void __launch_bounds__(256) head_gemm_simt_kernel(const T* __restrict__ x, long long ldx, long long x_head, const T* __restrict__ w, T* __restrict__ y, long long ldy, long long y_head,
+                                                             const T* __restrict__ gate, long long ldg, long long g_head, int rows, int M, int K) {
+  PG_PDL_ENTRY();
+  const int m0 = blockIdx.x * 64, t0 = blockIdx.y * 64, h = blockIdx.z;
+  const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+  float acc[4][4] = {};
+  simt_tile(x + h * x_head, w + (long long)h * M * K, t0, rows, m0, M, K, ldx, (long long)K, [](int t) { return t; }, acc);
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int t = t0 + ty * 4 + i, m = m0 + tx * 4 + j;
+      if (t >= rows || m >= M) continue;
+      float v = acc[i][j];
+      if (gate) v /= 1.f + __expf(-to_f32(gate[(long long)t * ldg + h * g_head + m]));
+      y[(long long)t * ldy + h * y_head + m] = from_f32<T>(v);
+    }
+}
+
+// Rows sorted by expert: y[r] = act(x[src(r)] w[e(r)]^T), src(r) = sorted_src[r] / k (token of the route) or r itself.
+// Grid y counts 64-row tiles of all experts; a tile finds its expert by walking the offsets.
+template <typename T>
+__global__ void __launch_bounds__(256) expert_gemm_simt_kernel(const T* __restrict__ x, long long ldx, const int* __restrict__ sorted_src, int k, const T* __restrict__ w, T* __restrict__ y,
+                                                               const int* __restrict__ offsets, int E, int M, int K, int relu2) {
+  PG_PDL_ENTRY();
+  __shared__ int s_e, s_row, s_end;
+  if (threadIdx.x == 0) {
+    int rem = blockIdx.y;
+    s_e = -1;
+    for (int e = 0; e < E; ++e) {
+      const int a = offsets[e], b = offsets[e + 1], tiles = (b - a + 63) / 64;
+      if (rem < tiles) {
+        s_e = e, s_row = a + rem * 64, s_end = b;
+        break;
+      }
+      rem -= tiles;
+    }
+  }
+  __syncthreads();
+  const int e = s_e;
+  if (e < 0) return;
+  const int m0 = blockIdx.x * 64, t0 = s_row, end = s_end;
+  const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+  float acc[4][4] = {};
+  simt_tile(x, w + (long long)e * M * K, t0, end, m0, M, K, ldx, (long long)K, [=](int r) { return sorted_src ? sorted_src[r] / k : r; }, acc);
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int t = t0 + ty * 4 + i, m = m0 + tx * 4 + j;
+      if (t >= end || m >= M) continue;
+      float v = acc[i][j];
+      if (relu2) v = v > 0.f ? v * v : 0.f;
+      y[(long long)t * M + m] = from_f32<T>(v);
     }
 }
 
@@ -291,6 +456,29 @@ extern "C" int pg_post_norm(const void* y, int y_f32, long long ldy, const void*
   return PG_OK;
 }
 
+// y: [tokens, ldy] rows, or with pos / weights [tokens, k] the expert rows that pos points into (their weighted sum is the
+// token's y).  x: f32 stream, updated in place (null: none, and then the norm itself goes to xt).
+extern "C" int pg_add_layer_norm(const void* y, int y_f32, long long ldy, const void* pos, const void* weights, int k, void* x, const void* w, void* xt, int xt_f32, long long ldxt, int tokens, int width,
+                                 float eps, cudaStream_t stream) {
+  PG_REQUIRE(y != nullptr && w != nullptr && (x || xt), "add_layer_norm: rows, the norm weight and a destination are required");
+  PG_REQUIRE((pos == nullptr) == (weights == nullptr) && (pos == nullptr || k >= 1), "add_layer_norm: row positions and weights come together");
+  if (tokens == 0) return PG_OK;
+  const int yb = y_f32 ? 4 : 2, tb = xt_f32 ? 4 : 2;
+  const bool v4 = width % 4 == 0 && al(w, 16) && (!x || al(x, 16)) && ldy % 4 == 0 && al(y, 4 * yb) && (!xt || (ldxt % 4 == 0 && al(xt, 4 * tb)));
+#define PG_LN(TY, TO, V)                                                                                                                                                                             \
+  launch_pdl(add_layer_norm_kernel<TY, TO, V>, dim3(tokens), dim3(256), (size_t)0, stream, RowSource<TY>{(const TY*)y, ldy, (const int*)pos, (const float*)weights, k}, (float*)x, (const float*)w, \
+             (TO*)xt, ldxt, width, eps)
+#define PG_LN2(TY, TO) (v4 ? PG_LN(TY, TO, 4) : PG_LN(TY, TO, 1))
+  if (y_f32)
+    PG_CUDA(xt_f32 ? PG_LN2(float, float) : PG_LN2(float, bf16));
+  else
+    PG_CUDA(xt_f32 ? PG_LN2(bf16, float) : PG_LN2(bf16, bf16));
+#undef PG_LN2
+#undef PG_LN
+  PG_LAUNCH_CHECK();
+  return PG_OK;
+}
+
 extern "C" int pg_gated_row_norm(const void* x, const void* gate, long long ldg, const void* w, void* y, int tokens, int heads, int dim, float eps, int is_f32, cudaStream_t stream) {
   if (tokens == 0) return PG_OK;
   const long long rows = (long long)tokens * heads;
@@ -341,6 +529,30 @@ extern "C" int pg_gemm_simt(const void* x, const void* w, int x_f32, void* y, in
   else
     PG_CUDA(y_f32 ? PG_SG(bf16, float) : PG_SG(bf16, bf16));
 #undef PG_SG
+  PG_LAUNCH_CHECK();
+  return PG_OK;
+}
+
+extern "C" int pg_head_gemm_simt(const void* x, long long ldx, long long x_head, const void* w, void* y, long long ldy, long long y_head, const void* gate, long long ldg, long long g_head, int heads,
+                                 int rows, int M, int K, int is_f32, cudaStream_t stream) {
+  PG_REQUIRE(heads > 0 && rows > 0 && M > 0 && K > 0, "head_gemm_simt: empty problem");
+  const dim3 grid((M + 63) / 64, (rows + 63) / 64, heads);
+  PG_REQUIRE(grid.y <= 65535u && grid.z <= 65535u, "head_gemm_simt: %d rows of %d heads", rows, heads);
+#define PG_HG(T) launch_pdl(head_gemm_simt_kernel<T>, grid, dim3(256), (size_t)0, stream, (const T*)x, ldx, x_head, (const T*)w, (T*)y, ldy, y_head, (const T*)gate, ldg, g_head, rows, M, K)
+  PG_CUDA(is_f32 ? PG_HG(float) : PG_HG(bf16));
+#undef PG_HG
+  PG_LAUNCH_CHECK();
+  return PG_OK;
+}
+
+extern "C" int pg_expert_gemm_simt(const void* x, long long ldx, const void* sorted_src, int k, const void* w, void* y, const void* offsets, int routes, int E, int M, int K, int relu2, int is_f32,
+                                   cudaStream_t stream) {
+  if (routes == 0) return PG_OK;
+  const dim3 grid((M + 63) / 64, (routes + 63) / 64 + (E < routes ? E : routes));
+  PG_REQUIRE(M > 0 && K > 0 && grid.y <= 65535u, "expert_gemm_simt: %d routes, %d x %d", routes, M, K);
+#define PG_EG(T) launch_pdl(expert_gemm_simt_kernel<T>, grid, dim3(256), (size_t)0, stream, (const T*)x, ldx, (const int*)sorted_src, k, (const T*)w, (T*)y, (const int*)offsets, E, M, K, relu2)
+  PG_CUDA(is_f32 ? PG_EG(float) : PG_EG(bf16));
+#undef PG_EG
   PG_LAUNCH_CHECK();
   return PG_OK;
 }

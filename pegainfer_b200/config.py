@@ -21,8 +21,10 @@ from typing import Optional
 @dataclass(frozen=True)
 class MixerSpec:
     """Token mixer of one layer, for families whose layers are listed one by one.  ``kind``: ``"attention"`` (all fields but
-    the recurrent ones), ``"lightning"`` (fixed decay per head) or ``"channel_delta"`` (gated delta rule with a decay per key
-    channel; ``conv`` taps, low-rank decay and output-gate projections of the given ranks)."""
+    the recurrent and latent ones), ``"lightning"`` (fixed decay per head), ``"channel_delta"`` (gated delta rule with a decay
+    per key channel; ``conv`` taps, low-rank decay and output-gate projections of the given ranks) or ``"latent"`` (attention
+    over a cached latent of ``kv_rank`` columns and, with ``rot_dims``, a shared rotated key part; queries through a latent of
+    ``q_rank``; a sliding window and an element-wise output gate are optional)."""
 
     kind: str
     heads: int
@@ -38,17 +40,36 @@ class MixerSpec:
     conv: int = 0
     decay_rank: int = 0
     gate_rank: int = 0
+    q_rank: int = 0
+    kv_rank: int = 0
+    window: int = 0  # a position sees itself and the window - 1 before it (0: all before it)
+    out_gate: bool = False
+    yarn: tuple = ()  # (factor, original, fast, slow) of the rotation, or none
+
+
+@dataclass(frozen=True)
+class ExpertsSpec:
+    """Mixture-of-experts feed-forward: softmax scores over ``experts``, the ``top`` best of the ``keep`` best of ``groups``
+    groups of neighbours (a group counts as its best expert), weights not renormalised; an expert of width ``ff`` is an up
+    projection, the squared ReLU and a down projection."""
+
+    experts: int
+    top: int
+    ff: int
+    groups: int = 1
+    keep: int = 1
 
 
 @dataclass(frozen=True)
 class LayerSpec:
     mixer: MixerSpec
     ff: int = 0  # width of the SwiGLU feed-forward (0: the layer has none)
+    moe: Optional[ExpertsSpec] = None
 
 
 @dataclass
 class ModelConfig:
-    family: str = "qwen3"  # qwen3 | qwen35 | deepseek_v2 | kimi_k2 | glm_dsa | gemma4 | kimi_k3 | nemipel
+    family: str = "qwen3"  # qwen3 | qwen35 | deepseek_v2 | kimi_k2 | glm_dsa | gemma4 | kimi_k3 | nemipel | vekalorn
     vocab_size: int = 1024
     hidden_size: int = 256
     num_layers: int = 2
@@ -116,7 +137,7 @@ class ModelConfig:
     attn_res_block: int = 0
     kda_gate_rank: int = 0
     kda_gate_lower_bound: float = -5.0
-    # families whose layers are listed one by one (Nemipel line): the mixer and feed-forward of every layer, the factor on
+    # families whose layers are listed one by one (Nemipel, Vekalorn lines): the mixer and feed-forward of every layer, the factor on
     # the stream in the norm after the sum; final_logit_softcapping caps the logits
     layer_specs: tuple = ()
     postln_alpha: float = 1.0
@@ -278,6 +299,22 @@ PRESETS["nemipel-8b-shape"] = _nemipel(4096, 151936, 12288, 32, 8, 128, 32, 128,
 PRESETS["qwen35-8b-shape"] = replace(PRESETS["small-qwen35"], vocab_size=151936, hidden_size=4096, num_layers=36, num_q_heads=32, num_kv_heads=8, head_dim=128, intermediate_size=12288,
                                      layer_types=("linear_attention", "full_attention", "linear_attention") * 12, partial_rotary_factor=0.5, gdn_num_k_heads=16, gdn_num_v_heads=32, gdn_head_dim=128,
                                      max_position=131072)
+def _vekalorn(width: int, vocab: int, heads: int, q_rank: int, kv_rank: int, dim: int, rot: int, vdim: int, window: int, experts: ExpertsSpec, periods: int, **kw) -> ModelConfig:
+    """A Vekalorn stack of ``periods`` x (full latent attention with rotation and gate, two windowed layers without
+    positions), a mixture of experts in every layer."""
+    full = MixerSpec("latent", heads, dim, vdim, scale=(dim + rot) ** -0.5, rot_dims=rot, rot_base=5e4, q_rank=q_rank, kv_rank=kv_rank, out_gate=True, yarn=(16.0, 4096, 32.0, 1.0))
+    local = MixerSpec("latent", heads, dim, vdim, scale=dim ** -0.5, q_rank=q_rank, kv_rank=kv_rank, window=window)
+    layers = tuple(LayerSpec(m, moe=experts) for _ in range(periods) for m in (full, local, local))
+    base = dict(family="vekalorn", vocab_size=vocab, hidden_size=width, num_layers=len(layers), num_q_heads=heads, num_kv_heads=1, head_dim=dim + rot, intermediate_size=experts.ff * experts.top,
+                rms_eps=1e-5, qk_norm=False, layer_specs=layers, max_position=65536)
+    base.update(kw)
+    return ModelConfig(**base)
+
+
+PRESETS["tiny-vekalorn"] = _vekalorn(88, 256, 3, 40, 48, 24, 8, 32, 20, ExpertsSpec(12, 3, 24, 3, 2), 2, max_position=4096)
+PRESETS["small-vekalorn"] = _vekalorn(1024, 4096, 16, 512, 512, 128, 64, 128, 256, ExpertsSpec(16, 4, 512, 4, 2), 2, max_position=8192)
+# layers of a mid-size latent-attention mixture of experts, for benchmarks (not a released configuration)
+PRESETS["vekalorn-16b-shape"] = _vekalorn(2048, 102400, 16, 1536, 512, 128, 64, 128, 1024, ExpertsSpec(64, 6, 2112, 8, 4), 9)
 PRESETS["small-glm-fp8"] = replace(PRESETS["small-glm"], expert_quant="fp8_block128", dense_quant="fp8_block128")
 for _name in ("tiny-dsv2", "small-dsv2", "dsv2-lite"):
     if _name in PRESETS:
@@ -292,8 +329,8 @@ def preset(name: str, **overrides) -> ModelConfig:
 
 def detect_family(cfg: dict) -> str:
     """Map a ``config.json`` to a model line (exactly one line must claim it)."""
-    if cfg.get("architecture") == "Nemipel":
-        return "nemipel"
+    if cfg.get("architecture") in ("Nemipel", "Vekalorn"):
+        return cfg["architecture"].lower()
     mt = cfg.get("model_type", "")
     archs = " ".join(cfg.get("architectures", []))
     if mt in ("qwen3",) or "Qwen3ForCausalLM" in archs:
@@ -409,11 +446,72 @@ def nemipel_to_json(cfg: ModelConfig) -> dict:
     return out
 
 
+# the two mixers of the Vekalorn line by the name config.json gives them: rotated and gated, or without positions and gate
+_LATENT_TYPES = {"latent_attention": False, "latent_attention_2": True}
+
+
+def _vekalorn_from_json(cfg: dict, model_dir: Optional[str]) -> ModelConfig:
+    """``config.json`` of the Vekalorn line: sizes and constants per layer."""
+    layers = []
+    for i, entry in enumerate(cfg["layers"]):
+        m, kind = entry["mixer"], entry["type"]
+        if kind not in _LATENT_TYPES:
+            raise ValueError(f"layer {i}: no mixer of type {kind!r}")
+        rotated = _LATENT_TYPES[kind]
+        rot, yarn = (m.get("rot") or {}) if rotated else {}, ()
+        if rotated:
+            if rot.get("dims", m["rot_dim"]) != m["rot_dim"] or m["rot_dim"] % 2:
+                raise ValueError(f"layer {i}: the rotated part has {m['rot_dim']} columns, {rot.get('dims')} are to be rotated")
+            if rot.get("scaling"):
+                yarn = tuple(rot["scaling"][k] for k in ("factor", "original", "fast", "slow"))
+        window = (m.get("mask") or {}).get("size", 0)
+        if not rotated and window < 1:
+            raise ValueError(f"layer {i}: a window of {window} positions")
+        spec = MixerSpec("latent", m["heads"], m["dim"], m["vdim"], scale=float(m["scale"]), rot_dims=m["rot_dim"] if rotated else 0, rot_base=float(rot.get("base", 1e4)), q_rank=m["q_rank"],
+                         kv_rank=m["kv_rank"], window=window, out_gate=rotated, yarn=yarn)
+        mlp, moe = entry.get("mlp"), None
+        if mlp is not None:
+            if mlp.get("kind", "moe") != "moe":
+                raise ValueError(f"layer {i}: no feed-forward of kind {mlp['kind']!r}")
+            r = mlp["router"]
+            g = r.get("groups") or dict(count=1, keep=1)
+            moe = ExpertsSpec(r["experts"], r["top"], mlp["expert"]["ff"], g["count"], g["keep"])
+            if moe.experts % moe.groups or not 1 <= moe.keep <= moe.groups or not 1 <= moe.top <= moe.experts // moe.groups * moe.keep:
+                raise ValueError(f"layer {i}: {moe.top} experts from {moe.keep} of {moe.groups} groups of {moe.experts}")
+        layers.append(LayerSpec(spec, moe=moe))
+    first = layers[0].mixer
+    return ModelConfig(family="vekalorn", vocab_size=cfg["vocab"], hidden_size=cfg["width"], num_layers=len(layers), num_q_heads=first.heads, num_kv_heads=1, head_dim=first.dim + first.rot_dims,
+                       intermediate_size=max([l.moe.ff * l.moe.top for l in layers if l.moe] or [0]), rms_eps=cfg["norm"]["eps"], qk_norm=False, layer_specs=tuple(layers), max_position=131072,
+                       eos_token_ids=_eos_ids(model_dir, cfg))
+
+
+def vekalorn_to_json(cfg: ModelConfig) -> dict:
+    """The ``config.json`` that ``_vekalorn_from_json`` reads back."""
+    layers = []
+    for l in cfg.layer_specs:
+        m, e = l.mixer, l.moe
+        mix = dict(heads=m.heads, dim=m.dim, vdim=m.vdim, q_rank=m.q_rank, kv_rank=m.kv_rank, scale=m.scale)
+        if m.window:
+            mix["mask"] = dict(size=m.window)
+        if m.out_gate:
+            mix.update(rot_dim=m.rot_dims, rot=dict(dims=m.rot_dims, base=m.rot_base))
+            if m.yarn:
+                mix["rot"]["scaling"] = dict(zip(("factor", "original", "fast", "slow"), m.yarn))
+        mlp = dict(kind="moe", expert=dict(ff=e.ff), router=dict(experts=e.experts, top=e.top, groups=dict(count=e.groups, keep=e.keep))) if e else None
+        layers.append(dict(type="latent_attention_2" if m.out_gate else "latent_attention", mixer=mix, mlp=mlp))
+    out = dict(architecture="Vekalorn", vocab=cfg.vocab_size, width=cfg.hidden_size, norm=dict(eps=cfg.rms_eps), layers=layers)
+    if cfg.eos_token_ids:
+        out["eos_token_id"] = list(cfg.eos_token_ids)
+    return out
+
+
 def from_hf(cfg: dict, model_dir: Optional[str] = None) -> ModelConfig:
     family = detect_family(cfg)
     top = cfg
     if family == "nemipel":
         return _nemipel_from_json(cfg, model_dir)
+    if family == "vekalorn":
+        return _vekalorn_from_json(cfg, model_dir)
     if family == "qwen35" and "text_config" in cfg:
         cfg = cfg["text_config"]
     if family == "kimi_k2" and "text_config" in cfg:

@@ -25,7 +25,7 @@ from .contract import EngineInfo, KvCapacity
 from .driver import Engine
 
 
-F32_FAMILIES = ("nemipel",)  # lines whose kernels also run in 32-bit on the GPU
+F32_FAMILIES = ("nemipel", "vekalorn")  # lines whose kernels also run in 32-bit on the GPU
 
 
 def resolve_model_config(ecfg: EngineConfig) -> ModelConfig:
@@ -114,13 +114,14 @@ def build_engine(ecfg: EngineConfig, mcfg: Optional[ModelConfig] = None, device=
     kv = model.make_kv(nblocks, page) if hasattr(model, "make_kv") else KvBuffer(KvLayout(page_size=page, num_pages=nblocks, dtype=dtype, **model.kv_geometry()), device)
     pool = BlockPool(nblocks, page, enable_prefix_cache=not ecfg.no_prefix_cache and getattr(model, "supports_prefix_cache", True))
     max_blocks_per_seq = (max_len + page - 1) // page
-    extra = {"state_slots": ecfg.state_slots} if ecfg.state_slots else {}
+    state_slots = ecfg.state_slots if hasattr(model, "make_state") else None  # lines without recurrent state have no slots to bound
+    extra = {"state_slots": state_slots} if state_slots else {}
     executor = (model.make_executor if hasattr(model, "make_executor") else TorchExecutor)(
         model, kv, page, cuda_graph=ecfg.cuda_graph, max_decode_batch=ecfg.max_decode_batch, max_blocks_per_seq=max_blocks_per_seq, seed=ecfg.seed, **extra
     )
     scfg = SchedulerConfig(
         max_prefill_tokens=ecfg.max_prefill_tokens,
-        max_decode_batch=min(ecfg.max_decode_batch, ecfg.state_slots or ecfg.max_decode_batch),
+        max_decode_batch=min(ecfg.max_decode_batch, state_slots or ecfg.max_decode_batch),
         max_model_len=max_len,
         eos_token_ids=tuple(mcfg.eos_token_ids),
         batch_invariant=ecfg.batch_invariant,
@@ -132,7 +133,7 @@ def build_engine(ecfg: EngineConfig, mcfg: Optional[ModelConfig] = None, device=
     )
     host_tier = None
     if ecfg.kv_offload:
-        if not getattr(model, "supports_prefix_cache", True):
+        if not getattr(model, "supports_prefix_cache", True) or not getattr(model, "supports_kv_offload", True):
             raise ValueError("KV offload needs whole pages per layer slab: this model's layers have different KV row widths (or keep recurrent state)")
         from ..kv.host_tier import HostTier
 

@@ -32,6 +32,7 @@ from ..loader.sources import RandomSource, WeightSource
 from ..ops.reference import AttnMeta, pair_rope_tables
 from ..parallel.tp import SINGLE, TPContext
 from ..sched.executor import HybridExecutor
+from .layers import FusedProjection, pad8
 
 
 def nemipel_shapes(cfg: ModelConfig) -> dict:
@@ -73,32 +74,9 @@ def nemipel_source(cfg: ModelConfig, seed: int = 0, dtype=torch.bfloat16) -> Ran
     return RandomSource(nemipel_shapes(cfg), seed=seed, dtype=dtype, kind=_kind)
 
 
-def _pad8(n: int) -> int:
-    return (n + 7) // 8 * 8
-
-
-class _Fused:
-    """Matrices that read the same rows, stacked with every part padded to a multiple of 8 rows."""
-
-    def __init__(self, parts: dict):
-        self.at, rows, out = {}, 0, []
-        for name, w in parts.items():
-            self.at[name] = (rows, rows + w.shape[0])
-            out.append(w)
-            pad = _pad8(w.shape[0]) - w.shape[0]
-            if pad:
-                out.append(torch.zeros((pad, w.shape[1]), dtype=w.dtype, device=w.device))
-            rows += w.shape[0] + pad
-        self.w = torch.cat(out, 0).contiguous()
-
-    def __call__(self, x):
-        y = ops.dense(x, self.w)
-        return {n: y[:, a:b] for n, (a, b) in self.at.items()}
-
-
 @dataclass
 class AttentionPart:
-    proj: _Fused
+    proj: FusedProjection
     q_norm: torch.Tensor
     k_norm: Optional[torch.Tensor]
     cos: torch.Tensor
@@ -108,7 +86,7 @@ class AttentionPart:
 
 @dataclass
 class LightningPart:
-    proj: _Fused
+    proj: FusedProjection
     decay: torch.Tensor
     norm: torch.Tensor
     state_index: int
@@ -116,7 +94,7 @@ class LightningPart:
 
 @dataclass
 class ChannelDeltaPart:
-    proj: _Fused
+    proj: FusedProjection
     conv_cols: int  # q | k | v columns of the projection that pass the convolution (with their padding)
     conv_w: torch.Tensor
     a2: torch.Tensor
@@ -177,12 +155,12 @@ class NemipelModel:
             else:
                 self._kv_of[i] = self._kv_of[m.kv_from]
             cos, sin = self._rope_tables(m)
-            part = AttentionPart(_Fused(mat("q", "k", "v", "g") if own else mat("q", "g")), src.get(p + "q.norm", dev, f32), src.get(p + "k.norm", dev, f32) if own else None, cos, sin, self._kv_of[i])
+            part = AttentionPart(FusedProjection(mat("q", "k", "v", "g") if own else mat("q", "g")), src.get(p + "q.norm", dev, f32), src.get(p + "k.norm", dev, f32) if own else None, cos, sin, self._kv_of[i])
         elif m.kind == "lightning":
-            part = LightningPart(_Fused(mat("q", "k", "v", "g")), torch.tensor(m.decay, dtype=f32, device=dev), src.get(p + "norm", dev, f32), len(self.state_geometries))
+            part = LightningPart(FusedProjection(mat("q", "k", "v", "g")), torch.tensor(m.decay, dtype=f32, device=dev), src.get(p + "norm", dev, f32), len(self.state_geometries))
             self.state_geometries.append((m.heads, m.dim, m.vdim, 0, 0))
         elif m.kind == "channel_delta":
-            proj = _Fused(mat("q", "k", "v", "b", "a1", "g1"))
+            proj = FusedProjection(mat("q", "k", "v", "b", "a1", "g1"))
             cols = proj.at["b"][0]
             conv = torch.zeros((cols, m.conv), dtype=f32, device=dev)
             for n in ("q", "k", "v"):
@@ -195,7 +173,7 @@ class NemipelModel:
         L = NemipelLayer(m, part, src.get(p + "o", dev, dt), src.get(f"l{i}.norm1", dev, f32))
         if spec.ff:
             q = f"l{i}.mlp."
-            pad = _pad8(spec.ff) - spec.ff  # zero rows: their activations are zero
+            pad = pad8(spec.ff) - spec.ff  # zero rows: their activations are zero
             g, u = (torch.nn.functional.pad(src.get(q + n, dev, dt), (0, 0, 0, pad)) for n in ("gate", "up"))
             L.gate_up = torch.stack((g, u), 1).reshape(-1, g.shape[1]).contiguous() if self.interleaved else torch.cat((g, u), 0)
             L.down = torch.nn.functional.pad(src.get(q + "down", dev, dt), (0, pad)).contiguous()

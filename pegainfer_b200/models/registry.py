@@ -54,12 +54,20 @@ def _nemipel(cfg, **kw):
     return NemipelModel(cfg, **kw)
 
 
-BUILDERS = {"nemipel": _nemipel, "kimi_k3": _k3, "gemma4": _gemma4, "glm_dsa": _glm_dsa, "qwen3": _qwen3, "qwen35": _qwen35, "deepseek_v2": _mla_moe, "kimi_k2": _mla_moe}
+def _vekalorn(cfg, **kw):
+    from .vekalorn import VekalornModel
+
+    kw.pop("ep", None)
+    return VekalornModel(cfg, **kw)
+
+
+BUILDERS = {"vekalorn": _vekalorn, "nemipel": _nemipel, "kimi_k3": _k3, "gemma4": _gemma4, "glm_dsa": _glm_dsa, "qwen3": _qwen3, "qwen35": _qwen35, "deepseek_v2": _mla_moe, "kimi_k2": _mla_moe}
 
 
 # Translation units (csrc/<name>.cu) that a family's kernels come from, for programs that build only what one model needs
 KERNEL_UNITS = {
     "nemipel": ("runtime", "gemm_sm100", "gemm2sm_sm100", "elementwise", "stream32", "attention", "attention_tc", "attention_general", "kda", "lightning", "sampling"),
+    "vekalorn": ("runtime", "gemm_sm100", "gemm2sm_sm100", "elementwise", "stream32", "mla", "mla_prefill", "moe_route", "moe_gemm", "sampling"),
 }
 
 
@@ -92,6 +100,10 @@ def shapes_for(cfg: ModelConfig) -> dict:
         from .nemipel import nemipel_shapes
 
         return nemipel_shapes(cfg)
+    if cfg.family == "vekalorn":
+        from .vekalorn import vekalorn_shapes
+
+        return vekalorn_shapes(cfg)
     raise ValueError(f"no tensor-shape table for family {cfg.family!r}")
 
 

@@ -584,7 +584,7 @@ _PREFILL_TC_MIN_KV = int(os.environ.get("PEGAINFER_PREFILL_TC_MIN_KV", "512"))
 
 
 # how often each tcgen05 prefill kernel was chosen (tests assert that long prompts really take them)
-PREFILL_TC_CALLS = {"hd128": 0, "hd256": 0, "mla": 0}
+PREFILL_TC_CALLS = {"hd128": 0, "hd256": 0, "mla": 0, "latent": 0}
 
 
 def set_prefill_tc(min_kv: int) -> int:
@@ -896,6 +896,32 @@ def stream_norm(x, w, eps: float, act_dtype):
     return _post_norm(None, x, None, w, eps, 1.0, act_dtype)
 
 
+def _add_layer_norm(y, pos, weights, x, w, eps, act_dtype):
+    t, width = weights.shape[0] if weights is not None else y.shape[0], y.shape[1]
+    assert w.dtype == torch.float32 and y.stride(1) == 1 and (x is None or (x.dtype == torch.float32 and x.is_contiguous() and x.shape == (t, width)))
+    f32 = act_dtype == torch.float32
+    xt = x if f32 and x is not None else torch.empty((t, width), dtype=act_dtype, device=y.device)
+    _check(lib().pg_add_layer_norm(_ptr(y), _ci(_is_f32(y)), _ll(y.stride(0)), _ptr(pos), _ptr(weights), _ci(weights.shape[1] if weights is not None else 0), _ptr(x), _ptr(w),
+                                   _vp(0) if xt is x else _ptr(xt), _ci(int(f32)), _ll(xt.stride(0)), _ci(t), _ci(width), _cf(eps), _stream()), ctx(y.device))
+    return xt
+
+
+def add_layer_norm(y, x, w, eps: float, act_dtype):
+    """``x += layer_norm(y) * w`` on the f32 stream, in place; returns the activation-dtype copy."""
+    return _add_layer_norm(y, None, None, x, w, eps, act_dtype)
+
+
+def add_layer_norm_rows(rows, pos, weights, x, w, eps: float, act_dtype):
+    """``add_layer_norm`` of the weighted sums of the tokens' expert rows, which are formed in the same kernel."""
+    assert weights.dtype == torch.float32 and weights.is_contiguous() and pos.dtype == torch.int32
+    return _add_layer_norm(rows, pos, weights, x, w, eps, act_dtype)
+
+
+def stream_layer_norm(x, w, eps: float, act_dtype):
+    """Layer norm of the f32 stream in the activation dtype."""
+    return _add_layer_norm(x, None, None, None, w, eps, act_dtype)
+
+
 def gated_row_norm(x, gate, w, eps: float):
     """``rms_norm(x) * w * sigmoid(gate)`` over the last axis of ``x`` [T, H, D]; ``gate`` [T, H * D], unit column stride."""
     t, h, d = x.shape
@@ -1086,7 +1112,7 @@ def decay_attention(q, k, v, decay, state, meta: AttnMeta, chunked: Optional[boo
 # ----------------------------------------------------------------------------------
 # mixture of experts
 # ----------------------------------------------------------------------------------
-def router_topk(logits, top_k, scoring="softmax", bias=None, n_group=1, topk_group=1, norm_topk_prob=False, scale=1.0):
+def router_topk(logits, top_k, scoring="softmax", bias=None, n_group=1, topk_group=1, norm_topk_prob=False, scale=1.0, group_top=2):
     assert logits.dtype == torch.float32 and logits.stride(-1) == 1
     t, e = logits.shape
     ids = torch.empty((t, top_k), dtype=torch.int32, device=logits.device)
@@ -1094,7 +1120,7 @@ def router_topk(logits, top_k, scoring="softmax", bias=None, n_group=1, topk_gro
     c = ctx(logits.device)
     b = bias.float().contiguous() if bias is not None else None
     rc = lib().pg_router_topk(_ptr(logits), _ll(logits.stride(0)), _ptr(b), _ptr(ids), _ptr(w), _ci(t), _ci(e), _ci(top_k), _ci(int(scoring == "sigmoid")), _ci(n_group),
-                              _ci(topk_group), _ci(int(norm_topk_prob)), _cf(scale), _stream())
+                              _ci(topk_group), _ci(group_top), _ci(int(norm_topk_prob)), _cf(scale), _stream())
     _check(rc, c)
     return ids, w
 
@@ -1152,9 +1178,10 @@ def repack_int4_pairs(packed):
     return out
 
 
-def grouped_gemm(xs, offsets, w, scales=None, bn: int = 16):
+def grouped_gemm(xs, offsets, w, scales=None, bn: int = 16, relu2: bool = False):
     """``xs`` [rows, K] sorted by expert; ``w`` bf16 [E, M, K], packed int32 [E, M, K/8] with bf16
-    scales [E, M, K/32], or FP8 e4m3 [E, M, K] with f32 ``scale_inv`` [E, ceil(M/128), ceil(K/128)]."""
+    scales [E, M, K/32], or FP8 e4m3 [E, M, K] with f32 ``scale_inv`` [E, ceil(M/128), ceil(K/128)].  ``relu2``: the squared
+    ReLU of the result (bf16 weights)."""
     rows, k = xs.shape
     e, m = w.shape[0], w.shape[1]
     mode = quant_code(w)
@@ -1165,6 +1192,10 @@ def grouped_gemm(xs, offsets, w, scales=None, bn: int = 16):
         assert scales.dtype == torch.float32 and scales.shape == (e, (m + 127) // 128, (k + 127) // 128), "FP8 experts need f32 scale_inv per 128x128 block"
     y = torch.empty((rows, m), dtype=torch.bfloat16, device=xs.device)
     c = ctx(xs.device)
+    if relu2:
+        assert mode == 0, "the squared ReLU is wired for bf16 expert weights"
+        _check(lib().pg_moe_grouped_gemm_relu2(_ptr(xs), _ll(xs.stride(0)), _ll(rows), _ptr(w), _ptr(y), _ll(y.stride(0)), _ptr(offsets), _ci(e), _ci(m), _ci(k), _ci(bn), _ptr(c.status), _stream()), c)
+        return y
     rc = lib().pg_moe_grouped_gemm(_ptr(xs), _ll(xs.stride(0)), _ll(rows), _ptr(w), _ptr(scales), _ci(mode), _ptr(y), _ll(y.stride(0)), _ptr(offsets), _ci(e), _ci(m),
                                    _ci(k), _ci(bn), _ptr(c.status), _stream())
     _check(rc, c)
@@ -1188,7 +1219,8 @@ def grouped_gemm_fp8(xq, x_scale, offsets, w_fp8, w_scale, bn: int = 16):
     return y
 
 
-def _moe_pipeline(x, ids, weights, w13, s13, w2, s2, expert_offset, act: str = "swiglu"):
+def _routed_rows(x, ids, w13, s13, w2, s2, expert_offset, act: str):
+    """Expert outputs of all local routes, sorted by expert, and every route's row among them."""
     _bf16(x)
     t, h = x.shape
     k = ids.shape[1]
@@ -1199,19 +1231,43 @@ def _moe_pipeline(x, ids, weights, w13, s13, w2, s2, expert_offset, act: str = "
     xs = torch.empty((routes, h), dtype=x.dtype, device=x.device)
     _check(lib().pg_moe_gather(_ptr(x), _ll(x.stride(0)), _ptr(sorted_src), _ptr(offsets), _ci(e_local), _ci(k), _ptr(xs), _ci(h), _ci(routes), _stream()), c)
     bn = _token_tile(routes, e_local)
-    assert act == "swiglu" or quant_code(w13) == 0, "the situ activation is wired for bf16 expert weights"
+    assert act == "swiglu" or quant_code(w13) == 0, "the situ and squared ReLU activations are wired for bf16 expert weights"
     if quant_code(w13) == 2 and _MOE_FP8_TC and h % 128 == 0 and w13.shape[1] % 256 == 0 and w2.shape[1] % 128 == 0:
         # both GEMMs on the FP8 tensor-core path: activations quantised per row and 128-wide k group
         xq, xsc = quant_fp8_1x128(xs)
         aq, asc = swiglu_quant_fp8_1x128(grouped_gemm_fp8(xq, xsc, offsets, w13, s13, bn))
-        y2 = grouped_gemm_fp8(aq, asc, offsets, w2, s2, bn)
+        return grouped_gemm_fp8(aq, asc, offsets, w2, s2, bn), route_pos
+    if act == "relu2":
+        mid = grouped_gemm(xs, offsets, w13, None, bn, relu2=True)
     else:
         y1 = grouped_gemm(xs, offsets, w13, s13, bn)
         mid = situ(y1) if act == "situ" else swiglu(y1)
-        y2 = grouped_gemm(mid, offsets, w2, s2, bn)
+    return grouped_gemm(mid, offsets, w2, s2, bn), route_pos
+
+
+def _moe_pipeline(x, ids, weights, w13, s13, w2, s2, expert_offset, act: str = "swiglu"):
+    (t, h), k = x.shape, ids.shape[1]
+    y2, route_pos = _routed_rows(x, ids, w13, s13, w2, s2, expert_offset, act)
     out = torch.empty((t, h), dtype=torch.float32, device=x.device)
-    _check(lib().pg_moe_combine(_ptr(y2), _ll(y2.stride(0)), _ptr(route_pos), _ptr(weights.contiguous()), _ci(t), _ci(k), _ptr(out), _ci(h), _ci(0), _stream()), c)
+    _check(lib().pg_moe_combine(_ptr(y2), _ll(y2.stride(0)), _ptr(route_pos), _ptr(weights.contiguous()), _ci(t), _ci(k), _ptr(out), _ci(h), _ci(0), _stream()), ctx(x.device))
     return out
+
+
+def expert_rows(x, ids, w1, w2, act: str = "relu2"):
+    """Unweighted expert outputs of every route and their rows (``reference.expert_rows``); f32 and sizes that TMA cannot
+    address run on the CUDA-core grouped GEMM (squared ReLU only)."""
+    (t, h), k, (e, inter) = x.shape, ids.shape[1], w1.shape[:2]
+    f32 = _is_f32(x)
+    if not f32 and h % 8 == 0 and inter % 8 == 0:
+        return _routed_rows(x, ids, w1, None, w2, None, 0, act)
+    assert act == "relu2" and x.stride(1) == 1 and w1.dtype == w2.dtype == x.dtype and w1.is_contiguous() and w2.is_contiguous()
+    offsets, sorted_src, route_pos = moe_route_plan(ids, 0, e)
+    c = ctx(x.device)
+    mid = torch.empty((t * k, inter), dtype=x.dtype, device=x.device)
+    out = torch.empty((t * k, h), dtype=x.dtype, device=x.device)
+    _check(lib().pg_expert_gemm_simt(_ptr(x), _ll(x.stride(0)), _ptr(sorted_src), _ci(k), _ptr(w1), _ptr(mid), _ptr(offsets), _ci(t * k), _ci(e), _ci(inter), _ci(h), _ci(1), _ci(f32), _stream()), c)
+    _check(lib().pg_expert_gemm_simt(_ptr(mid), _ll(inter), _vp(0), _ci(1), _ptr(w2), _ptr(out), _ptr(offsets), _ci(t * k), _ci(e), _ci(h), _ci(inter), _ci(0), _ci(f32), _stream()), c)
+    return out, route_pos
 
 
 def moe_experts(x, ids, weights, w13, w2, expert_offset=0, act: str = "swiglu"):
@@ -1409,6 +1465,120 @@ def mla_attention(q: "_MlaQ", w_uk, w_uv, latent_layer, meta: AttnMeta, scale, k
     vdim = w_uv.shape[1]
     out = torch.empty((t, h * vdim), dtype=torch.bfloat16, device=dev)
     _check(lib().pg_permute_021(_ptr(v_hm), _ptr(out), _ci(h), _ci(t), _ci(vdim), _stream()), c)
+    return out
+
+
+def latent_rows(zq, zkv, q_norm_w, kv_norm_w, cos, sin, meta: AttnMeta, cache, latent: int, eps: float):
+    """Query latent and cache rows of a latent attention layer (``reference.latent_rows``); ``zq`` and ``zkv`` are column
+    slices of one fused projection."""
+    t, qr = zq.shape
+    rot = zkv.shape[1] - latent
+    ld = _same_rows(zq, zkv)
+    assert zq.stride(1) == zkv.stride(1) == 1 and zq.dtype == zkv.dtype == cache.dtype and q_norm_w.dtype == kv_norm_w.dtype == torch.float32
+    assert cache.is_contiguous() and cache.shape[1] == meta.page_size * (latent + rot) and (rot == 0 or (cos.dtype == torch.float32 and 2 * cos.shape[1] == rot))
+    cq = torch.empty((t, qr), dtype=zq.dtype, device=zq.device)
+    c = ctx(zq.device)
+    _check(lib().pg_latent_rows(_ptr(zq), _ptr(zkv), _ll(ld), _ptr(q_norm_w), _ptr(kv_norm_w), _ptr(cos if rot else None), _ptr(sin if rot else None), _ptr(meta.positions), _ptr(meta.slot_mapping), _ptr(cq),
+                                _ptr(cache), _ci(t), _ci(qr), _ci(latent), _ci(rot), _ci(cos.shape[0] if rot else 0), _ll(cache.shape[0] * meta.page_size), _cf(eps), _ci(_is_f32(zq)), _ptr(c.status),
+                                _stream()), c)
+    return cq
+
+
+def _head_gemm(x, x_tok: int, x_head: int, w, y, gate=None):
+    """``y[t, h, :] = x[t, h, :] @ w[h].T`` (times ``sigmoid(gate[t, h, :])``); ``x`` a data pointer holder read by strides,
+    ``w`` [heads, M, K], ``y`` [rows, heads, M], ``gate`` [rows, heads * M] with any row stride."""
+    rows, heads, m = y.shape
+    k = w.shape[2]
+    c = ctx(y.device)
+    args = (_ptr(x), _ll(x_tok), _ll(x_head), _ptr(w), _ptr(y), _ll(heads * m), _ll(m), _ptr(gate), _ll(gate.stride(0) if gate is not None else 0), _ll(m), _ci(heads), _ci(rows), _ci(m), _ci(k))
+    if y.dtype == torch.bfloat16 and k % 8 == 0 and x_tok % 8 == 0 and x_head % 8 == 0 and x.data_ptr() % 16 == 0 and heads <= 512:
+        _check(lib().pg_head_gemm(*args, _ci(_token_tile(heads * rows, heads)), _ptr(c.status), _stream()), c)
+    else:
+        _check(lib().pg_head_gemm_simt(*args, _ci(_is_f32(y)), _stream()), c)
+
+
+def _latent_key_plan(meta: AttnMeta, n: int, window: int, device):
+    """Dense key rows of the step's first ``n`` sequences: row offsets, first positions and counts (device), their total;
+    with a window only the keys that some row of the sequence sees.  Made once per step and window."""
+    plans = meta.__dict__.setdefault("_pg_latent_plans", {})
+    key = (n, window)
+    if key not in plans:
+        qi, kvl = meta.h_q_indptr, meta.h_kv_lens
+        first = [max(0, kvl[b] - (qi[b + 1] - qi[b]) - window + 1) if window else 0 for b in range(n)]
+        ind = [0]
+        for b in range(n):
+            ind.append(ind[-1] + kvl[b] - first[b])
+        host = torch.tensor(ind + first + [kvl[b] - first[b] for b in range(n)], dtype=torch.int32).pin_memory()
+        dev = host.to(device, non_blocking=True)
+        plans[key] = (dev[: n + 1], dev[n + 1 : 2 * n + 1], dev[2 * n + 1 :], ind[-1], host)
+    return plans[key][:4]
+
+
+def latent_attention(q, uk_t, uv, ukv, cache, meta: AttnMeta, rot: int, scale: float, window: int = 0, cos=None, sin=None, gate=None):
+    """Latent attention over the paged cache (``reference.latent_attention``).  Long prompt portions of heads up to
+    128 + 64 / 128 columns run in the expanded form on tcgen05, single rows and short portions in the absorbed form on the
+    split-KV kernel (latents up to 512 + 64), f32 and other sizes on the CUDA-core kernel."""
+    heads, lat, dim = uk_t.shape
+    vdim, t = uv.shape[1], q.shape[0]
+    f32, dev = _is_f32(q), q.device
+    assert q.is_contiguous() and q.shape[1] == heads * (dim + rot) and uk_t.is_contiguous() and uv.is_contiguous() and cache.is_contiguous() and cache.dtype == q.dtype
+    assert cache.shape[1] == meta.page_size * (lat + rot) and (gate is None or (gate.dtype == q.dtype and gate.stride(1) == 1 and gate.shape == (t, heads * vdim)))
+    out = torch.empty((t, heads * vdim), dtype=q.dtype, device=dev)
+    if t == 0:
+        return out
+    c = ctx(dev)
+    max_pos = cos.shape[0] if rot else 0
+    cos, sin = (cos, sin) if rot else (None, None)
+    table, ps, qd = meta.block_table, meta.page_size, dim + rot
+    qi, kvl = meta.h_q_indptr, meta.h_kv_lens
+    aligned = not f32 and lat % 8 == 0 and rot % 8 == 0 and ps in (16, 32, 64)
+
+    n_pf = 0  # leading sequences in the expanded form: the prompt portions in front of the step's single rows
+    if aligned and not meta.decode_only and _PREFILL_TC and not _BATCH_INVARIANT and qi is not None and kvl is not None and dim % 8 == 0 and vdim % 8 == 0 and dim <= 128 and rot <= 64 and vdim <= 128 \
+            and (gate is None or (gate.data_ptr() % 16 == 0 and gate.stride(0) % 8 == 0)):
+        n_pf = meta.num_seqs
+        while n_pf > 0 and qi[n_pf] - qi[n_pf - 1] == 1:
+            n_pf -= 1
+        if n_pf and (max(qi[b + 1] - qi[b] for b in range(n_pf)) < _PREFILL_TC_MIN_ROWS or max(kvl[:n_pf]) < _PREFILL_TC_MIN_KV):
+            n_pf = 0
+    row0 = qi[n_pf] if n_pf else 0
+    if n_pf:
+        PREFILL_TC_CALLS["latent"] += 1
+        kv_indptr, starts, lens, total = _latent_key_plan(meta, n_pf, window, dev)
+        dense_rows = torch.empty((total, lat + rot), dtype=q.dtype, device=dev)
+        _check(lib().pg_latent_gather(_ptr(cache), _ci(ps), _ll(cache.shape[0]), _ci(lat + rot), _ptr(table), _ci(table.stride(0)), _ptr(kv_indptr), _ptr(starts), _ci(n_pf), _ci(total), _ptr(dense_rows),
+                                      _ptr(c.status), _stream()), c)
+        kv = linear(dense_rows[:, :lat], ukv)  # [total, heads * dim keys | heads * vdim values]
+        if rot:
+            _check(lib().pg_rotate_pairs(_ptr(q[:, dim:]), _ll(heads * qd), _ll(qd), _ptr(cos), _ptr(sin), _ptr(meta.positions), _ci(row0), _ci(heads), _ci(rot), _ci(max_pos), _ci(0), _stream()), c)
+        rc = lib().pg_latent_prefill_tc(_ptr(q), _ll(heads * qd), _ll(qd), _ptr(q[:, dim:]), _ll(heads * qd), _ll(qd), _ptr(kv), _ptr(kv[:, heads * dim :]), _ll(kv.stride(0)),
+                                        _ptr(dense_rows[:, lat:] if rot else None), _ll(lat + rot), _ptr(gate), _ll(gate.stride(0) if gate is not None else 0), _ptr(out), _ptr(meta.q_indptr),
+                                        _ptr(kv_indptr), _ptr(lens), _ci(n_pf), _ci(row0), _ci(total), _ci(heads), _ci(dim), _ci(rot), _ci(vdim), _cf(scale), _ci(window),
+                                        _ci(sum((qi[b + 1] - qi[b] + 255) // 256 for b in range(n_pf))), _ptr(c.status), _stream())
+        _check(rc, c)
+        if row0 == t:
+            return out
+    # absorbed form for the rows from row0 on
+    n = t - row0
+    qs = q[row0:]
+    q_abs = torch.empty((n, heads, lat), dtype=q.dtype, device=dev)
+    _head_gemm(qs, heads * qd, qd, uk_t, q_abs)
+    o = torch.empty((n, heads, lat), dtype=q.dtype, device=dev)
+    strides = (_ll(heads * lat), _ll(lat))
+    pe = (_ptr(qs[:, dim:] if rot else None), _ll(heads * qd), _ll(qd), _ptr(cos), _ptr(sin), _ci(max_pos))
+    where = (_ptr(cache), _ptr(o), *strides, _ptr(meta.q_indptr), _ptr(meta.kv_lens), _ptr(table), _ci(table.stride(0)), _ptr(_unit_seq(meta, dev)))
+    if aligned and lat <= 512 and rot <= 64:
+        longest = max(meta.max_kv_len, 1)
+        longest = min(longest, window + 31) if window else min(longest, 4096)
+        splits = max(1, min(16, (4 * c.sms) // (n * ((heads + 15) // 16)), (longest + 127) // 128))
+        splits = max(1, min(splits, c.attn_part.numel() // (n * heads * (lat + 1) * 4)))
+        rc = lib().pg_latent_attention(_ptr(q_abs), *strides, *pe, *where, _ci(row0), _ci(meta.num_seqs), _ci(n), _ci(heads), _ci(lat), _ci(rot), _ci(ps), _cf(scale), _ci(window), _ci(splits),
+                                       _ptr(c.attn_part), _ptr(c.attn_part[n * heads * splits * lat * 4 :]), _stream())
+        _check(rc, c, 2 if splits > 1 else 1)
+    else:
+        assert row0 == 0
+        _check(lib().pg_latent_attention_plain(_ptr(q_abs), *strides, *pe, *where, _ci(n), _ci(heads), _ci(lat), _ci(rot), _ci(ps), _cf(scale), _ci(window), _ci(f32), _stream()), c)
+    _head_gemm(o, heads * lat, lat, uv, out[row0:].view(n, heads, vdim), gate[row0:] if gate is not None else None)
     return out
 
 

@@ -101,6 +101,30 @@ def stream_norm(x, w, eps: float, act_dtype):
     return (x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps) * w.float()).to(act_dtype)
 
 
+def _layer_norm(y, w, eps: float):
+    d = y - y.mean(-1, keepdim=True)
+    return d * torch.rsqrt(d.pow(2).mean(-1, keepdim=True) + eps) * w.float()
+
+
+def add_layer_norm(y, x, w, eps: float, act_dtype):
+    """Norm before the sum, in f32: ``x += layer_norm(y) * w`` (in place on the f32 stream ``x``; mean and variance of the
+    row, no bias); returns the copy in the activation dtype.  ``y`` is a sublayer's output, f32 or the activation dtype."""
+    x.add_(_layer_norm(y.float(), w, eps))
+    return x.to(act_dtype)
+
+
+def add_layer_norm_rows(rows, pos, weights, x, w, eps: float, act_dtype):
+    """``add_layer_norm`` of the weighted sum of every token's expert rows (``expert_rows``): ``y[t] = sum_j weights[t, j] *
+    rows[pos[t, j]]``."""
+    t, k = weights.shape
+    return add_layer_norm((rows.float()[pos.long()].view(t, k, -1) * weights.unsqueeze(-1)).sum(1), x, w, eps, act_dtype)
+
+
+def stream_layer_norm(x, w, eps: float, act_dtype):
+    """Layer norm of the f32 stream in the activation dtype (the stream is left as it is)."""
+    return _layer_norm(x, w, eps).to(act_dtype)
+
+
 def gated_row_norm(x, gate, w, eps: float):
     """``rms_norm(x) * w * sigmoid(gate)`` over the last axis of ``x`` [T, H, D], rounded once; ``gate`` [T, H * D] may be a
     column slice of a wider projection."""
@@ -320,11 +344,19 @@ def qk_norm_rope_append(qkv, q_norm_w, k_norm_w, cos, sin, meta: AttnMeta, kv_la
 # ----------------------------------------------------------------------------------
 # attention
 # ----------------------------------------------------------------------------------
-def pair_rope_tables(max_pos: int, rotary_dim: int, theta: float, device="cpu"):
-    """f32 cos / sin ``[max_pos, rotary_dim / 2]``; the angles ``p * theta^(-2 i / rotary_dim)`` are formed in f64."""
+def pair_rope_tables(max_pos: int, rotary_dim: int, theta: float, device="cpu", yarn: tuple = ()):
+    """f32 cos / sin ``[max_pos, rotary_dim / 2]``; the angles ``p * theta^(-2 i / rotary_dim)`` are formed in f64.  ``yarn``
+    ``(factor, original, fast, slow)``: YaRN frequencies, and the attention factor ``0.1 ln(factor) + 1`` on both tables."""
     inv = theta ** (-torch.arange(0, rotary_dim, 2, dtype=torch.float64) / max(rotary_dim, 1))
+    gain = 1.0
+    if yarn:
+        factor, original, fast, slow = yarn
+        at = lambda turns: rotary_dim * math.log(original / (2 * math.pi * turns)) / (2 * math.log(theta))
+        lo, hi = max(math.floor(at(fast)), 0), min(math.ceil(at(slow)), rotary_dim - 1)
+        ramp = ((torch.arange(rotary_dim // 2, dtype=torch.float64) - lo) / max(hi - lo, 0.001)).clamp(0, 1)
+        inv, gain = inv / factor * ramp + inv * (1 - ramp), 0.1 * math.log(factor) + 1
     ang = torch.outer(torch.arange(max_pos, dtype=torch.float64), inv)
-    return ang.cos().float().to(device), ang.sin().float().to(device)
+    return (ang.cos() * gain).float().to(device), (ang.sin() * gain).float().to(device)
 
 
 def _pages_kv(kv_layer, kv_heads: int, dim: int, vdim: int, page_size: int):
@@ -498,13 +530,13 @@ def sample(logits, temperature, top_k, top_p, min_p, u):
 # ----------------------------------------------------------------------------------
 # MoE routing and experts
 # ----------------------------------------------------------------------------------
-def router_topk(logits, top_k, scoring="softmax", bias=None, n_group=1, topk_group=1, norm_topk_prob=False, scale=1.0):
+def router_topk(logits, top_k, scoring="softmax", bias=None, n_group=1, topk_group=1, norm_topk_prob=False, scale=1.0, group_top=2):
     """Expert selection.  ``logits`` [T, E] f32.  Returns (ids int32 [T,k], weights f32 [T,k]).
 
     softmax: probabilities over all experts, top-k by probability.
-    sigmoid: scores = sigmoid(logits); selection on ``scores + bias`` restricted to the
-    ``topk_group`` best of ``n_group`` expert groups (group score = sum of its two best
-    biased scores); weights come from the un-biased scores.
+    sigmoid: scores = sigmoid(logits).  Selection on ``scores + bias`` restricted to the
+    ``topk_group`` best of ``n_group`` expert groups (group score = sum of its ``group_top``,
+    1 or 2, best biased scores); weights come from the un-biased scores.
     Ties resolve to the lowest expert id; ids are returned in selection order
     (descending score).  Weights are renormalised to sum 1 when ``norm_topk_prob`` and
     multiplied by ``scale``."""
@@ -514,7 +546,7 @@ def router_topk(logits, top_k, scoring="softmax", bias=None, n_group=1, topk_gro
     choice = scores + bias.float() if bias is not None else scores
     if n_group > 1:
         g = choice.view(t, n_group, e // n_group)
-        gscore = g.topk(min(2, e // n_group), dim=-1).values.sum(-1)
+        gscore = g.topk(min(group_top, e // n_group), dim=-1).values.sum(-1)
         # stable: prefer lower group index on ties
         order = torch.argsort(-gscore, dim=-1, stable=True)[:, :topk_group]
         gmask = torch.zeros(t, n_group, dtype=torch.bool, device=lf.device).scatter_(1, order, True)
@@ -609,7 +641,8 @@ def moe_experts(x, ids, weights, w13, w2, expert_offset=0, act: str = "swiglu"):
     """Routed experts on local weights.  ``w13`` [E_local, 2I, H] (gate rows then up
     rows), ``w2`` [E_local, H, I].  Tokens routed to experts outside
     [expert_offset, expert_offset + E_local) contribute nothing.  Returns f32 [T, H]
-    (sum over the local selections of weight * expert(x)).  ``act``: ``swiglu`` or ``situ``."""
+    (sum over the local selections of weight * expert(x)).  ``act``: ``swiglu`` or ``situ``, or ``relu2`` (squared ReLU of
+    ``w13`` [E_local, I, H], no gate rows)."""
     t, h = x.shape
     e_local = w13.shape[0]
     out = torch.zeros(t, h, dtype=torch.float32, device=x.device)
@@ -619,11 +652,28 @@ def moe_experts(x, ids, weights, w13, w2, expert_offset=0, act: str = "swiglu"):
         if rows.numel() == 0:
             continue
         xe = x[rows]
-        mid = situ(linear(xe, w13[e])) if act == "situ" else swiglu(linear(xe, w13[e]))
-        ye = linear(mid, w2[e]).float()
+        ye = linear(_expert_act(linear(xe, w13[e], torch.float32) if act == "relu2" else linear(xe, w13[e]), act).to(x.dtype), w2[e]).float()
         we = (weights * sel.float()).sum(-1)[rows]
         out.index_add_(0, rows, ye * we.unsqueeze(-1))
     return out
+
+
+def _expert_act(y, act: str):
+    return torch.relu(y).square() if act == "relu2" else situ(y) if act == "situ" else swiglu(y)
+
+
+def expert_rows(x, ids, w1, w2, act: str = "relu2"):
+    """Every route's expert output, not yet weighted: ``(rows [T * k, H], pos int32 [T * k])`` with the output of choice ``j``
+    of token ``t`` in row ``pos[t * k + j]``.  Weights as in ``moe_experts``; the sum is left to ``add_layer_norm_rows``."""
+    t, k = ids.shape
+    rows = torch.zeros(t * k, w2.shape[1], dtype=x.dtype, device=x.device)
+    flat = ids.reshape(-1)
+    for e in range(w1.shape[0]):
+        at = (flat == e).nonzero().flatten()
+        if at.numel():
+            xe = x[at // k]
+            rows[at] = linear(_expert_act(linear(xe, w1[e], torch.float32) if act == "relu2" else linear(xe, w1[e]), act).to(x.dtype), w2[e])
+    return rows, torch.arange(t * k, dtype=torch.int32, device=x.device)
 
 
 # ----------------------------------------------------------------------------------
@@ -676,6 +726,60 @@ def mla_attention(q, w_uk, w_uv, latent_layer, meta: AttnMeta, scale, kv_lora):
         lo = torch.einsum("hqk,kc->qhc", p, ckv).to(q.dtype)
         out[q0:q1] = torch.einsum("qhc,hvc->qhv", lo.float(), w_uv.float()).to(q.dtype)
     return out.reshape(t, h * v)
+
+
+def _turn_pairs(x, cos, sin):
+    """Rotation of neighbouring pairs of the last axis of ``x`` [T, heads, R] by f32 ``cos`` / ``sin`` [T, R / 2], in f32."""
+    u, v = x[..., 0::2].float(), x[..., 1::2].float()
+    c, s = cos[:, None, :], sin[:, None, :]
+    return torch.stack((u * c - v * s, v * c + u * s), -1).flatten(-2)
+
+
+def latent_rows(zq, zkv, q_norm_w, kv_norm_w, cos, sin, meta: AttnMeta, cache, latent: int, eps: float):
+    """The token rows of a latent attention layer: returns the RMS-normed query latent of ``zq`` [T, q_rank] and appends to
+    the paged cache (``[pages, page_size * (latent + R)]``) the RMS-normed first ``latent`` columns of ``zkv`` and its last
+    ``R`` columns rotated in pairs.  ``cos`` / ``sin`` f32 [max_pos, R / 2], ``None`` without rotated columns."""
+    rms = lambda y, w: y.float() * torch.rsqrt(y.float().pow(2).mean(-1, keepdim=True) + eps) * w.float()
+    row = [rms(zkv[:, :latent], kv_norm_w)]
+    if zkv.shape[1] > latent:
+        pos = meta.positions.long()
+        row.append(_turn_pairs(zkv[:, None, latent:], cos[pos], sin[pos])[:, 0])
+    cache.view(-1, zkv.shape[1])[meta.slot_mapping.long()] = torch.cat(row, -1).to(cache.dtype)
+    return rms(zq, q_norm_w).to(zq.dtype)
+
+
+def latent_attention(q, uk_t, uv, ukv, cache, meta: AttnMeta, rot: int, scale: float, window: int = 0, cos=None, sin=None, gate=None):
+    """Latent attention over the paged cache of ``latent_rows``.  ``q`` [T, heads * (dim + rot)] per head unrotated columns,
+    then the columns that are rotated here (and in place, if at all); ``uk_t`` [heads, latent, dim] and ``uv`` [heads, vdim,
+    latent] up-projections of keys and values, ``ukv`` [heads * (dim + vdim), latent] the same stacked for the expanded form;
+    a row sees its last ``window`` keys (0: all).  ``gate`` [T, heads * vdim]: its sigmoid multiplies the output."""
+    heads, c, dim = uk_t.shape
+    vdim, t = uv.shape[1], q.shape[0]
+    q = q.view(t, heads, dim + rot)
+    rows = cache.view(-1, c + rot)
+    qa = torch.einsum("thd,hcd->thc", q[..., :dim].float(), uk_t.float()).to(q.dtype).float()
+    if rot:
+        pos = meta.positions.long()
+        qa = torch.cat((qa, _turn_pairs(q[..., dim:], cos[pos], sin[pos]).to(q.dtype).float()), -1)
+    lat = torch.zeros(t, heads, c, dtype=q.dtype, device=q.device)
+    qi = meta.h_q_indptr if meta.h_q_indptr is not None else meta.q_indptr.tolist()
+    kvl = meta.h_kv_lens if meta.h_kv_lens is not None else meta.kv_lens.tolist()
+    ps = meta.page_size
+    for b in range(meta.num_seqs):
+        q0, q1, n = qi[b], qi[b + 1], kvl[b]
+        if n == 0 or q1 == q0:
+            continue
+        at = torch.arange(n, device=q.device)
+        k = rows[meta.block_table[b].long()[at // ps] * ps + at % ps].float()
+        own = torch.arange(n - (q1 - q0), n, device=q.device)[:, None]
+        hide = (at > own) | (at <= own - window) if window else at > own
+        s = torch.einsum("thc,kc->htk", qa[q0:q1], k) * scale
+        p = torch.softmax(s.masked_fill(hide, float("-inf")), -1)
+        lat[q0:q1] = torch.einsum("htk,kc->thc", p, k[:, :c]).to(q.dtype)
+    out = torch.einsum("thc,hvc->thv", lat.float(), uv.float()).reshape(t, heads * vdim)
+    if gate is not None:
+        out = out * torch.sigmoid(gate.float())
+    return out.to(q.dtype)
 
 
 def quant_fp8_1x128(x):

@@ -282,7 +282,8 @@ class TorchExecutor(ModelExecutor):
             from ..ops import cuda as K
 
             geo = self.model.kv_geometry()
-            meta.plan = K.plan_decode_splits(len(seqs), geo["kv_heads"], min(self.max_blocks_per_seq * self.page_size, 2048), self.device)
+            if geo.get("split_plan", True):
+                meta.plan = K.plan_decode_splits(len(seqs), geo["kv_heads"], min(self.max_blocks_per_seq * self.page_size, 2048), self.device)
         return token_ids, meta
 
     def step_logits(self, batch: StepBatch, want: Sequence[Sequence[int]]) -> Optional[torch.Tensor]:

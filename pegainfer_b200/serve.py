@@ -63,6 +63,7 @@ LINES = [
     ModelLine("gemma4", ("gemma4",), frozenset()),
     ModelLine("kimi-k3", ("kimi_k3",), frozenset({"ep_backend"})),
     ModelLine("nemipel", ("nemipel",), frozenset({"dtype", "state_slots"})),
+    ModelLine("vekalorn", ("vekalorn",), frozenset({"dtype"})),
 ]
 LINES[0].validate = _qwen3_validate  # type: ignore[method-assign]
 

@@ -169,6 +169,8 @@ class DecodeGraphs:
 
     def _splits_for(self, b: int) -> int:
         geo = self.ex.model.kv_geometry()
+        if not geo.get("split_plan", True):  # the line's attention plans its KV splits itself
+            return None
         # fixed per bucket so the captured launch shape never changes; sized for ~2k context
         return _K().plan_decode_splits(b, geo["kv_heads"], min(self.width * self.page_size, 2048), self.device)
 
