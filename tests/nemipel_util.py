@@ -116,12 +116,12 @@ def replayer(cfg, W, device, dtype, max_tokens, requests=4, **kw):
     from pegainfer_b200.config import EngineConfig, from_hf
     from pegainfer_b200.engine.build import build_engine
     from pegainfer_b200.loader.sources import DictSource
-    from pegainfer_b200.models.nemipel import NemipelModel
+    from pegainfer_b200.models import registry
     from pegainfer_b200.replay import Replayer
 
     mcfg = from_hf(cfg)
     mcfg.max_position = 4096
-    model = NemipelModel(mcfg, source=DictSource(W), device=device, dtype=dtype)
+    model = registry.build(mcfg, source=DictSource(W), device=device, dtype=dtype)
     page = kw.pop("page", 16)
     ecfg = EngineConfig(kv_page_size=page, num_kv_blocks=(max_tokens + page - 1) // page + 1, max_decode_batch=requests, state_slots=requests, no_prefix_cache=True, run_ahead=False, **kw)
     return Replayer(build_engine(ecfg, mcfg, device=device, dtype=dtype, model=model, start=False))
