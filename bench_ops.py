@@ -6,7 +6,7 @@ distinct weight / KV buffers (larger than L2 in total, so every launch streams f
 HBM), replayed after warm-up and timed with CUDA events.  Fractions are against the
 measured peaks in MEASURED_PEAKS.json (copy bandwidth, cuBLAS bf16 throughput).
 
-    python bench_ops.py [--only gemm|attn|small|gdn|kda|nemipel|moe|mla] [--iters 16] [--json out.json]
+    python bench_ops.py [--only gemm|attn|small|gdn|kda|nemipel|vekalorn|moe|mla] [--iters 16] [--json out.json]
     python bench_ops.py --single gemm:64x4096x4096      # one op, few launches (ncu target)
 
 Plays the role of the reference's kernel/op report binaries
@@ -264,6 +264,77 @@ def nemipel_single(kind, n, length, iters):
         f, b, z = torch.randn(t, hq * d, device=DEV), bf(t, hq), torch.zeros(hq * d, device=DEV)
         fn = lambda i: K.channel_delta(q, k, v, f, b, z[:hq], z, st, meta)
     return kind, time_graph(fn, 1, iters), n * hq * d * d * 8 + t * 4 * hq * d * 2, 8.0 * t * hq * d * d
+
+
+def vekalorn_cases(iters):
+    """Kernels of the Vekalorn line, each beside the like kernel of the DeepSeek-V2 line at the same size (indented rows):
+    a latent of 512 + 64, heads of 128 + 64 / 128.  Decode attention with its per-head products and gate, prefill attention
+    with gather and expansion; windowed rows count only the keys a window holds."""
+    from pegainfer_b200.models.layers import LatentHeads
+    from pegainfer_b200.ops import cuda as K
+    from pegainfer_b200.ops.reference import pair_rope_tables, rope_tables
+
+    rows, page, c, r, d, v = [], 16, 512, 64, 128, 128
+    few = max(2, iters // 4)
+    bf = lambda *s: torch.randn(*s, device=DEV).bfloat16()
+    cos, sin = pair_rope_tables(16384, r, 1e4, DEV)
+    c16, s16 = rope_tables(16384, r, 1e4, torch.bfloat16, DEV)
+
+    def pair(name, like, new, old, by, by_old, fl, fl_old, nvar, it, timer=time_graph):
+        t = (lambda fn: timer(fn, nvar, it)) if timer is time_graph else (lambda fn: timer(lambda: fn(0), it))
+        rows.append((name, t(new), by, fl))
+        rows.append(("  " + like, t(old), by_old, fl_old))
+
+    for heads, bs, ctx, window in ((16, 64, 1024, 0), (64, 64, 1024, 0), (64, 16, 8192, 0), (16, 1, 8192, 0), (16, 64, 4096, 1024), (64, 16, 8192, 1024)):
+        rot = 0 if window else r
+        meta, pages = _meta_for([1] * bs, [ctx] * bs, page)
+        caches = [bf(pages, page * (c + rot)) for _ in range(3)]
+        old = [bf(pages, page, c + r) for _ in range(3)]
+        uk, uv, q, gate = bf(heads * d, c) * 0.05, bf(heads * v, c) * 0.05, bf(bs, heads * (d + rot)), bf(bs, heads * v)
+        w, q_old = LatentHeads(uk, uv, heads), bf(bs, heads, d + r)
+        uk3, uv3 = uk.view(heads, d, c).contiguous(), uv.view(heads, v, c).contiguous()
+        n, wb = min(ctx, window or ctx), heads * (d + v) * c * 2
+        pair(f"latent_attention decode {heads}h {bs}x{ctx}" + (f" window {window}" if window else " rot, gate"), "mla_rope_q + mla_attention", lambda i: K.latent_attention(q, w.uk_t, w.uv, w.ukv, caches[i], meta, rot, 0.07, window, cos, sin, None if window else gate),
+             lambda i: K.mla_attention(K.mla_rope_q(q_old, c16, s16, meta, d), uk3, uv3, old[i], meta, 0.07, c), bs * n * (c + rot) * 2 + wb, bs * ctx * (c + r) * 2 + wb, 2.0 * bs * n * heads * (2 * c + rot),
+             2.0 * bs * ctx * heads * (2 * c + r), 3, few)
+    for heads, ns, ql, window in ((16, 1, 4096, 0), (16, 8, 1024, 0), (64, 1, 4096, 0), (16, 1, 16384, 0), (16, 1, 4096, 1024), (64, 1, 16384, 1024)):
+        rot, t = 0 if window else r, ns * ql
+        meta, pages = _meta_for([ql] * ns, [ql] * ns, page)
+        cache, old, q, gate = bf(pages, page * (c + rot)), bf(pages, page, c + r), bf(t, heads * (d + rot)), bf(t, heads * v)
+        uk, uv, q_old = bf(heads * d, c) * 0.05, bf(heads * v, c) * 0.05, bf(t, heads, d + r)
+        w, uk3, uv3 = LatentHeads(uk, uv, heads), uk.view(heads, d, c).contiguous(), uv.view(heads, v, c).contiguous()
+        seen = (ql * ql / 2 if not window or window >= ql else window * ql - window * window / 2) * ns
+        up = 2.0 * t * c * heads * (d + v)
+        pair(f"latent_attention prefill {heads}h {ns}x{ql}" + (f" window {window}" if window else " rot, gate"), "mla_rope_q + mla_attention", lambda i: K.latent_attention(q, w.uk_t, w.uv, w.ukv, cache, meta, rot, 0.07, window, cos, sin, None if window else gate),
+             lambda i: K.mla_attention(K.mla_rope_q(q_old, c16, s16, meta, d), uk3, uv3, old, meta, 0.07, c), t * (c + r) * 2, t * (c + r) * 2, up + 2.0 * seen * heads * (d + rot + v),
+             up + 2.0 * ns * ql * ql / 2 * heads * (d + r + v), 1, few, time_eager)
+    for t, h, ff, e, k in ((64, 2048, 2112, 64, 6), (1, 2048, 2112, 64, 6), (4096, 2048, 2112, 64, 6), (64, 7168, 3072, 16, 4), (8192, 4096, 3072, 32, 4)):
+        x, lg = bf(t, h), torch.randn(t, e, device=DEV)
+        ids, wts = K.router_topk(lg, k, "softmax", None, 8, 4, group_top=1)
+        nv = 2
+        up, down = [bf(e, ff, h) * 0.02 for _ in range(nv)], [bf(e, h, ff) * 0.02 for _ in range(nv)]
+        i2 = ff * 2 // 3
+        w13, w2 = [bf(e, 2 * i2, h) * 0.02 for _ in range(nv)], [bf(e, h, i2) * 0.02 for _ in range(nv)]
+        res, r16, nw, nw16 = torch.randn(t, h, device=DEV), bf(t, h), torch.ones(h, device=DEV), torch.ones(h, device=DEV).bfloat16()
+        by, fl = min(e, t * k) * 2 * ff * h * 2, 2.0 * t * k * 2 * ff * h
+        pair(f"expert_rows + add_layer_norm_rows T{t} {h} / {ff}, {e} experts top {k}", "moe_experts + add_rms_norm", lambda i: K.add_layer_norm_rows(*K.expert_rows(x, ids, up[i], down[i]), wts, res, nw, 1e-5, torch.bfloat16),
+             lambda i: K.add_rms_norm(K.moe_experts(x, ids, wts, w13[i], w2[i]).to(torch.bfloat16), r16, nw16, 1e-5), by, by, fl, fl, nv, few)
+        pair(f"router_topk T{t} {e} experts, best of a group", "router_topk", lambda i: K.router_topk(lg, k, "softmax", None, 8, 4, group_top=1), lambda i: K.router_topk(lg, k, "softmax", None, 8, 4), t * e * 4, t * e * 4, 0, 0, 1, iters)
+    for t in (64, 4096):
+        for width in (2048, 7168):
+            y16, y32 = [bf(t, width) for _ in range(4)], [torch.randn(t, width, device=DEV) for _ in range(4)]
+            x32, r16, w32, w16 = [torch.randn(t, width, device=DEV) for _ in range(4)], [bf(t, width) for _ in range(4)], torch.ones(width, device=DEV), torch.ones(width, device=DEV).bfloat16()
+            y = y32 if t == 64 else y16
+            pair(f"add_layer_norm {t}x{width}", "add_rms_norm", lambda i: K.add_layer_norm(y[i], x32[i], w32, 1e-5, torch.bfloat16), lambda i: K.add_rms_norm(y16[i], r16[i], w16, 1e-5), t * width * (10 + y[0].element_size()),
+                 t * width * 8, 0, 0, 4, iters)
+        meta, pages = _meta_for([1] * 64 if t == 64 else [t], [1024] * 64 if t == 64 else [t], page)
+        qr = 1536
+        z, cache, old = [bf(t, qr + c + r) for _ in range(4)], bf(pages, page * (c + r)), bf(pages, page, c + r)
+        qw, kw, qw16, kw16 = torch.ones(qr, device=DEV), torch.ones(c, device=DEV), torch.ones(qr, device=DEV).bfloat16(), torch.ones(c, device=DEV).bfloat16()
+        by = t * (qr + c + r) * 4
+        pair(f"latent_rows {t} ({qr}, {c} + {r})", "rms_norm + mla_append", lambda i: K.latent_rows(z[i][:, :qr], z[i][:, qr:], qw, kw, cos, sin, meta, cache, c, 1e-5),
+             lambda i: (K.rms_norm(z[i][:, :qr], qw16, 1e-5), K.mla_append(z[i][:, qr:], kw16, c16, s16, meta, old, c, 1e-5)), by, by, 0, 0, 4, iters)
+    return rows
 
 
 def kda_cases(iters, only=None):
@@ -644,6 +715,8 @@ def main():
             rows.extend(kda_cases(args.iters))
         if args.only in (None, "nemipel"):
             rows.extend(nemipel_cases(args.iters))
+        if args.only in (None, "vekalorn"):
+            rows.extend(vekalorn_cases(args.iters))
         if args.only in (None, "moe"):
             rows.extend(moe_cases(args.iters))
         if args.only in (None, "mla"):
@@ -653,11 +726,12 @@ def main():
         if args.only in (None, "dsa"):
             rows.extend(dsa_cases(args.iters))
     out = []
-    print(f"{'op':58s} {'us':>9s} {'GB/s':>8s} {'%HBM':>6s} {'TFLOP/s':>8s} {'%bf16':>6s}   (peaks: {src} {hbm:.0f} GB/s, {tf:.0f} TFLOP/s)")
+    wide = max([58] + [len(r[0]) for r in rows])
+    print(f"{'op':{wide}s} {'us':>9s} {'GB/s':>8s} {'%HBM':>6s} {'TFLOP/s':>8s} {'%bf16':>6s}   (peaks: {src} {hbm:.0f} GB/s, {tf:.0f} TFLOP/s)")
     for name, ms, by, fl in rows:
         gbs = by / ms / 1e6
         tfl = fl / ms / 1e9
-        print(f"{name:58s} {ms * 1e3:9.1f} {gbs:8.0f} {100 * gbs / hbm:6.1f} {tfl:8.1f} {100 * tfl / tf:6.1f}")
+        print(f"{name:{wide}s} {ms * 1e3:9.1f} {gbs:8.0f} {100 * gbs / hbm:6.1f} {tfl:8.1f} {100 * tfl / tf:6.1f}")
         out.append(dict(op=name, us=ms * 1e3, gbs=gbs, frac_hbm=gbs / hbm, tflops=tfl, frac_bf16=tfl / tf, peaks=src))
     if args.json:
         os.makedirs(os.path.dirname(os.path.abspath(args.json)), exist_ok=True)

@@ -1,5 +1,8 @@
-"""Throughput of the Nemipel line beside the Qwen3.5 line (the closest: linear-attention layers with recurrent state
-interleaved with paged attention) at equal sizes, random weights: ``bench.py --line-speed``.
+"""Throughput of a model line beside its closest neighbour at equal sizes, random weights: ``bench.py --line-speed LINE``.
+
+* ``nemipel`` beside the Qwen3.5 line (linear-attention layers with recurrent state interleaved with paged attention).
+* ``vekalorn`` beside the DeepSeek-V2 line (latent attention and mixture of experts in every layer): the same heads, latents
+  and number of experts, and expert widths that give both the same expert weights (two matrices against three).
 
 Device time (CUDA events) of whole steps of the executor: prefill steps of the given batches, and replays of the decode graph
 at a batch and context.  Weights and state are larger than L2 at every size, so no flush is needed.
@@ -7,21 +10,47 @@ at a batch and context.  Weights and state are larger than L2 at every size, so 
 from __future__ import annotations
 
 import json
-from dataclasses import replace
-
-# (name, width, feed-forward, query heads, KV heads, recurrent heads); heads of 128, 12 layers each
-SIZES = (("2048", 2048, 6144, 16, 8, 16), ("4096", 4096, 12288, 32, 8, 32), ("5120", 5120, 17408, 40, 8, 40))
-PREFILL = ((1, 4096), (8, 1024))
-DECODE = ((64, 1024), (8, 1024), (1, 1024))
+from dataclasses import dataclass, replace
+from typing import Callable
 
 
-def configs(width, ff, heads, kv_heads, lin_heads, periods=4, vocab=32768):
+@dataclass(frozen=True)
+class Comparison:
+    other: str
+    names: tuple  # of the numbers that make a size
+    sizes: tuple  # (name, numbers)
+    prefill: tuple  # (sequences, tokens)
+    decode: tuple  # (sequences, context)
+    configs: Callable
+    fixed: tuple = ()
+
+
+def _nemipel_configs(width, ff, heads, kv_heads, lin_heads, periods=4, vocab=32768):
     from ..config import PRESETS, _nemipel
 
     a = _nemipel(width, vocab, ff, heads, kv_heads, 128, lin_heads, 128, 128, periods, lightning_ff=ff, max_position=16384)
     b = replace(PRESETS["qwen35-8b-shape"], vocab_size=vocab, hidden_size=width, num_layers=3 * periods, num_q_heads=heads, num_kv_heads=kv_heads, intermediate_size=ff,
                 layer_types=("linear_attention", "full_attention", "linear_attention") * periods, gdn_num_k_heads=lin_heads // 2, gdn_num_v_heads=lin_heads, max_position=16384)
     return {"nemipel": a, "qwen35": b}
+
+
+def _vekalorn_configs(width, heads, q_rank, window, experts, top, ff, periods, vocab=32768):
+    from ..config import PRESETS, ExpertsSpec, _vekalorn
+
+    a = _vekalorn(width, vocab, heads, q_rank, 512, 128, 64, 128, window, ExpertsSpec(experts, top, ff, 8, 4), periods, max_position=16384)
+    b = replace(PRESETS["dsv2-lite"], vocab_size=vocab, hidden_size=width, num_layers=3 * periods, num_q_heads=heads, num_kv_heads=heads, q_lora_rank=q_rank, n_routed_experts=experts, n_shared_experts=0,
+                num_experts_per_tok=top, moe_intermediate_size=ff * 2 // 3, first_k_dense_replace=0, n_group=8, topk_group=4, max_position=16384)
+    return {"vekalorn": a, "deepseek_v2": b}
+
+
+LINES = {
+    "nemipel": Comparison("qwen35", ("width", "ff", "heads", "kv_heads", "recurrent_heads"), (("2048", (2048, 6144, 16, 8, 16)), ("4096", (4096, 12288, 32, 8, 32)), ("5120", (5120, 17408, 40, 8, 40))),
+                          ((1, 4096), (8, 1024)), ((64, 1024), (8, 1024), (1, 1024)), _nemipel_configs, (("layers", 12), ("head_dim", 128))),
+    "vekalorn": Comparison("deepseek_v2", ("width", "heads", "q_rank", "window", "experts", "top", "ff", "periods"),
+                           (("2048", (2048, 16, 1536, 1024, 64, 6, 2112, 4)), ("4096", (4096, 32, 1536, 1024, 32, 4, 3072, 2)), ("7168", (7168, 64, 1536, 1024, 16, 4, 3072, 2))),
+                           ((1, 4096), (8, 1024)), ((64, 1024), (16, 8192), (8, 1024), (1, 1024)), _vekalorn_configs,
+                           (("kv_rank", 512), ("dim", 128), ("rot_dim", 64), ("vdim", 128), ("layers_per_period", "1 full + 2 windowed"))),
+}
 
 
 def _timed(fn, n, warmup):
@@ -39,7 +68,7 @@ def _timed(fn, n, warmup):
     return e0.elapsed_time(e1) / n
 
 
-def measure(mcfg, steps: int, warmup: int, device="cuda:0") -> dict:
+def measure(cmp: Comparison, mcfg, steps: int, warmup: int, device="cuda:0") -> dict:
     import torch
 
     from ..config import EngineConfig
@@ -48,8 +77,8 @@ def measure(mcfg, steps: int, warmup: int, device="cuda:0") -> dict:
     from ..sched.executor import SeqStep, build_meta
 
     page, out = 16, {}
-    longest = max(max(n for _, n in PREFILL), max(n for _, n in DECODE) + steps)
-    blocks = 64 * ((1024 + 2 * page) // page + 1) + longest // page + 8
+    longest = max(max(n for _, n in cmp.prefill), max(n for _, n in cmp.decode) + steps)
+    blocks = max(n * ((length + page - 1) // page + 1) for n, length in cmp.prefill + cmp.decode) + 8
     eng = build_engine(EngineConfig(num_kv_blocks=blocks, max_decode_batch=64, max_model_len=longest + page, no_prefix_cache=True), mcfg, device=device, dtype=torch.bfloat16, start=False)
     ex = eng.executor
     try:
@@ -59,7 +88,7 @@ def measure(mcfg, steps: int, warmup: int, device="cuda:0") -> dict:
             per = (length + page - 1) // page
             return [SeqStep(rid=i, input_tokens=[(7 * j + i) % mcfg.vocab_size for j in range(new)], start_pos=length - new, view=KvView(list(range(1 + i * per, 1 + (i + 1) * per)), length, page)) for i in range(n)]
 
-        for n, length in PREFILL:
+        for n, length in cmp.prefill:
             seqs = sequences(n, length, length)
             ids, meta = build_meta(seqs, page, device)
             ex.prepare_meta(seqs, meta)
@@ -68,7 +97,7 @@ def measure(mcfg, steps: int, warmup: int, device="cuda:0") -> dict:
             out[f"prefill_{n}x{length}_tok_s"] = round(n * length / ms * 1e3)
             for s in seqs:
                 ex.release_request(s.rid)
-        for n, ctx in DECODE:
+        for n, ctx in cmp.decode:
             seqs = sequences(n, ctx, 1)
             ex._graphs.run(seqs)
             b = next(x for x in ex._graphs.buckets if x >= n)
@@ -85,22 +114,23 @@ def measure(mcfg, steps: int, warmup: int, device="cuda:0") -> dict:
     return out
 
 
-def run(steps: int = 64, warmup: int = 8, sampler=None) -> int:
+def run(name: str, steps: int = 64, warmup: int = 8, sampler=None) -> int:
     import gc
 
     import torch
 
-    for name, *dims in SIZES:
-        line = {"metric": "prefill and decode tok/s, Nemipel line beside the Qwen3.5 line", "size": name, "config": dict(zip(("width", "ff", "heads", "kv_heads", "recurrent_heads"), dims), layers=12, head_dim=128), "dtype": "bf16",
+    cmp = LINES[name]
+    for size, numbers in cmp.sizes:
+        line = {"metric": f"prefill and decode tok/s, {name} line beside the {cmp.other} line", "size": size, "config": dict(zip(cmp.names, numbers), **dict(cmp.fixed)), "dtype": "bf16",
                 "data": "random-init weights, synthetic tokens", "steps": steps, "warmup": warmup}
         if sampler is not None:
             sampler.start()
-        for fam, cfg in configs(*dims).items():
-            line[fam] = measure(cfg, steps, warmup)
+        for fam, cfg in cmp.configs(*numbers).items():
+            line[fam] = measure(cmp, cfg, steps, warmup)
             gc.collect()
             torch.cuda.empty_cache()
         if sampler is not None:
             line["clocks"] = sampler.stop()
-        line["nemipel_over_qwen35"] = {k[:-6]: round(line["nemipel"][k] / line["qwen35"][k], 3) for k in line["nemipel"] if k.endswith("_tok_s")}
+        line[f"{name}_over_{cmp.other}"] = {k[:-6]: round(line[name][k] / line[cmp.other][k], 3) for k in line[name] if k.endswith("_tok_s")}
         print(json.dumps(line), flush=True)
     return 0
