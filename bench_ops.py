@@ -269,7 +269,8 @@ def nemipel_single(kind, n, length, iters):
 def vekalorn_cases(iters):
     """Kernels of the Vekalorn line, each beside the like kernel of the DeepSeek-V2 line at the same size (indented rows):
     a latent of 512 + 64, heads of 128 + 64 / 128.  Decode attention with its per-head products and gate, prefill attention
-    with gather and expansion; windowed rows count only the keys a window holds."""
+    with gather and expansion; windowed rows count only the keys a window holds, and in decoding stand beside the other
+    kernel at a context of the window's length."""
     from pegainfer_b200.models.layers import LatentHeads
     from pegainfer_b200.ops import cuda as K
     from pegainfer_b200.ops.reference import pair_rope_tables, rope_tables
@@ -288,15 +289,17 @@ def vekalorn_cases(iters):
     for heads, bs, ctx, window in ((16, 64, 1024, 0), (64, 64, 1024, 0), (64, 16, 8192, 0), (16, 1, 8192, 0), (16, 64, 4096, 1024), (64, 16, 8192, 1024)):
         rot = 0 if window else r
         meta, pages = _meta_for([1] * bs, [ctx] * bs, page)
+        n = min(ctx, window or ctx)
+        meta_old, pages_old = _meta_for([1] * bs, [n] * bs, page)
         caches = [bf(pages, page * (c + rot)) for _ in range(3)]
-        old = [bf(pages, page, c + r) for _ in range(3)]
+        old = [bf(pages_old, page, c + r) for _ in range(3)]
         uk, uv, q, gate = bf(heads * d, c) * 0.05, bf(heads * v, c) * 0.05, bf(bs, heads * (d + rot)), bf(bs, heads * v)
         w, q_old = LatentHeads(uk, uv, heads), bf(bs, heads, d + r)
         uk3, uv3 = uk.view(heads, d, c).contiguous(), uv.view(heads, v, c).contiguous()
-        n, wb = min(ctx, window or ctx), heads * (d + v) * c * 2
+        wb = heads * (d + v) * c * 2
         pair(f"latent_attention decode {heads}h {bs}x{ctx}" + (f" window {window}" if window else " rot, gate"), "mla_rope_q + mla_attention", lambda i: K.latent_attention(q, w.uk_t, w.uv, w.ukv, caches[i], meta, rot, 0.07, window, cos, sin, None if window else gate),
-             lambda i: K.mla_attention(K.mla_rope_q(q_old, c16, s16, meta, d), uk3, uv3, old[i], meta, 0.07, c), bs * n * (c + rot) * 2 + wb, bs * ctx * (c + r) * 2 + wb, 2.0 * bs * n * heads * (2 * c + rot),
-             2.0 * bs * ctx * heads * (2 * c + r), 3, few)
+             lambda i: K.mla_attention(K.mla_rope_q(q_old, c16, s16, meta_old, d), uk3, uv3, old[i], meta_old, 0.07, c), bs * n * (c + rot) * 2 + wb, bs * n * (c + r) * 2 + wb,
+             2.0 * bs * n * heads * (2 * c + rot), 2.0 * bs * n * heads * (2 * c + r), 3, few)
     for heads, ns, ql, window in ((16, 1, 4096, 0), (16, 8, 1024, 0), (64, 1, 4096, 0), (16, 1, 16384, 0), (16, 1, 4096, 1024), (64, 1, 16384, 1024)):
         rot, t = 0 if window else r, ns * ql
         meta, pages = _meta_for([ql] * ns, [ql] * ns, page)

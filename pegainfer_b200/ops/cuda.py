@@ -1492,7 +1492,10 @@ def _head_gemm(x, x_tok: int, x_head: int, w, y, gate=None):
     c = ctx(y.device)
     args = (_ptr(x), _ll(x_tok), _ll(x_head), _ptr(w), _ptr(y), _ll(heads * m), _ll(m), _ptr(gate), _ll(gate.stride(0) if gate is not None else 0), _ll(m), _ci(heads), _ci(rows), _ci(m), _ci(k))
     if y.dtype == torch.bfloat16 and k % 8 == 0 and x_tok % 8 == 0 and x_head % 8 == 0 and x.data_ptr() % 16 == 0 and heads <= 512:
-        _check(lib().pg_head_gemm(*args, _ci(_token_tile(heads * rows, heads)), _ptr(c.status), _stream()), c)
+        bn, tiles = _token_tile(heads * rows, heads), heads * ((m + 127) // 128)
+        while bn > 16 and tiles * ((rows + bn - 1) // bn) < c.sms:  # narrower token tiles until every SM has one (a head's weights come from L2 again)
+            bn //= 2
+        _check(lib().pg_head_gemm(*args, _ci(bn), _ptr(c.status), _stream()), c)
     else:
         _check(lib().pg_head_gemm_simt(*args, _ci(_is_f32(y)), _stream()), c)
 
