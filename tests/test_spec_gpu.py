@@ -9,6 +9,16 @@ from pegainfer_b200.engine.build import build_engine
 pytestmark = pytest.mark.gpu
 
 
+@pytest.fixture(autouse=True)
+def _restore_numeric_policy():
+    """The engines of this file run batch-invariant, a policy of the whole process."""
+    from pegainfer_b200.ops import cuda as K
+
+    before = K.batch_invariant()
+    yield
+    K.set_batch_invariant(before)
+
+
 def test_markov_step_argmax_kernel_matches_reference():
     from pegainfer_b200.ops import cuda as K
     from pegainfer_b200.ops import reference as R
