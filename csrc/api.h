@@ -62,7 +62,7 @@ int pg_ipc_close(void* p);
 int pg_gemm2sm_eligible(int T, int M, int K);
 int pg_gemm2sm_bf16_tn(const void* x, const void* w, void* y, int T, int M, int K, long long ldx, long long ldw, long long ldy, void* status,
                        cudaStream_t stream);
-int pg_gemm2sm_bf16_tn_swiglu(const void* x, const void* w, void* y, int T, int M, int K, long long ldx, long long ldw, long long ldy, void* status,
+int pg_gemm2sm_bf16_tn_swiglu(const void* x, const void* w, void* y, int T, int M, int K, long long ldx, long long ldw, long long ldy, int gelu, void* status,
                        cudaStream_t stream);
 int pg_make_tmap_bf16_2d(CUtensorMap* out, const void* ptr, long long rows, long long cols, long long ld, int box_rows, int box_cols);
 
@@ -97,8 +97,8 @@ int pg_prefill_attention_tc_capped(const void* q, const void* kv_layer, void* ou
 int pg_latent_gather(const void* latent_layer, int page_size, long long num_pages, int width, const void* table, int table_stride, const void* kv_indptr, const void* starts, int num_seqs, int total_kv,
                      void* out, void* status, cudaStream_t stream);
 int pg_latent_prefill_tc(const void* q, long long q_tok, long long q_head, const void* q_pe, long long pe_tok, long long pe_head, const void* k, const void* v, long long ld_kv, const void* k_pe,
-                         long long pe_ld, const void* gate, long long ld_gate, void* out, const void* q_indptr, const void* kv_indptr, const void* kv_lens, int num_seqs, int tokens, int total_kv, int heads,
-                         int dim, int rot, int vdim, float scale, int window, int q_tiles, void* status, cudaStream_t stream);
+                         long long pe_ld, const void* gate, long long ld_gate, int gate_cols, const void* sink, void* out, const void* q_indptr, const void* kv_indptr, const void* kv_lens, int num_seqs,
+                         int tokens, int total_kv, int heads, int dim, int rot, int vdim, float scale, int window, int q_tiles, void* status, cudaStream_t stream);
 
 // ---- block-scaled FP8 GEMM on tcgen05 kind::f8f6f4 (gemm_fp8_sm100.cu) --------------------
 long long pg_gemm_fp8_ws_bytes(int T, int M);
@@ -135,10 +135,11 @@ int pg_mla_attention(const void* q_abs, const void* q_pe, const void* latent, vo
 // sliding window, and rotation of neighbouring query columns inside the kernel; token / head strides in elements.
 int pg_latent_attention(const void* q_abs, long long q_tok, long long q_head, const void* q_pe, long long pe_tok, long long pe_head, const void* cos, const void* sin, int max_pos, const void* latent,
                         void* out, long long o_tok, long long o_head, const void* q_indptr, const void* kv_lens, const void* table, int table_stride, const void* unit_seq, int first_row, int num_seqs,
-                        int tokens, int heads, int c, int r, int page_size, float scale, int window, int splits, void* part_o, void* part_lse, cudaStream_t stream);
+                        int tokens, int heads, int c, int r, int page_size, float scale, int window, const void* sink, const void* head_gate, long long ld_gate, int splits, void* part_o, void* part_lse,
+                        cudaStream_t stream);
 int pg_latent_attention_plain(const void* q_abs, long long q_tok, long long q_head, const void* q_pe, long long pe_tok, long long pe_head, const void* cos, const void* sin, int max_pos, const void* latent,
                               void* out, long long o_tok, long long o_head, const void* q_indptr, const void* kv_lens, const void* table, int table_stride, const void* unit_seq, int tokens, int heads, int c,
-                              int r, int page_size, float scale, int window, int is_f32, cudaStream_t stream);
+                              int r, int page_size, float scale, int window, const void* sink, const void* head_gate, long long ld_gate, int is_f32, cudaStream_t stream);
 int pg_latent_rows(const void* zq, const void* zkv, long long ld, const void* q_w, const void* kv_w, const void* cos, const void* sin, const void* positions, const void* slots, void* cq, void* latent,
                    int tokens, int qr, int c, int r, int max_pos, long long num_slots, float eps, int is_f32, void* status, cudaStream_t stream);
 int pg_rotate_pairs(void* x, long long tok, long long head, const void* cos, const void* sin, const void* positions, int tokens, int heads, int r, int max_pos, int is_f32, cudaStream_t stream);
@@ -155,7 +156,7 @@ int pg_moe_combine(const void* y, long long ldy, const void* route_pos, const vo
 int pg_moe_grouped_gemm(const void* x, long long ldx, long long x_rows, const void* w, const void* scales, int quant, void* y, long long ldy,
                         const void* offsets, int E, int M, int K, int bn, void* status, cudaStream_t stream);
 
-int pg_moe_grouped_gemm_relu2(const void* x, long long ldx, long long x_rows, const void* w, void* y, long long ldy, const void* offsets, int E, int M, int K, int bn, void* status, cudaStream_t stream);
+int pg_moe_grouped_gemm_act(const void* x, long long ldx, long long x_rows, const void* w, void* y, long long ldy, const void* offsets, int E, int M, int K, int bn, int act, void* status, cudaStream_t stream);
 // Per-head products of strided activations: y[t, h, :] = x[t, h, :] w[h]^T (times the sigmoid of a gate)
 int pg_head_gemm(const void* x, long long ldx, long long x_head, const void* w, void* y, long long ldy, long long y_head, const void* gate, long long ldg, long long g_head, int heads, int rows, int M, int K,
                  int bn, void* status, cudaStream_t stream);
@@ -200,6 +201,13 @@ int pg_decay_recurrent(const void* q, const void* k, const void* v, long long ld
 // Chunk-wise (64-token) tensor-core form of decay_recurrent for sequences of >= min_len tokens, bf16 (lightning.cu).
 int pg_lightning_chunked(const void* q, const void* k, const void* v, long long ld, const void* decay, void* state, void* out, const void* q_indptr, const void* slots, int num_seqs,
                          int heads, int dk, int dv, int min_len, cudaStream_t stream);
+// wkv_recurrent: linear attention with a decay per token and key channel and a bonus for the current token.
+int pg_wkv_recurrent(const void* r, const void* k, const void* v, long long ld, const void* f, long long ldf, const void* w0, const void* u, void* state, void* out, const void* q_indptr,
+                     const void* slots, int num_seqs, int heads, int dk, int dv, int max_q_len, int skip_len, int is_f32, cudaStream_t stream);
+// ---- token shift and chunk-wise WKV (wkv.cu) ------------------------------------------
+// out[t, i] = h[t] + (h[t - 1] - h[t]) * mu[i]; carried [slots, width]: the row in front of a request's first one of the step.
+int pg_token_mix(const void* h, long long ldh, const void* mu, void* carried, void* out, const void* unit_seq, const void* q_indptr, const void* slots, int tokens, int n, int width, int is_f32,
+                 cudaStream_t stream);
 // Softmax mix of the first nb snapshot rows of each token (snaps [T, cap, hidden], ld_tok = cap * hidden) and its current row.
 int pg_attnres_mix(const void* cur, long long ld_cur, const void* snaps, long long ld_tok, const void* score_w, void* out, long long ld_out,
                    int tokens, int nb, int hidden, float eps, cudaStream_t stream);
@@ -223,22 +231,30 @@ int pg_attention_capped(const void* q, const void* kv, void* out, const void* q_
 int pg_row_norm_rope_append(const void* q, const void* k, const void* v, long long ld, const void* q_w, const void* k_w, const void* cos, const void* sin, int rot, int max_pos,
                             const void* positions, const void* slots, void* q_out, void* kv, int tokens, int hq, int hkv, int dim, int vdim, int page_size, long long num_pages, float eps,
                             int is_f32, void* status, cudaStream_t stream);
+int pg_head_norm_append(const void* q, const void* k, const void* v, long long ld, const void* q_w, const void* k_w, const void* temp, int max_pos, const void* positions, const void* slots,
+                        void* q_out, void* kv, int tokens, int hq, int hkv, int dim, int vdim, int page_size, long long num_pages, float eps, int is_f32, void* status, cudaStream_t stream);
 int pg_attention_plain(const void* q, const void* kv, void* out, const void* q_indptr, const void* kv_lens, const void* table, int table_stride, int tokens, int num_seqs, int hq, int hkv,
                        int dim, int vdim, int page_size, long long num_pages, float scale, float softcap, const void* gate, long long ld_gate, int is_f32, cudaStream_t stream);
 
 // ---- rows around an f32 residual stream (stream32.cu) --------------------------------
 int pg_embed_rows(const void* table, int table_f32, long long ldt, const void* ids, void* x_f32, void* xt, int xt_f32, long long ldxt, int tokens, int width, long long rows, void* status,
                   cudaStream_t stream);
+int pg_embed_pairs_norm(const void* table, int table_f32, long long ldt, const void* pairs, long long ldp, const void* ids, const void* unit_seq, const void* q_indptr, const void* slots, void* carried,
+                        float scale, long long buckets, long long mul_prev, long long mul_cur, const void* w, void* x, void* xt, int xt_f32, int tokens, int width, long long rows, float eps,
+                        void* status, cudaStream_t stream);
+int pg_residual_norm(const void* y, int y_f32, long long ldy, const void* pos, const void* weights, int k, const void* extra, int extra_f32, long long lde, const void* extra_gate, long long ldg,
+                     void* x, float mult, const void* w, void* xt, int xt_f32, long long ldxt, int tokens, int width, float eps, cudaStream_t stream);
+int pg_tanh_rows(const void* x, void* y, long long n, int is_f32, cudaStream_t stream);
 int pg_post_norm(const void* y, int y_f32, long long ldy, const void* x_in, void* x_out, float alpha, const void* w, void* xt, int xt_f32, long long ldxt, int tokens, int width, float eps,
                  cudaStream_t stream);
 int pg_add_layer_norm(const void* y, int y_f32, long long ldy, const void* pos, const void* weights, int k, void* x, const void* w, void* xt, int xt_f32, long long ldxt, int tokens, int width, float eps,
                       cudaStream_t stream);
 int pg_head_gemm_simt(const void* x, long long ldx, long long x_head, const void* w, void* y, long long ldy, long long y_head, const void* gate, long long ldg, long long g_head, int heads, int rows, int M,
                       int K, int is_f32, cudaStream_t stream);
-int pg_expert_gemm_simt(const void* x, long long ldx, const void* sorted_src, int k, const void* w, void* y, const void* offsets, int routes, int E, int M, int K, int relu2, int is_f32,
+int pg_expert_gemm_simt(const void* x, long long ldx, const void* sorted_src, int k, const void* w, void* y, const void* offsets, int routes, int E, int M, int K, int act, int is_f32,
                         cudaStream_t stream);
-int pg_gated_row_norm(const void* x, const void* gate, long long ldg, const void* w, void* y, int tokens, int heads, int dim, float eps, int is_f32, cudaStream_t stream);
-int pg_glu_rows_f32(const void* gu, void* out, int rows, int inter, long long ldin, cudaStream_t stream);
+int pg_gated_row_norm(const void* x, const void* gate, long long ldg, const void* w, void* y, int tokens, int heads, int dim, float eps, int silu, int w_heads, int is_f32, cudaStream_t stream);
+int pg_glu_rows_f32(const void* gu, void* out, int rows, int inter, long long ldin, int gelu, cudaStream_t stream);
 int pg_softcap_f32(const void* x, void* y, long long n, float cap, cudaStream_t stream);
 int pg_gemm_simt(const void* x, const void* w, int x_f32, void* y, int y_f32, int T, int M, int K, long long ldx, long long ldw, long long ldy, cudaStream_t stream);
 int pg_conv_silu(const void* x, long long ldx, const void* w, void* state, void* out, long long ldo, const void* q_indptr, const void* slots, int num_seqs, int channels, int taps,

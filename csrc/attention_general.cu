@@ -4,6 +4,8 @@
 //    pairs (2i, 2i + 1) of the first `rot` entries of every head with f32 cos / sin tables, then the queries go to a
 //    dense buffer and keys and values to the token's slot of the paged cache.  One CTA per token.  Without keys (a layer
 //    that reads another layer's cache) only the queries are made.
+//  * head_norm_append: RMS norm of every query and key head with a weight shared by the heads, queries times a factor per
+//    position; queries go to a dense buffer, keys and values (untouched; they may be the key projection itself) to the cache.
 //  * attention_plain: one CTA per (query row, head) on the CUDA cores, keys in chunks of 128 with an online softmax; any
 //    head size, value size and group.  It is the 32-bit path, and the path of head sizes the tensor-core kernels
 //    (attention.cu, attention_tc.cu) do not address.
@@ -134,6 +136,57 @@ __global__ void __launch_bounds__(256) row_norm_rope_append_kernel(const T* __re
   }
 }
 
+// TPR threads (16 or 32) per unit of a token: hq query heads, hkv key heads, hkv value heads.
+template <typename T, int V, int TPR>
+__global__ void __launch_bounds__(256) head_norm_append_kernel(const T* __restrict__ q, const T* __restrict__ k, const T* __restrict__ v, long long ld, const float* __restrict__ q_w, const float* __restrict__ k_w,
+                                                               const float* __restrict__ temp, int max_pos, const int* __restrict__ positions, const int* __restrict__ slots, T* __restrict__ q_out,
+                                                               T* __restrict__ kv, int hq, int hkv, int dim, int vdim, int page_size, long long num_pages, float eps, uint32_t* status) {
+  PG_PDL_ENTRY();
+  const long long t = blockIdx.x;
+  const int me = threadIdx.x % TPR, units = hq + 2 * hkv;
+  float factor = 1.f;
+  if (temp) {
+    int pos = positions[t];
+    if (pos < 0 || pos >= max_pos) {
+      if (threadIdx.x == 0) atomicCAS(status, PG_ST_OK, PG_ST_BOUNDS | (57u << 8));
+      pos = pos < 0 ? 0 : max_pos - 1;
+    }
+    factor = temp[pos];
+  }
+  const long long slot = slots[t];
+  const bool slot_ok = slot >= 0 && slot < num_pages * page_size;
+  if (!slot_ok && threadIdx.x == 0) atomicCAS(status, PG_ST_OK, PG_ST_BOUNDS | (58u << 8));
+  const long long page = slot / page_size, off = slot % page_size;
+  T* kpage = kv + page * page_size * hkv * (dim + vdim);
+  for (int u0 = 0; u0 < units; u0 += 256 / TPR) {  // all lanes of a warp take part in the sums
+    const int u = u0 + threadIdx.x / TPR;
+    const bool live = u < units && (u < hq || slot_ok), value = u >= hq + hkv;
+    const int h = u < hq ? u : value ? u - hq - hkv : u - hq, n = live ? (value ? vdim : dim) / V : 0;
+    const T* src = u < hq ? q + t * ld + (long long)h * dim : value ? v + t * ld + (long long)h * vdim : k + t * ld + (long long)h * dim;
+    T* dst = u < hq ? q_out + (t * hq + h) * dim : value ? kpage + (long long)page_size * hkv * dim + (off * hkv + h) * vdim : kpage + (off * hkv + h) * dim;
+    float f[V], ss = 0.f;
+    for (int i = me; i < n; i += TPR) {
+      load_vec<V>(src + i * V, f);
+#pragma unroll
+      for (int j = 0; j < V; ++j) ss += f[j] * f[j];
+    }
+#pragma unroll
+    for (int o = TPR / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    const float inv = rsqrtf(ss / (float)dim + eps) * (u < hq ? factor : 1.f);
+    const float* w = u < hq ? q_w : k_w;
+    for (int i = me; i < n; i += TPR) {
+      if (n > TPR) load_vec<V>(src + i * V, f);
+      if (!value) {
+        float wf[V];
+        load_vec<V>(w + i * V, wf);
+#pragma unroll
+        for (int j = 0; j < V; ++j) f[j] *= inv * wf[j];
+      }
+      store_vec<V>(dst + i * V, f);
+    }
+  }
+}
+
 constexpr int PL_KEYS = 128;  // keys per chunk, one per thread
 constexpr int PL_VMAX = 8;    // value columns per thread: vdim <= 1024
 
@@ -225,6 +278,24 @@ extern "C" int pg_row_norm_rope_append(const void* q, const void* k, const void*
   else
     PG_CUDA(v8 ? PG_RNR(bf16, 8) : PG_RNR(bf16, 1));
 #undef PG_RNR
+  PG_LAUNCH_CHECK();
+  return PG_OK;
+}
+
+// q, k, v: columns of rows of stride ld; temp f32 [max_pos] (or null); cache as above.
+extern "C" int pg_head_norm_append(const void* q, const void* k, const void* v, long long ld, const void* q_w, const void* k_w, const void* temp, int max_pos, const void* positions, const void* slots,
+                                   void* q_out, void* kv, int tokens, int hq, int hkv, int dim, int vdim, int page_size, long long num_pages, float eps, int is_f32, void* status, cudaStream_t stream) {
+  PG_REQUIRE(hq >= 1 && hkv >= 1 && dim >= 1 && vdim >= 1 && (temp == nullptr || max_pos > 0), "head_norm_append: heads %d / %d of %d / %d columns", hq, hkv, dim, vdim);
+  if (tokens == 0) return PG_OK;
+  const bool v8 = dim % 8 == 0 && vdim % 8 == 0 && ld % 8 == 0 && ((((uintptr_t)q | (uintptr_t)k | (uintptr_t)v | (uintptr_t)q_out | (uintptr_t)kv | (uintptr_t)q_w | (uintptr_t)k_w) & 15) == 0);
+#define PG_HN(T, V, TPR)                                                                                                                                                                            \
+  launch_pdl(head_norm_append_kernel<T, V, TPR>, dim3(tokens), dim3(256), (size_t)0, stream, (const T*)q, (const T*)k, (const T*)v, ld, (const float*)q_w, (const float*)k_w, (const float*)temp, max_pos, \
+             (const int*)positions, (const int*)slots, (T*)q_out, (T*)kv, hq, hkv, dim, vdim, page_size, num_pages, eps, (uint32_t*)status)
+  if (is_f32)
+    PG_CUDA(PG_HN(float, 1, 32));
+  else
+    PG_CUDA(v8 ? (dim <= 128 && vdim <= 128 ? PG_HN(bf16, 8, 16) : PG_HN(bf16, 8, 32)) : PG_HN(bf16, 1, 32));
+#undef PG_HN
   PG_LAUNCH_CHECK();
   return PG_OK;
 }

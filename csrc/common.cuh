@@ -74,6 +74,11 @@ __device__ __forceinline__ uint64_t globaltimer_ns() {
 }
 
 __device__ __forceinline__ float bf16_round(float x) { return __bfloat162float(__float2bfloat16(x)); }
+// Activation of a gated feed-forward: SiLU, or the tanh form of GELU (0.5 (1 + tanh(a)) is the logistic function of 2 a).
+__device__ __forceinline__ float glu_act(float z, bool gelu) {
+  const float t = gelu ? 1.5957691216057308f * (z + 0.044715f * z * z * z) : z;
+  return z / (1.f + __expf(-t));
+}
 
 struct __align__(16) bf16x8 {
   bf162 v[4];

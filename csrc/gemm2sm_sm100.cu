@@ -251,8 +251,8 @@ gemm2sm_bf16_tn_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_co
         tmem_ld16(t_row + c, v[0]);
         tmem_ld16(t_row + c + 16, v[1]);
         tmem_ld_wait();
-        if (p.epi == 1) {
-          // SwiGLU: lanes 2 i and 2 i + 1 hold gate and up of output column m / 2 (both rounded to bf16 first, as the
+        if (p.epi != 0) {
+          // SwiGLU (1) or its form with tanh-GELU (3): lanes 2 i and 2 i + 1 hold gate and up of output column m / 2 (both rounded to bf16 first, as the
           // separate kernel sees them); the shuffles run on all lanes, the even ones store
           bf16* ys = p.y + (m >> 1);
 #pragma unroll
@@ -263,7 +263,7 @@ gemm2sm_bf16_tn_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_co
               const float other = __shfl_xor_sync(0xFFFFFFFFu, mine, 1);
               const int n = n0 + c + h * 16 + j;
               if (!(lane & 1) && m < p.M && n < p.T) {
-                const float a = __bfloat162float(__float2bfloat16(mine / (1.f + __expf(-mine))));
+                const float a = bf16_round(glu_act(mine, p.epi == 3));
                 ys[(long long)n * p.ldy] = __float2bfloat16(a * other);
               }
             }
@@ -340,11 +340,11 @@ extern "C" int pg_gemm2sm_bf16_tn(const void* x, const void* w, void* y, int T, 
   return gemm2sm_impl(x, w, y, T, M, K, ldx, ldw, ldy, status, 0, stream);
 }
 
-// The same product with SwiGLU in the epilogue: w [M, K] with rows alternating (gate_i, up_i), y [T, M / 2].
-extern "C" int pg_gemm2sm_bf16_tn_swiglu(const void* x, const void* w, void* y, int T, int M, int K, long long ldx, long long ldw, long long ldy, void* status,
+// The same product with SwiGLU (gelu: tanh-GELU on the gate) in the epilogue: w [M, K] with rows alternating (gate_i, up_i), y [T, M / 2].
+extern "C" int pg_gemm2sm_bf16_tn_swiglu(const void* x, const void* w, void* y, int T, int M, int K, long long ldx, long long ldw, long long ldy, int gelu, void* status,
                                          cudaStream_t stream) {
   PG_REQUIRE(M % 2 == 0, "gemm2sm swiglu: M %d must be even (interleaved gate / up rows)", M);
-  return gemm2sm_impl(x, w, y, T, M, K, ldx, ldw, ldy, status, 1, stream);
+  return gemm2sm_impl(x, w, y, T, M, K, ldx, ldw, ldy, status, gelu ? 3 : 1, stream);
 }
 
 static int gemm2sm_impl(const void* x, const void* w, void* y, int T, int M, int K, long long ldx, long long ldw, long long ldy, void* status, int epi, cudaStream_t stream) {

@@ -91,6 +91,7 @@ struct FuseSpec {
   long long ld_res;
   const bf16* norm_w;   // EPI_RESID_NORMW: weight of the norm that the consumer completes
   int norm_offset;      // (1 + w) form
+  int gelu;             // EPI_SWIGLU: tanh-GELU in the place of SiLU
   float* out_ssp;       // EPI_RESID_NORMW: [T][out_ld], entry [n][m_tile]
   int out_ld;
 };
@@ -212,7 +213,7 @@ __device__ __forceinline__ float store_out4(const GemmParams& p, int n, int m, f
     // rows (m, m+1) = (gate, up) of feature m / 2, rows (m+2, m+3) of the next one
     if (m + 3 < p.M) {
       const float g0 = bf16_round(v.x), u0 = bf16_round(v.y), g1 = bf16_round(v.z), u1 = bf16_round(v.w);
-      const bf162 o = __floats2bfloat162_rn(bf16_round(g0 / (1.f + __expf(-g0))) * u0, bf16_round(g1 / (1.f + __expf(-g1))) * u1);
+      const bf162 o = __floats2bfloat162_rn(bf16_round(glu_act(g0, p.fuse.gelu)) * u0, bf16_round(glu_act(g1, p.fuse.gelu)) * u1);
       *reinterpret_cast<bf162*>(p.y + (size_t)n * p.ldy + (m >> 1)) = o;
     }
     return 0.f;
@@ -1318,7 +1319,7 @@ extern "C" int pg_tp_gemm_rs_norm_ag(const void* a, const void* w, int T, int hi
 
 // The decode-chain form of the GEMM (T <= 64): optional deferred-RMSNorm scaling of the input rows
 // (`in_ssp` [in_parts][T] sums of squares written by the producer, nullptr = none) and a fused
-// epilogue: 0 plain, 1 SwiGLU over interleaved (gate, up) weight rows (y is [T, M / 2]), 2 residual
+// epilogue: 0 plain, 1 SwiGLU over interleaved (gate, up) weight rows (y is [T, M / 2]), 3 the same with tanh-GELU, 2 residual
 // add + norm-weight product (y = xw [T, M], `residual` updated in place, `out_ssp` [ceil(M / 128)][T]
 // written).  Returns PG_ERR_UNSUPPORTED when the problem does not plan onto the on-chip split-K path;
 // the caller then runs the separate kernels.
@@ -1326,6 +1327,8 @@ extern "C" int pg_gemm_bf16_tn_fused(const void* x, const void* w, void* y, int 
                                      const void* in_ssp, int in_parts, int in_ld, int in_width, float in_eps, int epi, void* residual, long long ld_res,
                                      const void* norm_w, int norm_offset, void* out_ssp, int out_ld, void* ws, long long ws_bytes, void* counters,
                                      long long counter_bytes, void* status, cudaStream_t stream) {
+  const bool gelu = epi == 3;
+  if (gelu) epi = EPI_SWIGLU;
   PG_REQUIRE(epi >= EPI_PLAIN && epi <= EPI_RESID_NORMW, "gemm fused: unknown epilogue %d", epi);
   PG_REQUIRE(T <= 64, "gemm fused: built for decode steps of at most 64 token rows, got %d", T);
   PG_REQUIRE(in_ssp == nullptr || (in_parts > 0 && in_width > 0 && in_ld >= in_parts && in_ld % 4 == 0 && ((uintptr_t)in_ssp & 15) == 0),
@@ -1349,6 +1352,7 @@ extern "C" int pg_gemm_bf16_tn_fused(const void* x, const void* w, void* y, int 
   f.ld_res = ld_res;
   f.norm_w = (const bf16*)norm_w;
   f.norm_offset = norm_offset;
+  f.gelu = gelu;
   f.out_ssp = (float*)out_ssp;
   f.out_ld = out_ld;
   return gemm_impl(x, w, y, 0, T, M, K, ldx, ldw, ldy, ws, ws_bytes, counters, counter_bytes, status, 0, nullptr, nullptr, stream, nullptr, &f);

@@ -10,8 +10,10 @@
 //    quarter of its Dk elements in registers; a stage of 8 tokens is normalised into shared memory, then
 //    walked in order.  A decode step is one pass over the state (read + write).
 //    The same kernel runs two more rules (RULE below): the decay in its softplus form, exp(-exp(A_log) softplus(f + dt_bias)),
-//    with query / key heads shared by several value heads, and plain linear attention with one fixed decay per head
-//    (S = decay S + k (x) v, out = S^T q, SiLU on q, k and v).  Those take bf16 or f32 rows and any key width up to 256.
+//    with query / key heads shared by several value heads, plain linear attention with one fixed decay per head
+//    (S = decay S + k (x) v, out = S^T q, SiLU on q, k and v), and linear attention with a decay per token and key channel and a
+//    bonus for the current token (out = (S + diag(u) k (x) v)^T q in front of S = diag(dec) S + k (x) v, dec = exp(-exp(f + w0))).
+//    Those take bf16 or f32 rows and any key width up to 256.
 //  * attnres_mix: the attention-residual mix.  Every token keeps up to `cap` snapshot rows of its own residual
 //    stream; a mix scores each of the first nb snapshots and the current row with
 //    dot(x / rms(x), score_w) and returns the softmax-weighted sum of the un-normalised rows.
@@ -28,18 +30,19 @@ constexpr int KDA_STAGE = 8;
 constexpr int KDA_COLS = 32;
 
 // What a token does to the state.  BOUNDED and SOFTPLUS are the delta rule with a decay per key channel and two forms of
-// the decay; DECAY is linear attention with a fixed decay per head (no correction term).
-enum { RULE_BOUNDED = 0, RULE_SOFTPLUS = 1, RULE_DECAY = 2 };
+// the decay; DECAY is linear attention with a fixed decay per head (no correction term), WKV with a decay per token and key
+// channel, read in front of the update with a bonus for the current token.
+enum { RULE_BOUNDED = 0, RULE_SOFTPLUS = 1, RULE_DECAY = 2, RULE_WKV = 3 };
 
 template <typename T>
 struct RecArgs {
   const T *q, *k, *v;  // token rows of stride ld; q and k [kv_heads * dk], v [heads * dv]
   long long ld;
-  const void* f;  // raw decay projection [heads * dk]: T (BOUNDED) or f32 (SOFTPLUS)
+  const void* f;  // raw decay projection [heads * dk]: T (BOUNDED) or f32 (SOFTPLUS, WKV)
   long long ldf;
   const T* b;  // raw step-size projection [heads]
   long long ldb;
-  const float *a_log, *dt_bias, *decay;  // decay [heads]: DECAY only
+  const float *a_log, *dt_bias, *decay;  // decay [heads]: DECAY; WKV: dt_bias = w0 [heads * dk], decay = the bonus u [heads * dk]
   float lower;
   float* state;
   T* out;
@@ -61,8 +64,9 @@ __global__ void __launch_bounds__(128) kda_recurrent_kernel(const T* __restrict_
   constexpr int QK = DK / 4;   // state elements per thread
   constexpr int QS = QK + 4;   // padded quarter stride: the four quarters land in different banks
   constexpr int QL = DK / 32;  // elements per lane when a warp holds one token
-  constexpr bool DELTA = RULE != RULE_DECAY;
-  __shared__ __align__(16) float sq[KDA_STAGE][4 * QS], sk[KDA_STAGE][4 * QS], sd[DELTA ? KDA_STAGE : 1][4 * QS];
+  constexpr bool DELTA = RULE == RULE_BOUNDED || RULE == RULE_SOFTPLUS;
+  constexpr bool KEYED = RULE != RULE_DECAY;  // a decay per key channel
+  __shared__ __align__(16) float sq[KDA_STAGE][4 * QS], sk[KDA_STAGE][4 * QS], sd[KEYED ? KDA_STAGE : 1][4 * QS];
   __shared__ float sv[KDA_STAGE][KDA_COLS], sb[KDA_STAGE];
   __shared__ float red_kv[4][KDA_COLS], red_o[DELTA ? 1 : 2][4][KDA_COLS];
   const int dk = PAD ? dk_arg : DK;
@@ -84,7 +88,7 @@ __global__ void __launch_bounds__(128) kda_recurrent_kernel(const T* __restrict_
   const int kh = RULE == RULE_SOFTPLUS ? h * kv_heads / heads : h;
   const float q_scale = DELTA ? rsqrtf((float)dk) : 1.f;
   const float a = DELTA ? __expf(a_log[h]) : 0.f;
-  const float fixed = DELTA ? 0.f : decay[h];
+  const float fixed = RULE == RULE_DECAY ? decay[h] : 0.f;
 
   for (int t0 = q0; t0 < q1; t0 += KDA_STAGE) {
     const int nt = min(KDA_STAGE, q1 - t0);
@@ -102,6 +106,8 @@ __global__ void __launch_bounds__(128) kda_recurrent_kernel(const T* __restrict_
         if (DELTA) {
           qs += rq[i] * rq[i];
           ks += rk[i] * rk[i];
+        } else if (RULE == RULE_WKV) {
+          if (in) qs += rq[i] * rk[i] * decay[h * dk + lane + 32 * i];
         } else {  // the activation's result is what the layer works with, in the activation type
           rq[i] = to_f32(from_f32<T>(rq[i] / (1.f + __expf(-rq[i]))));
           rk[i] = to_f32(from_f32<T>(rk[i] / (1.f + __expf(-rk[i]))));
@@ -112,6 +118,10 @@ __global__ void __launch_bounds__(128) kda_recurrent_kernel(const T* __restrict_
         qs = warp_sum(qs);
         ks = warp_sum(ks);
         qn = rsqrtf(qs + 1e-6f) * q_scale, kn = rsqrtf(ks + 1e-6f);
+      }
+      if (RULE == RULE_WKV) {  // what the token's own value counts
+        qs = warp_sum(qs);
+        if (lane == 0) sb[j] = qs;
       }
 #pragma unroll
       for (int i = 0; i < QL; ++i) {
@@ -128,13 +138,15 @@ __global__ void __launch_bounds__(128) kda_recurrent_kernel(const T* __restrict_
             dec = __expf(-a * (raw > 20.f ? raw : log1pf(__expf(raw))));
           }
           sd[j][at] = dec;
+        } else if (RULE == RULE_WKV) {
+          sd[j][at] = !PAD || e < dk ? __expf(-__expf(((const float*)f)[row * ldf + (long long)h * dk + e] + dt_bias[h * dk + e])) : 1.f;
         }
       }
     }
     for (int idx = tid; idx < nt * KDA_COLS; idx += 128) {
       const int j = idx / KDA_COLS, d = cg * KDA_COLS + idx % KDA_COLS;
       float x = d < dv ? to_f32(v[(long long)(t0 + j) * ld + (long long)h * dv + d]) : 0.f;
-      if (!DELTA) x = to_f32(from_f32<T>(x / (1.f + __expf(-x))));
+      if (RULE == RULE_DECAY) x = to_f32(from_f32<T>(x / (1.f + __expf(-x))));
       sv[j][idx % KDA_COLS] = x;
     }
     if (DELTA && tid < nt) sb[tid] = 1.f / (1.f + __expf(-to_f32(b[(long long)(t0 + tid) * ldb + h])));
@@ -173,6 +185,18 @@ __global__ void __launch_bounds__(128) kda_recurrent_kernel(const T* __restrict_
 #pragma unroll
       for (int i = 0; i < QK / 4; ++i) {
         const float4 kk = kq[i], qv = qq[i];
+        if (RULE == RULE_WKV) {
+          const float4 dd = reinterpret_cast<const float4*>(&sd[KEYED ? j : 0][qtr * QS])[i];
+          o4.x += s_col[4 * i + 0] * qv.x;
+          o4.y += s_col[4 * i + 1] * qv.y;
+          o4.z += s_col[4 * i + 2] * qv.z;
+          o4.w += s_col[4 * i + 3] * qv.w;
+          s_col[4 * i + 0] = s_col[4 * i + 0] * dd.x + kk.x * delta;
+          s_col[4 * i + 1] = s_col[4 * i + 1] * dd.y + kk.y * delta;
+          s_col[4 * i + 2] = s_col[4 * i + 2] * dd.z + kk.z * delta;
+          s_col[4 * i + 3] = s_col[4 * i + 3] * dd.w + kk.w * delta;
+          continue;
+        }
         if (!DELTA) {
           s_col[4 * i + 0] *= fixed;
           s_col[4 * i + 1] *= fixed;
@@ -199,6 +223,7 @@ __global__ void __launch_bounds__(128) kda_recurrent_kernel(const T* __restrict_
         o += __shfl_xor_sync(0xffffffffu, o, 1);
         o += __shfl_xor_sync(0xffffffffu, o, 2);
       }
+      if (RULE == RULE_WKV) o += sb[j] * delta;
       if (owner && qtr == 0) out[((long long)(t0 + j) * heads + h) * dv + col] = from_f32<T>(o);
     }
     __syncthreads();
@@ -235,7 +260,9 @@ int run_rule(int rule, RecArgs<T> p, int num_seqs, int max_q_len, cudaStream_t s
   p.col_groups = (p.dv + KDA_COLS - 1) / KDA_COLS;
   const dim3 grid(p.heads * p.col_groups, num_seqs);
   const bool few = max_q_len <= 4;  // decode rows and verify steps: the row-coalesced mapping
-  PG_CUDA(rule == RULE_SOFTPLUS ? (launch_padded<T, RULE_SOFTPLUS>(p, grid, few, stream)) : (launch_padded<T, RULE_DECAY>(p, grid, few, stream)));
+  PG_CUDA(rule == RULE_SOFTPLUS ? (launch_padded<T, RULE_SOFTPLUS>(p, grid, few, stream))
+          : rule == RULE_WKV    ? (launch_padded<T, RULE_WKV>(p, grid, few, stream))
+                                : (launch_padded<T, RULE_DECAY>(p, grid, few, stream)));
   PG_LAUNCH_CHECK();
   return PG_OK;
 }
@@ -352,6 +379,23 @@ extern "C" int pg_decay_recurrent(const void* q, const void* k, const void* v, l
   RecArgs<bf16> p = {(const bf16*)q, (const bf16*)k, (const bf16*)v, ld, nullptr, 0, nullptr, 0, nullptr, nullptr, (const float*)decay, 0.f,
                      (float*)state, (bf16*)out, (const int*)q_indptr, (const int*)slots, heads, heads, dk, dv, 0, skip_len};
   return run_rule<bf16>(RULE_DECAY, p, num_seqs, max_q_len, stream);
+}
+
+// Linear attention with the decay exp(-exp(f + w0)) per token and key channel (f in f32) and the bonus u [heads, dk] for the
+// current token: o = (S + diag(u) k v^T)^T r, then S <- diag(decay) S + k v^T.
+extern "C" int pg_wkv_recurrent(const void* r, const void* k, const void* v, long long ld, const void* f, long long ldf, const void* w0, const void* u, void* state, void* out, const void* q_indptr,
+                                const void* slots, int num_seqs, int heads, int dk, int dv, int max_q_len, int skip_len, int is_f32, cudaStream_t stream) {
+  PG_REQUIRE(dk >= 1 && dk <= 256 && dv >= 1, "wkv_recurrent: key width %d (at most 256), value width %d", dk, dv);
+  PG_REQUIRE(num_seqs <= 65535, "wkv_recurrent: %d sequences", num_seqs);
+  if (num_seqs == 0) return PG_OK;
+  if (is_f32) {
+    RecArgs<float> p = {(const float*)r, (const float*)k, (const float*)v, ld, f, ldf, nullptr, 0, nullptr, (const float*)w0, (const float*)u, 0.f,
+                        (float*)state, (float*)out, (const int*)q_indptr, (const int*)slots, heads, heads, dk, dv, 0, skip_len};
+    return run_rule<float>(RULE_WKV, p, num_seqs, max_q_len, stream);
+  }
+  RecArgs<bf16> p = {(const bf16*)r, (const bf16*)k, (const bf16*)v, ld, f, ldf, nullptr, 0, nullptr, (const float*)w0, (const float*)u, 0.f,
+                     (float*)state, (bf16*)out, (const int*)q_indptr, (const int*)slots, heads, heads, dk, dv, 0, skip_len};
+  return run_rule<bf16>(RULE_WKV, p, num_seqs, max_q_len, stream);
 }
 
 extern "C" int pg_attnres_mix(const void* cur, long long ld_cur, const void* snaps, long long ld_tok, const void* score_w, void* out, long long ld_out,

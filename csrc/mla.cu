@@ -14,7 +14,10 @@
 //    (multiples of 8) fill the rest of the tile with zeros in shared memory only.  A sliding
 //    window skips the tiles in front of it.  Queries either come rotated, or their rotary part
 //    is turned by f32 tables on its way into the MMA fragments (pairs of neighbouring columns).
-//  * latent_rows: from one token's fused projection row, the RMS-normed query latent (dense) and
+//    A sink per head adds exp(sink) to the softmax's denominator, and the sigmoid of a gate per
+//    (token, head) may multiply the output: both where a row is divided by its sum (or merged).
+//  * latent_rows: from one token's fused projection row, the RMS-normed query latent (dense; none
+//    where queries have no latent) and
 //    the cache row: RMS-normed latent, then the shared key part rotated in pairs with f32 tables.
 //    rotate_pairs_: the same rotation in place on the query columns, for the expanded prefill form.
 //  * latent_attention_plain: the absorbed form on the CUDA cores for f32 and for sizes the tensor-core
@@ -146,9 +149,21 @@ struct MlaParams {
   float scale_log2;
   float* part_o;    // [tokens * heads, splits, C]
   float* part_lse;  // [tokens * heads, splits]
+  const float* sink;    // [H]: exp(sink) is part of a row's denominator (null: none)
+  const bf16* gate;     // [T, >= H] rows of stride ld_gate whose sigmoid multiplies a head's output (null: none)
+  long long ld_gate;
   const int* unit_seq;  // [first_row + T] sequence of each token row
   int first_row;        // number of this launch's first row in the step
 };
+
+// Factor on a row's sum of weighted values: 1 / (sum of weights + sink), times the gate.  `m` and `l`: maximum (log2) and sum.
+__device__ __forceinline__ float row_factor(const MlaParams& p, int t, int head, float m, float l) {
+  if (!(l > 0.f)) return 0.f;
+  if (p.sink) l += exp2f(p.sink[head] * LOG2E - m);
+  float f = 1.f / l;
+  if (p.gate) f /= 1.f + __expf(-__bfloat162float(p.gate[t * p.ld_gate + head]));
+  return f;
+}
 
 // CTA = (token row t, head group of 16, split).  C, R: sizes of the instance; EXACT: they are the problem's.
 template <int C, int R, bool EXACT>
@@ -361,7 +376,7 @@ __global__ void __launch_bounds__(128) mla_attn_kernel(const MlaParams p) {
     const int head = hg * 16 + g + rr * 8;
     if (head >= p.heads) continue;
     const float L = l_run[rr];
-    const float inv = L > 0.f ? 1.f / L : 0.f;
+    const float inv = p.splits == 1 ? row_factor(p, t, head, m_run[rr], L) : L > 0.f ? 1.f / L : 0.f;
     const int d0 = warp * VD + 2 * t4;
     if (p.splits == 1) {
       bf16* dst = p.out + t * p.o_tok + head * p.o_head + d0;
@@ -404,9 +419,10 @@ __global__ void __launch_bounds__(128) mla_merge_kernel(const MlaParams p) {
       if (lane + 32 * i < p.c) acc[i] += f * po[lane + 32 * i];
   }
   bf16* dst = p.out + t * p.o_tok + head * p.o_head;
+  const float inv = row_factor(p, t, head, M, Wsum);
 #pragma unroll
   for (int i = 0; i < C / 32; ++i)
-    if (lane + 32 * i < p.c) dst[lane + 32 * i] = __float2bfloat16(Wsum > 0.f ? acc[i] / Wsum : 0.f);
+    if (lane + 32 * i < p.c) dst[lane + 32 * i] = __float2bfloat16(acc[i] * inv);
 }
 
 // One CTA per token.  z row: [.. zq: qr ..][.. zkv: c + r ..] inside one fused projection row.
@@ -440,8 +456,10 @@ __global__ void __launch_bounds__(256) latent_rows_kernel(const T* __restrict__ 
       store_vec<V>(dst + i * V, f);
     }
   };
-  const float iq = rsqrtf(square_sum(qrow, qr) / (float)qr + eps);
-  write_norm(qrow, q_w, cq + t * qr, qr, iq);
+  if (qr > 0) {
+    const float iq = rsqrtf(square_sum(qrow, qr) / (float)qr + eps);
+    write_norm(qrow, q_w, cq + t * qr, qr, iq);
+  }
   const float ik = rsqrtf(square_sum(krow, c) / (float)c + eps);
   const long long slot = slots[t];
   if (slot < 0 || slot >= num_slots) {
@@ -491,7 +509,8 @@ template <typename T>
 __global__ void __launch_bounds__(128) latent_attention_plain_kernel(const T* __restrict__ q_abs, long long q_tok, long long q_head, const T* __restrict__ q_pe, long long pe_tok, long long pe_head,
                                                                      const float* __restrict__ cos, const float* __restrict__ sin, int max_pos, const T* __restrict__ latent, T* __restrict__ out,
                                                                      long long o_tok, long long o_head, const int* __restrict__ q_indptr, const int* __restrict__ kv_lens, const int* __restrict__ table,
-                                                                     int table_stride, const int* __restrict__ unit_seq, int c, int r, int page_size, float scale, int window) {
+                                                                     int table_stride, const int* __restrict__ unit_seq, int c, int r, int page_size, float scale, int window, const float* __restrict__ sink,
+                                                                     const T* __restrict__ gate, long long ld_gate) {
   PG_PDL_ENTRY();
   extern __shared__ __align__(16) float sm[];
   const int w = c + r;
@@ -552,7 +571,9 @@ __global__ void __launch_bounds__(128) latent_attention_plain_kernel(const T* __
     }
     __syncthreads();
   }
-  const float f = l > 0.f ? 1.f / l : 0.f;
+  if (sink && l > 0.f) l += __expf(sink[h] - m);
+  float f = l > 0.f ? 1.f / l : 0.f;
+  if (gate) f /= 1.f + __expf(-to_f32(gate[t * ld_gate + h]));
 #pragma unroll
   for (int i = 0; i < PL_VMAX; ++i)
     if (tid + 128 * i < c) out[t * o_tok + h * o_head + tid + 128 * i] = from_f32<T>(acc[i] * f);
@@ -615,16 +636,16 @@ extern "C" int pg_mla_attention(const void* q_abs, const void* q_pe, const void*
   PG_REQUIRE(heads % 16 == 0, "mla_attention: heads %d must be a multiple of 16", heads);
   // head-major absorbed queries and outputs, token-major rotated query parts
   return pg_latent_attention(q_abs, c, (long long)tokens * c, q_pe, (long long)heads * rope, rope, nullptr, nullptr, 0, latent, out, c, (long long)tokens * c, q_indptr, kv_lens, table, table_stride, unit_seq, 0,
-                             num_seqs, tokens, heads, c, rope, page_size, scale, 0, splits, part_o, part_lse, stream);
+                             num_seqs, tokens, heads, c, rope, page_size, scale, 0, nullptr, nullptr, 0, splits, part_o, part_lse, stream);
 }
 
 // q_abs, q_pe and out by token / head strides in elements; cos / sin f32 [max_pos, r / 2] turn the q_pe columns (null: they
-// come rotated); window > 0: a row sees its last `window` keys.  Row 0 of this
-// call is row `first_row` of the step that q_indptr and unit_seq describe.
+// come rotated); window > 0: a row sees its last `window` keys; sink f32 [heads] and head_gate bf16 [tokens, >= heads] as in
+// MlaParams (or null).  Row 0 of this call is row `first_row` of the step that q_indptr and unit_seq describe.
 extern "C" int pg_latent_attention(const void* q_abs, long long q_tok, long long q_head, const void* q_pe, long long pe_tok, long long pe_head, const void* cos, const void* sin, int max_pos,
                                    const void* latent, void* out, long long o_tok, long long o_head, const void* q_indptr, const void* kv_lens, const void* table, int table_stride,
-                                   const void* unit_seq, int first_row, int num_seqs, int tokens, int heads, int c, int r, int page_size, float scale, int window, int splits, void* part_o, void* part_lse,
-                                   cudaStream_t stream) {
+                                   const void* unit_seq, int first_row, int num_seqs, int tokens, int heads, int c, int r, int page_size, float scale, int window, const void* sink, const void* head_gate, long long ld_gate,
+                                   int splits, void* part_o, void* part_lse, cudaStream_t stream) {
   PG_REQUIRE(c % 8 == 0 && r % 8 == 0 && c >= 8 && c <= 512 && r >= 0 && r <= 64, "latent_attention: a latent of %d + %d columns is not supported (multiples of 8 up to 512 + 64)", c, r);
   PG_REQUIRE(page_size == 16 || page_size == 32 || page_size == 64, "latent_attention: pages of %d tokens", page_size);
   PG_REQUIRE(q_tok % 2 == 0 && q_head % 2 == 0 && pe_tok % 2 == 0 && pe_head % 2 == 0 && o_tok % 2 == 0 && o_head % 2 == 0, "latent_attention: strides must keep column pairs aligned");
@@ -637,6 +658,7 @@ extern "C" int pg_latent_attention(const void* q_abs, long long q_tok, long long
   p.latent = (const bf16*)latent;
   p.out = (bf16*)out, p.o_tok = o_tok, p.o_head = o_head;
   p.c = c, p.r = r, p.window = window;
+  p.sink = (const float*)sink, p.gate = (const bf16*)head_gate, p.ld_gate = ld_gate;
   p.q_indptr = (const int*)q_indptr;
   p.kv_lens = (const int*)kv_lens;
   p.table = (const int*)table;
@@ -661,14 +683,16 @@ extern "C" int pg_latent_attention(const void* q_abs, long long q_tok, long long
 
 extern "C" int pg_latent_attention_plain(const void* q_abs, long long q_tok, long long q_head, const void* q_pe, long long pe_tok, long long pe_head, const void* cos, const void* sin, int max_pos,
                                          const void* latent, void* out, long long o_tok, long long o_head, const void* q_indptr, const void* kv_lens, const void* table, int table_stride,
-                                         const void* unit_seq, int tokens, int heads, int c, int r, int page_size, float scale, int window, int is_f32, cudaStream_t stream) {
+                                         const void* unit_seq, int tokens, int heads, int c, int r, int page_size, float scale, int window, const void* sink, const void* head_gate, long long ld_gate, int is_f32,
+                                         cudaStream_t stream) {
   PG_REQUIRE(c >= 1 && c <= 128 * PL_VMAX && r >= 0 && r % 2 == 0 && r <= 2048 && heads <= 65535, "latent_attention_plain: %d heads over %d + %d columns", heads, c, r);
   PG_REQUIRE(r == 0 || (cos && sin && max_pos > 0), "latent_attention_plain: rotated columns need their tables");
   if (tokens == 0) return PG_OK;
   const size_t smem = (size_t)(c + r + PL_KEYS) * 4;
 #define PG_LAP(T)                                                                                                                                                                                   \
   launch_pdl(latent_attention_plain_kernel<T>, dim3(tokens, heads), dim3(128), smem, stream, (const T*)q_abs, q_tok, q_head, (const T*)q_pe, pe_tok, pe_head, (const float*)cos, (const float*)sin, \
-             max_pos, (const T*)latent, (T*)out, o_tok, o_head, (const int*)q_indptr, (const int*)kv_lens, (const int*)table, table_stride, (const int*)unit_seq, c, r, page_size, scale, window)
+             max_pos, (const T*)latent, (T*)out, o_tok, o_head, (const int*)q_indptr, (const int*)kv_lens, (const int*)table, table_stride, (const int*)unit_seq, c, r, page_size, scale, window, \
+             (const float*)sink, (const T*)head_gate, ld_gate)
   PG_CUDA(is_f32 ? PG_LAP(float) : PG_LAP(bf16));
 #undef PG_LAP
   PG_LAUNCH_CHECK();
@@ -677,7 +701,7 @@ extern "C" int pg_latent_attention_plain(const void* q_abs, long long q_tok, lon
 
 extern "C" int pg_latent_rows(const void* zq, const void* zkv, long long ld, const void* q_w, const void* kv_w, const void* cos, const void* sin, const void* positions, const void* slots, void* cq,
                               void* latent, int tokens, int qr, int c, int r, int max_pos, long long num_slots, float eps, int is_f32, void* status, cudaStream_t stream) {
-  PG_REQUIRE(qr >= 1 && c >= 1 && r >= 0 && r % 2 == 0 && (r == 0 || (cos && sin && max_pos > 0)), "latent_rows: sizes %d, %d + %d", qr, c, r);
+  PG_REQUIRE(qr >= 0 && c >= 1 && r >= 0 && r % 2 == 0 && (r == 0 || (cos && sin && max_pos > 0)), "latent_rows: sizes %d, %d + %d", qr, c, r);
   if (tokens == 0) return PG_OK;
   const bool v8 = !is_f32 && qr % 8 == 0 && c % 8 == 0 && r % 8 == 0 && ld % 8 == 0 && (((uintptr_t)zq | (uintptr_t)zkv | (uintptr_t)q_w | (uintptr_t)kv_w | (uintptr_t)cq | (uintptr_t)latent) & 15) == 0;
 #define PG_LR(T, V)                                                                                                                                                                                \

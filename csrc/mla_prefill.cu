@@ -12,7 +12,8 @@ namespace {
 // memory), with key tiles of 64 so that Q (2 x 48 KB) and two stages of K (24 KB) and V (16 KB) fit shared memory.  The
 // rotary block of Q and K comes through tensor maps of its own; an instance without it serves layers without positions.
 // Narrower heads are filled with zeros by TMA.  A sliding window drops the key tiles in front of the CTA's first row and
-// masks the tiles its lower edge crosses.  The sigmoid of a gate may multiply the output.
+// masks the tiles its lower edge crosses.  The sigmoid of a gate (per element or per head) may multiply the output, and a sink
+// per head adds its exponential to the softmax's denominator.
 //
 // Reference parity: pegainfer-kernels/csrc/k3/k3_flash_mla_prefill.cu (gather / expand, then a dense SM100 FMHA).
 constexpr int MV_BYTES = BKV2 * 128 * 2; // 16 KB: [2 blocks of 64 columns][64 rows][128 B]
@@ -26,6 +27,8 @@ struct MlaTcParams {
   int head_major;        // order of the two outer coordinates of the query maps: 1 (row, head), 0 (head, row)
   const bf16* gate;      // [T, heads * vdim] rows of stride ld_gate, or null
   long long ld_gate;
+  int gate_cols;         // columns of the gate per head: vdim, or 1 for a gate per (token, head)
+  const float* sink;     // [heads], or null
   float scale_log2;
   uint32_t* status;
 };
@@ -215,10 +218,12 @@ __global__ void __launch_bounds__(THREADS, 1) mla_prefill_tc_kernel(const __grid
       ok = mbar_wait(&sh->o_full[g], (uint32_t)((my_n - 1) & 1), abort_flag);
       tc_fence_after();
     }
-    const float inv = (ok && l > 0.f) ? 1.f / l : 0.f;
+    if (p.sink && l > 0.f) l += exp2f(p.sink[h] * 1.4426950408889634f - m);
+    float inv = (ok && l > 0.f) ? 1.f / l : 0.f;
     const long long row = q0 + row_base + g * 128 + r;
+    if (p.gate && p.gate_cols == 1 && r < rows_g) inv /= 1.f + __expf(-__bfloat162float(p.gate[row * p.ld_gate + h]));
     bf16* dst = p.out + (row * p.heads + h) * p.vdim;
-    const bf16* gate = p.gate ? p.gate + row * p.ld_gate + (long long)h * p.vdim : nullptr;
+    const bf16* gate = p.gate && p.gate_cols > 1 ? p.gate + row * p.ld_gate + (long long)h * p.vdim : nullptr;
 #pragma unroll 1
     for (int c = 0; c < p.vdim; c += 32) {
       uint32_t w[32];
@@ -295,14 +300,16 @@ extern "C" int pg_mla_gather_latent(const void* latent_layer, int page_size, lon
 // Expanded-form latent prefill on tcgen05.  q (unrotated columns) and q_pe (rotated ones) by token / head strides, k and v dense
 // [total_kv] rows of stride ld_kv with heads dim / vdim columns apart, k_pe rows of stride pe_ld; strides in elements,
 // multiples of 8.  kv_lens [num_seqs] counts a sequence's dense rows, which are its last keys; window > 0: a row sees its
-// last `window` keys.  out [T, heads * vdim]; gate (or null) rows of stride ld_gate.  `q_tiles` = sum over the sequences of
+// last `window` keys.  out [T, heads * vdim]; gate (or null) rows of stride ld_gate with gate_cols columns per head (vdim, or 1);
+// sink f32 [heads] (or null).  `q_tiles` = sum over the sequences of
 // ceil(query rows / 256).
 extern "C" int pg_latent_prefill_tc(const void* q, long long q_tok, long long q_head, const void* q_pe, long long pe_tok, long long pe_head, const void* k, const void* v, long long ld_kv, const void* k_pe,
-                                    long long pe_ld, const void* gate, long long ld_gate, void* out, const void* q_indptr, const void* kv_indptr, const void* kv_lens, int num_seqs, int tokens, int total_kv,
-                                    int heads, int dim, int rot, int vdim, float scale, int window, int q_tiles, void* status, cudaStream_t stream) {
+                                    long long pe_ld, const void* gate, long long ld_gate, int gate_cols, const void* sink, void* out, const void* q_indptr, const void* kv_indptr, const void* kv_lens, int num_seqs,
+                                    int tokens, int total_kv, int heads, int dim, int rot, int vdim, float scale, int window, int q_tiles, void* status, cudaStream_t stream) {
   PG_REQUIRE(dim % 8 == 0 && rot % 8 == 0 && vdim % 8 == 0 && dim >= 8 && vdim >= 8 && dim <= 128 && rot >= 0 && rot <= 64 && vdim <= 128,
              "tcgen05 latent prefill takes up to 128 + 64 query / key and 128 value columns (got %d + %d, %d)", dim, rot, vdim);
-  PG_REQUIRE(gate == nullptr || (((uintptr_t)gate & 15) == 0 && ld_gate % 8 == 0), "latent prefill: the gate must start and step on 16-byte boundaries");
+  PG_REQUIRE(gate == nullptr || gate_cols == 1 || gate_cols == vdim, "latent prefill: a gate of %d columns per head", gate_cols);
+  PG_REQUIRE(gate == nullptr || gate_cols == 1 || (((uintptr_t)gate & 15) == 0 && ld_gate % 8 == 0), "latent prefill: the gate must start and step on 16-byte boundaries");
   if (q_tiles == 0 || tokens == 0 || total_kv == 0) return PG_OK;
   CUtensorMap tm_qn, tm_qpe, tm_kn, tm_kpe, tm_v;
   auto map3 = [](CUtensorMap* m, const void* ptr, int cols, long long d1, long long s1, long long d2, long long s2, int b1, int b2) {
@@ -336,6 +343,8 @@ extern "C" int pg_latent_prefill_tc(const void* q, long long q_tok, long long q_
   p.head_major = head_major;
   p.gate = (const bf16*)gate;
   p.ld_gate = ld_gate;
+  p.gate_cols = gate_cols;
+  p.sink = (const float*)sink;
   p.scale_log2 = scale * 1.4426950408889634f;
   p.status = (uint32_t*)status;
   auto smem = [](int blocks) { return 1024 + (size_t)blocks * 128 * (GROUPS * 128 + 2 * BKV2) + 2 * (size_t)MV_BYTES + sizeof(TcSmem) + 64; };
@@ -357,6 +366,6 @@ extern "C" int pg_mla_prefill_tc(const void* q_nope_hm, long long q_nope_head_st
                                  const void* q_indptr, const void* kv_indptr, const void* kv_lens, int num_seqs, int tokens, int total_kv, int heads, int nope, int rope, int vdim,
                                  float scale, int q_tiles, void* status, cudaStream_t stream) {
   PG_REQUIRE(nope == 128 && rope == 64 && vdim == 128, "tcgen05 MLA prefill is built for 128 + 64 query / key and 128 value columns (got %d + %d, %d)", nope, rope, vdim);
-  return pg_latent_prefill_tc(q_nope_hm, 128, q_nope_head_stride, q_pe, (long long)heads * 64, 64, k_nope, v, (long long)heads * 128, (const bf16*)k_pe_rows + pe_col, pe_ld, nullptr, 0, out, q_indptr,
+  return pg_latent_prefill_tc(q_nope_hm, 128, q_nope_head_stride, q_pe, (long long)heads * 64, 64, k_nope, v, (long long)heads * 128, (const bf16*)k_pe_rows + pe_col, pe_ld, nullptr, 0, 0, nullptr, out, q_indptr,
                               kv_indptr, kv_lens, num_seqs, tokens, total_kv, heads, nope, rope, vdim, scale, 0, q_tiles, status, stream);
 }

@@ -10,7 +10,8 @@
 // derived on the device from `offsets`, so the launch shape does not depend on the
 // routing and the kernel can sit inside a captured graph.
 //
-// Two further forms of the bf16 kernel: the squared ReLU on the output (experts without a gate projection), and heads in
+// Further forms of the bf16 kernel: an activation on the output, the squared ReLU (experts without a gate projection) or
+// SiLU(gate) * up over weight rows that alternate (gate_i, up_i), whose two results sit in neighbouring lanes; and heads in
 // the place of experts (pg_head_gemm): every head has the same number of rows, taken from a strided [rows, heads, K]
 // activation through a tensor map of its own and stored strided, so that the per-head products around latent attention
 // read and write token-major buffers; a sigmoid gate may multiply the output.
@@ -68,7 +69,7 @@ struct MoeGemmParams {
   bf16* peer_out[8];
   uint32_t* peer_flags[8];
   int cap, rank, world, site;
-  int relu2;  // y = max(y, 0)^2
+  int act;  // 1: y = max(y, 0)^2; 2: y[:, m / 2] = silu(row m) * row m + 1
   // heads instead of experts: `head_rows` rows each (0: rows come from `offsets`), output of head h at y + h * y_head, and
   // an optional gate[row * ldg + h * g_head + m] whose sigmoid multiplies the output
   int head_rows;
@@ -281,9 +282,16 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant_
         uint32_t v[16];
         tmem_ld16(t_row + c, v);
         tmem_ld_wait();
-        if (m < p.M) {
+        if (p.act == 2) {  // the shuffles run on all lanes, the even ones store
+          bf16* dst = p.y + (long long)(it.row0 + c) * p.ldy + (m >> 1);
+#pragma unroll
+          for (int j = 0; j < 16; ++j) {
+            const float g = __uint_as_float(v[j]), u = __shfl_xor_sync(0xFFFFFFFFu, g, 1);
+            if (!(lane & 1) && m < p.M && c + j < it.rows) dst[j * p.ldy] = __float2bfloat16(g / (1.f + __expf(-g)) * u);
+          }
+        } else if (m < p.M) {
           if (p.scatter_src == nullptr) {
-            if (p.relu2) {
+            if (p.act == 1) {
 #pragma unroll
               for (int j = 0; j < 16; ++j) {
                 const float f = fmaxf(__uint_as_float(v[j]), 0.f);
@@ -493,7 +501,7 @@ struct HeadArgs {
 // `bn` is the token tile (multiple of 16, <= 256): pick it near the expected rows per expert.
 static int moe_gemm_impl(const void* x, long long ldx, long long x_rows, const void* w, const void* scales, int quant, void* y, long long ldy,
                          const void* offsets, int E, int M, int K, int bn, void* status, const void* scatter_src, void* const* peer_out,
-                         void* const* peer_flags, int cap, int rank, int world, int site, cudaStream_t stream, int relu2 = 0, const HeadArgs* heads = nullptr) {
+                         void* const* peer_flags, int cap, int rank, int world, int site, cudaStream_t stream, int act = 0, const HeadArgs* heads = nullptr) {
   PG_REQUIRE(E >= 1 && E <= MAX_EXPERTS, "moe gemm: %d experts not supported (<= %d)", E, MAX_EXPERTS);
   PG_REQUIRE(quant == 0 ? K % 8 == 0 : K % 64 == 0, "moe gemm: K=%d must be a multiple of %d", K, quant == 0 ? 8 : 64);
   PG_REQUIRE(bn >= 16 && bn <= 256 && bn % 16 == 0, "moe gemm: token tile %d must be a multiple of 16 in [16, 256]", bn);
@@ -531,7 +539,7 @@ static int moe_gemm_impl(const void* x, long long ldx, long long x_rows, const v
   p.scales = scales;
   p.offsets = (const int*)offsets;
   p.status = (uint32_t*)status;
-  p.relu2 = relu2;
+  p.act = act;
   if (heads) {
     p.head_rows = (int)x_rows;
     p.y_head = heads->y_head;
@@ -615,10 +623,12 @@ extern "C" int pg_moe_grouped_gemm(const void* x, long long ldx, long long x_row
   return moe_gemm_impl(x, ldx, x_rows, w, scales, quant, y, ldy, offsets, E, M, K, bn, status, nullptr, nullptr, nullptr, 0, 0, 1, 0, stream);
 }
 
-// bf16 experts with the squared ReLU on the output.
-extern "C" int pg_moe_grouped_gemm_relu2(const void* x, long long ldx, long long x_rows, const void* w, void* y, long long ldy, const void* offsets, int E, int M, int K, int bn, void* status,
-                                         cudaStream_t stream) {
-  return moe_gemm_impl(x, ldx, x_rows, w, nullptr, 0, y, ldy, offsets, E, M, K, bn, status, nullptr, nullptr, nullptr, 0, 0, 1, 0, stream, 1);
+// bf16 experts with an activation on the output: 1 the squared ReLU, 2 SiLU(gate) * up over alternating weight rows
+// (y is [rows, M / 2]).
+extern "C" int pg_moe_grouped_gemm_act(const void* x, long long ldx, long long x_rows, const void* w, void* y, long long ldy, const void* offsets, int E, int M, int K, int bn, int act, void* status,
+                                       cudaStream_t stream) {
+  PG_REQUIRE((act == 1 || act == 2) && (act == 1 || M % 2 == 0), "moe gemm: activation %d on %d rows", act, M);
+  return moe_gemm_impl(x, ldx, x_rows, w, nullptr, 0, y, ldy, offsets, E, M, K, bn, status, nullptr, nullptr, nullptr, 0, 0, 1, 0, stream, act);
 }
 
 // y[t, h, :] = x[t, h, :] w[h]^T, w [heads, M, K]; row / head strides in elements; gate (bf16, or null) strided like y.

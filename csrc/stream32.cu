@@ -1,6 +1,11 @@
 // Row kernels around a residual stream that is kept in 32 bits, for bf16 and f32 activations.
 //
 //  * embed_rows: table row -> f32 stream row (+ a copy in the activation type for the next projection).
+//  * embed_pairs_norm: scaled table row plus the row of the pair (previous token, token) -> f32 stream row and its RMS norm.
+//    The previous token of a step's first row comes from the request's slot, which then takes the step's last token.
+//  * residual_norm: the norm before the sublayer.  x += mult * y on the f32 stream, and the RMS norm of the sum, which the
+//    next sublayer reads, in the same pass.  y is a projection's output, or the weighted sum of a token's expert rows plus a
+//    further row times the sigmoid of a number per token (an expert that every token takes).
 //  * post_norm: the norm after the sum.  s = alpha * x + y; x = s / sqrt(mean(s^2) + eps) * w.  The stream x is read and
 //    written in f32, y is a projection's output (f32 or bf16), and the activation-type copy that the next projection
 //    reads is written in the same pass.  Without y and with alpha = 1 it is a plain RMS norm of the stream.
@@ -8,9 +13,9 @@
 //    on the f32 stream, with the activation-type copy of the new stream written in the same pass.  y is a projection's
 //    output, or the weighted sum of a token's expert rows, which is then formed here instead of by a kernel of its own.
 //    With y = x and no sum it is the plain layer norm of the stream.
-//  * gated_row_norm: RMS norm over a row (one head, or all heads of a token at once), times a weight, times the sigmoid
-//    of a gate row that may lie inside a wider projection output.
-//  * glu_rows: silu(gate) * up on f32 rows; softcap_f32: cap * tanh(x / cap) on f32 values.
+//  * gated_row_norm: RMS norm over a row (one head, or all heads of a token at once), times a weight, times the sigmoid or
+//    the SiLU of a gate row that may lie inside a wider projection output.
+//  * glu_rows: silu(gate) * up or gelu(gate) * up on f32 rows; softcap_f32: cap * tanh(x / cap) on f32 values; tanh_rows.
 //  * gemm_simt: y = x w^T on the CUDA cores with f32 accumulation, for f32 operands (the 32-bit mode) and for bf16
 //    problems whose rows the TMA kernels cannot address (an inner size that is not a multiple of 8).  head_gemm_simt is the
 //    same per attention head (strided operands, sigmoid gate on the output), expert_gemm_simt per expert over sorted rows.
@@ -35,6 +40,73 @@ __global__ void __launch_bounds__(256) embed_rows_kernel(const TI* __restrict__ 
     const float v = to_f32(table[id * ldt + i]);
     if (x) x[(long long)t * width + i] = v;
     if (xt) xt[(long long)t * ldxt + i] = from_f32<TO>(v);
+  }
+}
+
+// One CTA per row.  `unit_seq[t]`: sequence of row t.  The CTA of a sequence's first row is the only one that touches its slot.
+template <typename T, typename TO, int V>
+__global__ void __launch_bounds__(256) embed_pairs_norm_kernel(const T* __restrict__ table, long long ldt, const T* __restrict__ pairs, long long ldp, const int* __restrict__ ids, const int* __restrict__ unit_seq,
+                                                               const int* __restrict__ q_indptr, const int* __restrict__ slots, int* __restrict__ carried, float scale, long long buckets, long long mul_prev,
+                                                               long long mul_cur, const float* __restrict__ w, float* __restrict__ x, TO* __restrict__ xt, int width, long long rows, float eps,
+                                                               uint32_t* status) {
+  PG_PDL_ENTRY();
+  __shared__ float red[32];
+  __shared__ long long s_pair;
+  const int t = blockIdx.x;
+  long long id = ids[t];
+  if (threadIdx.x == 0) {
+    if (id < 0 || id >= rows) atomicCAS(status, PG_ST_OK, PG_ST_BOUNDS | (56u << 8));
+    if (pairs) {
+      const int b = unit_seq[t], q0 = q_indptr[b], slot = slots[b];
+      long long prev = t > q0 ? (long long)ids[t - 1] : slot >= 0 ? (long long)carried[slot] - 1 : -1;
+      if (t == q0 && slot >= 0) carried[slot] = ids[q_indptr[b + 1] - 1] + 1;
+      const long long sum = prev * mul_prev + (id < 0 ? 0 : id) * mul_cur;
+      s_pair = prev < 0 || sum < 0 ? buckets : sum % buckets;
+    }
+  }
+  if (id < 0 || id >= rows) id = 0;
+  __syncthreads();
+  const T* row = table + id * ldt;
+  const T* pair = pairs ? pairs + s_pair * ldp : nullptr;
+  constexpr int KEEP = 8;
+  const int nv = width / V;
+  float s[KEEP][V], ss = 0.f;
+  auto sum_at = [&](int i, float* o) {
+    load_vec<V>(row + i * V, o);
+#pragma unroll
+    for (int j = 0; j < V; ++j) o[j] *= scale;
+    if (pair) {
+      float f[V];
+      load_vec<V>(pair + i * V, f);
+#pragma unroll
+      for (int j = 0; j < V; ++j) o[j] += f[j];
+    }
+#pragma unroll
+    for (int j = 0; j < V; ++j) ss += o[j] * o[j];
+    store_vec<V>(x + (long long)t * width + i * V, o);
+  };
+#pragma unroll
+  for (int k = 0; k < KEEP; ++k)
+    if (threadIdx.x + k * 256 < nv) sum_at(threadIdx.x + k * 256, s[k]);
+  for (int i = threadIdx.x + KEEP * 256; i < nv; i += 256) {  // wider rows: read back below
+    float o[V];
+    sum_at(i, o);
+  }
+  const float inv = rsqrtf(block_sum(ss, red) / (float)width + eps);
+  auto put = [&](int i, const float* o) {
+    float wf[V], r[V];
+    load_vec<V>(w + i * V, wf);
+#pragma unroll
+    for (int j = 0; j < V; ++j) r[j] = o[j] * inv * wf[j];
+    store_vec<V>(xt + (long long)t * width + i * V, r);
+  };
+#pragma unroll
+  for (int k = 0; k < KEEP; ++k)
+    if (threadIdx.x + k * 256 < nv) put(threadIdx.x + k * 256, s[k]);
+  for (int i = threadIdx.x + KEEP * 256; i < nv; i += 256) {
+    float o[V];
+    load_vec<V>(x + (long long)t * width + i * V, o);
+    put(i, o);
   }
 }
 
@@ -128,6 +200,63 @@ struct RowSource {
   }
 };
 
+// One CTA per row.  x += mult * (src row + sigmoid(extra_gate[row]) * extra row); xt = rms_norm(x) * w.
+template <typename TY, typename TO, int V>
+__global__ void __launch_bounds__(256) residual_norm_kernel(const RowSource<TY> src, const void* __restrict__ extra, int extra_f32, long long lde, const float* __restrict__ extra_gate, long long ldg,
+                                                            float* __restrict__ x, float mult, const float* __restrict__ w, TO* __restrict__ xt, long long ldxt, int width, float eps) {
+  PG_PDL_ENTRY();
+  __shared__ float red[32];
+  constexpr int KEEP = 8;
+  const long long row = blockIdx.x;
+  const int nv = width / V;
+  float* xr = x + row * width;
+  const float gate = extra ? (extra_gate ? 1.f / (1.f + __expf(-extra_gate[row * ldg])) : 1.f) : 0.f;
+  float s[KEEP][V], ss = 0.f;
+  auto sum_at = [&](int i, float* o) {
+    float y[V];
+    src.template load<V>(row, i * V, y);
+    if (extra) {
+      float f[V];
+      if (extra_f32)
+        load_vec<V>(reinterpret_cast<const float*>(extra) + row * lde + i * V, f);
+      else
+        load_vec<V>(reinterpret_cast<const bf16*>(extra) + row * lde + i * V, f);
+#pragma unroll
+      for (int j = 0; j < V; ++j) y[j] = fmaf(gate, f[j], y[j]);
+    }
+    load_vec<V>(xr + i * V, o);
+#pragma unroll
+    for (int j = 0; j < V; ++j) {
+      o[j] = fmaf(mult, y[j], o[j]);
+      ss += o[j] * o[j];
+    }
+    store_vec<V>(xr + i * V, o);
+  };
+#pragma unroll
+  for (int k = 0; k < KEEP; ++k)
+    if (threadIdx.x + k * 256 < nv) sum_at(threadIdx.x + k * 256, s[k]);
+  for (int i = threadIdx.x + KEEP * 256; i < nv; i += 256) {  // wider rows: read back below
+    float o[V];
+    sum_at(i, o);
+  }
+  const float inv = rsqrtf(block_sum(ss, red) / (float)width + eps);
+  auto put = [&](int i, const float* o) {
+    float wf[V], r[V];
+    load_vec<V>(w + i * V, wf);
+#pragma unroll
+    for (int j = 0; j < V; ++j) r[j] = o[j] * inv * wf[j];
+    store_vec<V>(xt + row * ldxt + i * V, r);
+  };
+#pragma unroll
+  for (int k = 0; k < KEEP; ++k)
+    if (threadIdx.x + k * 256 < nv) put(threadIdx.x + k * 256, s[k]);
+  for (int i = threadIdx.x + KEEP * 256; i < nv; i += 256) {
+    float o[V];
+    load_vec<V>(xr + i * V, o);
+    put(i, o);
+  }
+}
+
 // One CTA per row.  x (f32 stream) is read and written; x == nullptr: only the norm goes to xt.
 template <typename TY, typename TO, int V>
 __global__ void __launch_bounds__(256) add_layer_norm_kernel(const RowSource<TY> src, float* __restrict__ x, const float* __restrict__ w, TO* __restrict__ xt, long long ldxt, int width, float eps) {
@@ -196,7 +325,7 @@ __global__ void __launch_bounds__(256) add_layer_norm_kernel(const RowSource<TY>
 // TPR threads per row (16, 32 or 256); row r = token * heads + head; the gate row of (token, head) is gate + token * ldg + head * dim.
 template <typename T, int V, int TPR>
 __global__ void __launch_bounds__(256) gated_row_norm_kernel(const T* __restrict__ x, const T* __restrict__ gate, long long ldg, const float* __restrict__ w, T* __restrict__ y, long long rows, int heads, int dim,
-                                                             float eps) {
+                                                             float eps, int silu, int w_heads) {
   PG_PDL_ENTRY();
   __shared__ float red[32];
   const long long row = TPR == 256 ? (long long)blockIdx.x : (long long)blockIdx.x * (256 / TPR) + threadIdx.x / TPR;
@@ -204,6 +333,7 @@ __global__ void __launch_bounds__(256) gated_row_norm_kernel(const T* __restrict
   const bool live = row < rows;  // with TPR == 256 the grid has no spare blocks
   const T* xr = x + row * dim;
   const T* gr = gate + (row / heads) * ldg + (row % heads) * dim;
+  if (w_heads) w += (row % heads) * dim;  // a weight per head
   constexpr int KEEP = 4;
   const int nv = live ? dim / V : 0;
   float f[KEEP][V], ss = 0.f;
@@ -234,7 +364,7 @@ __global__ void __launch_bounds__(256) gated_row_norm_kernel(const T* __restrict
     load_vec<V>(gr + i * V, g);
     load_vec<V>(w + i * V, wf);
 #pragma unroll
-    for (int j = 0; j < V; ++j) r[j] = o[j] * inv * wf[j] / (1.f + __expf(-g[j]));
+    for (int j = 0; j < V; ++j) r[j] = o[j] * inv * wf[j] * (silu ? g[j] : 1.f) / (1.f + __expf(-g[j]));
     store_vec<V>(y + row * dim + i * V, r);
   };
 #pragma unroll
@@ -249,14 +379,20 @@ __global__ void __launch_bounds__(256) gated_row_norm_kernel(const T* __restrict
   }
 }
 
-__global__ void glu_rows_kernel(const float* __restrict__ gu, float* __restrict__ out, int rows, int inter, long long ldin) {
+__global__ void glu_rows_kernel(const float* __restrict__ gu, float* __restrict__ out, int rows, int inter, long long ldin, int gelu) {
   PG_PDL_ENTRY();
   const long long total = (long long)rows * inter;
   for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (long long)gridDim.x * blockDim.x) {
     const long long r = i / inter, c = i % inter;
     const float g = gu[r * ldin + c], u = gu[r * ldin + inter + c];
-    out[i] = g / (1.f + __expf(-g)) * u;
+    out[i] = glu_act(g, gelu) * u;
   }
+}
+
+template <typename T>
+__global__ void tanh_rows_kernel(const T* __restrict__ x, T* __restrict__ y, long long n) {
+  PG_PDL_ENTRY();
+  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x) y[i] = from_f32<T>(tanh_full(to_f32(x[i])));
 }
 
 __global__ void softcap_f32_kernel(const float* __restrict__ x, float* __restrict__ y, long long n, float cap) {
@@ -329,10 +465,11 @@ __global__ void __launch_bounds__(256) head_gemm_simt_kernel(const T* __restrict
 }
 
 // Rows sorted by expert: y[r] = act(x[src(r)] w[e(r)]^T), src(r) = sorted_src[r] / k (token of the route) or r itself.
+// act: 0 none, 1 squared ReLU, 2 SiLU(gate) * up over weight rows that alternate (gate_i, up_i), y [rows, M / 2].
 // Grid y counts 64-row tiles of all experts; a tile finds its expert by walking the offsets.
 template <typename T>
 __global__ void __launch_bounds__(256) expert_gemm_simt_kernel(const T* __restrict__ x, long long ldx, const int* __restrict__ sorted_src, int k, const T* __restrict__ w, T* __restrict__ y,
-                                                               const int* __restrict__ offsets, int E, int M, int K, int relu2) {
+                                                               const int* __restrict__ offsets, int E, int M, int K, int act) {
   PG_PDL_ENTRY();
   __shared__ int s_e, s_row, s_end;
   if (threadIdx.x == 0) {
@@ -361,7 +498,11 @@ __global__ void __launch_bounds__(256) expert_gemm_simt_kernel(const T* __restri
       const int t = t0 + ty * 4 + i, m = m0 + tx * 4 + j;
       if (t >= end || m >= M) continue;
       float v = acc[i][j];
-      if (relu2) v = v > 0.f ? v * v : 0.f;
+      if (act == 2) {
+        if (!(j & 1)) y[(long long)t * (M / 2) + m / 2] = from_f32<T>(glu_act(v, false) * acc[i][j | 1]);
+        continue;
+      }
+      if (act == 1) v = v > 0.f ? v * v : 0.f;
       y[(long long)t * M + m] = from_f32<T>(v);
     }
 }
@@ -456,6 +597,61 @@ extern "C" int pg_post_norm(const void* y, int y_f32, long long ldy, const void*
   return PG_OK;
 }
 
+// table and pairs of one type; x f32 [tokens, width], xt [tokens, width]; carried int32 per slot: 1 + the previous token (0: none).
+extern "C" int pg_embed_pairs_norm(const void* table, int table_f32, long long ldt, const void* pairs, long long ldp, const void* ids, const void* unit_seq, const void* q_indptr, const void* slots, void* carried,
+                                   float scale, long long buckets, long long mul_prev, long long mul_cur, const void* w, void* x, void* xt, int xt_f32, int tokens, int width, long long rows, float eps,
+                                   void* status, cudaStream_t stream) {
+  PG_REQUIRE(pairs == nullptr || (buckets >= 1 && mul_prev >= 0 && mul_cur >= 0 && mul_prev < (1ll << 31) && mul_cur < (1ll << 31) && carried && unit_seq && q_indptr && slots),
+             "embed_pairs: %lld buckets, multipliers %lld and %lld", buckets, mul_prev, mul_cur);
+  if (tokens == 0) return PG_OK;
+  const int ib = table_f32 ? 4 : 2, ob = xt_f32 ? 4 : 2;
+  const bool v4 = width % 4 == 0 && al(table, 4 * ib) && ldt % 4 == 0 && (!pairs || (al(pairs, 4 * ib) && ldp % 4 == 0)) && al(w, 16) && al(x, 16) && al(xt, 4 * ob);
+#define PG_EP(T, TO, V)                                                                                                                                                                            \
+  launch_pdl(embed_pairs_norm_kernel<T, TO, V>, dim3(tokens), dim3(256), (size_t)0, stream, (const T*)table, ldt, (const T*)pairs, ldp, (const int*)ids, (const int*)unit_seq, (const int*)q_indptr, \
+             (const int*)slots, (int*)carried, scale, buckets, mul_prev, mul_cur, (const float*)w, (float*)x, (TO*)xt, width, rows, eps, (uint32_t*)status)
+#define PG_EP2(T, TO) (v4 ? PG_EP(T, TO, 4) : PG_EP(T, TO, 1))
+  if (table_f32)
+    PG_CUDA(xt_f32 ? PG_EP2(float, float) : PG_EP2(float, bf16));
+  else
+    PG_CUDA(xt_f32 ? PG_EP2(bf16, float) : PG_EP2(bf16, bf16));
+#undef PG_EP2
+#undef PG_EP
+  PG_LAUNCH_CHECK();
+  return PG_OK;
+}
+
+// y as in pg_add_layer_norm; extra (or null): a further row per token, times the sigmoid of extra_gate[token * ldg] (f32).
+extern "C" int pg_residual_norm(const void* y, int y_f32, long long ldy, const void* pos, const void* weights, int k, const void* extra, int extra_f32, long long lde, const void* extra_gate, long long ldg,
+                                void* x, float mult, const void* w, void* xt, int xt_f32, long long ldxt, int tokens, int width, float eps, cudaStream_t stream) {
+  PG_REQUIRE(y != nullptr && w != nullptr && x != nullptr && xt != nullptr, "residual_norm: rows, the stream, the norm weight and a destination are required");
+  PG_REQUIRE((pos == nullptr) == (weights == nullptr) && (pos == nullptr || k >= 1), "residual_norm: row positions and weights come together");
+  if (tokens == 0) return PG_OK;
+  const int yb = y_f32 ? 4 : 2, tb = xt_f32 ? 4 : 2, eb = extra_f32 ? 4 : 2;
+  const bool v4 = width % 4 == 0 && al(w, 16) && al(x, 16) && ldy % 4 == 0 && al(y, 4 * yb) && ldxt % 4 == 0 && al(xt, 4 * tb) && (!extra || (lde % 4 == 0 && al(extra, 4 * eb)));
+#define PG_RN(TY, TO, V)                                                                                                                                                                           \
+  launch_pdl(residual_norm_kernel<TY, TO, V>, dim3(tokens), dim3(256), (size_t)0, stream, RowSource<TY>{(const TY*)y, ldy, (const int*)pos, (const float*)weights, k}, extra, extra_f32, lde,       \
+             (const float*)extra_gate, ldg, (float*)x, mult, (const float*)w, (TO*)xt, ldxt, width, eps)
+#define PG_RN2(TY, TO) (v4 ? PG_RN(TY, TO, 4) : PG_RN(TY, TO, 1))
+  if (y_f32)
+    PG_CUDA(xt_f32 ? PG_RN2(float, float) : PG_RN2(float, bf16));
+  else
+    PG_CUDA(xt_f32 ? PG_RN2(bf16, float) : PG_RN2(bf16, bf16));
+#undef PG_RN2
+#undef PG_RN
+  PG_LAUNCH_CHECK();
+  return PG_OK;
+}
+
+extern "C" int pg_tanh_rows(const void* x, void* y, long long n, int is_f32, cudaStream_t stream) {
+  if (n == 0) return PG_OK;
+  long long blocks = (n + 255) / 256;
+  if (blocks > 148 * 16) blocks = 148 * 16;
+  PG_CUDA(is_f32 ? launch_pdl(tanh_rows_kernel<float>, dim3((unsigned)blocks), dim3(256), (size_t)0, stream, (const float*)x, (float*)y, n)
+                 : launch_pdl(tanh_rows_kernel<bf16>, dim3((unsigned)blocks), dim3(256), (size_t)0, stream, (const bf16*)x, (bf16*)y, n));
+  PG_LAUNCH_CHECK();
+  return PG_OK;
+}
+
 // y: [tokens, ldy] rows, or with pos / weights [tokens, k] the expert rows that pos points into (their weighted sum is the
 // token's y).  x: f32 stream, updated in place (null: none, and then the norm itself goes to xt).
 extern "C" int pg_add_layer_norm(const void* y, int y_f32, long long ldy, const void* pos, const void* weights, int k, void* x, const void* w, void* xt, int xt_f32, long long ldxt, int tokens, int width,
@@ -479,14 +675,15 @@ extern "C" int pg_add_layer_norm(const void* y, int y_f32, long long ldy, const 
   return PG_OK;
 }
 
-extern "C" int pg_gated_row_norm(const void* x, const void* gate, long long ldg, const void* w, void* y, int tokens, int heads, int dim, float eps, int is_f32, cudaStream_t stream) {
+extern "C" int pg_gated_row_norm(const void* x, const void* gate, long long ldg, const void* w, void* y, int tokens, int heads, int dim, float eps, int silu, int w_heads, int is_f32,
+                                 cudaStream_t stream) {
   if (tokens == 0) return PG_OK;
   const long long rows = (long long)tokens * heads;
   const bool wide = dim > 512;
   const bool v8 = !is_f32 && dim % 8 == 0 && ldg % 8 == 0 && al(x, 16) && al(gate, 16) && al(w, 16) && al(y, 16);
   const bool half = v8 && dim <= 128;  // a half warp covers the row with one access per lane
   const dim3 grid((unsigned)(wide ? rows : half ? (rows + 15) / 16 : (rows + 7) / 8));
-#define PG_GRN(T, V, TPR) launch_pdl(gated_row_norm_kernel<T, V, TPR>, grid, dim3(256), (size_t)0, stream, (const T*)x, (const T*)gate, ldg, (const float*)w, (T*)y, rows, heads, dim, eps)
+#define PG_GRN(T, V, TPR) launch_pdl(gated_row_norm_kernel<T, V, TPR>, grid, dim3(256), (size_t)0, stream, (const T*)x, (const T*)gate, ldg, (const float*)w, (T*)y, rows, heads, dim, eps, silu, w_heads)
   if (is_f32) {
     PG_CUDA(wide ? PG_GRN(float, 1, 256) : PG_GRN(float, 1, 32));
   } else {
@@ -500,11 +697,11 @@ extern "C" int pg_gated_row_norm(const void* x, const void* gate, long long ldg,
   return PG_OK;
 }
 
-extern "C" int pg_glu_rows_f32(const void* gu, void* out, int rows, int inter, long long ldin, cudaStream_t stream) {
+extern "C" int pg_glu_rows_f32(const void* gu, void* out, int rows, int inter, long long ldin, int gelu, cudaStream_t stream) {
   if (rows == 0 || inter == 0) return PG_OK;
   long long blocks = ((long long)rows * inter + 255) / 256;
   if (blocks > 148 * 16) blocks = 148 * 16;
-  PG_CUDA(launch_pdl(glu_rows_kernel, dim3((unsigned)blocks), dim3(256), (size_t)0, stream, (const float*)gu, (float*)out, rows, inter, ldin));
+  PG_CUDA(launch_pdl(glu_rows_kernel, dim3((unsigned)blocks), dim3(256), (size_t)0, stream, (const float*)gu, (float*)out, rows, inter, ldin, gelu));
   PG_LAUNCH_CHECK();
   return PG_OK;
 }
@@ -545,12 +742,13 @@ extern "C" int pg_head_gemm_simt(const void* x, long long ldx, long long x_head,
   return PG_OK;
 }
 
-extern "C" int pg_expert_gemm_simt(const void* x, long long ldx, const void* sorted_src, int k, const void* w, void* y, const void* offsets, int routes, int E, int M, int K, int relu2, int is_f32,
+extern "C" int pg_expert_gemm_simt(const void* x, long long ldx, const void* sorted_src, int k, const void* w, void* y, const void* offsets, int routes, int E, int M, int K, int act, int is_f32,
                                    cudaStream_t stream) {
+  PG_REQUIRE(act != 2 || M % 2 == 0, "expert_gemm_simt: %d rows are not pairs of gate and up", M);
   if (routes == 0) return PG_OK;
   const dim3 grid((M + 63) / 64, (routes + 63) / 64 + (E < routes ? E : routes));
   PG_REQUIRE(M > 0 && K > 0 && grid.y <= 65535u, "expert_gemm_simt: %d routes, %d x %d", routes, M, K);
-#define PG_EG(T) launch_pdl(expert_gemm_simt_kernel<T>, grid, dim3(256), (size_t)0, stream, (const T*)x, ldx, (const int*)sorted_src, k, (const T*)w, (T*)y, (const int*)offsets, E, M, K, relu2)
+#define PG_EG(T) launch_pdl(expert_gemm_simt_kernel<T>, grid, dim3(256), (size_t)0, stream, (const T*)x, ldx, (const int*)sorted_src, k, (const T*)w, (T*)y, (const int*)offsets, E, M, K, act)
   PG_CUDA(is_f32 ? PG_EG(float) : PG_EG(bf16));
 #undef PG_EG
   PG_LAUNCH_CHECK();

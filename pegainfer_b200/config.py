@@ -24,7 +24,9 @@ class MixerSpec:
     the recurrent and latent ones), ``"lightning"`` (fixed decay per head), ``"channel_delta"`` (gated delta rule with a decay
     per key channel; ``conv`` taps, low-rank decay and output-gate projections of the given ranks) or ``"latent"`` (attention
     over a cached latent of ``kv_rank`` columns and, with ``rot_dims``, a shared rotated key part; queries through a latent of
-    ``q_rank``; a sliding window and an element-wise output gate are optional)."""
+    ``q_rank``, or straight from the stream without one; a sliding window, an element-wise or per-head output gate and a sink
+    are optional) or ``"wkv"`` (token-shift mixes, a decay per key channel from a low-rank projection of ``decay_rank``, a bonus
+    for the current token)."""
 
     kind: str
     heads: int
@@ -45,31 +47,46 @@ class MixerSpec:
     window: int = 0  # a position sees itself and the window - 1 before it (0: all before it)
     out_gate: bool = False
     yarn: tuple = ()  # (factor, original, fast, slow) of the rotation, or none
+    head_gate: bool = False  # latent: the sigmoid of one number per head multiplies the head's output
+    sink: bool = False  # latent: a learned number per head in the softmax's denominator
+    head_norm: bool = False  # attention: query and key norms per head (False: over the whole projection)
+    values_are_keys: bool = False  # attention: no value projection, the values are the projected keys before their norm
+    q_temp: tuple = ()  # attention: (coef, every): queries at position p times 1 + coef * ln(floor((p + 1) / every) + 1)
 
 
 @dataclass(frozen=True)
 class ExpertsSpec:
-    """Mixture-of-experts feed-forward: softmax scores over ``experts``, the ``top`` best of the ``keep`` best of ``groups``
-    groups of neighbours (a group counts as its best expert), weights not renormalised; an expert of width ``ff`` is an up
-    projection, the squared ReLU and a down projection."""
+    """Mixture-of-experts feed-forward: ``scoring`` (softmax or sigmoid) over ``experts``, the ``top`` best of the ``keep`` best
+    of ``groups`` groups of neighbours (a group counts as its best expert); with ``correction`` a learned number per expert is
+    added for the choice only; the chosen scores are the weights, divided by their sum with ``norm`` and times ``scale``.  An
+    expert of width ``ff`` is an up projection, the squared ReLU and a down projection (``act`` relu2), or gate and up
+    projections with SiLU (``act`` swiglu).  ``shared_ff``: width of an expert that runs for every token, times the sigmoid of
+    one number per token (0: none)."""
 
     experts: int
     top: int
     ff: int
     groups: int = 1
     keep: int = 1
+    scoring: str = "softmax"
+    correction: bool = False
+    norm: bool = False
+    scale: float = 1.0
+    act: str = "relu2"
+    shared_ff: int = 0
 
 
 @dataclass(frozen=True)
 class LayerSpec:
     mixer: MixerSpec
-    ff: int = 0  # width of the SwiGLU feed-forward (0: the layer has none)
+    ff: int = 0  # width of the gated feed-forward (0: the layer has none)
     moe: Optional[ExpertsSpec] = None
+    act: str = "silu"  # of the feed-forward's gate: silu or gelu_tanh
 
 
 @dataclass
 class ModelConfig:
-    family: str = "qwen3"  # qwen3 | qwen35 | deepseek_v2 | kimi_k2 | glm_dsa | gemma4 | kimi_k3 | nemipel | vekalorn
+    family: str = "qwen3"  # qwen3 | qwen35 | deepseek_v2 | kimi_k2 | glm_dsa | gemma4 | kimi_k3 | nemipel | vekalorn | zeripel
     vocab_size: int = 1024
     hidden_size: int = 256
     num_layers: int = 2
@@ -137,10 +154,14 @@ class ModelConfig:
     attn_res_block: int = 0
     kda_gate_rank: int = 0
     kda_gate_lower_bound: float = -5.0
-    # families whose layers are listed one by one (Nemipel, Vekalorn lines): the mixer and feed-forward of every layer, the factor on
+    # families whose layers are listed one by one (Nemipel, Vekalorn, Zeripel lines): the mixer and feed-forward of every layer, the factor on
     # the stream in the norm after the sum; final_logit_softcapping caps the logits
     layer_specs: tuple = ()
     postln_alpha: float = 1.0
+    # Zeripel line: factor on the token embedding, table of token pairs (buckets, mul_prev, mul_cur), factor on a sublayer's output
+    embed_scale: float = 1.0
+    bigram: tuple = ()
+    residual_mult: float = 1.0
 
     # -- derived ---------------------------------------------------------------
     @property
@@ -315,6 +336,33 @@ PRESETS["tiny-vekalorn"] = _vekalorn(88, 256, 3, 40, 48, 24, 8, 32, 20, ExpertsS
 PRESETS["small-vekalorn"] = _vekalorn(1024, 4096, 16, 512, 512, 128, 64, 128, 256, ExpertsSpec(16, 4, 512, 4, 2), 2, max_position=8192)
 # layers of a mid-size latent-attention mixture of experts, for benchmarks (not a released configuration)
 PRESETS["vekalorn-16b-shape"] = _vekalorn(2048, 102400, 16, 1536, 512, 128, 64, 128, 1024, ExpertsSpec(64, 6, 2112, 8, 4), 9)
+
+
+def _zeripel(width: int, vocab: int, ff: int, heads: int, kv_heads: int, dim: int, kv_rank: int, nope: int, rot: int, vdim: int, rec_heads: int, rec_dim: int, rank: int, experts: ExpertsSpec,
+             periods: int, **kw) -> ModelConfig:
+    """A Zeripel stack of ``periods`` x (latent attention, latent attention over the same cache, WKV, attention); the first
+    layer's feed-forward is dense."""
+    latent = MixerSpec("latent", heads, nope, vdim, scale=(nope + rot) ** -0.5, rot_dims=rot, rot_base=1e5, kv_rank=kv_rank, head_gate=True, sink=True)
+    wkv = MixerSpec("wkv", rec_heads, rec_dim, rec_dim, decay_rank=rank)
+    attn = MixerSpec("attention", heads, dim, dim, kv_heads=kv_heads, scale=dim ** -0.5, head_norm=True, values_are_keys=True, q_temp=(0.1, 4096))
+    layers = []
+    for n in range(periods):
+        layers += [LayerSpec(m, moe=experts) for m in (latent, replace(latent, kv_from=4 * n), wkv, attn)]
+    layers[0] = LayerSpec(latent, ff, act="gelu_tanh")
+    base = dict(family="zeripel", vocab_size=vocab, hidden_size=width, num_layers=len(layers), num_q_heads=heads, num_kv_heads=kv_heads, head_dim=dim, intermediate_size=ff, rms_eps=1e-6, qk_norm=False,
+                layer_specs=tuple(layers), embed_scale=width ** 0.5, bigram=(vocab * 2 - 3, 31, 5), residual_mult=0.5, max_position=65536)
+    base.update(kw)
+    return ModelConfig(**base)
+
+
+def _zeripel_experts(experts: int, top: int, ff: int, shared_ff: int, scale: float) -> ExpertsSpec:
+    return ExpertsSpec(experts, top, ff, scoring="sigmoid", correction=True, norm=True, scale=scale, act="swiglu", shared_ff=shared_ff)
+
+
+PRESETS["tiny-zeripel"] = _zeripel(80, 256, 112, 4, 2, 24, 40, 16, 8, 32, 3, 16, 12, _zeripel_experts(10, 2, 24, 40, 2.0), 1, max_position=4096)
+PRESETS["small-zeripel"] = _zeripel(1024, 4096, 2048, 16, 4, 128, 512, 128, 64, 128, 8, 128, 64, _zeripel_experts(16, 4, 512, 512, 2.5), 2, max_position=8192)
+# layers of a mid-size hybrid mixture of experts, for benchmarks (not a released configuration)
+PRESETS["zeripel-16b-shape"] = _zeripel(2048, 102400, 8192, 16, 4, 128, 512, 128, 64, 128, 16, 128, 64, _zeripel_experts(64, 6, 1408, 2816, 2.5), 7)
 PRESETS["small-glm-fp8"] = replace(PRESETS["small-glm"], expert_quant="fp8_block128", dense_quant="fp8_block128")
 for _name in ("tiny-dsv2", "small-dsv2", "dsv2-lite"):
     if _name in PRESETS:
@@ -329,7 +377,7 @@ def preset(name: str, **overrides) -> ModelConfig:
 
 def detect_family(cfg: dict) -> str:
     """Map a ``config.json`` to a model line (exactly one line must claim it)."""
-    if cfg.get("architecture") in ("Nemipel", "Vekalorn"):
+    if cfg.get("architecture") in ("Nemipel", "Vekalorn", "Zeripel"):
         return cfg["architecture"].lower()
     mt = cfg.get("model_type", "")
     archs = " ".join(cfg.get("architectures", []))
@@ -505,6 +553,89 @@ def vekalorn_to_json(cfg: ModelConfig) -> dict:
     return out
 
 
+def _zeripel_mixer(i: int, kind: str, m: dict, layers: list) -> MixerSpec:
+    if kind == "wkv":
+        return MixerSpec("wkv", m["heads"], m["dim"], m["dim"])
+    if kind == "attention":
+        if m.get("vdim", m["dim"]) != m["dim"]:
+            raise ValueError(f"layer {i}: values of {m['vdim']} columns, which are keys of {m['dim']}")
+        if m["heads"] % m["kv_heads"]:
+            raise ValueError(f"layer {i}: {m['heads']} query heads over {m['kv_heads']} key heads")
+        t = m.get("q_temp")
+        if t and (t["every"] != int(t["every"]) or t["every"] < 1):
+            raise ValueError(f"layer {i}: the query temperature steps every {t['every']} positions")
+        return MixerSpec("attention", m["heads"], m["dim"], m["dim"], kv_heads=m["kv_heads"], scale=float(m["scale"]), head_norm=True, values_are_keys=True,
+                         q_temp=(float(t["coef"]), int(t["every"])) if t else ())
+    if kind == "latent_attention":
+        rot, src = m.get("rot") or {}, m.get("kv_from")
+        if rot.get("dims", m["rot_dim"]) != m["rot_dim"] or m["rot_dim"] % 2:
+            raise ValueError(f"layer {i}: the rotated part has {m['rot_dim']} columns, {rot.get('dims')} are to be rotated")
+        spec = MixerSpec("latent", m["heads"], m["dim"], m["vdim"], scale=float(m["scale"]), rot_dims=m["rot_dim"], rot_base=float(rot.get("base", 1e4)), kv_rank=m["kv_rank"],
+                         kv_from=-1 if src is None else src, head_gate=True, sink=True)
+        if src is not None:
+            own = layers[src].mixer if 0 <= src < i else None
+            if own is None or own.kind != "latent" or own.kv_from >= 0 or (own.kv_rank, own.rot_dims, own.rot_base) != (spec.kv_rank, spec.rot_dims, spec.rot_base):
+                raise ValueError(f"layer {i}: kv_from={src} is not an earlier latent attention layer with a cache of the same shape and rotation")
+        return spec
+    raise ValueError(f"layer {i}: no mixer of type {kind!r}")
+
+
+def _zeripel_from_json(cfg: dict, model_dir: Optional[str]) -> ModelConfig:
+    """``config.json`` of the Zeripel line: sizes and constants per layer."""
+    layers = []
+    for i, entry in enumerate(cfg["layers"]):
+        mixer, mlp = _zeripel_mixer(i, entry["type"], entry["mixer"], layers), entry.get("mlp")
+        if mlp is None:
+            layers.append(LayerSpec(mixer))
+        elif mlp.get("kind", "dense") == "dense":
+            layers.append(LayerSpec(mixer, mlp["ff"], act="gelu_tanh"))
+        elif mlp["kind"] == "moe":
+            r = mlp["router"]
+            if not 1 <= r["top"] <= r["experts"]:
+                raise ValueError(f"layer {i}: {r['top']} of {r['experts']} experts")
+            layers.append(LayerSpec(mixer, moe=_zeripel_experts(r["experts"], r["top"], mlp["expert"]["ff"], (mlp.get("shared") or {}).get("ff", 0), float(r.get("scale", 1.0)))))
+        else:
+            raise ValueError(f"layer {i}: no feed-forward of kind {mlp['kind']!r}")
+    attn = [l.mixer for l in layers if l.mixer.kind == "attention"] or [layers[0].mixer]
+    emb = cfg.get("embedding") or {}
+    big = emb.get("bigram")
+    return ModelConfig(family="zeripel", vocab_size=cfg["vocab"], hidden_size=cfg["width"], num_layers=len(layers), num_q_heads=attn[0].heads, num_kv_heads=max(attn[0].kv_heads, 1), head_dim=attn[0].dim,
+                       intermediate_size=max([l.ff for l in layers] + [l.moe.ff * l.moe.top + l.moe.shared_ff for l in layers if l.moe]), rms_eps=cfg["norm"]["eps"], qk_norm=False,
+                       layer_specs=tuple(layers), embed_scale=float(emb.get("scale", 1.0)), bigram=(big["buckets"], big["mul_prev"], big["mul_cur"]) if big else (),
+                       residual_mult=float(cfg.get("residual_mult", 1.0)), max_position=131072, eos_token_ids=_eos_ids(model_dir, cfg))
+
+
+def zeripel_to_json(cfg: ModelConfig) -> dict:
+    """The ``config.json`` that ``_zeripel_from_json`` reads back."""
+    layers = []
+    for l in cfg.layer_specs:
+        m, e = l.mixer, l.moe
+        mix = dict(heads=m.heads, dim=m.dim)
+        if m.kind == "attention":
+            mix.update(vdim=m.vdim, kv_heads=m.kv_heads, scale=m.scale)
+            if m.q_temp:
+                mix["q_temp"] = dict(coef=m.q_temp[0], every=m.q_temp[1])
+        elif m.kind == "latent":
+            mix.update(vdim=m.vdim, rot_dim=m.rot_dims, kv_rank=m.kv_rank, scale=m.scale, rot=dict(dims=m.rot_dims, base=m.rot_base))
+            if m.kv_from >= 0:
+                mix["kv_from"] = m.kv_from
+        mlp = None
+        if e:
+            mlp = dict(kind="moe", expert=dict(ff=e.ff), router=dict(experts=e.experts, top=e.top, scale=e.scale))
+            if e.shared_ff:
+                mlp["shared"] = dict(ff=e.shared_ff)
+        elif l.ff:
+            mlp = dict(kind="dense", ff=l.ff)
+        layers.append(dict(type="latent_attention" if m.kind == "latent" else m.kind, mixer=mix, mlp=mlp))
+    emb = dict(scale=cfg.embed_scale)
+    if cfg.bigram:
+        emb["bigram"] = dict(zip(("buckets", "mul_prev", "mul_cur"), cfg.bigram))
+    out = dict(architecture="Zeripel", vocab=cfg.vocab_size, width=cfg.hidden_size, norm=dict(eps=cfg.rms_eps), residual_mult=cfg.residual_mult, embedding=emb, layers=layers)
+    if cfg.eos_token_ids:
+        out["eos_token_id"] = list(cfg.eos_token_ids)
+    return out
+
+
 def from_hf(cfg: dict, model_dir: Optional[str] = None) -> ModelConfig:
     family = detect_family(cfg)
     top = cfg
@@ -512,6 +643,8 @@ def from_hf(cfg: dict, model_dir: Optional[str] = None) -> ModelConfig:
         return _nemipel_from_json(cfg, model_dir)
     if family == "vekalorn":
         return _vekalorn_from_json(cfg, model_dir)
+    if family == "zeripel":
+        return _zeripel_from_json(cfg, model_dir)
     if family == "qwen35" and "text_config" in cfg:
         cfg = cfg["text_config"]
     if family == "kimi_k2" and "text_config" in cfg:

@@ -4,7 +4,9 @@
 cleared when it is taken.  ``RecurrentState`` holds the state of models whose linear layers are all alike (one convolution
 tensor and one state tensor over the layers), ``LayerStates`` that of models whose layers differ (a state tensor per layer,
 and a convolution tensor where the layer has short convolutions).  A layer's state is f32 ``[slots, heads, dk, dv]``, its
-carried convolution inputs ``[slots, channels, taps - 1]`` in the activation dtype.
+carried convolution inputs ``[slots, channels, taps - 1]`` in the activation dtype.  The previous row that a token-shift mix
+reads is kept as the carried input of a two-tap convolution; ``LayerStates.token`` (where the model's embedding looks at the
+previous token) is int32 ``[slots]``, 1 + that token, 0 before the first.
 
 Reference parity: pegainfer-qwen35/src/recurrent_state.rs:16-170.
 """
@@ -52,10 +54,11 @@ class RecurrentState(StateSlots):
 
 
 class LayerStates(StateSlots):
-    def __init__(self, num_slots: int, geometries, dtype, device):
+    def __init__(self, num_slots: int, geometries, dtype, device, token: bool = False):
         """``geometries``: ``(heads, dk, dv, conv_channels, taps)`` of every recurrent layer, ``taps == 0`` without
         short convolutions."""
         super().__init__(num_slots)
+        self.token = torch.zeros(num_slots, dtype=torch.int32, device=device) if token else None
         self.ssm = [torch.zeros((num_slots, h, dk, dv), dtype=torch.float32, device=device) for h, dk, dv, _, _ in geometries]
         self.conv = [torch.zeros((num_slots, c, max(taps - 1, 0)), dtype=dtype, device=device) if taps else None for _, _, _, c, taps in geometries]
 
@@ -63,3 +66,5 @@ class LayerStates(StateSlots):
         live = [t[slot] for t in self.ssm] + [t[slot] for t in self.conv if t is not None and t.numel()]
         if live:
             torch._foreach_zero_(live)
+        if self.token is not None:
+            self.token[slot].zero_()

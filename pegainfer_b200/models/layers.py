@@ -1,9 +1,14 @@
 """Weight layouts shared by the model lines whose layers are listed one by one."""
 from __future__ import annotations
 
+from typing import Optional
+
 import torch
 
 from .. import ops
+from ..kv.buffer import MixedKvBuffer
+from ..kv.state import LayerStates
+from ..sched.executor import HybridExecutor
 
 
 def pad8(n: int) -> int:
@@ -39,3 +44,34 @@ class LatentHeads:
         self.ukv = torch.cat((uk, uv), 0).contiguous()
         self.uv = self.ukv[uk.shape[0] :].view(heads, -1, uk.shape[1])
         self.uk_t = uk.view(heads, -1, uk.shape[1]).transpose(1, 2).contiguous()
+
+
+class HybridLayers:
+    """Cache, state and executor of a model whose layers are listed one by one, some with pages, some with recurrent state:
+    ``kv_geometries`` ``(kv_heads, dim, vdim)`` of the layers that own a cache, ``state_geometries`` as in ``LayerStates``."""
+
+    supports_prefix_cache = False  # recurrent state is per request and not cached
+    carries_token = False  # the embedding reads the previous token
+    rec: Optional[LayerStates] = None
+
+    def kv_geometry(self) -> dict:
+        g = self.kv_geometries or [(1, 8, 8)]
+        # KV heads of the attention layers times the groups of up to eight query heads that one CTA of the decode kernel takes
+        attn = [l.mixer for l in self.cfg.layer_specs if l.mixer.kind == "attention"]
+        return dict(num_layers=len(g), kv_heads=max([m.kv_heads * ((m.heads // m.kv_heads + 7) // 8) for m in attn] or [1]), head_dim=max(max(d, v) for _, d, v in g),
+                    bytes_per_block=lambda page: max(1, MixedKvBuffer.bytes_per_block(self.kv_geometries, page, self.dtype)))
+
+    def make_kv(self, num_pages: int, page_size: int) -> MixedKvBuffer:
+        return MixedKvBuffer(self.kv_geometries, num_pages, page_size, self.dtype, self.device)
+
+    def state_bytes(self, slots: int) -> int:
+        elem = torch.empty((), dtype=self.dtype).element_size()
+        return (slots + 1) * (4 * self.carries_token + sum(4 * h * dk * dv + elem * c * max(taps - 1, 0) for h, dk, dv, c, taps in self.state_geometries))
+
+    def make_state(self, num_slots: int) -> LayerStates:
+        self.rec = LayerStates(num_slots + 1, self.state_geometries, self.dtype, self.device, token=self.carries_token)
+        return self.rec
+
+    @staticmethod
+    def make_executor(model, kv, page_size, cuda_graph=False, max_decode_batch=256, max_blocks_per_seq=0, seed=0, state_slots=None):
+        return HybridExecutor(model, kv, page_size, state_slots=state_slots or max_decode_batch, cuda_graph=cuda_graph, max_decode_batch=max_decode_batch, max_blocks_per_seq=max_blocks_per_seq, seed=seed)

@@ -26,13 +26,10 @@ import torch
 
 from .. import ops
 from ..config import MixerSpec, ModelConfig
-from ..kv.buffer import MixedKvBuffer
-from ..kv.state import LayerStates
 from ..loader.sources import RandomSource, WeightSource
 from ..ops.reference import AttnMeta, pair_rope_tables
 from ..parallel.tp import SINGLE, TPContext
-from ..sched.executor import HybridExecutor
-from .layers import FusedProjection, pad8
+from .layers import FusedProjection, HybridLayers, pad8
 
 
 def nemipel_shapes(cfg: ModelConfig) -> dict:
@@ -116,15 +113,13 @@ class NemipelLayer:
     norm2: Optional[torch.Tensor] = None
 
 
-class NemipelModel:
+class NemipelModel(HybridLayers):
     family = "nemipel"
-    supports_prefix_cache = False  # recurrent state is per request and not cached
 
     def __init__(self, cfg: ModelConfig, source: Optional[WeightSource] = None, device="cpu", dtype=torch.bfloat16, tp: TPContext = SINGLE, seed: int = 0):
         if tp.world != 1:
             raise ValueError("the Nemipel line runs on one GPU")
         self.cfg, self.device, self.dtype, self.tp = cfg, torch.device(device), dtype, tp
-        self.rec: Optional[LayerStates] = None
         self.kv_geometries, self.state_geometries = [], []
         self._kv_of = {}  # layer -> index of the cache it reads
         self._rope = {}
@@ -179,34 +174,6 @@ class NemipelModel:
             L.down = torch.nn.functional.pad(src.get(q + "down", dev, dt), (0, pad)).contiguous()
             L.norm2 = src.get(f"l{i}.norm2", dev, f32)
         return L
-
-    # -- geometry / executor -------------------------------------------------------------
-    def kv_geometry(self) -> dict:
-        g = self.kv_geometries or [(1, 8, 8)]
-        return dict(num_layers=len(g), kv_heads=max(h * self._parts(h) for h, _, _ in g), head_dim=max(max(d, v) for _, d, v in g),
-                    bytes_per_block=lambda page: max(1, MixedKvBuffer.bytes_per_block(self.kv_geometries, page, self.dtype)))
-
-    def _parts(self, kv_heads: int) -> int:
-        """Groups of up to eight query heads per KV head (what one CTA of the decode kernel takes)."""
-        return max([(l.mixer.heads // l.mixer.kv_heads + 7) // 8 for l in self.cfg_attention() if l.mixer.kv_heads == kv_heads] or [1])
-
-    def cfg_attention(self):
-        return [l for l in self.cfg.layer_specs if l.mixer.kind == "attention"]
-
-    def make_kv(self, num_pages: int, page_size: int) -> MixedKvBuffer:
-        return MixedKvBuffer(self.kv_geometries, num_pages, page_size, self.dtype, self.device)
-
-    def state_bytes(self, slots: int) -> int:
-        elem = torch.empty((), dtype=self.dtype).element_size()
-        return (slots + 1) * sum(4 * h * dk * dv + elem * c * max(taps - 1, 0) for h, dk, dv, c, taps in self.state_geometries)
-
-    def make_state(self, num_slots: int) -> LayerStates:
-        self.rec = LayerStates(num_slots + 1, self.state_geometries, self.dtype, self.device)
-        return self.rec
-
-    @staticmethod
-    def make_executor(model, kv, page_size, cuda_graph=False, max_decode_batch=256, max_blocks_per_seq=0, seed=0, state_slots=None):
-        return HybridExecutor(model, kv, page_size, state_slots=state_slots or max_decode_batch, cuda_graph=cuda_graph, max_decode_batch=max_decode_batch, max_blocks_per_seq=max_blocks_per_seq, seed=seed)
 
     # -- mixers ----------------------------------------------------------------------------
     def attention(self, L: NemipelLayer, x, meta: AttnMeta, kv):

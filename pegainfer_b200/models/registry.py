@@ -61,13 +61,21 @@ def _vekalorn(cfg, **kw):
     return VekalornModel(cfg, **kw)
 
 
-BUILDERS = {"vekalorn": _vekalorn, "nemipel": _nemipel, "kimi_k3": _k3, "gemma4": _gemma4, "glm_dsa": _glm_dsa, "qwen3": _qwen3, "qwen35": _qwen35, "deepseek_v2": _mla_moe, "kimi_k2": _mla_moe}
+def _zeripel(cfg, **kw):
+    from .zeripel import ZeripelModel
+
+    kw.pop("ep", None)
+    return ZeripelModel(cfg, **kw)
+
+
+BUILDERS = {"zeripel": _zeripel, "vekalorn": _vekalorn, "nemipel": _nemipel, "kimi_k3": _k3, "gemma4": _gemma4, "glm_dsa": _glm_dsa, "qwen3": _qwen3, "qwen35": _qwen35, "deepseek_v2": _mla_moe, "kimi_k2": _mla_moe}
 
 
 # Translation units (csrc/<name>.cu) that a family's kernels come from, for programs that build only what one model needs
 KERNEL_UNITS = {
     "nemipel": ("runtime", "gemm_sm100", "gemm2sm_sm100", "elementwise", "stream32", "attention", "attention_tc", "attention_general", "kda", "lightning", "sampling"),
     "vekalorn": ("runtime", "gemm_sm100", "gemm2sm_sm100", "elementwise", "stream32", "mla", "mla_prefill", "moe_route", "moe_gemm", "sampling"),
+    "zeripel": ("runtime", "gemm_sm100", "gemm2sm_sm100", "elementwise", "stream32", "attention", "attention_tc", "attention_general", "kda", "wkv", "mla", "mla_prefill", "moe_route", "moe_gemm", "sampling"),
 }
 
 
@@ -104,6 +112,10 @@ def shapes_for(cfg: ModelConfig) -> dict:
         from .vekalorn import vekalorn_shapes
 
         return vekalorn_shapes(cfg)
+    if cfg.family == "zeripel":
+        from .zeripel import zeripel_shapes
+
+        return zeripel_shapes(cfg)
     raise ValueError(f"no tensor-shape table for family {cfg.family!r}")
 
 

@@ -214,13 +214,13 @@ def swiglu(gate_up, interleaved: bool = False):
     return out.view(*gate_up.shape[:-1], inter)
 
 
-def geglu(gate_up):
-    """``bf16(gelu_tanh(gate)) * up`` on a fused ``[T, 2 I]`` buffer, gate half first."""
+def geglu(gate_up, interleaved: bool = False):
+    """``bf16(gelu_tanh(gate)) * up`` on a fused ``[T, 2 I]`` buffer, gate half first, or columns alternating (gate_i, up_i)."""
     _bf16(gate_up)
     g2 = _rows2d(gate_up)
     inter = g2.shape[1] // 2
     out = torch.empty((g2.shape[0], inter), dtype=g2.dtype, device=g2.device)
-    _check(lib().pg_swiglu(_ptr(g2), _ptr(out), _ci(g2.shape[0]), _ci(inter), _ll(g2.stride(0)), _ll(out.stride(0)), _ci(2), _stream()), ctx(g2.device))
+    _check(lib().pg_swiglu(_ptr(g2), _ptr(out), _ci(g2.shape[0]), _ci(inter), _ll(g2.stride(0)), _ll(out.stride(0)), _ci(2 + int(interleaved)), _stream()), ctx(g2.device))
     return out.view(*gate_up.shape[:-1], inter)
 
 
@@ -268,7 +268,7 @@ class DeferredNorm:
 
 
 FUSED_MAX_ROWS = 64
-EPI_PLAIN, EPI_SWIGLU, EPI_RESID_NORMW = 0, 1, 2
+EPI_PLAIN, EPI_SWIGLU, EPI_RESID_NORMW, EPI_GEGLU = 0, 1, 2, 3
 
 
 def fused_plan_ok(t: int, m: int, k: int) -> bool:
@@ -278,7 +278,7 @@ def fused_plan_ok(t: int, m: int, k: int) -> bool:
 
 def linear_fused(x, w, epilogue: int = EPI_PLAIN, residual=None, norm_w=None, norm_offset: bool = False, eps: float = 0.0):
     """Decode-chain GEMM.  ``x``: a bf16 ``[T, K]`` tensor or a ``DeferredNorm``.  ``epilogue``:
-    ``EPI_PLAIN`` -> ``[T, M]``; ``EPI_SWIGLU`` (interleaved gate/up weight rows) -> ``[T, M / 2]``;
+    ``EPI_PLAIN`` -> ``[T, M]``; ``EPI_SWIGLU``, ``EPI_GEGLU`` (interleaved gate/up weight rows) -> ``[T, M / 2]``;
     ``EPI_RESID_NORMW`` -> updates ``residual`` in place and returns a ``DeferredNorm`` for the norm
     with weight ``norm_w`` (its consumer completes it)."""
     dn = x if isinstance(x, DeferredNorm) else None
@@ -289,7 +289,7 @@ def linear_fused(x, w, epilogue: int = EPI_PLAIN, residual=None, norm_w=None, no
     m = w.shape[0]
     assert w.shape[1] == k and xin.stride(-1) == 1 and w.stride(-1) == 1
     c = ctx(xin.device)
-    out = torch.empty((t, m // 2 if epilogue == EPI_SWIGLU else m), dtype=torch.bfloat16, device=xin.device)
+    out = torch.empty((t, m // 2 if epilogue in (EPI_SWIGLU, EPI_GEGLU) else m), dtype=torch.bfloat16, device=xin.device)
     ssp = None
     if epilogue == EPI_RESID_NORMW:
         assert residual is not None and norm_w is not None and residual.stride(-1) == 1
@@ -433,8 +433,8 @@ def linear_2sm(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
     return out.view(*x.shape[:-1], m)
 
 
-def linear_swiglu_2sm(x: torch.Tensor, w: torch.Tensor) -> Optional[torch.Tensor]:
-    """``swiglu(x @ w.T)`` for a gate_up weight whose rows alternate (gate_i, up_i), with SwiGLU in the epilogue of the
+def linear_swiglu_2sm(x: torch.Tensor, w: torch.Tensor, gelu: bool = False) -> Optional[torch.Tensor]:
+    """``swiglu(x @ w.T)`` (``gelu``: with tanh-GELU on the gate) for a gate_up weight whose rows alternate (gate_i, up_i), with SwiGLU in the epilogue of the
     two-SM GEMM (prefill-sized steps); ``None`` when the two-SM kernel does not take the problem."""
     _bf16(x)
     x2 = _rows2d(x)
@@ -444,7 +444,7 @@ def linear_swiglu_2sm(x: torch.Tensor, w: torch.Tensor) -> Optional[torch.Tensor
         return None
     out = torch.empty((t, m // 2), dtype=torch.bfloat16, device=x.device)
     c = ctx(x.device)
-    rc = lib().pg_gemm2sm_bf16_tn_swiglu(_ptr(x2), _ptr(w), _ptr(out), _ci(t), _ci(m), _ci(k), _ll(x2.stride(0)), _ll(w.stride(0)), _ll(out.stride(0)), _ptr(c.status), _stream())
+    rc = lib().pg_gemm2sm_bf16_tn_swiglu(_ptr(x2), _ptr(w), _ptr(out), _ci(t), _ci(m), _ci(k), _ll(x2.stride(0)), _ll(w.stride(0)), _ll(out.stride(0)), _ci(int(gelu)), _ptr(c.status), _stream())
     _check(rc, c)
     return out.view(*x.shape[:-1], m // 2)
 
@@ -875,6 +875,78 @@ def embed_stream(ids, table, act_dtype):
     return x, xt
 
 
+def embed_pairs_norm(ids, table, pairs, scale: float, bigram, carried, w, eps: float, meta: AttnMeta, act_dtype):
+    """Stream of scaled table rows plus token-pair rows, and its RMS norm (``reference.embed_pairs_norm``)."""
+    ids = ids.to(torch.int32).contiguous()
+    t, width = ids.numel(), table.shape[1]
+    assert table.stride(1) == 1 and w.dtype == torch.float32 and (pairs is None or (pairs.dtype == table.dtype and pairs.stride(1) == 1 and pairs.shape == (bigram[0] + 1, width)))
+    x = torch.empty((t, width), dtype=torch.float32, device=table.device)
+    h = torch.empty((t, width), dtype=act_dtype, device=table.device)
+    c = ctx(table.device)
+    big = pairs is not None
+    assert not big or carried.dtype == torch.int32
+    _check(lib().pg_embed_pairs_norm(_ptr(table), _ci(_is_f32(table)), _ll(table.stride(0)), _ptr(pairs), _ll(pairs.stride(0) if big else 0), _ptr(ids), _ptr(_unit_seq(meta, table.device) if big else None),
+                                     _ptr(meta.q_indptr), _ptr(meta.state_slots if big else None), _ptr(carried if big else None), _cf(scale), *(_ll(n) for n in (bigram if big else (0, 0, 0))), _ptr(w),
+                                     _ptr(x), _ptr(h), _ci(int(act_dtype == torch.float32)), _ci(t), _ci(width), _ll(table.shape[0]), _cf(eps), _ptr(c.status), _stream()), c)
+    return x, h
+
+
+def _residual_norm(y, pos, weights, extra, extra_gate, x, w, eps, mult, act_dtype):
+    t, width = x.shape
+    assert x.dtype == w.dtype == torch.float32 and x.is_contiguous() and y.stride(1) == 1 and y.shape[1] == width and (weights is not None or y.shape[0] == t)
+    assert extra is None or (extra.shape == x.shape and extra.stride(1) == 1 and (extra_gate is None or extra_gate.dtype == torch.float32))
+    h = torch.empty((t, width), dtype=act_dtype, device=x.device)
+    _check(lib().pg_residual_norm(_ptr(y), _ci(_is_f32(y)), _ll(y.stride(0)), _ptr(pos), _ptr(weights), _ci(weights.shape[1] if weights is not None else 0), _ptr(extra),
+                                  _ci(_is_f32(extra) if extra is not None else 0), _ll(extra.stride(0) if extra is not None else 0), _ptr(extra_gate), _ll(extra_gate.stride(0) if extra_gate is not None else 0),
+                                  _ptr(x), _cf(mult), _ptr(w), _ptr(h), _ci(int(act_dtype == torch.float32)), _ll(width), _ci(t), _ci(width), _cf(eps), _stream()), ctx(x.device))
+    return h
+
+
+def residual_norm(y, x, w, eps: float, mult: float, act_dtype):
+    """``x += mult * y`` on the f32 stream, in place; returns the RMS norm of the sum in the activation dtype."""
+    return _residual_norm(y, None, None, None, None, x, w, eps, mult, act_dtype)
+
+
+def residual_norm_rows(rows, pos, weights, shared, shared_gate, x, w, eps: float, mult: float, act_dtype):
+    """``residual_norm`` of a mixture of experts (``reference.residual_norm_rows``): the weighted sum of the tokens' expert rows
+    and the gated shared row are formed in the same kernel."""
+    assert weights.dtype == torch.float32 and weights.is_contiguous() and pos.dtype == torch.int32
+    return _residual_norm(rows, pos, weights, shared, shared_gate, x, w, eps, mult, act_dtype)
+
+
+def token_mix(h, mu, carried, meta: AttnMeta):
+    """Mixes of every row with its predecessor (``reference.token_mix``)."""
+    t, width = h.shape
+    n = mu.shape[0]
+    assert h.stride(1) == 1 and mu.dtype == torch.float32 and mu.is_contiguous() and mu.shape[1] == width and carried.is_contiguous() and carried.dtype == h.dtype and carried[0].numel() == width
+    out = torch.empty((t, n, width), dtype=h.dtype, device=h.device)
+    _check(lib().pg_token_mix(_ptr(h), _ll(h.stride(0)), _ptr(mu), _ptr(carried), _ptr(out), _ptr(_unit_seq(meta, h.device)), _ptr(meta.q_indptr), _ptr(meta.state_slots), _ci(t), _ci(n), _ci(width),
+                              _ci(_is_f32(h)), _stream()), ctx(h.device))
+    return out
+
+
+def multi_dense(x, w):
+    """``y[t, i] = w[i] x[t, i]``: one batched launch, or the two-SM GEMM per matrix where it serves the problem."""
+    (t, n, k), m = x.shape, w.shape[1]
+    assert w.shape == (n, m, k) and w.is_contiguous() and x.stride(2) == 1 and x.dtype == w.dtype
+    y = torch.empty((t, n, m), dtype=x.dtype, device=x.device)
+    if t == 0:
+        return y
+    if not _is_f32(x) and k % 8 == 0 and x.stride(0) % 8 == 0 and x.stride(1) % 8 == 0 and not _BATCH_INVARIANT and m % 8 == 0 and lib().pg_gemm2sm_eligible(_ci(t), _ci(m), _ci(k)):
+        for i in range(n):
+            linear(x[:, i], w[i], out=y[:, i])
+        return y
+    _head_gemm(x, x.stride(0), x.stride(1), w, y)
+    return y
+
+
+def tanh_rows(x):
+    x = x.contiguous()
+    y = torch.empty_like(x)
+    _check(lib().pg_tanh_rows(_ptr(x), _ptr(y), _ll(x.numel()), _ci(_is_f32(x)), _stream()), ctx(x.device))
+    return y
+
+
 def _post_norm(y, x, x_out, w, eps, alpha, act_dtype):
     t, width = x.shape
     assert x.dtype == torch.float32 and w.dtype == torch.float32 and x.is_contiguous() and (y is None or (y.shape == x.shape and y.stride(1) == 1))
@@ -922,12 +994,14 @@ def stream_layer_norm(x, w, eps: float, act_dtype):
     return _add_layer_norm(x, None, None, None, w, eps, act_dtype)
 
 
-def gated_row_norm(x, gate, w, eps: float):
-    """``rms_norm(x) * w * sigmoid(gate)`` over the last axis of ``x`` [T, H, D]; ``gate`` [T, H * D], unit column stride."""
+def gated_row_norm(x, gate, w, eps: float, act: str = "sigmoid"):
+    """``rms_norm(x) * w * act(gate)`` over the last axis of ``x`` [T, H, D]; ``gate`` [T, H * D], unit column stride; ``w`` [D]
+    or [H * D]; ``act``: sigmoid or silu."""
     t, h, d = x.shape
-    assert x.is_contiguous() and gate.shape == (t, h * d) and gate.stride(1) == 1 and gate.dtype == x.dtype and w.dtype == torch.float32
+    assert x.is_contiguous() and gate.shape == (t, h * d) and gate.stride(1) == 1 and gate.dtype == x.dtype and w.dtype == torch.float32 and w.numel() in (d, h * d) and act in ("sigmoid", "silu")
     y = torch.empty((t, h, d), dtype=x.dtype, device=x.device)
-    _check(lib().pg_gated_row_norm(_ptr(x), _ptr(gate), _ll(gate.stride(0)), _ptr(w), _ptr(y), _ci(t), _ci(h), _ci(d), _cf(eps), _ci(_is_f32(x)), _stream()), ctx(x.device))
+    _check(lib().pg_gated_row_norm(_ptr(x), _ptr(gate), _ll(gate.stride(0)), _ptr(w), _ptr(y), _ci(t), _ci(h), _ci(d), _cf(eps), _ci(int(act == "silu")), _ci(int(w.numel() > d)), _ci(_is_f32(x)), _stream()),
+           ctx(x.device))
     return y
 
 
@@ -949,24 +1023,25 @@ def dense(x, w, out_dtype=None):
     return y
 
 
-def dense_glu(x, gate_up, interleaved: bool = False):
-    """``silu(gate) * up`` of the fused projection ``x @ gate_up.T``: in the GEMM's epilogue where a kernel has it (decode
+def dense_glu(x, gate_up, interleaved: bool = False, act: str = "silu"):
+    """``act(gate) * up`` (silu or gelu_tanh) of the fused projection ``x @ gate_up.T``: in the GEMM's epilogue where a kernel has it (decode
     steps on the on-chip split-K path, prefill-sized steps on the two-SM kernel; interleaved rows), else two launches."""
+    gelu = act == "gelu_tanh"
     if _is_f32(x):
         gu = dense(x, gate_up)
         assert not interleaved
         out = torch.empty((x.shape[0], gu.shape[1] // 2), dtype=torch.float32, device=x.device)
-        _check(lib().pg_glu_rows_f32(_ptr(gu), _ptr(out), _ci(gu.shape[0]), _ci(out.shape[1]), _ll(gu.stride(0)), _stream()), ctx(x.device))
+        _check(lib().pg_glu_rows_f32(_ptr(gu), _ptr(out), _ci(gu.shape[0]), _ci(out.shape[1]), _ll(gu.stride(0)), _ci(int(gelu)), _stream()), ctx(x.device))
         return out
     t, k = x.shape
     m = gate_up.shape[0]
     if interleaved and k % 8 == 0 and x.stride(0) % 8 == 0:
         if m % 4 == 0 and fused_plan_ok(t, m, k):
-            return linear_fused(x, gate_up, EPI_SWIGLU)
-        act = linear_swiglu_2sm(x, gate_up)
-        if act is not None:
-            return act
-    return swiglu(dense(x, gate_up), interleaved)
+            return linear_fused(x, gate_up, EPI_GEGLU if gelu else EPI_SWIGLU)
+        y = linear_swiglu_2sm(x, gate_up, gelu)
+        if y is not None:
+            return y
+    return geglu(dense(x, gate_up), interleaved) if gelu else swiglu(dense(x, gate_up), interleaved)
 
 
 def softcap_rows(logits, cap: float):
@@ -990,6 +1065,21 @@ def row_norm_rope_append(q, k, v, q_norm_w, k_norm_w, cos, sin, meta: AttnMeta, 
     _check(lib().pg_row_norm_rope_append(_ptr(q), _ptr(k), _ptr(v), _ll(q.stride(0)), _ptr(q_norm_w), _ptr(k_norm_w if k is not None else None), _ptr(cos), _ptr(sin), _ci(2 * cos.shape[1]), _ci(cos.shape[0]),
                                          _ptr(meta.positions), _ptr(meta.slot_mapping), _ptr(out), _ptr(kv_layer if k is not None else None), _ci(t), _ci(heads), _ci(kv_heads), _ci(dim), _ci(vdim),
                                          _ci(meta.page_size), _ll(kv_layer.shape[0] if k is not None else 0), _cf(eps), _ci(_is_f32(q)), _ptr(c.status), _stream()), c)
+    return out
+
+
+def head_norm_append(q, k, v, q_norm_w, k_norm_w, temp, meta: AttnMeta, kv_layer, heads: int, kv_heads: int, dim: int, vdim: int, eps: float):
+    """Per-head query and key norms, query temperature and paged append (``reference.head_norm_append``)."""
+    t = q.shape[0]
+    ld = _same_rows(q, k, v)
+    assert q.stride(1) == k.stride(1) == v.stride(1) == 1 and q.dtype == k.dtype == v.dtype == kv_layer.dtype and q_norm_w.dtype == k_norm_w.dtype == torch.float32
+    assert q.shape[1] == heads * dim and k.shape[1] == kv_heads * dim and v.shape[1] == kv_heads * vdim and kv_layer.is_contiguous() and kv_layer.shape[1] == meta.page_size * kv_heads * (dim + vdim)
+    assert temp is None or (temp.dtype == torch.float32 and temp.is_contiguous())
+    out = torch.empty((t, heads, dim), dtype=q.dtype, device=q.device)
+    c = ctx(q.device)
+    _check(lib().pg_head_norm_append(_ptr(q), _ptr(k), _ptr(v), _ll(ld), _ptr(q_norm_w), _ptr(k_norm_w), _ptr(temp), _ci(temp.shape[0] if temp is not None else 0), _ptr(meta.positions),
+                                     _ptr(meta.slot_mapping), _ptr(out), _ptr(kv_layer), _ci(t), _ci(heads), _ci(kv_heads), _ci(dim), _ci(vdim), _ci(meta.page_size), _ll(kv_layer.shape[0]), _cf(eps),
+                                     _ci(_is_f32(q)), _ptr(c.status), _stream()), c)
     return out
 
 
@@ -1036,10 +1126,13 @@ def capped_attention(q, kv_layer, kv_heads: int, vdim: int, meta: AttnMeta, scal
     if (n_pf > 0 and dim == vdim == 128 and _PREFILL_TC and not _BATCH_INVARIANT and max(qi[b + 1] - qi[b] for b in range(n_pf)) >= _PREFILL_TC_MIN_ROWS
             and (meta.h_kv_lens is None or max(meta.h_kv_lens[:n_pf]) >= _PREFILL_TC_MIN_KV)):
         PREFILL_TC_CALLS["hd128"] += 1
-        rc = lib().pg_prefill_attention_tc_capped(_ptr(q), _ptr(kv_layer), _ptr(out), _ptr(meta.q_indptr), _ptr(meta.kv_lens), _ptr(table), _ci(table.stride(0)), _ci(n_pf), _ci(qi[n_pf]), _ci(hq),
-                                                  _ci(kv_heads), _ci(ps), _ll(pages), _cf(scale), _cf(softcap), *gate_args, _ci(sum((qi[b + 1] - qi[b] + 255) // 256 for b in range(n_pf))),
-                                                  _ptr(c.status), _stream())
-        _check(rc, c)
+        tiles = _ci(sum((qi[b + 1] - qi[b] + 255) // 256 for b in range(n_pf)))
+        if softcap == 0.0 and gate is None:
+            _check(lib().pg_prefill_attention_tc(_ptr(q), _ptr(kv_layer), _ptr(out), _ptr(meta.q_indptr), _ptr(meta.kv_lens), _ptr(table), _ci(table.stride(0)), _ci(n_pf), _ci(qi[n_pf]), _ci(hq), _ci(kv_heads),
+                                                 _ci(dim), _ci(ps), _ll(pages), _cf(scale), tiles, _ci(0), _ptr(c.status), _stream()), c)
+        else:
+            _check(lib().pg_prefill_attention_tc_capped(_ptr(q), _ptr(kv_layer), _ptr(out), _ptr(meta.q_indptr), _ptr(meta.kv_lens), _ptr(table), _ci(table.stride(0)), _ci(n_pf), _ci(qi[n_pf]), _ci(hq),
+                                                  _ci(kv_heads), _ci(ps), _ll(pages), _cf(scale), _cf(softcap), *gate_args, tiles, _ptr(c.status), _stream()), c)
     elif n_pf > 0:
         run(0, n_pf, 1, 1, sum((qi[b + 1] - qi[b] + 63) // 64 for b in range(n_pf)))
     if n_pf < meta.num_seqs:
@@ -1106,6 +1199,19 @@ def decay_attention(q, k, v, decay, state, meta: AttnMeta, chunked: Optional[boo
         _check(lib().pg_lightning_chunked(*args, _ci(_GDN_CHUNK_MIN), _stream()), c)
     if not chunked or _has_short_rows(meta, _GDN_CHUNK_MIN):
         _check(lib().pg_decay_recurrent(*args, _ci(int(meta.max_q_len)), _ci(_GDN_CHUNK_MIN if chunked else 0), _ci(f32), _stream()), c)
+    return out
+
+
+def wkv_attention(r, k, v, f, w0, u, state, meta: AttnMeta):
+    """Linear attention with a decay per token and key channel and a bonus for the current token (``reference.wkv_attention``);
+    ``r, k, v`` share a row stride."""
+    t, h, dk = r.shape
+    dv = v.shape[2]
+    assert r.stride(2) == 1 and r.stride(1) == dk and k.stride(1) == dk and v.stride(1) == dv and f.dtype == torch.float32 and f.stride(1) == 1 and f.shape[1] == h * dk
+    assert state.is_contiguous() and state.dtype == w0.dtype == u.dtype == torch.float32 and w0.is_contiguous() and u.is_contiguous()
+    out = torch.empty((t, h, dv), dtype=r.dtype, device=r.device)
+    _check(lib().pg_wkv_recurrent(_ptr(r), _ptr(k), _ptr(v), _ll(_same_rows(r, k, v)), _ptr(f), _ll(f.stride(0)), _ptr(w0), _ptr(u), _ptr(state), _ptr(out), _ptr(meta.q_indptr), _ptr(meta.state_slots),
+                                  _ci(meta.num_seqs), _ci(h), _ci(dk), _ci(dv), _ci(int(meta.max_q_len)), _ci(0), _ci(_is_f32(r)), _stream()), ctx(r.device))
     return out
 
 
@@ -1178,10 +1284,10 @@ def repack_int4_pairs(packed):
     return out
 
 
-def grouped_gemm(xs, offsets, w, scales=None, bn: int = 16, relu2: bool = False):
+def grouped_gemm(xs, offsets, w, scales=None, bn: int = 16, act: str = ""):
     """``xs`` [rows, K] sorted by expert; ``w`` bf16 [E, M, K], packed int32 [E, M, K/8] with bf16
-    scales [E, M, K/32], or FP8 e4m3 [E, M, K] with f32 ``scale_inv`` [E, ceil(M/128), ceil(K/128)].  ``relu2``: the squared
-    ReLU of the result (bf16 weights)."""
+    scales [E, M, K/32], or FP8 e4m3 [E, M, K] with f32 ``scale_inv`` [E, ceil(M/128), ceil(K/128)].  ``act`` (bf16
+    weights): ``relu2`` the squared ReLU of the result, ``glu`` [rows, M / 2] SiLU(gate) * up over alternating weight rows."""
     rows, k = xs.shape
     e, m = w.shape[0], w.shape[1]
     mode = quant_code(w)
@@ -1190,11 +1296,12 @@ def grouped_gemm(xs, offsets, w, scales=None, bn: int = 16, relu2: bool = False)
         w = paired_int4(w)
     if mode == 2:
         assert scales.dtype == torch.float32 and scales.shape == (e, (m + 127) // 128, (k + 127) // 128), "FP8 experts need f32 scale_inv per 128x128 block"
-    y = torch.empty((rows, m), dtype=torch.bfloat16, device=xs.device)
+    y = torch.empty((rows, m // 2 if act == "glu" else m), dtype=torch.bfloat16, device=xs.device)
     c = ctx(xs.device)
-    if relu2:
-        assert mode == 0, "the squared ReLU is wired for bf16 expert weights"
-        _check(lib().pg_moe_grouped_gemm_relu2(_ptr(xs), _ll(xs.stride(0)), _ll(rows), _ptr(w), _ptr(y), _ll(y.stride(0)), _ptr(offsets), _ci(e), _ci(m), _ci(k), _ci(bn), _ptr(c.status), _stream()), c)
+    if act:
+        assert mode == 0 and w.is_contiguous(), "activations are wired for bf16 expert weights"
+        _check(lib().pg_moe_grouped_gemm_act(_ptr(xs), _ll(xs.stride(0)), _ll(rows), _ptr(w), _ptr(y), _ll(y.stride(0)), _ptr(offsets), _ci(e), _ci(m), _ci(k), _ci(bn), _ci({"relu2": 1, "glu": 2}[act]), _ptr(c.status),
+                                             _stream()), c)
         return y
     rc = lib().pg_moe_grouped_gemm(_ptr(xs), _ll(xs.stride(0)), _ll(rows), _ptr(w), _ptr(scales), _ci(mode), _ptr(y), _ll(y.stride(0)), _ptr(offsets), _ci(e), _ci(m),
                                    _ci(k), _ci(bn), _ptr(c.status), _stream())
@@ -1231,14 +1338,14 @@ def _routed_rows(x, ids, w13, s13, w2, s2, expert_offset, act: str):
     xs = torch.empty((routes, h), dtype=x.dtype, device=x.device)
     _check(lib().pg_moe_gather(_ptr(x), _ll(x.stride(0)), _ptr(sorted_src), _ptr(offsets), _ci(e_local), _ci(k), _ptr(xs), _ci(h), _ci(routes), _stream()), c)
     bn = _token_tile(routes, e_local)
-    assert act == "swiglu" or quant_code(w13) == 0, "the situ and squared ReLU activations are wired for bf16 expert weights"
+    assert act == "swiglu" or quant_code(w13) == 0, "the situ, interleaved and squared ReLU activations are wired for bf16 expert weights"
     if quant_code(w13) == 2 and _MOE_FP8_TC and h % 128 == 0 and w13.shape[1] % 256 == 0 and w2.shape[1] % 128 == 0:
         # both GEMMs on the FP8 tensor-core path: activations quantised per row and 128-wide k group
         xq, xsc = quant_fp8_1x128(xs)
         aq, asc = swiglu_quant_fp8_1x128(grouped_gemm_fp8(xq, xsc, offsets, w13, s13, bn))
         return grouped_gemm_fp8(aq, asc, offsets, w2, s2, bn), route_pos
-    if act == "relu2":
-        mid = grouped_gemm(xs, offsets, w13, None, bn, relu2=True)
+    if act in ("relu2", "glu"):
+        mid = grouped_gemm(xs, offsets, w13, None, bn, act)
     else:
         y1 = grouped_gemm(xs, offsets, w13, s13, bn)
         mid = situ(y1) if act == "situ" else swiglu(y1)
@@ -1255,17 +1362,19 @@ def _moe_pipeline(x, ids, weights, w13, s13, w2, s2, expert_offset, act: str = "
 
 def expert_rows(x, ids, w1, w2, act: str = "relu2"):
     """Unweighted expert outputs of every route and their rows (``reference.expert_rows``); f32 and sizes that TMA cannot
-    address run on the CUDA-core grouped GEMM (squared ReLU only)."""
-    (t, h), k, (e, inter) = x.shape, ids.shape[1], w1.shape[:2]
+    address run on the CUDA-core grouped GEMM."""
+    (t, h), k, e, inter = x.shape, ids.shape[1], w1.shape[0], w2.shape[2]
     f32 = _is_f32(x)
+    assert act in ("relu2", "swiglu") and w1.shape[1] == inter * (2 if act == "swiglu" else 1)
     if not f32 and h % 8 == 0 and inter % 8 == 0:
-        return _routed_rows(x, ids, w1, None, w2, None, 0, act)
-    assert act == "relu2" and x.stride(1) == 1 and w1.dtype == w2.dtype == x.dtype and w1.is_contiguous() and w2.is_contiguous()
+        return _routed_rows(x, ids, w1, None, w2, None, 0, "glu" if act == "swiglu" else act)
+    assert x.stride(1) == 1 and w1.dtype == w2.dtype == x.dtype and w1.is_contiguous() and w2.is_contiguous()
     offsets, sorted_src, route_pos = moe_route_plan(ids, 0, e)
     c = ctx(x.device)
     mid = torch.empty((t * k, inter), dtype=x.dtype, device=x.device)
     out = torch.empty((t * k, h), dtype=x.dtype, device=x.device)
-    _check(lib().pg_expert_gemm_simt(_ptr(x), _ll(x.stride(0)), _ptr(sorted_src), _ci(k), _ptr(w1), _ptr(mid), _ptr(offsets), _ci(t * k), _ci(e), _ci(inter), _ci(h), _ci(1), _ci(f32), _stream()), c)
+    _check(lib().pg_expert_gemm_simt(_ptr(x), _ll(x.stride(0)), _ptr(sorted_src), _ci(k), _ptr(w1), _ptr(mid), _ptr(offsets), _ci(t * k), _ci(e), _ci(w1.shape[1]), _ci(h), _ci(2 if act == "swiglu" else 1),
+                                     _ci(f32), _stream()), c)
     _check(lib().pg_expert_gemm_simt(_ptr(mid), _ll(inter), _vp(0), _ci(1), _ptr(w2), _ptr(out), _ptr(offsets), _ci(t * k), _ci(e), _ci(h), _ci(inter), _ci(0), _ci(f32), _stream()), c)
     return out, route_pos
 
@@ -1470,16 +1579,16 @@ def mla_attention(q: "_MlaQ", w_uk, w_uv, latent_layer, meta: AttnMeta, scale, k
 
 def latent_rows(zq, zkv, q_norm_w, kv_norm_w, cos, sin, meta: AttnMeta, cache, latent: int, eps: float):
     """Query latent and cache rows of a latent attention layer (``reference.latent_rows``); ``zq`` and ``zkv`` are column
-    slices of one fused projection."""
-    t, qr = zq.shape
+    slices of one fused projection; without ``zq`` only the cache rows are made."""
+    t, qr = zkv.shape[0], zq.shape[1] if zq is not None else 0
     rot = zkv.shape[1] - latent
-    ld = _same_rows(zq, zkv)
-    assert zq.stride(1) == zkv.stride(1) == 1 and zq.dtype == zkv.dtype == cache.dtype and q_norm_w.dtype == kv_norm_w.dtype == torch.float32
+    ld = _same_rows(zkv, zq) if zq is not None else zkv.stride(0)
+    assert zkv.stride(1) == 1 and zkv.dtype == cache.dtype and kv_norm_w.dtype == torch.float32 and (zq is None or (zq.stride(1) == 1 and zq.dtype == zkv.dtype and q_norm_w.dtype == torch.float32))
     assert cache.is_contiguous() and cache.shape[1] == meta.page_size * (latent + rot) and (rot == 0 or (cos.dtype == torch.float32 and 2 * cos.shape[1] == rot))
-    cq = torch.empty((t, qr), dtype=zq.dtype, device=zq.device)
-    c = ctx(zq.device)
+    cq = torch.empty((t, qr), dtype=zkv.dtype, device=zkv.device) if zq is not None else None
+    c = ctx(zkv.device)
     _check(lib().pg_latent_rows(_ptr(zq), _ptr(zkv), _ll(ld), _ptr(q_norm_w), _ptr(kv_norm_w), _ptr(cos if rot else None), _ptr(sin if rot else None), _ptr(meta.positions), _ptr(meta.slot_mapping), _ptr(cq),
-                                _ptr(cache), _ci(t), _ci(qr), _ci(latent), _ci(rot), _ci(cos.shape[0] if rot else 0), _ll(cache.shape[0] * meta.page_size), _cf(eps), _ci(_is_f32(zq)), _ptr(c.status),
+                                _ptr(cache), _ci(t), _ci(qr), _ci(latent), _ci(rot), _ci(cos.shape[0] if rot else 0), _ll(cache.shape[0] * meta.page_size), _cf(eps), _ci(_is_f32(zkv)), _ptr(c.status),
                                 _stream()), c)
     return cq
 
@@ -1517,19 +1626,20 @@ def _latent_key_plan(meta: AttnMeta, n: int, window: int, device):
     return plans[key][:4]
 
 
-def latent_attention(q, uk_t, uv, ukv, cache, meta: AttnMeta, rot: int, scale: float, window: int = 0, cos=None, sin=None, gate=None):
-    """Latent attention over the paged cache (``reference.latent_attention``).  Long prompt portions of heads up to
+def latent_attention(q, uk_t, uv, ukv, cache, meta: AttnMeta, rot: int, scale: float, window: int = 0, cos=None, sin=None, gate=None, head_gate=None, sink=None):
+    """Latent attention over the paged cache (``reference.latent_attention``; ``q`` may be columns of a wider row).  Long prompt portions of heads up to
     128 + 64 / 128 columns run in the expanded form on tcgen05, single rows and short portions in the absorbed form on the
     split-KV kernel (latents up to 512 + 64), f32 and other sizes on the CUDA-core kernel."""
     heads, lat, dim = uk_t.shape
     vdim, t = uv.shape[1], q.shape[0]
     f32, dev = _is_f32(q), q.device
-    assert q.is_contiguous() and q.shape[1] == heads * (dim + rot) and uk_t.is_contiguous() and uv.is_contiguous() and cache.is_contiguous() and cache.dtype == q.dtype
+    assert q.stride(1) == 1 and q.shape[1] == heads * (dim + rot) and uk_t.is_contiguous() and uv.is_contiguous() and cache.is_contiguous() and cache.dtype == q.dtype
     assert cache.shape[1] == meta.page_size * (lat + rot) and (gate is None or (gate.dtype == q.dtype and gate.stride(1) == 1 and gate.shape == (t, heads * vdim)))
+    assert (head_gate is None or (gate is None and head_gate.dtype == q.dtype and head_gate.stride(1) == 1 and head_gate.shape == (t, heads))) and (sink is None or (sink.dtype == torch.float32 and sink.numel() == heads))
     out = torch.empty((t, heads * vdim), dtype=q.dtype, device=dev)
     if t == 0:
         return out
-    c = ctx(dev)
+    c, ldq = ctx(dev), q.stride(0)
     max_pos = cos.shape[0] if rot else 0
     cos, sin = (cos, sin) if rot else (None, None)
     table, ps, qd = meta.block_table, meta.page_size, dim + rot
@@ -1537,8 +1647,8 @@ def latent_attention(q, uk_t, uv, ukv, cache, meta: AttnMeta, rot: int, scale: f
     aligned = not f32 and lat % 8 == 0 and rot % 8 == 0 and ps in (16, 32, 64)
 
     n_pf = 0  # leading sequences in the expanded form: the prompt portions in front of the step's single rows
-    if aligned and not meta.decode_only and _PREFILL_TC and not _BATCH_INVARIANT and qi is not None and kvl is not None and dim % 8 == 0 and vdim % 8 == 0 and dim <= 128 and rot <= 64 and vdim <= 128 \
-            and (gate is None or (gate.data_ptr() % 16 == 0 and gate.stride(0) % 8 == 0)):
+    if aligned and not meta.decode_only and _PREFILL_TC and not _BATCH_INVARIANT and qi is not None and kvl is not None and dim % 8 == 0 and vdim % 8 == 0 and dim <= 128 and rot <= 64 and vdim <= 128 and lat <= 512 \
+            and q.data_ptr() % 16 == 0 and ldq % 8 == 0 and (gate is None or (gate.data_ptr() % 16 == 0 and gate.stride(0) % 8 == 0)):
         n_pf = meta.num_seqs
         while n_pf > 0 and qi[n_pf] - qi[n_pf - 1] == 1:
             n_pf -= 1
@@ -1553,10 +1663,11 @@ def latent_attention(q, uk_t, uv, ukv, cache, meta: AttnMeta, rot: int, scale: f
                                       _ptr(c.status), _stream()), c)
         kv = linear(dense_rows[:, :lat], ukv)  # [total, heads * dim keys | heads * vdim values]
         if rot:
-            _check(lib().pg_rotate_pairs(_ptr(q[:, dim:]), _ll(heads * qd), _ll(qd), _ptr(cos), _ptr(sin), _ptr(meta.positions), _ci(row0), _ci(heads), _ci(rot), _ci(max_pos), _ci(0), _stream()), c)
-        rc = lib().pg_latent_prefill_tc(_ptr(q), _ll(heads * qd), _ll(qd), _ptr(q[:, dim:]), _ll(heads * qd), _ll(qd), _ptr(kv), _ptr(kv[:, heads * dim :]), _ll(kv.stride(0)),
-                                        _ptr(dense_rows[:, lat:] if rot else None), _ll(lat + rot), _ptr(gate), _ll(gate.stride(0) if gate is not None else 0), _ptr(out), _ptr(meta.q_indptr),
-                                        _ptr(kv_indptr), _ptr(lens), _ci(n_pf), _ci(row0), _ci(total), _ci(heads), _ci(dim), _ci(rot), _ci(vdim), _cf(scale), _ci(window),
+            _check(lib().pg_rotate_pairs(_ptr(q[:, dim:]), _ll(ldq), _ll(qd), _ptr(cos), _ptr(sin), _ptr(meta.positions), _ci(row0), _ci(heads), _ci(rot), _ci(max_pos), _ci(0), _stream()), c)
+        eg = gate if gate is not None else head_gate
+        rc = lib().pg_latent_prefill_tc(_ptr(q), _ll(ldq), _ll(qd), _ptr(q[:, dim:]), _ll(ldq), _ll(qd), _ptr(kv), _ptr(kv[:, heads * dim :]), _ll(kv.stride(0)),
+                                        _ptr(dense_rows[:, lat:] if rot else None), _ll(lat + rot), _ptr(eg), _ll(eg.stride(0) if eg is not None else 0), _ci(vdim if gate is not None else 1), _ptr(sink),
+                                        _ptr(out), _ptr(meta.q_indptr), _ptr(kv_indptr), _ptr(lens), _ci(n_pf), _ci(row0), _ci(total), _ci(heads), _ci(dim), _ci(rot), _ci(vdim), _cf(scale), _ci(window),
                                         _ci(sum((qi[b + 1] - qi[b] + 255) // 256 for b in range(n_pf))), _ptr(c.status), _stream())
         _check(rc, c)
         if row0 == t:
@@ -1565,22 +1676,24 @@ def latent_attention(q, uk_t, uv, ukv, cache, meta: AttnMeta, rot: int, scale: f
     n = t - row0
     qs = q[row0:]
     q_abs = torch.empty((n, heads, lat), dtype=q.dtype, device=dev)
-    _head_gemm(qs, heads * qd, qd, uk_t, q_abs)
+    _head_gemm(qs, ldq, qd, uk_t, q_abs)
     o = torch.empty((n, heads, lat), dtype=q.dtype, device=dev)
     strides = (_ll(heads * lat), _ll(lat))
-    pe = (_ptr(qs[:, dim:] if rot else None), _ll(heads * qd), _ll(qd), _ptr(cos), _ptr(sin), _ci(max_pos))
+    hg = head_gate[row0:] if head_gate is not None else None
+    extra = (_ptr(sink), _ptr(hg), _ll(hg.stride(0) if hg is not None else 0))
+    pe = (_ptr(qs[:, dim:] if rot else None), _ll(ldq), _ll(qd), _ptr(cos), _ptr(sin), _ci(max_pos))
     where = (_ptr(cache), _ptr(o), *strides, _ptr(meta.q_indptr), _ptr(meta.kv_lens), _ptr(table), _ci(table.stride(0)), _ptr(_unit_seq(meta, dev)))
     if aligned and lat <= 512 and rot <= 64:
         longest = max(meta.max_kv_len, 1)
         longest = min(longest, window + 31) if window else min(longest, 4096)
         splits = max(1, min(16, (4 * c.sms) // (n * ((heads + 15) // 16)), (longest + 127) // 128))
         splits = max(1, min(splits, c.attn_part.numel() // (n * heads * (lat + 1) * 4)))
-        rc = lib().pg_latent_attention(_ptr(q_abs), *strides, *pe, *where, _ci(row0), _ci(meta.num_seqs), _ci(n), _ci(heads), _ci(lat), _ci(rot), _ci(ps), _cf(scale), _ci(window), _ci(splits),
+        rc = lib().pg_latent_attention(_ptr(q_abs), *strides, *pe, *where, _ci(row0), _ci(meta.num_seqs), _ci(n), _ci(heads), _ci(lat), _ci(rot), _ci(ps), _cf(scale), _ci(window), *extra, _ci(splits),
                                        _ptr(c.attn_part), _ptr(c.attn_part[n * heads * splits * lat * 4 :]), _stream())
         _check(rc, c, 2 if splits > 1 else 1)
     else:
         assert row0 == 0
-        _check(lib().pg_latent_attention_plain(_ptr(q_abs), *strides, *pe, *where, _ci(n), _ci(heads), _ci(lat), _ci(rot), _ci(ps), _cf(scale), _ci(window), _ci(f32), _stream()), c)
+        _check(lib().pg_latent_attention_plain(_ptr(q_abs), *strides, *pe, *where, _ci(n), _ci(heads), _ci(lat), _ci(rot), _ci(ps), _cf(scale), _ci(window), *extra, _ci(f32), _stream()), c)
     _head_gemm(o, heads * lat, lat, uv, out[row0:].view(n, heads, vdim), gate[row0:] if gate is not None else None)
     return out
 

@@ -88,6 +88,71 @@ def embed_stream(ids, table, act_dtype):
     return x, x.to(act_dtype)
 
 
+def embed_pairs_norm(ids, table, pairs, scale: float, bigram, carried, w, eps: float, meta: AttnMeta, act_dtype):
+    """Residual stream of scaled table rows plus the rows of token pairs, and its RMS norm: ``x = table[id] * scale +
+    pairs[(previous * mul_prev + id * mul_cur) mod buckets]`` in f32, the last row of ``pairs`` for a sequence's first token.
+    ``bigram``: (buckets, mul_prev, mul_cur).  ``carried`` int32 [slots]: 1 + the last token of the request in the slot (0: none
+    yet), read and replaced.  ``pairs`` ``None``: the scaled rows only.  Returns the f32 stream and the normed rows in the
+    activation dtype."""
+    x = table[ids.long()].float() * scale
+    if pairs is not None:
+        buckets, mul_prev, mul_cur = bigram
+        qi, slots = meta.h_q_indptr, meta.h_state_slots
+        tok, rows = ids.tolist(), []
+        for b in range(meta.num_seqs):
+            prev = int(carried[slots[b]]) - 1
+            for i in range(qi[b], qi[b + 1]):
+                rows.append((prev * mul_prev + tok[i] * mul_cur) % buckets if prev >= 0 else buckets)
+                prev = tok[i]
+            carried[slots[b]] = prev + 1
+        x = x + pairs[torch.tensor(rows, dtype=torch.long, device=x.device)].float()
+    return x, stream_norm(x, w, eps, act_dtype)
+
+
+def residual_norm(y, x, w, eps: float, mult: float, act_dtype):
+    """``x += mult * y`` on the f32 stream, in place, and the RMS norm of the sum in the activation dtype (the input of the
+    next sublayer).  ``y`` is a sublayer's output, f32 or the activation dtype."""
+    x.add_(y.float() * mult)
+    return stream_norm(x, w, eps, act_dtype)
+
+
+def residual_norm_rows(rows, pos, weights, shared, shared_gate, x, w, eps: float, mult: float, act_dtype):
+    """``residual_norm`` of a mixture of experts: ``y[t] = sum_j weights[t, j] * rows[pos[t, j]] + sigmoid(shared_gate[t]) *
+    shared[t]`` (``expert_rows``; ``shared`` ``None``: the sum alone)."""
+    t, k = weights.shape
+    y = (rows.float()[pos.long()].view(t, k, -1) * weights.unsqueeze(-1)).sum(1)
+    if shared is not None:
+        y = y + shared.float() * torch.sigmoid(shared_gate.float().view(t, 1))
+    return residual_norm(y, x, w, eps, mult, act_dtype)
+
+
+def token_mix(h, mu, carried, meta: AttnMeta):
+    """Mixes of every row with its predecessor, ``h + (h' - h) * mu[i]``: ``h`` [T, W], ``mu`` f32 [n, W] -> [T, n, W].
+    ``carried`` [slots, W, 1]: the last row of the request in the slot (zeros: none yet), read and replaced."""
+    t, w = h.shape
+    out = torch.empty(t, mu.shape[0], w, dtype=h.dtype, device=h.device)
+    qi, slots = meta.h_q_indptr, meta.h_state_slots
+    for b in range(meta.num_seqs):
+        q0, q1 = qi[b], qi[b + 1]
+        if q1 == q0 or slots[b] < 0:
+            continue
+        own = h[q0:q1].float()
+        back = torch.cat((carried[slots[b], :, 0][None].float(), own[:-1]))
+        out[q0:q1] = (own[:, None] + (back - own)[:, None] * mu).to(h.dtype)
+        carried[slots[b], :, 0] = h[q1 - 1]
+    return out
+
+
+def multi_dense(x, w):
+    """``y[t, i] = w[i] x[t, i]``: ``x`` [T, n, K] (columns of a wider row, if need be), ``w`` [n, M, K]."""
+    return torch.einsum("tnk,nmk->tnm", x.float(), w.float()).to(x.dtype)
+
+
+def tanh_rows(x):
+    """``tanh(x)`` in the dtype of ``x``, formed in f32."""
+    return torch.tanh(x.float()).to(x.dtype)
+
+
 def post_norm(y, x, w, eps: float, alpha: float, act_dtype):
     """Norm after the sum, in f32: ``x <- rms_norm(alpha * x + y) * w`` (in place on the f32 stream ``x``); returns the
     copy in the activation dtype.  ``y`` is a sublayer's output, f32 or the activation dtype."""
@@ -125,12 +190,13 @@ def stream_layer_norm(x, w, eps: float, act_dtype):
     return _layer_norm(x, w, eps).to(act_dtype)
 
 
-def gated_row_norm(x, gate, w, eps: float):
-    """``rms_norm(x) * w * sigmoid(gate)`` over the last axis of ``x`` [T, H, D], rounded once; ``gate`` [T, H * D] may be a
-    column slice of a wider projection."""
-    xf = x.float()
-    n = xf * torch.rsqrt(xf.pow(2).mean(-1, keepdim=True) + eps) * w.float()
-    return (n * torch.sigmoid(gate.float().reshape(x.shape))).to(x.dtype)
+def gated_row_norm(x, gate, w, eps: float, act: str = "sigmoid"):
+    """``rms_norm(x) * w * act(gate)`` over the last axis of ``x`` [T, H, D], rounded once; ``gate`` [T, H * D] may be a
+    column slice of a wider projection, ``w`` [D] shared by the heads or [H * D]; ``act``: sigmoid or silu."""
+    xf, g = x.float(), gate.float().reshape(x.shape)
+    n = xf * torch.rsqrt(xf.pow(2).mean(-1, keepdim=True) + eps)
+    n = n * w.float().view((x.shape[1], -1) if w.numel() > x.shape[2] else (-1,))
+    return (n * torch.sigmoid(g) * (g if act == "silu" else 1.0)).to(x.dtype)
 
 
 def dense(x, w, out_dtype=None):
@@ -139,9 +205,12 @@ def dense(x, w, out_dtype=None):
     return y.to(out_dtype or x.dtype)
 
 
-def dense_glu(x, gate_up, interleaved: bool = False):
-    """``silu(gate) * up`` of the fused projection ``x @ gate_up.T``."""
-    return swiglu(dense(x, gate_up), interleaved)
+def dense_glu(x, gate_up, interleaved: bool = False, act: str = "silu"):
+    """``act(gate) * up`` of the fused projection ``x @ gate_up.T``; ``act``: silu or gelu_tanh."""
+    y = dense(x, gate_up)
+    if act == "gelu_tanh":
+        return geglu(torch.cat((y[:, 0::2], y[:, 1::2]), 1) if interleaved else y)
+    return swiglu(y, interleaved)
 
 
 def softcap_rows(logits, cap: float):
@@ -386,6 +455,27 @@ def row_norm_rope_append(q, k, v, q_norm_w, k_norm_w, cos, sin, meta: AttnMeta, 
         kp[page, off] = make(k, k_norm_w, kv_heads).to(kv_layer.dtype)
         vp[page, off] = v.reshape(t, kv_heads, vdim).to(kv_layer.dtype)
     return make(q, q_norm_w, heads)
+
+
+def temperature_table(max_pos: int, coef: float, every: int, device="cpu"):
+    """f32 ``1 + coef * ln(floor((p + 1) / every) + 1)`` for positions ``p`` below ``max_pos`` (formed in f64)."""
+    p = torch.arange(1, max_pos + 1, dtype=torch.int64, device=device)
+    return (1.0 + coef * torch.log((p // every + 1).double())).float()
+
+
+def head_norm_append(q, k, v, q_norm_w, k_norm_w, temp, meta: AttnMeta, kv_layer, heads: int, kv_heads: int, dim: int, vdim: int, eps: float):
+    """RMS norm of every query and key head with weights [dim] shared by the heads, queries times ``temp[position]`` (``None``:
+    1); keys and the values ``v`` (as they are) go to the paged cache.  Returns queries [T, heads, dim]."""
+    t, ps = q.shape[0], meta.page_size
+    norm = lambda z, n, w: (lambda f: f * torch.rsqrt(f.pow(2).mean(-1, keepdim=True) + eps) * w.float())(z.float().reshape(t, n, dim))
+    qn = norm(q, heads, q_norm_w)
+    if temp is not None:
+        qn = qn * temp[meta.positions.long()][:, None, None]
+    kp, vp = _pages_kv(kv_layer, kv_heads, dim, vdim, ps)
+    slots = meta.slot_mapping.long()
+    kp[slots // ps, slots % ps] = norm(k, kv_heads, k_norm_w).to(kv_layer.dtype)
+    vp[slots // ps, slots % ps] = v.reshape(t, kv_heads, vdim).to(kv_layer.dtype)
+    return qn.to(q.dtype)
 
 
 def capped_attention(q, kv_layer, kv_heads: int, vdim: int, meta: AttnMeta, scale: float, softcap: float = 0.0, gate=None):
@@ -664,15 +754,16 @@ def _expert_act(y, act: str):
 
 def expert_rows(x, ids, w1, w2, act: str = "relu2"):
     """Every route's expert output, not yet weighted: ``(rows [T * k, H], pos int32 [T * k])`` with the output of choice ``j``
-    of token ``t`` in row ``pos[t * k + j]``.  Weights as in ``moe_experts``; the sum is left to ``add_layer_norm_rows``."""
+    of token ``t`` in row ``pos[t * k + j]``.  ``act`` relu2: weights as in ``moe_experts``; swiglu: the rows of ``w1``
+    [E, 2 I, H] alternate (gate_i, up_i).  The sum is left to ``add_layer_norm_rows`` or ``residual_norm_rows``."""
     t, k = ids.shape
     rows = torch.zeros(t * k, w2.shape[1], dtype=x.dtype, device=x.device)
     flat = ids.reshape(-1)
     for e in range(w1.shape[0]):
         at = (flat == e).nonzero().flatten()
         if at.numel():
-            xe = x[at // k]
-            rows[at] = linear(_expert_act(linear(xe, w1[e], torch.float32) if act == "relu2" else linear(xe, w1[e]), act).to(x.dtype), w2[e])
+            y = linear(x[at // k], w1[e], torch.float32)
+            rows[at] = linear((_expert_act(y, act) if act == "relu2" else F.silu(y[:, 0::2]) * y[:, 1::2]).to(x.dtype), w2[e])
     return rows, torch.arange(t * k, dtype=torch.int32, device=x.device)
 
 
@@ -738,24 +829,26 @@ def _turn_pairs(x, cos, sin):
 def latent_rows(zq, zkv, q_norm_w, kv_norm_w, cos, sin, meta: AttnMeta, cache, latent: int, eps: float):
     """The token rows of a latent attention layer: returns the RMS-normed query latent of ``zq`` [T, q_rank] and appends to
     the paged cache (``[pages, page_size * (latent + R)]``) the RMS-normed first ``latent`` columns of ``zkv`` and its last
-    ``R`` columns rotated in pairs.  ``cos`` / ``sin`` f32 [max_pos, R / 2], ``None`` without rotated columns."""
+    ``R`` columns rotated in pairs.  ``cos`` / ``sin`` f32 [max_pos, R / 2], ``None`` without rotated columns; ``zq`` ``None``:
+    the layer's queries have no latent, and nothing is returned."""
     rms = lambda y, w: y.float() * torch.rsqrt(y.float().pow(2).mean(-1, keepdim=True) + eps) * w.float()
     row = [rms(zkv[:, :latent], kv_norm_w)]
     if zkv.shape[1] > latent:
         pos = meta.positions.long()
         row.append(_turn_pairs(zkv[:, None, latent:], cos[pos], sin[pos])[:, 0])
     cache.view(-1, zkv.shape[1])[meta.slot_mapping.long()] = torch.cat(row, -1).to(cache.dtype)
-    return rms(zq, q_norm_w).to(zq.dtype)
+    return rms(zq, q_norm_w).to(zq.dtype) if zq is not None else None
 
 
-def latent_attention(q, uk_t, uv, ukv, cache, meta: AttnMeta, rot: int, scale: float, window: int = 0, cos=None, sin=None, gate=None):
+def latent_attention(q, uk_t, uv, ukv, cache, meta: AttnMeta, rot: int, scale: float, window: int = 0, cos=None, sin=None, gate=None, head_gate=None, sink=None):
     """Latent attention over the paged cache of ``latent_rows``.  ``q`` [T, heads * (dim + rot)] per head unrotated columns,
     then the columns that are rotated here (and in place, if at all); ``uk_t`` [heads, latent, dim] and ``uv`` [heads, vdim,
     latent] up-projections of keys and values, ``ukv`` [heads * (dim + vdim), latent] the same stacked for the expanded form;
-    a row sees its last ``window`` keys (0: all).  ``gate`` [T, heads * vdim]: its sigmoid multiplies the output."""
+    a row sees its last ``window`` keys (0: all).  ``gate`` [T, heads * vdim]: its sigmoid multiplies the output; ``head_gate``
+    [T, heads]: the same with one number per head.  ``sink`` f32 [heads]: ``exp(sink)`` is part of the softmax's denominator."""
     heads, c, dim = uk_t.shape
     vdim, t = uv.shape[1], q.shape[0]
-    q = q.view(t, heads, dim + rot)
+    q = q.reshape(t, heads, dim + rot)
     rows = cache.view(-1, c + rot)
     qa = torch.einsum("thd,hcd->thc", q[..., :dim].float(), uk_t.float()).to(q.dtype).float()
     if rot:
@@ -774,7 +867,12 @@ def latent_attention(q, uk_t, uv, ukv, cache, meta: AttnMeta, rot: int, scale: f
         own = torch.arange(n - (q1 - q0), n, device=q.device)[:, None]
         hide = (at > own) | (at <= own - window) if window else at > own
         s = torch.einsum("thc,kc->htk", qa[q0:q1], k) * scale
-        p = torch.softmax(s.masked_fill(hide, float("-inf")), -1)
+        s = s.masked_fill(hide, float("-inf"))
+        if sink is not None:
+            s = torch.cat((s, sink.float().view(heads, 1, 1).expand(heads, q1 - q0, 1)), -1)
+        p = torch.softmax(s, -1)[..., :n]
+        if head_gate is not None:
+            p = p * torch.sigmoid(head_gate[q0:q1].float()).t()[:, :, None]
         lat[q0:q1] = torch.einsum("htk,kc->thc", p, k[:, :c]).to(q.dtype)
     out = torch.einsum("thc,hvc->thv", lat.float(), uv.float()).reshape(t, heads * vdim)
     if gate is not None:
@@ -1098,6 +1196,28 @@ def decay_attention(q, k, v, decay, state, meta: AttnMeta):
         for i in range(qi[s], qi[s + 1]):
             S = S * decay.view(h, 1, 1) + torch.einsum("hk,hv->hkv", kf[i], vf[i])
             out[i] = torch.einsum("hkv,hk->hv", S, qf[i]).to(q.dtype)
+        state[slots[s]] = S
+    return out
+
+
+def wkv_attention(r, k, v, f, w0, u, state, meta: AttnMeta):
+    """Linear attention with a decay per token and key channel and a bonus for the current token.  ``r, k`` [T, H, Dk], ``v``
+    [T, H, Dv]; the decay is ``exp(-exp(f + w0))`` with ``f`` f32 [T, H * Dk] and ``w0`` f32 [H * Dk]; ``o = (S + diag(u) k
+    v^T)^T r``, then ``S <- diag(decay) S + k v^T`` over the f32 ``state`` [slots, H, Dk, Dv]; ``u`` f32 [H, Dk]."""
+    t, h, dk = r.shape
+    rf, kf, vf = r.float(), k.float(), v.float()
+    dec = torch.exp(-torch.exp(f.float() + w0)).view(t, h, dk)
+    bonus = (rf * u.view(1, h, dk) * kf).sum(-1, keepdim=True) * vf
+    out = torch.zeros(t, h, v.shape[2], dtype=r.dtype, device=r.device)
+    qi = meta.h_q_indptr if meta.h_q_indptr is not None else meta.q_indptr.tolist()
+    slots = meta.h_state_slots if meta.h_state_slots is not None else meta.state_slots.tolist()
+    for s in range(meta.num_seqs):
+        if slots[s] < 0:
+            continue
+        S = state[slots[s]]
+        for i in range(qi[s], qi[s + 1]):
+            out[i] = (torch.einsum("hkv,hk->hv", S, rf[i]) + bonus[i]).to(r.dtype)
+            S = S * dec[i].unsqueeze(-1) + torch.einsum("hk,hv->hkv", kf[i], vf[i])
         state[slots[s]] = S
     return out
 

@@ -64,6 +64,7 @@ LINES = [
     ModelLine("kimi-k3", ("kimi_k3",), frozenset({"ep_backend"})),
     ModelLine("nemipel", ("nemipel",), frozenset({"dtype", "state_slots"})),
     ModelLine("vekalorn", ("vekalorn",), frozenset({"dtype"})),
+    ModelLine("zeripel", ("zeripel",), frozenset({"dtype", "state_slots"})),
 ]
 LINES[0].validate = _qwen3_validate  # type: ignore[method-assign]
 
