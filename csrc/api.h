@@ -205,6 +205,9 @@ int pg_lightning_chunked(const void* q, const void* k, const void* v, long long 
 int pg_wkv_recurrent(const void* r, const void* k, const void* v, long long ld, const void* f, long long ldf, const void* w0, const void* u, void* state, void* out, const void* q_indptr,
                      const void* slots, int num_seqs, int heads, int dk, int dv, int max_q_len, int skip_len, int is_f32, cudaStream_t stream);
 // ---- token shift and chunk-wise WKV (wkv.cu) ------------------------------------------
+// The recurrence of pg_wkv_recurrent in blocks of 16 tokens on the tensor cores, for sequences of >= min_len tokens, bf16.
+int pg_wkv_block(const void* r, const void* k, const void* v, long long ld, const void* f, long long ldf, const void* w0, const void* u, void* state, void* out, const void* q_indptr, const void* slots,
+                 int num_seqs, int heads, int dk, int dv, int min_len, cudaStream_t stream);
 // out[t, i] = h[t] + (h[t - 1] - h[t]) * mu[i]; carried [slots, width]: the row in front of a request's first one of the step.
 int pg_token_mix(const void* h, long long ldh, const void* mu, void* carried, void* out, const void* unit_seq, const void* q_indptr, const void* slots, int tokens, int n, int width, int is_f32,
                  cudaStream_t stream);

@@ -1202,16 +1202,26 @@ def decay_attention(q, k, v, decay, state, meta: AttnMeta, chunked: Optional[boo
     return out
 
 
-def wkv_attention(r, k, v, f, w0, u, state, meta: AttnMeta):
+_WKV_BLOCK_MIN = 8  # sequences of at least this many tokens take the block kernel
+
+
+def wkv_attention(r, k, v, f, w0, u, state, meta: AttnMeta, blocks: Optional[bool] = None):
     """Linear attention with a decay per token and key channel and a bonus for the current token (``reference.wkv_attention``);
-    ``r, k, v`` share a row stride."""
+    ``r, k, v`` share a row stride.  Sequences of eight tokens or more run in blocks on the tensor cores (bf16, sizes that are
+    multiples of 8), shorter ones on the recurrence."""
     t, h, dk = r.shape
     dv = v.shape[2]
     assert r.stride(2) == 1 and r.stride(1) == dk and k.stride(1) == dk and v.stride(1) == dv and f.dtype == torch.float32 and f.stride(1) == 1 and f.shape[1] == h * dk
     assert state.is_contiguous() and state.dtype == w0.dtype == u.dtype == torch.float32 and w0.is_contiguous() and u.is_contiguous()
     out = torch.empty((t, h, dv), dtype=r.dtype, device=r.device)
-    _check(lib().pg_wkv_recurrent(_ptr(r), _ptr(k), _ptr(v), _ll(_same_rows(r, k, v)), _ptr(f), _ll(f.stride(0)), _ptr(w0), _ptr(u), _ptr(state), _ptr(out), _ptr(meta.q_indptr), _ptr(meta.state_slots),
-                                  _ci(meta.num_seqs), _ci(h), _ci(dk), _ci(dv), _ci(int(meta.max_q_len)), _ci(0), _ci(_is_f32(r)), _stream()), ctx(r.device))
+    f32, ld, c = _is_f32(r), _same_rows(r, k, v), ctx(r.device)
+    args = (_ptr(r), _ptr(k), _ptr(v), _ll(ld), _ptr(f), _ll(f.stride(0)), _ptr(w0), _ptr(u), _ptr(state), _ptr(out), _ptr(meta.q_indptr), _ptr(meta.state_slots), _ci(meta.num_seqs), _ci(h), _ci(dk), _ci(dv))
+    aligned = dk % 8 == 0 and dv % 8 == 0 and dk <= 128 and ld % 8 == 0 and f.stride(0) % 4 == 0 and all(x.data_ptr() % 16 == 0 for x in (r, k, v, f))
+    blocks = (_LINEAR_CHUNKED if blocks is None else blocks) and int(meta.max_q_len) >= _WKV_BLOCK_MIN and not f32 and aligned
+    if blocks:
+        _check(lib().pg_wkv_block(*args, _ci(_WKV_BLOCK_MIN), _stream()), c)
+    if not blocks or _has_short_rows(meta, _WKV_BLOCK_MIN):
+        _check(lib().pg_wkv_recurrent(*args, _ci(int(meta.max_q_len)), _ci(_WKV_BLOCK_MIN if blocks else 0), _ci(f32), _stream()), c)
     return out
 
 
