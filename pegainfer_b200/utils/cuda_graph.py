@@ -22,6 +22,7 @@ attention path), pegainfer-core/src/cuda_graph/dump.rs:24-135 (DOT export).
 """
 from __future__ import annotations
 
+import gc
 import os
 import time
 from typing import Optional
@@ -193,11 +194,16 @@ class DecodeGraphs:
             if self.pool is None:
                 self.pool = torch.cuda.graph_pool_handle()
             trace0 = len(_K().GemmTrace.names)
+            # a graph of an engine that is gone, freed by the collector in the middle of a capture, would invalidate it
+            collecting = gc.isenabled()
+            gc.disable()
             g.capture_begin(pool=self.pool)
             try:
                 logits = self._forward(b, greedy, splits)
             finally:
                 g.capture_end()
+                if collecting:
+                    gc.enable()
             self.trace_range[key] = (trace0, len(_K().GemmTrace.names))  # GEMM trace slots of this graph (debug aid)
             # The first launch of an instantiated graph uploads it to the device (measured: 50 - 70 ms
             # for a whole-step graph).  Pay that here, on the padding inputs the capture ran on, and not
