@@ -6,7 +6,7 @@ distinct weight / KV buffers (larger than L2 in total, so every launch streams f
 HBM), replayed after warm-up and timed with CUDA events.  Fractions are against the
 measured peaks in MEASURED_PEAKS.json (copy bandwidth, cuBLAS bf16 throughput).
 
-    python bench_ops.py [--only gemm|attn|small|gdn|kda|nemipel|vekalorn|moe|mla] [--iters 16] [--json out.json]
+    python bench_ops.py [--only gemm|attn|small|gdn|kda|nemipel|vekalorn|zeripel|moe|mla] [--iters 16] [--json out.json]
     python bench_ops.py --single gemm:64x4096x4096      # one op, few launches (ncu target)
 
 Plays the role of the reference's kernel/op report binaries
@@ -340,6 +340,112 @@ def vekalorn_cases(iters):
     return rows
 
 
+def zeripel_cases(iters):
+    """Kernels of the Zeripel line, each beside the like kernel of the closest line at the same size (indented rows): latent
+    attention with a sink and a head gate beside the Vekalorn line's, WKV beside the Nemipel line's channel delta, attention
+    whose values are its keys beside plain paged attention, gated experts with a shared one beside the DeepSeek-V2 line's."""
+    from pegainfer_b200.models.layers import LatentHeads
+    from pegainfer_b200.ops import cuda as K
+    from pegainfer_b200.ops.reference import pair_rope_tables, temperature_table
+
+    rows, page, c, r, d = [], 16, 512, 64, 128
+    few = max(2, iters // 4)
+    bf = lambda *s: torch.randn(*s, device=DEV).bfloat16()
+    f32 = lambda *s: torch.randn(*s, device=DEV)
+    cos, sin = pair_rope_tables(16384, r, 1e4, DEV)
+
+    def pair(name, like, new, old, by, by_old, fl, fl_old, nvar, it, timer=time_graph):
+        t = (lambda fn: timer(fn, nvar, it)) if timer is time_graph else (lambda fn: timer(lambda: fn(0), it))
+        rows.append((name, t(new), by, fl))
+        rows.append(("  " + like, t(old), by_old, fl_old))
+
+    for heads, bs, ctx in ((16, 64, 1024), (32, 64, 1024), (64, 16, 8192), (16, 1, 8192)):
+        meta, pages = _meta_for([1] * bs, [ctx] * bs, page)
+        caches = [bf(pages, page * (c + r)) for _ in range(3)]
+        uk, uv, q, gate, hg, sink = bf(heads * d, c) * 0.05, bf(heads * d, c) * 0.05, bf(bs, heads * (d + r)), bf(bs, heads * d), bf(bs, heads), f32(heads)
+        w = LatentHeads(uk, uv, heads)
+        by, fl = bs * ctx * (c + r) * 2 + heads * 2 * d * c * 2, 2.0 * bs * ctx * heads * (2 * c + r)
+        pair(f"latent_attention decode {heads}h {bs}x{ctx} sink, head gate", "latent_attention gate", lambda i: K.latent_attention(q, w.uk_t, w.uv, w.ukv, caches[i], meta, r, 0.07, 0, cos, sin, None, hg, sink),
+             lambda i: K.latent_attention(q, w.uk_t, w.uv, w.ukv, caches[i], meta, r, 0.07, 0, cos, sin, gate), by, by, fl, fl, 3, few)
+    for heads, ns, ql in ((16, 1, 4096), (16, 8, 1024), (64, 1, 4096), (16, 1, 16384)):
+        t = ns * ql
+        meta, pages = _meta_for([ql] * ns, [ql] * ns, page)
+        cache, q, gate, hg, sink = bf(pages, page * (c + r)), bf(t, heads * (d + r)), bf(t, heads * d), bf(t, heads), f32(heads)
+        w = LatentHeads(bf(heads * d, c) * 0.05, bf(heads * d, c) * 0.05, heads)
+        fl = 2.0 * t * c * heads * 2 * d + ns * ql * ql * heads * (2.0 * d + r)
+        pair(f"latent_attention prefill {heads}h {ns}x{ql} sink, head gate", "latent_attention gate", lambda i: K.latent_attention(q, w.uk_t, w.uv, w.ukv, cache, meta, r, 0.07, 0, cos, sin, None, hg, sink),
+             lambda i: K.latent_attention(q, w.uk_t, w.uv, w.ukv, cache, meta, r, 0.07, 0, cos, sin, gate), t * (c + r) * 2, t * (c + r) * 2, fl, fl, 1, few, time_eager)
+    h = 32
+    for name, lens in (("decode 64", [1] * 64), ("decode 8", [1] * 8), ("decode 1", [1]), ("prefill 1x4096", [4096]), ("prefill 8x1024", [1024] * 8), ("prefill 16x256", [256] * 16), ("prefill 64x16", [16] * 64)):
+        rows.extend(wkv_rows(name, lens, h, d, few))
+    for hq, hkv, bs, ctx in ((32, 8, 64, 1152), (32, 8, 64, 4096), (32, 8, 1, 1152), (64, 8, 64, 4096)):
+        meta, pages = _meta_for([1] * bs, [ctx] * bs, page)
+        kv, q = [bf(pages, 2, page, hkv, d) for _ in range(1 if bs * ctx > 1 << 16 else 4)], bf(bs, hq, d)
+        by, fl = bs * ctx * 2 * hkv * d * 2, 4.0 * bs * ctx * hq * d
+        pair(f"capped_attention (no cap) decode {bs}x{ctx} {hq}/{hkv}", "paged_attention", lambda i: K.capped_attention(q, kv[i].view(pages, -1), hkv, d, meta, d ** -0.5), lambda i: K.paged_attention(q, kv[i], meta), by, by, fl, fl,
+             len(kv), iters)
+    for ns, ql in ((4, 1024), (1, 4096), (1, 16384), (16, 256)):
+        meta, pages = _meta_for([ql] * ns, [ql] * ns, page)
+        kv, q = bf(pages, 2, page, 8, d), bf(ns * ql, 32, d)
+        by, fl = ns * ql * (2 * 32 + 2 * 8) * d * 2, 2.0 * ns * ql * ql * 32 * d
+        pair(f"capped_attention (no cap) prefill {ns}x{ql}", "paged_attention", lambda i: K.capped_attention(q, kv.view(pages, -1), 8, d, meta, d ** -0.5), lambda i: K.paged_attention(q, kv, meta), by, by, fl, fl, 1, few)
+    for t, w, ff, e, k in ((64, 2048, 1408, 64, 6), (1, 2048, 1408, 64, 6), (4096, 2048, 1408, 64, 6), (64, 7168, 2048, 16, 4), (8192, 4096, 2048, 32, 4)):
+        x, lg, bias = bf(t, w), f32(t, e + 1), f32(e) * 0.1
+        ids, wts = K.router_topk(lg[:, :e], k, "sigmoid", bias, 1, 1, True, 2.5)
+        gu, w2, sh, gate = [bf(e, 2 * ff, w) * 0.02 for _ in range(2)], [bf(e, w, ff) * 0.02 for _ in range(2)], bf(t, w), lg[:, e:]
+        res, r16, nw, nw16 = f32(t, w), bf(t, w), torch.ones(w, device=DEV), torch.ones(w, device=DEV).bfloat16()
+        by, fl = min(e, t * k) * 3 * ff * w * 2, 2.0 * t * k * 3 * ff * w
+        pair(f"expert_rows swiglu + residual_norm_rows T{t} {w} / {ff}, {e} experts top {k}", "moe_experts + add_rms_norm",
+             lambda i: K.residual_norm_rows(*K.expert_rows(x, ids, gu[i], w2[i], "swiglu"), wts, sh, gate, res, nw, 1e-5, 0.7, torch.bfloat16),
+             lambda i: K.add_rms_norm(K.moe_experts(x, ids, wts, gu[i], w2[i]).to(torch.bfloat16), r16, nw16, 1e-5), by, by, fl, fl, 2, few)
+    for t in (64, 4096):
+        w = 4096
+        meta, pages = _meta_for([1] * 64 if t == 64 else [1024] * 4, [1024] * 64 if t == 64 else [1024] * 4, page)
+        n = meta.num_seqs
+        meta.state_slots = torch.arange(n, dtype=torch.int32, device=DEV)
+        x32, y32, x16, w32, w16 = [f32(t, w) for _ in range(4)], [f32(t, w) for _ in range(4)], [bf(t, w) for _ in range(4)], torch.ones(w, device=DEV), torch.ones(w, device=DEV).bfloat16()
+        y = y32 if t == 64 else x16
+        pair(f"residual_norm {t}x{w}", "post_norm", lambda i: K.residual_norm(y[i], x32[i], w32, 1e-6, 0.5, torch.bfloat16), lambda i: K.post_norm(y[i], x32[i], w32, 1e-6, 2.0, torch.bfloat16),
+             *[t * w * (10 + y[0].element_size())] * 2, 0, 0, 4, iters)
+        o, gt, wh = [bf(t, 32, 128) for _ in range(4)], [bf(t, 4096) for _ in range(4)], torch.ones(4096, device=DEV)
+        pair(f"gated_row_norm silu {t}x32x128", "gated_row_norm sigmoid", lambda i: K.gated_row_norm(o[i], gt[i], wh, 1e-6, "silu"), lambda i: K.gated_row_norm(o[i], gt[i], wh[:128], 1e-6), *[t * w * 6] * 2, 0, 0, 4, iters)
+        mu, car, cw, cs = torch.rand(5, w, device=DEV), bf(n, w, 1), f32(w, 4), bf(n, w, 3)
+        pair(f"token_mix {t}x{w}, 5 mixes", "conv_silu", lambda i: K.token_mix(x16[i], mu, car, meta), lambda i: K.conv_silu(x16[i], cw, cs, meta), t * w * 12, t * w * 4, 0, 0, 4, iters)
+        table, pairs, tok = bf(65536, w), bf(65537, w), torch.zeros(n, dtype=torch.int32, device=DEV)
+        ids = torch.randint(0, 65536, (t,), dtype=torch.int32, device=DEV)
+        pair(f"embed_pairs_norm {t}x{w}", "embed_stream", lambda i: K.embed_pairs_norm(ids, table, pairs, 64.0, (65536, 31, 7), tok, w32, 1e-6, meta, torch.bfloat16), lambda i: K.embed_stream(ids, table, torch.bfloat16),
+             t * w * 10, t * w * 8, 0, 0, 1, iters)
+        z = [bf(t, 40 * d + 8 * d) for _ in range(4)]
+        kv, one, qn, kn, temp = bf(pages, 2 * page * 8 * d), torch.ones(d, device=DEV), torch.ones(32 * d, device=DEV), torch.ones(8 * d, device=DEV), temperature_table(8192, 0.1, 4096, DEV)
+        c32, s32 = pair_rope_tables(8192, d, 1e4, DEV)
+        cut = lambda x: (x[:, : 32 * d], x[:, 32 * d : 40 * d], x[:, 40 * d :])
+        pair(f"head_norm_append {t}", "row_norm_rope_append", lambda i: K.head_norm_append(*cut(z[i]), one, one, temp, meta, kv, 32, 8, d, d, 1e-6),
+             lambda i: K.row_norm_rope_append(*cut(z[i]), qn, kn, c32, s32, meta, kv, 32, 8, d, d, 1e-6), *[t * 48 * d * 4] * 2, 0, 0, 4, iters)
+        mats = [bf(4, w, w) * 0.02 for _ in range(3)]
+        xm, by, fl = bf(t, 5, w), 4 * w * w * 2 + t * 8 * w * 2, 2.0 * t * 4 * w * w
+        pair(f"multi_dense {t} x 4 x {w} x {w}", "linear of the stacked matrices", lambda i: K.multi_dense(xm[:, :4], mats[i]), lambda i: K.linear(xm[:, 0], mats[i].view(4 * w, w)), by, by, fl, fl, 3, few)
+        gup = [bf(24576, w) * 0.02 for _ in range(3)]
+        by, fl = 24576 * w * 2 + t * (w + 12288) * 2, 2.0 * t * w * 24576
+        pair(f"dense_glu gelu {t} x 12288 x {w}", "dense_glu silu", lambda i: K.dense_glu(x16[0], gup[i], True, "gelu_tanh"), lambda i: K.dense_glu(x16[0], gup[i], True), by, by, fl, fl, 3, few)
+    return rows
+
+
+def wkv_rows(name, lens, h, d, iters):
+    """The WKV recurrence and, beside it, the channel-delta one at the same sizes."""
+    from pegainfer_b200.ops import cuda as K
+
+    meta, _ = _meta_for(lens, lens, 16)
+    t, n = sum(lens), len(lens)
+    meta.state_slots = torch.arange(n, dtype=torch.int32, device=DEV)
+    st, x = [torch.zeros(n, h, d, d, device=DEV) for _ in range(3)], torch.randn(t, 4 * h * d, device=DEV).bfloat16()
+    q, k, v = (x[:, j * h * d : (j + 1) * h * d].view(t, h, d) for j in range(3))
+    f, w0, u = torch.randn(t, h * d, device=DEV), torch.linspace(-6, 0, h * d, device=DEV), torch.rand(h, d, device=DEV)
+    b, a_log, dt = torch.randn(t, h, device=DEV).bfloat16(), torch.zeros(h, device=DEV), torch.zeros(h * d, device=DEV)
+    by, fl = n * h * d * d * 8 + t * h * d * 12, 4.0 * t * h * d * d
+    return [(f"wkv_attention {name}", time_graph(lambda i: K.wkv_attention(q, k, v, f, w0, u, st[i], meta), 3, iters), by, fl),
+            ("  channel_delta", time_graph(lambda i: K.channel_delta(q, k, v, f, b, a_log, dt, st[i], meta), 3, iters), by, 2 * fl)]
+
+
 def kda_cases(iters, only=None):
     """KDA recurrence (decay per key channel, gate arithmetic in the kernel) and the attention-residual mix at the Kimi-K3
     shape: 96 heads with a 128x128 f32 state, hidden 7168, 8 snapshots."""
@@ -659,6 +765,8 @@ def main():
             name, ms, by, fl = gdn_cases(args.iters, only=[("single", [dims[1]] * dims[0])])[0]
         elif kind in ("capped", "lightning", "chdelta"):  # sequences x tokens: one prompt step of the Nemipel line's kernel
             name, ms, by, fl = nemipel_single(kind, dims[0], dims[1], args.iters)
+        elif kind == "wkv":
+            name, ms, by, fl = wkv_rows("single", [dims[1]] * dims[0], 32, 128, args.iters)[0]
         elif kind == "chain":
             ms, by, fl = chain_case(dims[0], dims[1], dims[2], dims[3], args.iters)
         elif kind == "fp8":
@@ -720,6 +828,8 @@ def main():
             rows.extend(nemipel_cases(args.iters))
         if args.only in (None, "vekalorn"):
             rows.extend(vekalorn_cases(args.iters))
+        if args.only in (None, "zeripel"):
+            rows.extend(zeripel_cases(args.iters))
         if args.only in (None, "moe"):
             rows.extend(moe_cases(args.iters))
         if args.only in (None, "mla"):

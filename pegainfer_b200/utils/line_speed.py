@@ -3,6 +3,9 @@
 * ``nemipel`` beside the Qwen3.5 line (linear-attention layers with recurrent state interleaved with paged attention).
 * ``vekalorn`` beside the DeepSeek-V2 line (latent attention and mixture of experts in every layer): the same heads, latents
   and number of experts, and expert widths that give both the same expert weights (two matrices against three).
+* ``zeripel`` beside the Kimi-K3 line (a recurrence with a decay per key channel, latent attention and sigmoid-routed experts
+  with a shared one): the same layer order, heads, latents and expert weights; its full-attention layers stand in for both
+  kinds of Zeripel attention, and its routed experts work behind two further projections of the stream's width.
 
 Device time (CUDA events) of whole steps of the executor: prefill steps of the given batches, and replays of the decode graph
 at a batch and context.  Weights and state are larger than L2 at every size, so no flush is needed.
@@ -43,6 +46,16 @@ def _vekalorn_configs(width, heads, q_rank, window, experts, top, ff, periods, v
     return {"vekalorn": a, "deepseek_v2": b}
 
 
+def _zeripel_configs(width, ff, heads, kv_heads, experts, top, expert_ff, shared_ff, periods, vocab=32768):
+    from ..config import PRESETS, _zeripel, _zeripel_experts
+
+    a = _zeripel(width, vocab, ff, heads, kv_heads, 128, 512, 128, 64, 128, heads, 128, 128, _zeripel_experts(experts, top, expert_ff, shared_ff, 2.5), periods, max_position=16384)
+    b = replace(PRESETS["kimi-k3"], vocab_size=vocab, hidden_size=width, num_layers=4 * periods, layer_types=("full_attention", "full_attention", "linear_attention", "full_attention") * periods,
+                num_q_heads=heads, num_kv_heads=heads, intermediate_size=ff, n_routed_experts=experts, num_experts_per_tok=top, n_shared_experts=shared_ff // expert_ff, moe_intermediate_size=expert_ff,
+                latent_moe_dim=width, attn_res_block=4, expert_quant="bf16", max_position=16384)
+    return {"zeripel": a, "kimi_k3": b}
+
+
 LINES = {
     "nemipel": Comparison("qwen35", ("width", "ff", "heads", "kv_heads", "recurrent_heads"), (("2048", (2048, 6144, 16, 8, 16)), ("4096", (4096, 12288, 32, 8, 32)), ("5120", (5120, 17408, 40, 8, 40))),
                           ((1, 4096), (8, 1024)), ((64, 1024), (8, 1024), (1, 1024)), _nemipel_configs, (("layers", 12), ("head_dim", 128))),
@@ -50,6 +63,10 @@ LINES = {
                            (("2048", (2048, 16, 1536, 1024, 64, 6, 2112, 4)), ("4096", (4096, 32, 1536, 1024, 32, 4, 3072, 2)), ("7168", (7168, 64, 1536, 1024, 16, 4, 3072, 2))),
                            ((1, 4096), (8, 1024)), ((64, 1024), (16, 8192), (8, 1024), (1, 1024)), _vekalorn_configs,
                            (("kv_rank", 512), ("dim", 128), ("rot_dim", 64), ("vdim", 128), ("layers_per_period", "1 full + 2 windowed"))),
+    "zeripel": Comparison("kimi_k3", ("width", "ff", "heads", "kv_heads", "experts", "top", "expert_ff", "shared_ff", "periods"),
+                          (("2048", (2048, 8192, 16, 4, 64, 6, 1408, 2816, 3)), ("4096", (4096, 12288, 32, 8, 32, 4, 2048, 4096, 2)), ("7168", (7168, 18432, 64, 8, 16, 4, 2048, 2048, 2))),
+                          ((1, 4096), (8, 1024)), ((64, 1024), (16, 8192), (8, 1024), (1, 1024)), _zeripel_configs,
+                          (("kv_rank", 512), ("dim", 128), ("rot_dim", 64), ("layers_per_period", "latent, latent over the same cache, WKV, attention"))),
 }
 
 
