@@ -26,7 +26,10 @@ class MixerSpec:
     over a cached latent of ``kv_rank`` columns and, with ``rot_dims``, a shared rotated key part; queries through a latent of
     ``q_rank``, or straight from the stream without one; a sliding window, an element-wise or per-head output gate and a sink
     are optional) or ``"wkv"`` (token-shift mixes, a decay per key channel from a low-rank projection of ``decay_rank``, a bonus
-    for the current token)."""
+    for the current token), ``"ssd"`` (state-space duality: one decay per token and head, ``dim`` state rows, ``kv_heads`` groups
+    of heads that share them, a convolution, a gate in front of a norm in ``norm_groups`` parts), ``"lru"`` (gated linear
+    recurrence per channel over ``heads`` blocks of ``dim`` channels, a convolution, a GELU branch) or ``"parallel"`` (the mixers
+    ``parts`` side by side over one input, each times its ``part_scales``)."""
 
     kind: str
     heads: int
@@ -52,6 +55,16 @@ class MixerSpec:
     head_norm: bool = False  # attention: query and key norms per head (False: over the whole projection)
     values_are_keys: bool = False  # attention: no value projection, the values are the projected keys before their norm
     q_temp: tuple = ()  # attention: (coef, every): queries at position p times 1 + coef * ln(floor((p + 1) / every) + 1)
+    bias: bool = False  # attention: query, key and value projections have biases
+    head_temp: bool = False  # attention: a learned factor per head on the scores
+    slopes: tuple = ()  # attention: per head, what the (capped) score loses per position of distance
+    norm_groups: int = 0
+    parts: tuple = ()
+    part_scales: tuple = ()
+
+    def flat(self) -> tuple:
+        """The mixer, or those it has side by side."""
+        return self.parts or (self,)
 
 
 @dataclass(frozen=True)
@@ -81,12 +94,12 @@ class LayerSpec:
     mixer: MixerSpec
     ff: int = 0  # width of the gated feed-forward (0: the layer has none)
     moe: Optional[ExpertsSpec] = None
-    act: str = "silu"  # of the feed-forward's gate: silu or gelu_tanh
+    act: str = "silu"  # of the feed-forward's gate: silu or gelu_tanh; xielu (two learned numbers): a feed-forward without gate
 
 
 @dataclass
 class ModelConfig:
-    family: str = "qwen3"  # qwen3 | qwen35 | deepseek_v2 | kimi_k2 | glm_dsa | gemma4 | kimi_k3 | nemipel | vekalorn | zeripel
+    family: str = "qwen3"  # qwen3 | qwen35 | deepseek_v2 | kimi_k2 | glm_dsa | gemma4 | kimi_k3 | nemipel | vekalorn | zeripel | nonetar
     vocab_size: int = 1024
     hidden_size: int = 256
     num_layers: int = 2
@@ -154,7 +167,7 @@ class ModelConfig:
     attn_res_block: int = 0
     kda_gate_rank: int = 0
     kda_gate_lower_bound: float = -5.0
-    # families whose layers are listed one by one (Nemipel, Vekalorn, Zeripel lines): the mixer and feed-forward of every layer, the factor on
+    # families whose layers are listed one by one (Nemipel, Vekalorn, Zeripel, Nonetar lines): the mixer and feed-forward of every layer, the factor on
     # the stream in the norm after the sum; final_logit_softcapping caps the logits
     layer_specs: tuple = ()
     postln_alpha: float = 1.0
@@ -162,6 +175,9 @@ class ModelConfig:
     embed_scale: float = 1.0
     bigram: tuple = ()
     residual_mult: float = 1.0
+    # Nonetar line: copies of the residual stream, factor on the logits
+    streams: int = 1
+    logit_scale: float = 1.0
 
     # -- derived ---------------------------------------------------------------
     @property
@@ -363,6 +379,36 @@ PRESETS["tiny-zeripel"] = _zeripel(80, 256, 112, 4, 2, 24, 40, 16, 8, 32, 3, 16,
 PRESETS["small-zeripel"] = _zeripel(1024, 4096, 2048, 16, 4, 128, 512, 128, 64, 128, 8, 128, 64, _zeripel_experts(16, 4, 512, 512, 2.5), 2, max_position=8192)
 # layers of a mid-size hybrid mixture of experts, for benchmarks (not a released configuration)
 PRESETS["zeripel-16b-shape"] = _zeripel(2048, 102400, 8192, 16, 4, 128, 512, 128, 64, 128, 16, 128, 64, _zeripel_experts(64, 6, 1408, 2816, 2.5), 7)
+
+
+def alibi_slopes(heads: int) -> tuple:
+    """Score lost per position of distance, a geometric row over the heads that ends at 2^-8."""
+    return tuple(2.0 ** (-8.0 * (h + 1) / heads) for h in range(heads))
+
+
+def _nonetar_parallel(heads: int, kv_heads: int, dim: int, vdim: int, scale: float, softcap: float, window: int, width: int, blocks: int, conv: int, scales: tuple) -> MixerSpec:
+    left = MixerSpec("attention", heads, dim, vdim, kv_heads=kv_heads, scale=scale, softcap=softcap, window=window, head_norm=True, bias=True, head_temp=True, slopes=alibi_slopes(heads))
+    return MixerSpec("parallel", 0, 0, 0, parts=(left, MixerSpec("lru", blocks, width // blocks, width // blocks, conv=conv)), part_scales=scales)
+
+
+def _nonetar_ssd(heads: int, vdim: int, state: int, groups: int, norm_groups: int, conv: int) -> MixerSpec:
+    return MixerSpec("ssd", heads, state, vdim, kv_heads=groups, norm_groups=norm_groups, conv=conv)
+
+
+def _nonetar(width: int, vocab: int, ff: int, streams: int, parallel: MixerSpec, ssd: MixerSpec, periods: int, **kw) -> ModelConfig:
+    """A Nonetar stack of ``periods`` x (attention beside a recurrent block, twice, then state-space duality)."""
+    layers = tuple(LayerSpec(m, ff, act="xielu") for _ in range(periods) for m in (parallel, parallel, ssd))
+    left = parallel.parts[0]
+    base = dict(family="nonetar", vocab_size=vocab, hidden_size=width, num_layers=len(layers), num_q_heads=left.heads, num_kv_heads=left.kv_heads, head_dim=left.dim, intermediate_size=ff, rms_eps=1e-6,
+                qk_norm=False, layer_specs=layers, streams=streams, logit_scale=0.5, max_position=65536)
+    base.update(kw)
+    return ModelConfig(**base)
+
+
+PRESETS["tiny-nonetar"] = _nonetar(72, 256, 104, 3, _nonetar_parallel(4, 2, 24, 32, 0.25, 30.0, 40, 96, 3, 4, (0.9, 0.6)), _nonetar_ssd(6, 16, 24, 3, 2, 4), 1, max_position=4096)
+PRESETS["small-nonetar"] = _nonetar(1024, 4096, 4096, 2, _nonetar_parallel(8, 2, 128, 128, 128 ** -0.5, 50.0, 256, 1024, 8, 4, (1.0, 0.5)), _nonetar_ssd(32, 64, 128, 4, 4, 4), 2, max_position=8192)
+# layers as wide as those of an 8 B-parameter model, for benchmarks (not a released configuration)
+PRESETS["nonetar-8b-shape"] = _nonetar(4096, 102400, 16384, 4, _nonetar_parallel(32, 8, 128, 128, 128 ** -0.5, 50.0, 2048, 4096, 16, 4, (1.0, 0.5)), _nonetar_ssd(128, 64, 128, 8, 8, 4), 10)
 PRESETS["small-glm-fp8"] = replace(PRESETS["small-glm"], expert_quant="fp8_block128", dense_quant="fp8_block128")
 for _name in ("tiny-dsv2", "small-dsv2", "dsv2-lite"):
     if _name in PRESETS:
@@ -377,7 +423,7 @@ def preset(name: str, **overrides) -> ModelConfig:
 
 def detect_family(cfg: dict) -> str:
     """Map a ``config.json`` to a model line (exactly one line must claim it)."""
-    if cfg.get("architecture") in ("Nemipel", "Vekalorn", "Zeripel"):
+    if cfg.get("architecture") in ("Nemipel", "Vekalorn", "Zeripel", "Nonetar"):
         return cfg["architecture"].lower()
     mt = cfg.get("model_type", "")
     archs = " ".join(cfg.get("architectures", []))
@@ -636,6 +682,62 @@ def zeripel_to_json(cfg: ModelConfig) -> dict:
     return out
 
 
+def _nonetar_mixer(i: int, kind: str, m: dict) -> MixerSpec:
+    if kind == "parallel":
+        a, b = m["left"], m["right"]
+        window = (a.get("mask") or {}).get("size", 0)
+        if a["heads"] % a["kv_heads"]:
+            raise ValueError(f"layer {i}: {a['heads']} query heads over {a['kv_heads']} key heads")
+        if a.get("mask") and window < 1:
+            raise ValueError(f"layer {i}: a window of {window} positions")
+        if b["width"] % b["blocks"]:
+            raise ValueError(f"layer {i}: {b['width']} channels in {b['blocks']} blocks")
+        return _nonetar_parallel(a["heads"], a["kv_heads"], a["dim"], a["vdim"], float(a["scale"]), float(a.get("softcap") or 0.0), window, b["width"], b["blocks"], b["conv"],
+                                 (float(m.get("left_scale", 1.0)), float(m.get("right_scale", 1.0))))
+    if kind == "mamba2":
+        if m["heads"] % m["groups"] or m["heads"] * m["vdim"] % m["norm_groups"]:
+            raise ValueError(f"layer {i}: {m['heads']} heads of {m['vdim']} in {m['groups']} groups, normed in {m['norm_groups']} parts")
+        return _nonetar_ssd(m["heads"], m["vdim"], m["state"], m["groups"], m["norm_groups"], m["conv"])
+    raise ValueError(f"layer {i}: no mixer of type {kind!r}")
+
+
+def _nonetar_from_json(cfg: dict, model_dir: Optional[str]) -> ModelConfig:
+    """``config.json`` of the Nonetar line: sizes and constants per layer."""
+    layers = []
+    for i, entry in enumerate(cfg["layers"]):
+        mlp = entry.get("mlp")
+        if mlp is not None and mlp.get("kind", "dense") != "dense":
+            raise ValueError(f"layer {i}: no feed-forward of kind {mlp['kind']!r}")
+        layers.append(LayerSpec(_nonetar_mixer(i, entry["type"], entry["mixer"]), mlp["ff"] if mlp else 0, act="xielu"))
+    flat = [m for l in layers for m in l.mixer.flat()]
+    attn = [m for m in flat if m.kind == "attention"] or flat[:1]
+    return ModelConfig(family="nonetar", vocab_size=cfg["vocab"], hidden_size=cfg["width"], num_layers=len(layers), num_q_heads=attn[0].heads, num_kv_heads=max(attn[0].kv_heads, 1), head_dim=attn[0].dim,
+                       intermediate_size=max(l.ff for l in layers), rms_eps=cfg["norm"]["eps"], qk_norm=False, layer_specs=tuple(layers), streams=cfg.get("streams", 1),
+                       logit_scale=float(cfg.get("logit_scale", 1.0)), max_position=131072, eos_token_ids=_eos_ids(model_dir, cfg))
+
+
+def nonetar_to_json(cfg: ModelConfig) -> dict:
+    """The ``config.json`` that ``_nonetar_from_json`` reads back."""
+    layers = []
+    for l in cfg.layer_specs:
+        m = l.mixer
+        if m.kind == "parallel":
+            a, b = m.parts
+            left = dict(heads=a.heads, kv_heads=a.kv_heads, dim=a.dim, vdim=a.vdim, scale=a.scale)
+            if a.softcap:
+                left["softcap"] = a.softcap
+            if a.window:
+                left["mask"] = dict(size=a.window)
+            mix = dict(left=left, right=dict(width=b.heads * b.dim, blocks=b.heads, conv=b.conv), left_scale=m.part_scales[0], right_scale=m.part_scales[1])
+        else:
+            mix = dict(heads=m.heads, vdim=m.vdim, state=m.dim, groups=m.kv_heads, norm_groups=m.norm_groups, conv=m.conv)
+        layers.append(dict(type="parallel" if m.kind == "parallel" else "mamba2", mixer=mix, mlp=dict(kind="dense", ff=l.ff) if l.ff else None))
+    out = dict(architecture="Nonetar", vocab=cfg.vocab_size, width=cfg.hidden_size, norm=dict(eps=cfg.rms_eps), streams=cfg.streams, logit_scale=cfg.logit_scale, layers=layers)
+    if cfg.eos_token_ids:
+        out["eos_token_id"] = list(cfg.eos_token_ids)
+    return out
+
+
 def from_hf(cfg: dict, model_dir: Optional[str] = None) -> ModelConfig:
     family = detect_family(cfg)
     top = cfg
@@ -645,6 +747,8 @@ def from_hf(cfg: dict, model_dir: Optional[str] = None) -> ModelConfig:
         return _vekalorn_from_json(cfg, model_dir)
     if family == "zeripel":
         return _zeripel_from_json(cfg, model_dir)
+    if family == "nonetar":
+        return _nonetar_from_json(cfg, model_dir)
     if family == "qwen35" and "text_config" in cfg:
         cfg = cfg["text_config"]
     if family == "kimi_k2" and "text_config" in cfg:

@@ -25,7 +25,7 @@ from .contract import EngineInfo, KvCapacity
 from .driver import Engine
 
 
-F32_FAMILIES = ("nemipel", "vekalorn", "zeripel")  # lines whose kernels also run in 32-bit on the GPU
+F32_FAMILIES = ("nemipel", "vekalorn", "zeripel", "nonetar")  # lines whose kernels also run in 32-bit on the GPU
 
 
 def resolve_model_config(ecfg: EngineConfig) -> ModelConfig:

@@ -56,14 +56,14 @@ class RecurrentState(StateSlots):
 class LayerStates(StateSlots):
     def __init__(self, num_slots: int, geometries, dtype, device, token: bool = False):
         """``geometries``: ``(heads, dk, dv, conv_channels, taps)`` of every recurrent layer, ``taps == 0`` without
-        short convolutions."""
+        short convolutions.  What a layer carries per channel in 32 bits is a state of ``dk == 1``; a layer may have several."""
         super().__init__(num_slots)
         self.token = torch.zeros(num_slots, dtype=torch.int32, device=device) if token else None
         self.ssm = [torch.zeros((num_slots, h, dk, dv), dtype=torch.float32, device=device) for h, dk, dv, _, _ in geometries]
         self.conv = [torch.zeros((num_slots, c, max(taps - 1, 0)), dtype=dtype, device=device) if taps else None for _, _, _, c, taps in geometries]
 
     def clear(self, slot: int) -> None:
-        live = [t[slot] for t in self.ssm] + [t[slot] for t in self.conv if t is not None and t.numel()]
+        live = [t[slot] for t in (*self.ssm, *self.conv) if t is not None and t.numel()]
         if live:
             torch._foreach_zero_(live)
         if self.token is not None:

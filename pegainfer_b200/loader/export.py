@@ -59,6 +59,10 @@ def default_source(cfg: ModelConfig, seed: int = 0, dtype=torch.bfloat16):
         from ..models.zeripel import zeripel_source
 
         return zeripel_source(cfg, seed=seed, dtype=dtype)
+    if cfg.family == "nonetar":
+        from ..models.nonetar import nonetar_source
+
+        return nonetar_source(cfg, seed=seed, dtype=dtype)
     from ..models import registry
 
     shapes = registry.shapes_for(cfg)
@@ -83,6 +87,10 @@ def to_hf_config(cfg: ModelConfig) -> dict:
         from ..config import zeripel_to_json
 
         return zeripel_to_json(cfg)
+    if cfg.family == "nonetar":
+        from ..config import nonetar_to_json
+
+        return nonetar_to_json(cfg)
     arch = {"qwen3": ("qwen3", "Qwen3ForCausalLM"), "qwen35": ("qwen3_5", "Qwen3_5ForCausalLM"), "deepseek_v2": ("deepseek_v2", "DeepseekV2ForCausalLM"),
             "kimi_k2": ("kimi_k2", "DeepseekV3ForCausalLM")}.get(cfg.family, (cfg.family, cfg.family))
     out = {

@@ -57,7 +57,7 @@ class HybridLayers:
     def kv_geometry(self) -> dict:
         g = self.kv_geometries or [(1, 8, 8)]
         # KV heads of the attention layers times the groups of up to eight query heads that one CTA of the decode kernel takes
-        attn = [l.mixer for l in self.cfg.layer_specs if l.mixer.kind == "attention"]
+        attn = [m for l in self.cfg.layer_specs for m in l.mixer.flat() if m.kind == "attention"]
         return dict(num_layers=len(g), kv_heads=max([m.kv_heads * ((m.heads // m.kv_heads + 7) // 8) for m in attn] or [1]), head_dim=max(max(d, v) for _, d, v in g),
                     bytes_per_block=lambda page: max(1, MixedKvBuffer.bytes_per_block(self.kv_geometries, page, self.dtype)))
 

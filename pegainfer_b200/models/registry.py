@@ -68,7 +68,14 @@ def _zeripel(cfg, **kw):
     return ZeripelModel(cfg, **kw)
 
 
-BUILDERS = {"zeripel": _zeripel, "vekalorn": _vekalorn, "nemipel": _nemipel, "kimi_k3": _k3, "gemma4": _gemma4, "glm_dsa": _glm_dsa, "qwen3": _qwen3, "qwen35": _qwen35, "deepseek_v2": _mla_moe, "kimi_k2": _mla_moe}
+def _nonetar(cfg, **kw):
+    from .nonetar import NonetarModel
+
+    kw.pop("ep", None)
+    return NonetarModel(cfg, **kw)
+
+
+BUILDERS = {"nonetar": _nonetar, "zeripel": _zeripel, "vekalorn": _vekalorn, "nemipel": _nemipel, "kimi_k3": _k3, "gemma4": _gemma4, "glm_dsa": _glm_dsa, "qwen3": _qwen3, "qwen35": _qwen35, "deepseek_v2": _mla_moe, "kimi_k2": _mla_moe}
 
 
 # Translation units (csrc/<name>.cu) that a family's kernels come from, for programs that build only what one model needs
@@ -76,6 +83,7 @@ KERNEL_UNITS = {
     "nemipel": ("runtime", "gemm_sm100", "gemm2sm_sm100", "elementwise", "stream32", "attention", "attention_tc", "attention_general", "kda", "lightning", "sampling"),
     "vekalorn": ("runtime", "gemm_sm100", "gemm2sm_sm100", "elementwise", "stream32", "mla", "mla_prefill", "moe_route", "moe_gemm", "sampling"),
     "zeripel": ("runtime", "gemm_sm100", "gemm2sm_sm100", "elementwise", "stream32", "attention", "attention_tc", "attention_general", "kda", "wkv", "mla", "mla_prefill", "moe_route", "moe_gemm", "sampling"),
+    "nonetar": ("runtime", "gemm_sm100", "gemm2sm_sm100", "elementwise", "stream32", "streams", "attention", "attention_tc", "attention_general", "kda", "lightning", "lru", "moe_gemm", "sampling"),
 }
 
 
@@ -116,6 +124,10 @@ def shapes_for(cfg: ModelConfig) -> dict:
         from .zeripel import zeripel_shapes
 
         return zeripel_shapes(cfg)
+    if cfg.family == "nonetar":
+        from .nonetar import nonetar_shapes
+
+        return nonetar_shapes(cfg)
     raise ValueError(f"no tensor-shape table for family {cfg.family!r}")
 
 

@@ -88,6 +88,62 @@ def embed_stream(ids, table, act_dtype):
     return x, x.to(act_dtype)
 
 
+POSITION_FINE = 256  # positions of one fine table; a coarse row is that many positions further
+
+
+def position_tables(max_pos: int, width: int, device="cpu"):
+    """Sines and cosines (formed in f64) whose angles add up to those of every position: coarse f32 [ceil(max_pos / 256), pairs,
+    2] at multiples of 256 and fine [256, pairs, 2]; pair i turns at ``10000 ** (-2 i / width)``, sine first."""
+    rate = 10000.0 ** (-2.0 * torch.arange((width + 1) // 2, dtype=torch.float64) / width)
+    make = lambda n, step: (lambda a: torch.stack((a.sin(), a.cos()), -1).float().to(device))(torch.outer(torch.arange(n, dtype=torch.float64) * step, rate))
+    return make(-(-max_pos // POSITION_FINE), POSITION_FINE), make(POSITION_FINE, 1)
+
+
+def embed_positions(ids, table, tables, meta: AttnMeta):
+    """f32 rows ``table[id]`` plus the sinusoids of their positions (``position_tables``): sines at even, cosines at odd places."""
+    coarse, fine = tables
+    p = meta.positions.long()
+    a, b = coarse[p // POSITION_FINE], fine[p % POSITION_FINE]
+    pos = torch.stack((a[..., 0] * b[..., 1] + a[..., 1] * b[..., 0], a[..., 1] * b[..., 1] - a[..., 0] * b[..., 0]), -1).flatten(1)
+    return table[ids.long()].float() + pos[:, : table.shape[1]]
+
+
+class StreamMix:
+    """Coefficients between two sublayers of a residual stream kept in several copies: ``x'[t] = sum_s mix[s, t] x[s] + out[t] y``
+    from the old copies and a sublayer's output, and the next sublayer's input ``u = sum_t gather[t] x'[t]``.  f32; ``mix``
+    [s_in, s_out].  ``packed``: mix, out, and ``u``'s coefficients over the OLD copies and y, which is how it is formed."""
+
+    def __init__(self, mix, out, gather):
+        self.mix, self.out, self.gather = mix, out, gather
+        d = lambda z: z.double()
+        self.old, self.new = (d(mix) @ d(gather)).float(), (d(out) * d(gather)).sum().float()
+        self.packed = torch.cat((mix.reshape(-1), out, self.old, self.new.view(1))).contiguous()
+
+
+def streams_norm(x, y, m: StreamMix, w, eps: float, act_dtype, shift=None, carried=None, meta: Optional[AttnMeta] = None, keep: bool = True):
+    """Hyper-connection step: ``x`` f32 [T, s_in, W] and a sublayer's output ``y`` [T, W] (``None``: nothing is added) to the new
+    copies [T, s_out, W] (``None`` without ``keep``; ``x`` itself without ``y``) and to the RMS norm of their ``gather`` sum times
+    ``w``, in the activation dtype.  With ``shift`` f32 [W] every normed row moves towards its predecessor by that much, in f32;
+    ``carried`` f32 [slots, 1, 1, W] holds the last row (in front of the move) of the request in the slot, read and replaced."""
+    u = torch.einsum("s,tsw->tw", m.old, x)
+    new = x
+    if y is not None:
+        u = u + m.new * y.float()
+        new = torch.einsum("sn,tsw->tnw", m.mix, x) + m.out[None, :, None] * y.float()[:, None] if keep else None
+    h = u * torch.rsqrt(u.pow(2).mean(-1, keepdim=True) + eps) * w.float()
+    if shift is not None:
+        qi, slots, moved = meta.h_q_indptr, meta.h_state_slots, torch.empty_like(h)
+        for b in range(meta.num_seqs):
+            q0, q1 = qi[b], qi[b + 1]
+            if q1 == q0:
+                continue
+            back = torch.cat((carried[slots[b]].view(1, -1), h[q0 : q1 - 1]))
+            moved[q0:q1] = h[q0:q1] + (back - h[q0:q1]) * shift
+            carried[slots[b]] = h[q1 - 1]
+        h = moved
+    return new, h.to(act_dtype)
+
+
 def embed_pairs_norm(ids, table, pairs, scale: float, bigram, carried, w, eps: float, meta: AttnMeta, act_dtype):
     """Residual stream of scaled table rows plus the rows of token pairs, and its RMS norm: ``x = table[id] * scale +
     pairs[(previous * mul_prev + id * mul_cur) mod buckets]`` in f32, the last row of ``pairs`` for a sequence's first token.
@@ -143,9 +199,9 @@ def token_mix(h, mu, carried, meta: AttnMeta):
     return out
 
 
-def multi_dense(x, w):
+def multi_dense(x, w, out_dtype=None):
     """``y[t, i] = w[i] x[t, i]``: ``x`` [T, n, K] (columns of a wider row, if need be), ``w`` [n, M, K]."""
-    return torch.einsum("tnk,nmk->tnm", x.float(), w.float()).to(x.dtype)
+    return torch.einsum("tnk,nmk->tnm", x.float(), w.float()).to(out_dtype or x.dtype)
 
 
 def tanh_rows(x):
@@ -190,13 +246,16 @@ def stream_layer_norm(x, w, eps: float, act_dtype):
     return _layer_norm(x, w, eps).to(act_dtype)
 
 
-def gated_row_norm(x, gate, w, eps: float, act: str = "sigmoid"):
+def gated_row_norm(x, gate, w, eps: float, act: str = "sigmoid", gate_first: bool = False):
     """``rms_norm(x) * w * act(gate)`` over the last axis of ``x`` [T, H, D], rounded once; ``gate`` [T, H * D] may be a
-    column slice of a wider projection, ``w`` [D] shared by the heads or [H * D]; ``act``: sigmoid or silu."""
+    column slice of a wider projection, ``w`` [D] shared by the heads or [H * D]; ``act``: sigmoid or silu.  ``gate_first``:
+    ``rms_norm(x * act(gate)) * w``."""
     xf, g = x.float(), gate.float().reshape(x.shape)
+    if gate_first:
+        xf, g = xf * torch.sigmoid(g) * (g if act == "silu" else 1.0), None
     n = xf * torch.rsqrt(xf.pow(2).mean(-1, keepdim=True) + eps)
     n = n * w.float().view((x.shape[1], -1) if w.numel() > x.shape[2] else (-1,))
-    return (n * torch.sigmoid(g) * (g if act == "silu" else 1.0)).to(x.dtype)
+    return n.to(x.dtype) if g is None else (n * torch.sigmoid(g) * (g if act == "silu" else 1.0)).to(x.dtype)
 
 
 def dense(x, w, out_dtype=None):
@@ -211,6 +270,17 @@ def dense_glu(x, gate_up, interleaved: bool = False, act: str = "silu"):
     if act == "gelu_tanh":
         return geglu(torch.cat((y[:, 0::2], y[:, 1::2]), 1) if interleaved else y)
     return swiglu(y, interleaved)
+
+
+def xielu(z, p, q):
+    """``softplus(p) z^2 + z / 2`` above zero, ``(1/2 + softplus(q)) (e^z - 1 - z) + z / 2`` below, in f32."""
+    z = z.float()
+    return torch.where(z > 0, F.softplus(p.float()) * z * z, (0.5 + F.softplus(q.float())) * (torch.expm1(z.clamp(max=0)) - z)) + 0.5 * z
+
+
+def dense_xielu(x, w, act):
+    """``xielu(x @ w.T, *act)`` with ``act`` f32 [2]."""
+    return xielu(x.float() @ w.float().t(), act[0], act[1]).to(x.dtype)
 
 
 def softcap_rows(logits, cap: float):
@@ -463,10 +533,13 @@ def temperature_table(max_pos: int, coef: float, every: int, device="cpu"):
     return (1.0 + coef * torch.log((p // every + 1).double())).float()
 
 
-def head_norm_append(q, k, v, q_norm_w, k_norm_w, temp, meta: AttnMeta, kv_layer, heads: int, kv_heads: int, dim: int, vdim: int, eps: float):
-    """RMS norm of every query and key head with weights [dim] shared by the heads, queries times ``temp[position]`` (``None``:
-    1); keys and the values ``v`` (as they are) go to the paged cache.  Returns queries [T, heads, dim]."""
+def head_norm_append(q, k, v, q_norm_w, k_norm_w, temp, meta: AttnMeta, kv_layer, heads: int, kv_heads: int, dim: int, vdim: int, eps: float, bias=None):
+    """RMS norm of every query and key head with weights [dim] shared by the heads ([heads, dim]: one per query head), queries
+    times ``temp[position]`` (``None``: 1); keys and the values ``v`` (as they are) go to the paged cache.  ``bias``: f32 vectors
+    that are added to q, k and v first.  Returns queries [T, heads, dim]."""
     t, ps = q.shape[0], meta.page_size
+    if bias is not None:
+        q, k, v = ((z.float() + b).to(z.dtype if z is v else torch.float32) for z, b in zip((q, k, v), bias))
     norm = lambda z, n, w: (lambda f: f * torch.rsqrt(f.pow(2).mean(-1, keepdim=True) + eps) * w.float())(z.float().reshape(t, n, dim))
     qn = norm(q, heads, q_norm_w)
     if temp is not None:
@@ -475,18 +548,20 @@ def head_norm_append(q, k, v, q_norm_w, k_norm_w, temp, meta: AttnMeta, kv_layer
     slots = meta.slot_mapping.long()
     kp[slots // ps, slots % ps] = norm(k, kv_heads, k_norm_w).to(kv_layer.dtype)
     vp[slots // ps, slots % ps] = v.reshape(t, kv_heads, vdim).to(kv_layer.dtype)
-    return qn.to(q.dtype)
+    return qn.to(kv_layer.dtype)
 
 
-def capped_attention(q, kv_layer, kv_heads: int, vdim: int, meta: AttnMeta, scale: float, softcap: float = 0.0, gate=None):
+def capped_attention(q, kv_layer, kv_heads: int, vdim: int, meta: AttnMeta, scale: float, softcap: float = 0.0, gate=None, window: int = 0, slopes=None, out_scale: float = 1.0, out=None):
     """Causal attention over the paged cache with different key and value sizes, an optional soft cap on the scaled scores
-    and an optional sigmoid gate per (token, head) (``gate`` [T, >= heads]).  Returns ``[T, heads * vdim]``."""
+    and an optional sigmoid gate per (token, head) (``gate`` [T, >= heads]).  ``window``: a row sees itself and the ``window -
+    1`` keys in front of it (0: all); ``slopes`` f32 [heads]: what a capped score loses per position of distance.  The result
+    times ``out_scale``, ``[T, heads * vdim]``, goes to ``out`` (columns of a wider buffer) or a new tensor."""
     t, hq, dim = q.shape
     rep = hq // kv_heads
     kp, vp = _pages_kv(kv_layer, kv_heads, dim, vdim, meta.page_size)
     qi = meta.h_q_indptr if meta.h_q_indptr is not None else meta.q_indptr.tolist()
     kl = meta.h_kv_lens if meta.h_kv_lens is not None else meta.kv_lens.tolist()
-    out = torch.zeros(t, hq, vdim, dtype=torch.float32, device=q.device)
+    o = torch.zeros(t, hq, vdim, dtype=torch.float32, device=q.device)
     for b in range(meta.num_seqs):
         q0, q1, n = qi[b], qi[b + 1], kl[b]
         if n == 0 or q1 == q0:
@@ -497,12 +572,15 @@ def capped_attention(q, kv_layer, kv_heads: int, vdim: int, meta: AttnMeta, scal
         s = torch.einsum("qhd,khd->hqk", q[q0:q1].float(), k) * scale
         if softcap:
             s = torch.tanh(s / softcap) * softcap
-        pos = torch.arange(n - (q1 - q0), n, device=q.device)
-        s = s.masked_fill(torch.arange(n, device=q.device)[None, None, :] > pos[None, :, None], float("-inf"))
-        out[q0:q1] = torch.einsum("hqk,khd->qhd", torch.softmax(s, -1), v)
+        dist = torch.arange(n - (q1 - q0), n, device=q.device)[:, None] - torch.arange(n, device=q.device)
+        if slopes is not None:
+            s = s - slopes.view(hq, 1, 1) * dist
+        s = s.masked_fill((dist < 0) | (dist >= window) if window else dist < 0, float("-inf"))
+        o[q0:q1] = torch.einsum("hqk,khd->qhd", torch.softmax(s, -1), v)
     if gate is not None:
-        out = out * torch.sigmoid(gate[:, :hq].float())[:, :, None]
-    return out.to(q.dtype).reshape(t, hq * vdim)
+        o = o * torch.sigmoid(gate[:, :hq].float())[:, :, None]
+    o = (o * out_scale).to(q.dtype).reshape(t, hq * vdim)
+    return o if out is None else out.copy_(o)
 
 
 def _gather_kv(kv_layer, pages, kv_len, page_size):
@@ -1138,8 +1216,16 @@ def kda_recurrent(q, k, v, f, b, a_log, dt_bias, lower: float, state, meta: Attn
 def conv_silu(x, conv_w, conv_state, meta: AttnMeta):
     """Causal depthwise convolution of any length + SiLU, rounded once; ``conv_w`` f32 [C, taps], ``conv_state``
     [slots, C, taps - 1] holds the last inputs of each sequence and is updated in place."""
+    return short_conv(x, conv_w, None, conv_state, meta)
+
+
+def short_conv(x, conv_w, bias, conv_state, meta: AttnMeta, act: str = "silu", in_bias=None):
+    """``conv_silu`` with an f32 bias per channel (or ``None``), ``act`` silu or none, and ``in_bias`` f32 [C] that is added to the
+    inputs (those in front of a sequence's start are zero all the same)."""
     taps = conv_w.shape[1]
     out = torch.zeros(x.shape, dtype=x.dtype, device=x.device)
+    if in_bias is not None:
+        x = (x.float() + in_bias).to(x.dtype)
     qi = meta.h_q_indptr if meta.h_q_indptr is not None else meta.q_indptr.tolist()
     slots = meta.h_state_slots if meta.h_state_slots is not None else meta.state_slots.tolist()
     for b in range(meta.num_seqs):
@@ -1148,7 +1234,9 @@ def conv_silu(x, conv_w, conv_state, meta: AttnMeta):
             continue
         seq = torch.cat([conv_state[slots[b]].t().to(x.dtype), x[q0:q1]], 0)
         pre = (seq.float().unfold(0, taps, 1) * conv_w.float()).sum(-1)
-        out[q0:q1] = (pre * torch.sigmoid(pre)).to(x.dtype)
+        if bias is not None:
+            pre = pre + bias
+        out[q0:q1] = (pre * torch.sigmoid(pre) if act == "silu" else pre).to(x.dtype)
         conv_state[slots[b]] = seq[seq.shape[0] - (taps - 1) :].t().to(conv_state.dtype)
     return out
 
@@ -1220,6 +1308,54 @@ def wkv_attention(r, k, v, f, w0, u, state, meta: AttnMeta):
             S = S * dec[i].unsqueeze(-1) + torch.einsum("hk,hv->hkv", kf[i], vf[i])
         state[slots[s]] = S
     return out
+
+
+def ssd_attention(x, B, C, dt, dt_bias, a_log, D, state, meta: AttnMeta):
+    """State-space duality (Mamba-2): with ``d = softplus(dt + dt_bias)`` per token and head, ``S <- exp(-exp(a_log) d) S + d B x^T``
+    over the f32 ``state`` [slots, H, N, Dv] and ``S^T C + D x``.  ``x`` [T, H, Dv], ``B, C`` [T, G, N] (head h reads group ``h //
+    (H / G)``), ``dt`` [T, H] raw.  Returns [T, H, Dv]."""
+    t, h, dv = x.shape
+    rep = h // B.shape[1]
+    xf, Bf, Cf = x.float(), B.float().repeat_interleave(rep, 1), C.float().repeat_interleave(rep, 1)
+    d = F.softplus(dt.float() + dt_bias)
+    dec = torch.exp(-torch.exp(a_log) * d)
+    out = torch.zeros(t, h, dv, dtype=x.dtype, device=x.device)
+    qi = meta.h_q_indptr if meta.h_q_indptr is not None else meta.q_indptr.tolist()
+    slots = meta.h_state_slots if meta.h_state_slots is not None else meta.state_slots.tolist()
+    for s in range(meta.num_seqs):
+        if slots[s] < 0:
+            continue
+        S = state[slots[s]]
+        for i in range(qi[s], qi[s + 1]):
+            S = S * dec[i].view(h, 1, 1) + torch.einsum("hk,hv->hkv", Bf[i], xf[i] * d[i].unsqueeze(-1))
+            out[i] = (torch.einsum("hkv,hk->hv", S, Cf[i]) + D.view(h, 1) * xf[i]).to(x.dtype)
+        state[slots[s]] = S
+    return out
+
+
+def gated_lru(gates, gate_bias, u, lam, y, y_bias, state, meta: AttnMeta, scale: float = 1.0, out=None):
+    """Real-gated linear recurrence per channel (Griffin): ``log a = -8 sigmoid(r) softplus(lam)``, ``S <- a S + sqrt(1 - a^2)
+    sigmoid(i) u``; returns ``S * gelu(y + y_bias) * scale`` in the dtype of ``u``, in ``out`` (columns of a wider buffer) or a new
+    tensor.  ``gates`` f32 [T, blocks, 2 * (W / blocks)]: a block's r, then its i, to which ``gate_bias`` f32 of the same columns is
+    added; ``u, y`` [T, W]; ``lam, y_bias`` f32 [W]; ``state`` f32 [slots, 1, 1, W]."""
+    t, w = u.shape
+    g = torch.sigmoid(gates + gate_bias.view(1, *gates.shape[1:])).view(t, gates.shape[1], 2, -1)
+    r, i = g[:, :, 0].reshape(t, w), g[:, :, 1].reshape(t, w)
+    e = torch.expm1(-8.0 * r * F.softplus(lam))
+    a, b = 1 + e, torch.sqrt(-e * (2 + e)) * i * u.float()
+    o = torch.zeros(t, w, dtype=torch.float32, device=u.device)
+    qi = meta.h_q_indptr if meta.h_q_indptr is not None else meta.q_indptr.tolist()
+    slots = meta.h_state_slots if meta.h_state_slots is not None else meta.state_slots.tolist()
+    for s in range(meta.num_seqs):
+        if slots[s] < 0:
+            continue
+        S = state[slots[s]].view(w)
+        for j in range(qi[s], qi[s + 1]):
+            S = a[j] * S + b[j]
+            o[j] = S
+        state[slots[s]] = S.view(1, 1, w)
+    o = (o * F.gelu(y.float() + y_bias, approximate="tanh") * scale).to(u.dtype)
+    return o if out is None else out.copy_(o)
 
 
 def markov_step_argmax(base, bias, block: int, step: int, next_tokens, drafts):

@@ -65,6 +65,7 @@ LINES = [
     ModelLine("nemipel", ("nemipel",), frozenset({"dtype", "state_slots"})),
     ModelLine("vekalorn", ("vekalorn",), frozenset({"dtype"})),
     ModelLine("zeripel", ("zeripel",), frozenset({"dtype", "state_slots"})),
+    ModelLine("nonetar", ("nonetar",), frozenset({"dtype", "state_slots"})),
 ]
 LINES[0].validate = _qwen3_validate  # type: ignore[method-assign]
 
