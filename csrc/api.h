@@ -43,6 +43,9 @@ int pg_gemm_bf16_tn_fused(const void* x, const void* w, void* y, int T, int M, i
                           const void* in_ssp, int in_parts, int in_ld, int in_width, float in_eps, int epi, void* residual, long long ld_res,
                           const void* norm_w, int norm_offset, void* out_ssp, int out_ld, void* ws, long long ws_bytes, void* counters,
                           long long counter_bytes, void* status, cudaStream_t stream);
+// xIELU (constants in act) in the epilogue of the plain GEMM, whatever kernel serves the problem.
+int pg_gemm_bf16_tn_xielu(const void* x, const void* w, void* y, int T, int M, int K, long long ldx, long long ldw, long long ldy, const void* act, void* ws, long long ws_bytes,
+                          void* counters, long long counter_bytes, void* status, int force_splits, cudaStream_t stream);
 // Decode chain (decode_chain.cu): up to four dependent GEMMs of a layer in one persistent kernel for
 // steps of at most 64 rows.  One PgChainPhase per GEMM; see decode_chain.cu for the fields.
 struct PgChainPhase;
@@ -64,6 +67,8 @@ int pg_gemm2sm_bf16_tn(const void* x, const void* w, void* y, int T, int M, int 
                        cudaStream_t stream);
 int pg_gemm2sm_bf16_tn_swiglu(const void* x, const void* w, void* y, int T, int M, int K, long long ldx, long long ldw, long long ldy, int gelu, void* status,
                        cudaStream_t stream);
+int pg_gemm2sm_bf16_tn_xielu(const void* x, const void* w, void* y, int T, int M, int K, long long ldx, long long ldw, long long ldy, const void* act, void* status,
+                             cudaStream_t stream);
 int pg_make_tmap_bf16_2d(CUtensorMap* out, const void* ptr, long long rows, long long cols, long long ld, int box_rows, int box_cols);
 
 // ---- row kernels (elementwise.cu) --------------------------------------------------
@@ -158,8 +163,8 @@ int pg_moe_grouped_gemm(const void* x, long long ldx, long long x_rows, const vo
 
 int pg_moe_grouped_gemm_act(const void* x, long long ldx, long long x_rows, const void* w, void* y, long long ldy, const void* offsets, int E, int M, int K, int bn, int act, void* status, cudaStream_t stream);
 // Per-head products of strided activations: y[t, h, :] = x[t, h, :] w[h]^T (times the sigmoid of a gate)
-int pg_head_gemm(const void* x, long long ldx, long long x_head, const void* w, void* y, long long ldy, long long y_head, const void* gate, long long ldg, long long g_head, int heads, int rows, int M, int K,
-                 int bn, void* status, cudaStream_t stream);
+int pg_head_gemm(const void* x, long long ldx, long long x_head, const void* w, void* y, int y_f32, long long ldy, long long y_head, const void* gate, long long ldg, long long g_head,
+                 int heads, int rows, int M, int K, int bn, void* status, cudaStream_t stream);
 int pg_moe_grouped_gemm_return(const void* x, long long ldx, long long x_rows, const void* w, const void* scales, int quant, long long ldy,
                                const void* offsets, int E, int M, int K, int bn, void* status, const void* scatter_src, void* const* peer_out,
                                void* const* peer_flags, int cap, int rank, int world, int site, cudaStream_t stream);
@@ -204,6 +209,12 @@ int pg_lightning_chunked(const void* q, const void* k, const void* v, long long 
 // wkv_recurrent: linear attention with a decay per token and key channel and a bonus for the current token.
 int pg_wkv_recurrent(const void* r, const void* k, const void* v, long long ld, const void* f, long long ldf, const void* w0, const void* u, void* state, void* out, const void* q_indptr,
                      const void* slots, int num_seqs, int heads, int dk, int dv, int max_q_len, int skip_len, int is_f32, cudaStream_t stream);
+// ssd_recurrent: state-space duality, one decay per token and head; ssd_chunked (lightning.cu): the same in chunks on the tensor cores.
+int pg_ssd_recurrent(const void* C, const void* B, const void* x, long long ld, const void* dt, long long lddt, const void* a_log, const void* dt_bias, const void* D, void* state,
+                     void* out, const void* q_indptr, const void* slots, int num_seqs, int heads, int groups, int n, int dv, int max_q_len, int skip_len, int is_f32,
+                     cudaStream_t stream);
+int pg_ssd_chunked(const void* C_, const void* B, const void* x, long long ld, const void* dt, long long lddt, const void* a_log, const void* dt_bias, const void* D, void* state,
+                   void* out, const void* q_indptr, const void* slots, int num_seqs, int heads, int groups, int n, int dv, int min_len, cudaStream_t stream);
 // ---- token shift and chunk-wise WKV (wkv.cu) ------------------------------------------
 // The recurrence of pg_wkv_recurrent in blocks of 16 tokens on the tensor cores, for sequences of >= min_len tokens, bf16.
 int pg_wkv_block(const void* r, const void* k, const void* v, long long ld, const void* f, long long ldf, const void* w0, const void* u, void* state, void* out, const void* q_indptr, const void* slots,
@@ -227,17 +238,19 @@ int pg_paged_attention(const void* q, const void* kv, void* out, const void* q_i
                        void* part_o, void* part_lse, int q_tiles, int window, void* status, cudaStream_t stream);
 
 int pg_attention_capped(const void* q, const void* kv, void* out, const void* q_indptr, const void* kv_lens, const void* table, int table_stride, int num_seqs, int hq, int hkv, int dim,
-                        int vdim, int page_size, long long num_pages, float scale, float softcap, const void* gate, long long ld_gate, int mode, int splits, void* part_o, void* part_lse,
-                        int q_tiles, void* status, cudaStream_t stream);
+                        int vdim, int page_size, long long num_pages, float scale, float softcap, const void* gate, long long ld_gate, int window, const void* slopes, float out_scale,
+                        long long ld_out, int mode, int splits, void* part_o, void* part_lse, int q_tiles, void* status, cudaStream_t stream);
 
 // ---- layers with runtime head sizes, bf16 or f32 (attention_general.cu) -----------------
 int pg_row_norm_rope_append(const void* q, const void* k, const void* v, long long ld, const void* q_w, const void* k_w, const void* cos, const void* sin, int rot, int max_pos,
                             const void* positions, const void* slots, void* q_out, void* kv, int tokens, int hq, int hkv, int dim, int vdim, int page_size, long long num_pages, float eps,
                             int is_f32, void* status, cudaStream_t stream);
-int pg_head_norm_append(const void* q, const void* k, const void* v, long long ld, const void* q_w, const void* k_w, const void* temp, int max_pos, const void* positions, const void* slots,
-                        void* q_out, void* kv, int tokens, int hq, int hkv, int dim, int vdim, int page_size, long long num_pages, float eps, int is_f32, void* status, cudaStream_t stream);
-int pg_attention_plain(const void* q, const void* kv, void* out, const void* q_indptr, const void* kv_lens, const void* table, int table_stride, int tokens, int num_seqs, int hq, int hkv,
-                       int dim, int vdim, int page_size, long long num_pages, float scale, float softcap, const void* gate, long long ld_gate, int is_f32, cudaStream_t stream);
+int pg_head_norm_append(const void* q, const void* k, const void* v, long long ld, const void* q_w, int q_w_heads, const void* k_w, const void* q_b, const void* k_b, const void* v_b,
+                        const void* temp, int max_pos, const void* positions, const void* slots, void* q_out, void* kv, int tokens, int hq, int hkv, int dim, int vdim, int page_size,
+                        long long num_pages, float eps, int is_f32, void* status, cudaStream_t stream);
+int pg_attention_plain(const void* q, const void* kv, void* out, const void* q_indptr, const void* kv_lens, const void* table, int table_stride, int tokens, int num_seqs, int hq,
+                       int hkv, int dim, int vdim, int page_size, long long num_pages, float scale, float softcap, const void* gate, long long ld_gate, int window, const void* slopes,
+                       float out_scale, long long ld_out, int is_f32, cudaStream_t stream);
 
 // ---- rows around an f32 residual stream (stream32.cu) --------------------------------
 int pg_embed_rows(const void* table, int table_f32, long long ldt, const void* ids, void* x_f32, void* xt, int xt_f32, long long ldxt, int tokens, int width, long long rows, void* status,
@@ -252,16 +265,27 @@ int pg_post_norm(const void* y, int y_f32, long long ldy, const void* x_in, void
                  cudaStream_t stream);
 int pg_add_layer_norm(const void* y, int y_f32, long long ldy, const void* pos, const void* weights, int k, void* x, const void* w, void* xt, int xt_f32, long long ldxt, int tokens, int width, float eps,
                       cudaStream_t stream);
-int pg_head_gemm_simt(const void* x, long long ldx, long long x_head, const void* w, void* y, long long ldy, long long y_head, const void* gate, long long ldg, long long g_head, int heads, int rows, int M,
-                      int K, int is_f32, cudaStream_t stream);
+int pg_head_gemm_simt(const void* x, long long ldx, long long x_head, const void* w, void* y, long long ldy, long long y_head, const void* gate, long long ldg, long long g_head,
+                      int heads, int rows, int M, int K, int y_f32, int is_f32, cudaStream_t stream);
 int pg_expert_gemm_simt(const void* x, long long ldx, const void* sorted_src, int k, const void* w, void* y, const void* offsets, int routes, int E, int M, int K, int act, int is_f32,
                         cudaStream_t stream);
-int pg_gated_row_norm(const void* x, const void* gate, long long ldg, const void* w, void* y, int tokens, int heads, int dim, float eps, int silu, int w_heads, int is_f32, cudaStream_t stream);
+int pg_gated_row_norm(const void* x, const void* gate, long long ldg, const void* w, void* y, int tokens, int heads, int dim, float eps, int silu, int w_heads, int gate_first,
+                      int is_f32, cudaStream_t stream);
 int pg_glu_rows_f32(const void* gu, void* out, int rows, int inter, long long ldin, int gelu, cudaStream_t stream);
+int pg_xielu_rows(const void* x, void* y, const void* act, long long n, int is_f32, cudaStream_t stream);
 int pg_softcap_f32(const void* x, void* y, long long n, float cap, cudaStream_t stream);
 int pg_gemm_simt(const void* x, const void* w, int x_f32, void* y, int y_f32, int T, int M, int K, long long ldx, long long ldw, long long ldy, cudaStream_t stream);
-int pg_conv_silu(const void* x, long long ldx, const void* w, void* state, void* out, long long ldo, const void* q_indptr, const void* slots, int num_seqs, int channels, int taps,
-                 long long slot_stride, int max_q_len, int is_f32, cudaStream_t stream);
+// causal depthwise convolution over ragged sequences with carried inputs; biases on the inputs and the sum, SiLU optional
+int pg_short_conv(const void* x, long long ldx, const void* w, const void* bias, const void* in_bias, void* state, void* out, long long ldo, const void* q_indptr, const void* slots,
+                  int num_seqs, int channels, int taps, long long slot_stride, int max_q_len, int silu, int is_f32, cudaStream_t stream);
+
+// ---- residual stream in several copies (streams.cu), gated linear recurrence per channel (lru.cu) ----
+int pg_embed_positions(const void* table, int table_f32, long long ldt, const void* coarse, int coarse_rows, const void* fine, const void* ids, const void* positions, void* x,
+                       int tokens, int width, long long rows, void* status, cudaStream_t stream);
+int pg_streams_norm(const void* x, int s_in, const void* y, int y_f32, long long ldy, const void* coef, void* x_out, int s_out, const void* w, void* h, int h_f32, const void* shift,
+                    void* carried, const void* unit_seq, const void* q_indptr, const void* slots, int tokens, int width, float eps, cudaStream_t stream);
+int pg_gated_lru(const void* gates, const void* gate_bias, const void* u, long long ldu, const void* lam, const void* y, long long ldy, const void* y_bias, void* state, void* out,
+                 long long ldo, const void* q_indptr, const void* slots, int num_seqs, int width, int blocks, float scale, int max_q_len, int is_f32, cudaStream_t stream);
 
 // ---- sampling (sampling.cu) --------------------------------------------------------
 long long pg_argmax_scratch_bytes(int rows, int vocab);

@@ -84,6 +84,9 @@ struct AttnParams {
   float cap_in, cap_out;     // cap_in > 0: score = cap_out * tanh(cap_in * dot), already times log2(e)
   const bf16* gate;          // [T, >= hq] rows of stride ld_gate, or null
   long long ld_gate;
+  const float* slopes;       // [hq]: a (capped) score loses slope * distance; or null
+  float out_scale;           // on the output
+  long long ld_out;          // row stride of out
 };
 
 // A score in units of log2(e): scaled, and capped when the layer has a cap.  tanh(x) = 1 - 2 / (1 + e^2x), whose absolute
@@ -92,6 +95,11 @@ template <bool GEN>
 __device__ __forceinline__ float score_of(const AttnParams& p, float dot) {
   if (GEN && p.cap_in > 0.f) return p.cap_out - __fdividef(2.f * p.cap_out, 1.f + exp2f(dot * p.cap_in * 2.f * LOG2E));
   return dot * p.scale_log2;
+}
+// What the distance costs a score of head hq, in units of log2(e).
+template <bool GEN>
+__device__ __forceinline__ float slope_of(const AttnParams& p, int hq) {
+  return GEN && p.slopes ? p.slopes[hq] * LOG2E : 0.f;
 }
 __device__ __forceinline__ float head_gate(const AttnParams& p, long long row, int hq) {
   return 1.f / (1.f + __expf(-__bfloat162float(p.gate[row * p.ld_gate + hq])));
@@ -415,6 +423,7 @@ __global__ void __launch_bounds__(128, D <= 128 ? 2 : 1) decode_attn_persistent_
 #pragma unroll
     for (int n = 0; n < NT; ++n) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f;
     float m_run = NEG_BIG, l_run = 0.f;
+    const float slope = slope_of<GEN>(p, head0 + min(g, Gu - 1));  // of this lane's row
     for (int tile = uc.t_begin + warp; tile < uc.t_end; tile += 4, ++it) {
       cp_async_wait<STAGES - 2>();
       __syncwarp();
@@ -441,6 +450,10 @@ __global__ void __launch_bounds__(128, D <= 128 ? 2 : 1) decode_attn_persistent_
       sv[1] = (tok0 + 1 < uc.kv_len && tok0 + 1 >= uc.kv_lo) ? score_of<GEN>(p, s_acc[0][1]) : NEG_BIG;
       sv[2] = (tok0 + 8 < uc.kv_len && tok0 + 8 >= uc.kv_lo) ? score_of<GEN>(p, s_acc[1][0]) : NEG_BIG;
       sv[3] = (tok0 + 9 < uc.kv_len && tok0 + 9 >= uc.kv_lo) ? score_of<GEN>(p, s_acc[1][1]) : NEG_BIG;
+      if (GEN) {
+        const float d0 = (float)(uc.kv_len - 1 - tok0);  // a masked score stays below NEG_BIG
+        sv[0] -= slope * fmaxf(d0, 0.f), sv[1] -= slope * fmaxf(d0 - 1.f, 0.f), sv[2] -= slope * fmaxf(d0 - 8.f, 0.f), sv[3] -= slope * fmaxf(d0 - 9.f, 0.f);
+      }
       float mx = fmaxf(fmaxf(sv[0], sv[1]), fmaxf(sv[2], sv[3]));
       mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
       mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
@@ -498,8 +511,9 @@ __global__ void __launch_bounds__(128, D <= 128 ? 2 : 1) decode_attn_persistent_
       const int hq = head0 + row;
       float val = L > 0.f ? O / L : 0.f;
       if (p.splits == 1) {
+        if (GEN) val *= p.out_scale;
         if (GEN && p.gate) val *= head_gate(p, uc.qrow, hq);
-        p.out[((long long)uc.qrow * p.hq + hq) * dv + d] = __float2bfloat16(val);
+        p.out[GEN ? uc.qrow * p.ld_out + hq * dv + d : ((long long)uc.qrow * p.hq + hq) * dv + d] = __float2bfloat16(val);
       } else {
         p.part_o[(((long long)uc.b * p.hq + hq) * p.splits + uc.split) * dv + d] = val;
         if (d == 0) p.part_lse[((long long)uc.b * p.hq + hq) * p.splits + uc.split] = L > 0.f ? M + log2f(L) : NEG_BIG;
@@ -538,8 +552,8 @@ __global__ void __launch_bounds__(128) decode_merge_kernel(const AttnParams p) {
       if (!GEN || lane + 32 * i < dv) acc[i] += f * po[lane + 32 * i];
   }
   const int qrow = p.q_indptr[b];
-  bf16* out = p.out + ((long long)qrow * p.hq + hq) * dv;
-  const float gate = GEN && p.gate ? head_gate(p, qrow, hq) : 1.f;
+  bf16* out = p.out + (GEN ? qrow * p.ld_out + hq * dv : ((long long)qrow * p.hq + hq) * dv);
+  const float gate = (GEN ? p.out_scale : 1.f) * (GEN && p.gate ? head_gate(p, qrow, hq) : 1.f);
 #pragma unroll
   for (int i = 0; i < D / 32; ++i) {
     float v = W > 0.f ? acc[i] / W : 0.f;
@@ -591,7 +605,7 @@ __global__ void __launch_bounds__(128, MINB) prefill_attn_kernel(const AttnParam
   const int pos_base = kv_len - q_len + row_base;  // absolute position of that row
   if (kv_len == 0) {
     for (int idx = threadIdx.x; idx < rows_here * dv; idx += 128)
-      p.out[((long long)(q0 + row_base + idx / dv) * p.hq + hq) * dv + idx % dv] = __float2bfloat16(0.f);
+      p.out[(q0 + row_base + idx / dv) * (GEN ? p.ld_out : (long long)p.hq * dv) + hq * dv + idx % dv] = __float2bfloat16(0.f);
     return;
   }
 
@@ -663,6 +677,7 @@ __global__ void __launch_bounds__(128, MINB) prefill_attn_kernel(const AttnParam
     cp_async_commit();
   };
 
+  const float slope = slope_of<GEN>(p, hq);
   issue(0, 0);
   const int qpos0 = pos_base + warp * 16 + g;  // position of this lane's row g; row g+8 is +8
   for (int kt = 0; kt < n_kv_tiles; ++kt) {
@@ -692,13 +707,14 @@ __global__ void __launch_bounds__(128, MINB) prefill_attn_kernel(const AttnParam
     float mx[2] = {NEG_BIG, NEG_BIG};
     // every key of the tile is visible to every row of this warp (all but the tiles on the
     // diagonal of a causal prompt): no per-element position tests
-    const bool full_tile = window <= 0 && tok_base + BKV - 1 <= pos_base + warp * 16 && tok_base + BKV <= kv_end;
+    const bool full_tile = (window <= 0 || (GEN && tok_base > pos_base + warp * 16 + 15 - window)) && tok_base + BKV - 1 <= pos_base + warp * 16 && tok_base + BKV <= kv_end;
     if (full_tile) {
 #pragma unroll
       for (int n = 0; n < BKV / 8; ++n) {
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-          const float v = score_of<GEN>(p, s_acc[n][e]);
+          float v = score_of<GEN>(p, s_acc[n][e]);
+          if (GEN) v -= slope * (float)(qpos0 + (e >> 1) * 8 - (tok_base + n * 8 + 2 * t4 + (e & 1)));
           s_acc[n][e] = v;
           mx[e >> 1] = fmaxf(mx[e >> 1], v);
         }
@@ -712,7 +728,11 @@ __global__ void __launch_bounds__(128, MINB) prefill_attn_kernel(const AttnParam
           const int qp = qpos0 + (e >> 1) * 8;
           bool ok = tok <= qp && tok < kv_end;
           if (window > 0) ok = ok && tok > qp - window;
-          const float v = ok ? score_of<GEN>(p, s_acc[n][e]) : NEG_BIG;
+          float v = NEG_BIG;
+          if (ok) {
+            v = score_of<GEN>(p, s_acc[n][e]);
+            if (GEN) v -= slope * (float)(qp - tok);
+          }
           s_acc[n][e] = v;
           mx[e >> 1] = fmaxf(mx[e >> 1], v);
         }
@@ -775,8 +795,9 @@ __global__ void __launch_bounds__(128, MINB) prefill_attn_kernel(const AttnParam
     const int r = warp * 16 + g + rr * 8;
     if (r < rows_here) {
       float inv = l_run[rr] > 0.f ? 1.f / l_run[rr] : 0.f;
+      if (GEN) inv *= p.out_scale;
       if (GEN && p.gate) inv *= head_gate(p, q0 + row_base + r, hq);
-      bf16* dst = p.out + ((long long)(q0 + row_base + r) * p.hq + hq) * dv;
+      bf16* dst = p.out + (q0 + row_base + r) * (GEN ? p.ld_out : (long long)p.hq * dv) + hq * dv;
 #pragma unroll
       for (int n = 0; n < NT; ++n) {
         if (!GEN || n * 8 < dv) *reinterpret_cast<uint32_t*>(dst + n * 8 + 2 * t4) = pack_bf16(o[n][rr * 2] * inv, o[n][rr * 2 + 1] * inv);
@@ -941,11 +962,13 @@ extern "C" int pg_paged_attention(const void* q, const void* kv, void* out, cons
 }
 
 // The general form: key / query size `dim` and value size `vdim` (multiples of 8, up to 256), any group, softcap > 0 caps
-// the scores, `gate` (bf16 rows [T, >= hq] of stride ld_gate, or null) multiplies a head's output by its sigmoid.
+// the scores, `gate` (bf16 rows [T, >= hq] of stride ld_gate, or null) multiplies a head's output by its sigmoid, `window` > 0
+// keeps a row's last keys, `slopes` (f32 [hq], or null) takes slope * distance off a score; out rows of stride ld_out, times out_scale.
 // KV page: [page_size, hkv, dim] keys, then [page_size, hkv, vdim] values.  Modes as above.
 extern "C" int pg_attention_capped(const void* q, const void* kv, void* out, const void* q_indptr, const void* kv_lens, const void* table, int table_stride, int num_seqs, int hq, int hkv, int dim,
-                                   int vdim, int page_size, long long num_pages, float scale, float softcap, const void* gate, long long ld_gate, int mode, int splits, void* part_o, void* part_lse,
-                                   int q_tiles, void* status, cudaStream_t stream) {
+                                   int vdim, int page_size, long long num_pages, float scale, float softcap, const void* gate, long long ld_gate, int window, const void* slopes, float out_scale, long long ld_out,
+                                   int mode, int splits, void* part_o, void* part_lse, int q_tiles, void* status, cudaStream_t stream) {
+  PG_REQUIRE(window >= 0 && ld_out % 2 == 0 && ld_out >= (long long)hq * vdim, "attention_capped: a window of %d keys, output rows of %lld", window, ld_out);
   PG_REQUIRE(dim % 8 == 0 && vdim % 8 == 0 && dim >= 8 && vdim >= 8 && dim <= 256 && vdim <= 256, "attention_capped: head sizes %d / %d not supported (multiples of 8 up to 256)", dim, vdim);
   PG_REQUIRE(hq % hkv == 0, "attention_capped: %d query heads over %d KV heads", hq, hkv);
   PG_REQUIRE(page_size == 16 || page_size == 32 || page_size == 64, "attention_capped: page size %d not supported", page_size);
@@ -977,6 +1000,10 @@ extern "C" int pg_attention_capped(const void* q, const void* kv, void* out, con
   p.cap_out = softcap * LOG2E;
   p.gate = (const bf16*)gate;
   p.ld_gate = ld_gate;
+  p.window = mode == 0 ? window : 0;
+  p.slopes = (const float*)slopes;
+  p.out_scale = out_scale;
+  p.ld_out = ld_out;
   const int wide = dim > vdim ? dim : vdim;
   if (mode == 0) {
     PG_REQUIRE(p.splits == 1 || (part_o && part_lse), "attention_capped: split-KV decode needs partial buffers");
@@ -986,7 +1013,7 @@ extern "C" int pg_attention_capped(const void* q, const void* kv, void* out, con
   }
   if (q_tiles == 0) return PG_OK;
   PG_REQUIRE(hq <= 65535, "attention_capped: %d heads", hq);
-  if (wide <= 64) return launch_prefill_b<64, 2, true>(p, q_tiles, 0, stream);
-  if (wide <= 128) return launch_prefill_b<128, 2, true>(p, q_tiles, 0, stream);
-  return launch_prefill_b<256, 1, true>(p, q_tiles, 0, stream);
+  if (wide <= 64) return launch_prefill_b<64, 2, true>(p, q_tiles, window, stream);
+  if (wide <= 128) return launch_prefill_b<128, 2, true>(p, q_tiles, window, stream);
+  return launch_prefill_b<256, 1, true>(p, q_tiles, window, stream);
 }

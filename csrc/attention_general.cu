@@ -4,13 +4,15 @@
 //    pairs (2i, 2i + 1) of the first `rot` entries of every head with f32 cos / sin tables, then the queries go to a
 //    dense buffer and keys and values to the token's slot of the paged cache.  One CTA per token.  Without keys (a layer
 //    that reads another layer's cache) only the queries are made.
-//  * head_norm_append: RMS norm of every query and key head with a weight shared by the heads, queries times a factor per
-//    position; queries go to a dense buffer, keys and values (untouched; they may be the key projection itself) to the cache.
+//  * head_norm_append: RMS norm of every query and key head with a weight shared by the heads (or one per query head), queries
+//    times a factor per position; queries go to a dense buffer, keys and values (untouched; they may be the key projection
+//    itself) to the cache.  The projections' biases, if there are any, are added first.
 //  * attention_plain: one CTA per (query row, head) on the CUDA cores, keys in chunks of 128 with an online softmax; any
 //    head size, value size and group.  It is the 32-bit path, and the path of head sizes the tensor-core kernels
 //    (attention.cu, attention_tc.cu) do not address.
 //
-// Score = dot(q, k) * scale, then softcap * tanh(score / softcap) when a cap is given; the head's output is multiplied by
+// Score = dot(q, k) * scale, then softcap * tanh(score / softcap) when a cap is given, less slope[head] * distance when
+// slopes are given, over the last `window` keys (0: all); the head's output is multiplied by out_scale and by
 // sigmoid(gate[token, head]) when a gate is given.  Cache page of one layer: [page_size, kv_heads, dim] keys, then
 // [page_size, kv_heads, vdim] values.
 #include "api.h"
@@ -138,8 +140,8 @@ __global__ void __launch_bounds__(256) row_norm_rope_append_kernel(const T* __re
 
 // TPR threads (16 or 32) per unit of a token: hq query heads, hkv key heads, hkv value heads.
 template <typename T, int V, int TPR>
-__global__ void __launch_bounds__(256) head_norm_append_kernel(const T* __restrict__ q, const T* __restrict__ k, const T* __restrict__ v, long long ld, const float* __restrict__ q_w, const float* __restrict__ k_w,
-                                                               const float* __restrict__ temp, int max_pos, const int* __restrict__ positions, const int* __restrict__ slots, T* __restrict__ q_out,
+__global__ void __launch_bounds__(256) head_norm_append_kernel(const T* __restrict__ q, const T* __restrict__ k, const T* __restrict__ v, long long ld, const float* __restrict__ q_w, int q_w_heads,
+                                                               const float* __restrict__ k_w, const float* __restrict__ q_b, const float* __restrict__ k_b, const float* __restrict__ v_b, const float* __restrict__ temp, int max_pos, const int* __restrict__ positions, const int* __restrict__ slots, T* __restrict__ q_out,
                                                                T* __restrict__ kv, int hq, int hkv, int dim, int vdim, int page_size, long long num_pages, float eps, uint32_t* status) {
   PG_PDL_ENTRY();
   const long long t = blockIdx.x;
@@ -164,18 +166,27 @@ __global__ void __launch_bounds__(256) head_norm_append_kernel(const T* __restri
     const int h = u < hq ? u : value ? u - hq - hkv : u - hq, n = live ? (value ? vdim : dim) / V : 0;
     const T* src = u < hq ? q + t * ld + (long long)h * dim : value ? v + t * ld + (long long)h * vdim : k + t * ld + (long long)h * dim;
     T* dst = u < hq ? q_out + (t * hq + h) * dim : value ? kpage + (long long)page_size * hkv * dim + (off * hkv + h) * vdim : kpage + (off * hkv + h) * dim;
+    const float* bias = u < hq ? q_b : value ? v_b : k_b;
+    if (bias) bias += h * (value ? vdim : dim);
     float f[V], ss = 0.f;
-    for (int i = me; i < n; i += TPR) {
+    auto get = [&](int i) {
       load_vec<V>(src + i * V, f);
+      if (bias) {
+#pragma unroll
+        for (int j = 0; j < V; ++j) f[j] += bias[i * V + j];
+      }
+    };
+    for (int i = me; i < n; i += TPR) {
+      get(i);
 #pragma unroll
       for (int j = 0; j < V; ++j) ss += f[j] * f[j];
     }
 #pragma unroll
     for (int o = TPR / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
     const float inv = rsqrtf(ss / (float)dim + eps) * (u < hq ? factor : 1.f);
-    const float* w = u < hq ? q_w : k_w;
+    const float* w = u < hq ? q_w + (q_w_heads ? h * dim : 0) : k_w;
     for (int i = me; i < n; i += TPR) {
-      if (n > TPR) load_vec<V>(src + i * V, f);
+      if (n > TPR) get(i);
       if (!value) {
         float wf[V];
         load_vec<V>(w + i * V, wf);
@@ -193,7 +204,8 @@ constexpr int PL_VMAX = 8;    // value columns per thread: vdim <= 1024
 template <typename T>
 __global__ void __launch_bounds__(128) attention_plain_kernel(const T* __restrict__ q, const T* __restrict__ kv, T* __restrict__ out, const int* __restrict__ q_indptr, const int* __restrict__ kv_lens,
                                                               const int* __restrict__ table, int table_stride, int num_seqs, int hq, int hkv, int dim, int vdim, int page_size, long long num_pages,
-                                                              float scale, float softcap, const T* __restrict__ gate, long long ld_gate) {
+                                                              float scale, float softcap, const T* __restrict__ gate, long long ld_gate, int window, const float* __restrict__ slopes, float out_scale,
+                                                              long long ld_out) {
   PG_PDL_ENTRY();
   extern __shared__ float sm[];
   float* sq = sm;         // [dim]
@@ -217,7 +229,9 @@ __global__ void __launch_bounds__(128) attention_plain_kernel(const T* __restric
   float m = -INFINITY, l = 0.f, acc[PL_VMAX];
 #pragma unroll
   for (int i = 0; i < PL_VMAX; ++i) acc[i] = 0.f;
-  for (int k0 = 0; k0 < n; k0 += PL_KEYS) {
+  const int first = window > 0 ? max(0, n - window) : 0;  // visible keys: first .. n - 1
+  const float slope = slopes ? slopes[h] : 0.f;
+  for (int k0 = first; k0 < n; k0 += PL_KEYS) {
     const int key = k0 + tid;
     float s = -INFINITY;
     if (key < n) {
@@ -226,6 +240,7 @@ __global__ void __launch_bounds__(128) attention_plain_kernel(const T* __restric
       for (int i = 0; i < dim; ++i) a = fmaf(sq[i], to_f32(kr[i]), a);
       s = a * scale;
       if (softcap > 0.f) s = softcap * tanh_full(s / softcap);
+      s -= slope * (float)(n - 1 - key);
     }
     float mx = warp_max(s);
     if (lane == 0) red[warp] = mx;
@@ -254,11 +269,11 @@ __global__ void __launch_bounds__(128) attention_plain_kernel(const T* __restric
     }
     __syncthreads();
   }
-  float f = l > 0.f ? 1.f / l : 0.f;
+  float f = l > 0.f ? out_scale / l : 0.f;
   if (gate) f /= 1.f + __expf(-to_f32(gate[(long long)t * ld_gate + h]));
 #pragma unroll
   for (int i = 0; i < PL_VMAX; ++i)
-    if (tid + 128 * i < vdim) out[((long long)t * hq + h) * vdim + tid + 128 * i] = from_f32<T>(acc[i] * f);
+    if (tid + 128 * i < vdim) out[t * ld_out + (long long)h * vdim + tid + 128 * i] = from_f32<T>(acc[i] * f);
 }
 
 }  // namespace
@@ -282,14 +297,15 @@ extern "C" int pg_row_norm_rope_append(const void* q, const void* k, const void*
   return PG_OK;
 }
 
-// q, k, v: columns of rows of stride ld; temp f32 [max_pos] (or null); cache as above.
-extern "C" int pg_head_norm_append(const void* q, const void* k, const void* v, long long ld, const void* q_w, const void* k_w, const void* temp, int max_pos, const void* positions, const void* slots,
+// q, k, v: columns of rows of stride ld; q_w f32 [dim], or [hq, dim] with q_w_heads; q_b, k_b, v_b: biases in f32 (or null); temp f32
+// [max_pos] (or null); cache as above.
+extern "C" int pg_head_norm_append(const void* q, const void* k, const void* v, long long ld, const void* q_w, int q_w_heads, const void* k_w, const void* q_b, const void* k_b, const void* v_b, const void* temp, int max_pos, const void* positions, const void* slots,
                                    void* q_out, void* kv, int tokens, int hq, int hkv, int dim, int vdim, int page_size, long long num_pages, float eps, int is_f32, void* status, cudaStream_t stream) {
   PG_REQUIRE(hq >= 1 && hkv >= 1 && dim >= 1 && vdim >= 1 && (temp == nullptr || max_pos > 0), "head_norm_append: heads %d / %d of %d / %d columns", hq, hkv, dim, vdim);
   if (tokens == 0) return PG_OK;
   const bool v8 = dim % 8 == 0 && vdim % 8 == 0 && ld % 8 == 0 && ((((uintptr_t)q | (uintptr_t)k | (uintptr_t)v | (uintptr_t)q_out | (uintptr_t)kv | (uintptr_t)q_w | (uintptr_t)k_w) & 15) == 0);
 #define PG_HN(T, V, TPR)                                                                                                                                                                            \
-  launch_pdl(head_norm_append_kernel<T, V, TPR>, dim3(tokens), dim3(256), (size_t)0, stream, (const T*)q, (const T*)k, (const T*)v, ld, (const float*)q_w, (const float*)k_w, (const float*)temp, max_pos, \
+  launch_pdl(head_norm_append_kernel<T, V, TPR>, dim3(tokens), dim3(256), (size_t)0, stream, (const T*)q, (const T*)k, (const T*)v, ld, (const float*)q_w, q_w_heads, (const float*)k_w, (const float*)q_b, (const float*)k_b, (const float*)v_b, (const float*)temp, max_pos, \
              (const int*)positions, (const int*)slots, (T*)q_out, (T*)kv, hq, hkv, dim, vdim, page_size, num_pages, eps, (uint32_t*)status)
   if (is_f32)
     PG_CUDA(PG_HN(float, 1, 32));
@@ -301,13 +317,14 @@ extern "C" int pg_head_norm_append(const void* q, const void* k, const void* v, 
 }
 
 extern "C" int pg_attention_plain(const void* q, const void* kv, void* out, const void* q_indptr, const void* kv_lens, const void* table, int table_stride, int tokens, int num_seqs, int hq, int hkv,
-                                  int dim, int vdim, int page_size, long long num_pages, float scale, float softcap, const void* gate, long long ld_gate, int is_f32, cudaStream_t stream) {
+                                  int dim, int vdim, int page_size, long long num_pages, float scale, float softcap, const void* gate, long long ld_gate, int window, const void* slopes, float out_scale, long long ld_out,
+                                  int is_f32, cudaStream_t stream) {
   PG_REQUIRE(hq % hkv == 0 && dim <= 8192 && vdim <= 128 * PL_VMAX, "attention_plain: heads %d / %d, sizes %d / %d not supported", hq, hkv, dim, vdim);
   if (tokens == 0) return PG_OK;
   const size_t smem = (size_t)(dim + PL_KEYS) * 4;
 #define PG_AP(T)                                                                                                                                                                                    \
   launch_pdl(attention_plain_kernel<T>, dim3(tokens, hq), dim3(128), smem, stream, (const T*)q, (const T*)kv, (T*)out, (const int*)q_indptr, (const int*)kv_lens, (const int*)table, table_stride,    \
-             num_seqs, hq, hkv, dim, vdim, page_size, num_pages, scale, softcap, (const T*)gate, ld_gate)
+             num_seqs, hq, hkv, dim, vdim, page_size, num_pages, scale, softcap, (const T*)gate, ld_gate, window, (const float*)slopes, out_scale, ld_out)
   if (is_f32)
     PG_CUDA(PG_AP(float));
   else

@@ -80,6 +80,12 @@ __device__ __forceinline__ float glu_act(float z, bool gelu) {
   return z / (1.f + __expf(-t));
 }
 
+// xIELU with its learned constants in the form a = softplus(p), b = 1/2 + softplus(q).
+__device__ __forceinline__ float xielu(float z, float a, float b) {
+  const float m = fminf(z, 0.f);
+  return (z > 0.f ? a * z * z : b * (expm1f(m) - m)) + 0.5f * z;
+}
+
 struct __align__(16) bf16x8 {
   bf162 v[4];
 };

@@ -49,6 +49,7 @@ struct Gemm2Params {
   uint32_t tmem_cols;
   uint32_t* status;
   int epi;  // 0: y = x W^T; 1: the weight rows alternate (gate_i, up_i) and y [T, M / 2] = bf16(silu(gate)) * up
+  const float* xielu;  // epi 0: the two constants of xIELU on every output (nullptr = none)
 };
 
 // Work item -> (weight-row pair, token tile).  Items walk RASTER_GROUP weight-row pairs across
@@ -269,6 +270,13 @@ gemm2sm_bf16_tn_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_co
             }
           }
         } else if (m < p.M) {
+          if (p.xielu != nullptr) {
+            const float a = p.xielu[0], b = p.xielu[1];
+#pragma unroll
+            for (int h = 0; h < 2; ++h)
+#pragma unroll
+              for (int j = 0; j < 16; ++j) v[h][j] = __float_as_uint(xielu(__uint_as_float(v[h][j]), a, b));
+          }
 #pragma unroll
           for (int h = 0; h < 2; ++h) {
 #pragma unroll
@@ -333,7 +341,7 @@ extern "C" int pg_gemm2sm_eligible(int T, int M, int K) {
   return (long long)ceil_div(M, 2 * BM) * ceil_div(T, 256) >= 64 ? 1 : 0;
 }
 
-static int gemm2sm_impl(const void* x, const void* w, void* y, int T, int M, int K, long long ldx, long long ldw, long long ldy, void* status, int epi, cudaStream_t stream);
+static int gemm2sm_impl(const void* x, const void* w, void* y, int T, int M, int K, long long ldx, long long ldw, long long ldy, void* status, int epi, cudaStream_t stream, const void* xielu = nullptr);
 
 extern "C" int pg_gemm2sm_bf16_tn(const void* x, const void* w, void* y, int T, int M, int K, long long ldx, long long ldw, long long ldy, void* status,
                                   cudaStream_t stream) {
@@ -347,7 +355,12 @@ extern "C" int pg_gemm2sm_bf16_tn_swiglu(const void* x, const void* w, void* y, 
   return gemm2sm_impl(x, w, y, T, M, K, ldx, ldw, ldy, status, gelu ? 3 : 1, stream);
 }
 
-static int gemm2sm_impl(const void* x, const void* w, void* y, int T, int M, int K, long long ldx, long long ldw, long long ldy, void* status, int epi, cudaStream_t stream) {
+// The same product with xIELU in the epilogue; act: f32 softplus(p), 1/2 + softplus(q).
+extern "C" int pg_gemm2sm_bf16_tn_xielu(const void* x, const void* w, void* y, int T, int M, int K, long long ldx, long long ldw, long long ldy, const void* act, void* status, cudaStream_t stream) {
+  return gemm2sm_impl(x, w, y, T, M, K, ldx, ldw, ldy, status, 0, stream, act);
+}
+
+static int gemm2sm_impl(const void* x, const void* w, void* y, int T, int M, int K, long long ldx, long long ldw, long long ldy, void* status, int epi, cudaStream_t stream, const void* xielu) {
   PG_REQUIRE(T > 0 && M > 0 && K > 0 && K % 8 == 0, "gemm2sm: bad problem %dx%dx%d", T, M, K);
   PG_REQUIRE(status != nullptr, "gemm2sm: a device status word is required");
   int dev = 0;
@@ -411,6 +424,7 @@ static int gemm2sm_impl(const void* x, const void* w, void* y, int T, int M, int
   p.tmem_cols = 2 * p.bn > 256 ? 512u : 256u;
   p.status = (uint32_t*)status;
   p.epi = epi;
+  p.xielu = (const float*)xielu;
   const size_t smem = 1024 + (size_t)p.stages * stage_bytes + tail;
   CUtensorMap tm_w, tm_x;
   int rc = pg_make_tmap_bf16_2d(&tm_w, w, M, K, ldw, BM, BK);

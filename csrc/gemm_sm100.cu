@@ -94,6 +94,7 @@ struct FuseSpec {
   int gelu;             // EPI_SWIGLU: tanh-GELU in the place of SiLU
   float* out_ssp;       // EPI_RESID_NORMW: [T][out_ld], entry [n][m_tile]
   int out_ld;
+  const float* xielu;   // EPI_PLAIN: the two constants of xIELU on every output (nullptr = none); any launch shape
 };
 
 struct GemmParams {
@@ -125,6 +126,7 @@ struct GemmParams {
 // local memory only.
 __device__ __forceinline__ void store_out(const GemmParams& p, int n, int m, float v, const float* s_inv = nullptr, int n_local = 0) {
   if (s_inv) v *= s_inv[n_local];
+  if (p.fuse.xielu) v = xielu(v, p.fuse.xielu[0], p.fuse.xielu[1]);
   if (p.tp.enabled) {
     const TpFuse& tp = p.tp;
     if (tp.one_shot) {
@@ -246,6 +248,10 @@ __device__ __forceinline__ float store_out4(const GemmParams& p, int n, int m, f
     for (int i = 0; i < 4; ++i)
       if (m + i < p.M) store_out(p, n, m + i, f[i]);
     return 0.f;
+  }
+  if (EPI == EPI_PLAIN && p.fuse.xielu) {
+    const float a = p.fuse.xielu[0], b = p.fuse.xielu[1];
+    v = make_float4(xielu(v.x, a, b), xielu(v.y, a, b), xielu(v.z, a, b), xielu(v.w, a, b));
   }
   if (p.tp.enabled) {
     const TpFuse& tp = p.tp;
@@ -1263,6 +1269,18 @@ extern "C" int pg_gemm_bf16_tn(const void* x, const void* w, void* y, int y_is_f
   // serving) keeps every problem size on this one kernel
   if (!y_is_f32 && force_splits <= 0 && pg_gemm2sm_eligible(T, M, K)) return pg_gemm2sm_bf16_tn(x, w, y, T, M, K, ldx, ldw, ldy, status, stream);
   return gemm_impl(x, w, y, y_is_f32, T, M, K, ldx, ldw, ldy, ws, ws_bytes, counters, counter_bytes, status, force_splits, nullptr, nullptr, stream);
+}
+
+// xIELU of the product in the epilogue; act: f32 softplus(p), 1/2 + softplus(q).
+extern "C" int pg_gemm_bf16_tn_xielu(const void* x, const void* w, void* y, int T, int M, int K, long long ldx, long long ldw, long long ldy, const void* act, void* ws, long long ws_bytes, void* counters,
+                                     long long counter_bytes, void* status, int force_splits, cudaStream_t stream) {
+  PG_REQUIRE(act != nullptr, "gemm xielu: the activation's constants are required");
+  if (force_splits <= 0 && pg_gemm2sm_eligible(T, M, K)) return pg_gemm2sm_bf16_tn_xielu(x, w, y, T, M, K, ldx, ldw, ldy, act, status, stream);
+  FuseSpec f;
+  memset(&f, 0, sizeof(f));
+  f.epi = EPI_PLAIN;
+  f.xielu = (const float*)act;
+  return gemm_impl(x, w, y, 0, T, M, K, ldx, ldw, ldy, ws, ws_bytes, counters, counter_bytes, status, force_splits, nullptr, nullptr, stream, nullptr, &f);
 }
 
 // Same GEMM, but X rows are being all-gathered into `x` by peers: the TMA producer streams

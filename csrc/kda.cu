@@ -12,7 +12,9 @@
 //    The same kernel runs two more rules (RULE below): the decay in its softplus form, exp(-exp(A_log) softplus(f + dt_bias)),
 //    with query / key heads shared by several value heads, plain linear attention with one fixed decay per head
 //    (S = decay S + k (x) v, out = S^T q, SiLU on q, k and v), and linear attention with a decay per token and key channel and a
-//    bonus for the current token (out = (S + diag(u) k (x) v)^T q in front of S = diag(dec) S + k (x) v, dec = exp(-exp(f + w0))).
+//    bonus for the current token (out = (S + diag(u) k (x) v)^T q in front of S = diag(dec) S + k (x) v, dec = exp(-exp(f + w0))), and
+//    state-space duality, one decay per token and head (d = softplus(f + dt_bias), S = exp(-exp(A_log) d) S + d k (x) v, out = S^T q +
+//    D v, keys and queries shared by a group of heads).
 //    Those take bf16 or f32 rows and any key width up to 256.
 //  * attnres_mix: the attention-residual mix.  Every token keeps up to `cap` snapshot rows of its own residual
 //    stream; a mix scores each of the first nb snapshots and the current row with
@@ -31,18 +33,18 @@ constexpr int KDA_COLS = 32;
 
 // What a token does to the state.  BOUNDED and SOFTPLUS are the delta rule with a decay per key channel and two forms of
 // the decay; DECAY is linear attention with a fixed decay per head (no correction term), WKV with a decay per token and key
-// channel, read in front of the update with a bonus for the current token.
-enum { RULE_BOUNDED = 0, RULE_SOFTPLUS = 1, RULE_DECAY = 2, RULE_WKV = 3 };
+// channel, read in front of the update with a bonus for the current token, SSD with a decay and a step size per token and head.
+enum { RULE_BOUNDED = 0, RULE_SOFTPLUS = 1, RULE_DECAY = 2, RULE_WKV = 3, RULE_SSD = 4 };
 
 template <typename T>
 struct RecArgs {
   const T *q, *k, *v;  // token rows of stride ld; q and k [kv_heads * dk], v [heads * dv]
   long long ld;
-  const void* f;  // raw decay projection [heads * dk]: T (BOUNDED) or f32 (SOFTPLUS, WKV)
+  const void* f;  // raw decay projection [heads * dk]: T (BOUNDED) or f32 (SOFTPLUS, WKV); SSD: raw step sizes T [heads]
   long long ldf;
   const T* b;  // raw step-size projection [heads]
   long long ldb;
-  const float *a_log, *dt_bias, *decay;  // decay [heads]: DECAY; WKV: dt_bias = w0 [heads * dk], decay = the bonus u [heads * dk]
+  const float *a_log, *dt_bias, *decay;  // decay [heads]: DECAY; WKV: dt_bias = w0 [heads * dk], decay = the bonus u [heads * dk]; SSD: dt_bias [heads], decay = D [heads]
   float lower;
   float* state;
   T* out;
@@ -65,9 +67,9 @@ __global__ void __launch_bounds__(128) kda_recurrent_kernel(const T* __restrict_
   constexpr int QS = QK + 4;   // padded quarter stride: the four quarters land in different banks
   constexpr int QL = DK / 32;  // elements per lane when a warp holds one token
   constexpr bool DELTA = RULE == RULE_BOUNDED || RULE == RULE_SOFTPLUS;
-  constexpr bool KEYED = RULE != RULE_DECAY;  // a decay per key channel
+  constexpr bool KEYED = RULE != RULE_DECAY && RULE != RULE_SSD;  // a decay per key channel
   __shared__ __align__(16) float sq[KDA_STAGE][4 * QS], sk[KDA_STAGE][4 * QS], sd[KEYED ? KDA_STAGE : 1][4 * QS];
-  __shared__ float sv[KDA_STAGE][KDA_COLS], sb[KDA_STAGE];
+  __shared__ float sv[KDA_STAGE][KDA_COLS], sb[KDA_STAGE], se[RULE == RULE_SSD ? KDA_STAGE : 1];
   __shared__ float red_kv[4][KDA_COLS], red_o[DELTA ? 1 : 2][4][KDA_COLS];
   const int dk = PAD ? dk_arg : DK;
   const int h = blockIdx.x / col_groups, cg = blockIdx.x % col_groups, seq = blockIdx.y;
@@ -85,10 +87,10 @@ __global__ void __launch_bounds__(128) kda_recurrent_kernel(const T* __restrict_
   float s_col[QK];
 #pragma unroll
   for (int i = 0; i < QK; ++i) s_col[i] = owner && (!PAD || qtr * QK + i < dk) ? S[(long long)(qtr * QK + i) * dv + col] : 0.f;
-  const int kh = RULE == RULE_SOFTPLUS ? h * kv_heads / heads : h;
+  const int kh = RULE == RULE_SOFTPLUS || RULE == RULE_SSD ? h * kv_heads / heads : h;
   const float q_scale = DELTA ? rsqrtf((float)dk) : 1.f;
-  const float a = DELTA ? __expf(a_log[h]) : 0.f;
-  const float fixed = RULE == RULE_DECAY ? decay[h] : 0.f;
+  const float a = DELTA || RULE == RULE_SSD ? __expf(a_log[h]) : 0.f;
+  const float fixed = RULE == RULE_DECAY || RULE == RULE_SSD ? decay[h] : 0.f;
 
   for (int t0 = q0; t0 < q1; t0 += KDA_STAGE) {
     const int nt = min(KDA_STAGE, q1 - t0);
@@ -108,7 +110,7 @@ __global__ void __launch_bounds__(128) kda_recurrent_kernel(const T* __restrict_
           ks += rk[i] * rk[i];
         } else if (RULE == RULE_WKV) {
           if (in) qs += rq[i] * rk[i] * decay[h * dk + lane + 32 * i];
-        } else {  // the activation's result is what the layer works with, in the activation type
+        } else if (RULE == RULE_DECAY) {  // the activation's result is what the layer works with, in the activation type
           rq[i] = to_f32(from_f32<T>(rq[i] / (1.f + __expf(-rq[i]))));
           rk[i] = to_f32(from_f32<T>(rk[i] / (1.f + __expf(-rk[i]))));
         }
@@ -149,12 +151,17 @@ __global__ void __launch_bounds__(128) kda_recurrent_kernel(const T* __restrict_
       if (RULE == RULE_DECAY) x = to_f32(from_f32<T>(x / (1.f + __expf(-x))));
       sv[j][idx % KDA_COLS] = x;
     }
+    if (RULE == RULE_SSD && tid < nt) {
+      const float raw = to_f32(((const T*)f)[(long long)(t0 + tid) * ldf + h]) + dt_bias[h], d = raw > 20.f ? raw : log1pf(__expf(raw));
+      sb[tid] = d;
+      se[tid] = __expf(-a * d);
+    }
     if (DELTA && tid < nt) sb[tid] = 1.f / (1.f + __expf(-to_f32(b[(long long)(t0 + tid) * ldb + h])));
     __syncthreads();
     for (int j = 0; j < nt; ++j) {
       const float4* kq = reinterpret_cast<const float4*>(&sk[j][qtr * QS]);
       const float4* qq = reinterpret_cast<const float4*>(&sq[j][qtr * QS]);
-      float delta = sv[j][lc];
+      float delta = RULE == RULE_SSD ? sv[j][lc] * sb[j] : sv[j][lc];
       if (DELTA) {
         const float4* dq = reinterpret_cast<const float4*>(&sd[DELTA ? j : 0][qtr * QS]);
         float4 kv4 = make_float4(0.f, 0.f, 0.f, 0.f);
@@ -198,10 +205,11 @@ __global__ void __launch_bounds__(128) kda_recurrent_kernel(const T* __restrict_
           continue;
         }
         if (!DELTA) {
-          s_col[4 * i + 0] *= fixed;
-          s_col[4 * i + 1] *= fixed;
-          s_col[4 * i + 2] *= fixed;
-          s_col[4 * i + 3] *= fixed;
+          const float dec = RULE == RULE_SSD ? se[RULE == RULE_SSD ? j : 0] : fixed;
+          s_col[4 * i + 0] *= dec;
+          s_col[4 * i + 1] *= dec;
+          s_col[4 * i + 2] *= dec;
+          s_col[4 * i + 3] *= dec;
         }
         s_col[4 * i + 0] += kk.x * delta;
         s_col[4 * i + 1] += kk.y * delta;
@@ -224,6 +232,7 @@ __global__ void __launch_bounds__(128) kda_recurrent_kernel(const T* __restrict_
         o += __shfl_xor_sync(0xffffffffu, o, 2);
       }
       if (RULE == RULE_WKV) o += sb[j] * delta;
+      if (RULE == RULE_SSD) o += fixed * sv[j][lc];
       if (owner && qtr == 0) out[((long long)(t0 + j) * heads + h) * dv + col] = from_f32<T>(o);
     }
     __syncthreads();
@@ -262,6 +271,7 @@ int run_rule(int rule, RecArgs<T> p, int num_seqs, int max_q_len, cudaStream_t s
   const bool few = max_q_len <= 4;  // decode rows and verify steps: the row-coalesced mapping
   PG_CUDA(rule == RULE_SOFTPLUS ? (launch_padded<T, RULE_SOFTPLUS>(p, grid, few, stream))
           : rule == RULE_WKV    ? (launch_padded<T, RULE_WKV>(p, grid, few, stream))
+          : rule == RULE_SSD    ? (launch_padded<T, RULE_SSD>(p, grid, few, stream))
                                 : (launch_padded<T, RULE_DECAY>(p, grid, few, stream)));
   PG_LAUNCH_CHECK();
   return PG_OK;
@@ -396,6 +406,23 @@ extern "C" int pg_wkv_recurrent(const void* r, const void* k, const void* v, lon
   RecArgs<bf16> p = {(const bf16*)r, (const bf16*)k, (const bf16*)v, ld, f, ldf, nullptr, 0, nullptr, (const float*)w0, (const float*)u, 0.f,
                      (float*)state, (bf16*)out, (const int*)q_indptr, (const int*)slots, heads, heads, dk, dv, 0, skip_len};
   return run_rule<bf16>(RULE_WKV, p, num_seqs, max_q_len, stream);
+}
+
+// State-space duality: x [T, heads, dv] rows of stride ld, B and C [T, groups, n] rows of the same stride, dt [T, heads] raw step sizes of
+// stride lddt; d = softplus(dt + dt_bias): S <- exp(-exp(a_log) d) S + d B x^T, out = S^T C + D x.
+extern "C" int pg_ssd_recurrent(const void* C, const void* B, const void* x, long long ld, const void* dt, long long lddt, const void* a_log, const void* dt_bias, const void* D, void* state, void* out,
+                                const void* q_indptr, const void* slots, int num_seqs, int heads, int groups, int n, int dv, int max_q_len, int skip_len, int is_f32, cudaStream_t stream) {
+  PG_REQUIRE(n >= 1 && n <= 256 && dv >= 1 && heads % groups == 0, "ssd_recurrent: heads %d / %d, state width %d (at most 256), value width %d", heads, groups, n, dv);
+  PG_REQUIRE(num_seqs <= 65535, "ssd_recurrent: %d sequences", num_seqs);
+  if (num_seqs == 0) return PG_OK;
+  if (is_f32) {
+    RecArgs<float> p = {(const float*)C, (const float*)B, (const float*)x, ld, dt, lddt, nullptr, 0, (const float*)a_log, (const float*)dt_bias, (const float*)D, 0.f,
+                        (float*)state, (float*)out, (const int*)q_indptr, (const int*)slots, heads, groups, n, dv, 0, skip_len};
+    return run_rule<float>(RULE_SSD, p, num_seqs, max_q_len, stream);
+  }
+  RecArgs<bf16> p = {(const bf16*)C, (const bf16*)B, (const bf16*)x, ld, dt, lddt, nullptr, 0, (const float*)a_log, (const float*)dt_bias, (const float*)D, 0.f,
+                     (float*)state, (bf16*)out, (const int*)q_indptr, (const int*)slots, heads, groups, n, dv, 0, skip_len};
+  return run_rule<bf16>(RULE_SSD, p, num_seqs, max_q_len, stream);
 }
 
 extern "C" int pg_attnres_mix(const void* cur, long long ld_cur, const void* snaps, long long ld_tok, const void* score_w, void* out, long long ld_out,

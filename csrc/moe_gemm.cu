@@ -76,6 +76,7 @@ struct MoeGemmParams {
   long long y_head;
   const bf16* gate;
   long long ldg, g_head;
+  float* y_f32;  // heads: the output in f32 in the place of y
 };
 
 struct Item {
@@ -298,7 +299,15 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant_
                 v[j] = __float_as_uint(f * f);
               }
             }
-            bf16* dst = p.y + (p.head_rows ? it.e * p.y_head : 0ll) + (long long)(it.row0 + c) * p.ldy + m;
+            const long long at = (p.head_rows ? it.e * p.y_head : 0ll) + (long long)(it.row0 + c) * p.ldy + m;
+            if (p.y_f32 != nullptr) {
+              float* dst = p.y_f32 + at;
+#pragma unroll
+              for (int j = 0; j < 16; ++j)
+                if (c + j < it.rows) dst[(long long)j * p.ldy] = __uint_as_float(v[j]);
+              continue;
+            }
+            bf16* dst = p.y + at;
             if (p.gate != nullptr) {
               const bf16* gp = p.gate + it.e * p.g_head + (long long)(it.row0 + c) * p.ldg + m;
               float gv[16];
@@ -493,6 +502,7 @@ std::mutex g_mu;
 struct HeadArgs {
   long long x_head, y_head, g_head, ldg;
   const void* gate;
+  int y_f32;
 };
 
 // x [rows, K] bf16 (rows sorted by expert), offsets [E+1] device int32, y [rows, M] bf16.
@@ -546,6 +556,7 @@ static int moe_gemm_impl(const void* x, long long ldx, long long x_rows, const v
     p.gate = (const bf16*)heads->gate;
     p.ldg = heads->ldg;
     p.g_head = heads->g_head;
+    if (heads->y_f32) p.y_f32 = (float*)y;
   }
   p.scatter_src = (const int*)scatter_src;
   if (scatter_src) {
@@ -631,10 +642,12 @@ extern "C" int pg_moe_grouped_gemm_act(const void* x, long long ldx, long long x
   return moe_gemm_impl(x, ldx, x_rows, w, nullptr, 0, y, ldy, offsets, E, M, K, bn, status, nullptr, nullptr, nullptr, 0, 0, 1, 0, stream, act);
 }
 
-// y[t, h, :] = x[t, h, :] w[h]^T, w [heads, M, K]; row / head strides in elements; gate (bf16, or null) strided like y.
-extern "C" int pg_head_gemm(const void* x, long long ldx, long long x_head, const void* w, void* y, long long ldy, long long y_head, const void* gate, long long ldg, long long g_head, int heads, int rows,
-                            int M, int K, int bn, void* status, cudaStream_t stream) {
+// y[t, h, :] = x[t, h, :] w[h]^T, w [heads, M, K]; row / head strides in elements; y bf16 or f32; gate (bf16, or null) strided like y.
+extern "C" int pg_head_gemm(const void* x, long long ldx, long long x_head, const void* w, void* y, int y_f32, long long ldy, long long y_head, const void* gate, long long ldg, long long g_head, int heads,
+                            int rows, int M, int K, int bn, void* status, cudaStream_t stream) {
+  PG_REQUIRE(!y_f32 || gate == nullptr, "head gemm: a gate multiplies a bf16 output only");
   HeadArgs a;
+  a.y_f32 = y_f32;
   a.x_head = x_head, a.y_head = y_head, a.g_head = g_head, a.ldg = ldg, a.gate = gate;
   return moe_gemm_impl(x, ldx, rows, w, nullptr, 0, y, ldy, nullptr, heads, M, K, bn, status, nullptr, nullptr, nullptr, 0, 0, 1, 0, stream, 0, &a);
 }

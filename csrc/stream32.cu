@@ -14,12 +14,13 @@
 //    output, or the weighted sum of a token's expert rows, which is then formed here instead of by a kernel of its own.
 //    With y = x and no sum it is the plain layer norm of the stream.
 //  * gated_row_norm: RMS norm over a row (one head, or all heads of a token at once), times a weight, times the sigmoid or
-//    the SiLU of a gate row that may lie inside a wider projection output.
-//  * glu_rows: silu(gate) * up or gelu(gate) * up on f32 rows; softcap_f32: cap * tanh(x / cap) on f32 values; tanh_rows.
+//    the SiLU of a gate row that may lie inside a wider projection output; or the gate in front of the norm.
+//  * glu_rows: silu(gate) * up or gelu(gate) * up on f32 rows; softcap_f32: cap * tanh(x / cap) on f32 values; tanh_rows; xielu_rows.
 //  * gemm_simt: y = x w^T on the CUDA cores with f32 accumulation, for f32 operands (the 32-bit mode) and for bf16
 //    problems whose rows the TMA kernels cannot address (an inner size that is not a multiple of 8).  head_gemm_simt is the
 //    same per attention head (strided operands, sigmoid gate on the output), expert_gemm_simt per expert over sorted rows.
-//  * conv_silu: causal depthwise convolution of any length + SiLU over ragged sequences with carried inputs.
+//  * short_conv: causal depthwise convolution of any length over ragged sequences with carried inputs; biases on the inputs and on
+//    the sum and a SiLU are optional.
 #include "api.h"
 #include "common.cuh"
 #include "types.cuh"
@@ -325,7 +326,7 @@ __global__ void __launch_bounds__(256) add_layer_norm_kernel(const RowSource<TY>
 // TPR threads per row (16, 32 or 256); row r = token * heads + head; the gate row of (token, head) is gate + token * ldg + head * dim.
 template <typename T, int V, int TPR>
 __global__ void __launch_bounds__(256) gated_row_norm_kernel(const T* __restrict__ x, const T* __restrict__ gate, long long ldg, const float* __restrict__ w, T* __restrict__ y, long long rows, int heads, int dim,
-                                                             float eps, int silu, int w_heads) {
+                                                             float eps, int silu, int w_heads, int gate_first) {
   PG_PDL_ENTRY();
   __shared__ float red[32];
   const long long row = TPR == 256 ? (long long)blockIdx.x : (long long)blockIdx.x * (256 / TPR) + threadIdx.x / TPR;
@@ -337,18 +338,27 @@ __global__ void __launch_bounds__(256) gated_row_norm_kernel(const T* __restrict
   constexpr int KEEP = 4;
   const int nv = live ? dim / V : 0;
   float f[KEEP][V], ss = 0.f;
+  auto get = [&](int i, float* o) {
+    load_vec<V>(xr + i * V, o);
+    if (gate_first) {
+      float g[V];
+      load_vec<V>(gr + i * V, g);
+#pragma unroll
+      for (int j = 0; j < V; ++j) o[j] *= (silu ? g[j] : 1.f) / (1.f + __expf(-g[j]));
+    }
+  };
 #pragma unroll
   for (int k = 0; k < KEEP; ++k) {
     const int i = me + k * TPR;
     if (i < nv) {
-      load_vec<V>(xr + i * V, f[k]);
+      get(i, f[k]);
 #pragma unroll
       for (int j = 0; j < V; ++j) ss += f[k][j] * f[k][j];
     }
   }
   for (int i = me + KEEP * TPR; i < nv; i += TPR) {
     float o[V];
-    load_vec<V>(xr + i * V, o);
+    get(i, o);
 #pragma unroll
     for (int j = 0; j < V; ++j) ss += o[j] * o[j];
   }
@@ -361,10 +371,15 @@ __global__ void __launch_bounds__(256) gated_row_norm_kernel(const T* __restrict
   const float inv = rsqrtf(ss / (float)dim + eps);
   auto put = [&](int i, const float* o) {
     float g[V], wf[V], r[V];
-    load_vec<V>(gr + i * V, g);
     load_vec<V>(w + i * V, wf);
+    if (gate_first) {
 #pragma unroll
-    for (int j = 0; j < V; ++j) r[j] = o[j] * inv * wf[j] * (silu ? g[j] : 1.f) / (1.f + __expf(-g[j]));
+      for (int j = 0; j < V; ++j) r[j] = o[j] * inv * wf[j];
+    } else {
+      load_vec<V>(gr + i * V, g);
+#pragma unroll
+      for (int j = 0; j < V; ++j) r[j] = o[j] * inv * wf[j] * (silu ? g[j] : 1.f) / (1.f + __expf(-g[j]));
+    }
     store_vec<V>(y + row * dim + i * V, r);
   };
 #pragma unroll
@@ -374,9 +389,16 @@ __global__ void __launch_bounds__(256) gated_row_norm_kernel(const T* __restrict
   }
   for (int i = me + KEEP * TPR; i < nv; i += TPR) {
     float o[V];
-    load_vec<V>(xr + i * V, o);
+    get(i, o);
     put(i, o);
   }
+}
+
+template <typename T>
+__global__ void xielu_rows_kernel(const T* __restrict__ x, T* __restrict__ y, const float* __restrict__ act, long long n) {
+  PG_PDL_ENTRY();
+  const float a = act[0], b = act[1];
+  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x) y[i] = from_f32<T>(xielu(to_f32(x[i]), a, b));
 }
 
 __global__ void glu_rows_kernel(const float* __restrict__ gu, float* __restrict__ out, int rows, int inter, long long ldin, int gelu) {
@@ -444,8 +466,8 @@ __global__ void __launch_bounds__(256) gemm_simt_kernel(const TX* __restrict__ x
 }
 
 // Head h (grid z): y[t, h, :] = x[t, h, :] w[h]^T, times sigmoid(gate[t, h, :]) when a gate is given.
-template <typename T>
-__global__ void __launch_bounds__(256) head_gemm_simt_kernel(const T* __restrict__ x, long long ldx, long long x_head, const T* __restrict__ w, T* __restrict__ y, long long ldy, long long y_head,
+template <typename T, typename TY>
+__global__ void __launch_bounds__(256) head_gemm_simt_kernel(const T* __restrict__ x, long long ldx, long long x_head, const T* __restrict__ w, TY* __restrict__ y, long long ldy, long long y_head,
                                                              const T* __restrict__ gate, long long ldg, long long g_head, int rows, int M, int K) {
   PG_PDL_ENTRY();
   const int m0 = blockIdx.x * 64, t0 = blockIdx.y * 64, h = blockIdx.z;
@@ -460,7 +482,7 @@ __global__ void __launch_bounds__(256) head_gemm_simt_kernel(const T* __restrict
       if (t >= rows || m >= M) continue;
       float v = acc[i][j];
       if (gate) v /= 1.f + __expf(-to_f32(gate[(long long)t * ldg + h * g_head + m]));
-      y[(long long)t * ldy + h * y_head + m] = from_f32<T>(v);
+      y[(long long)t * ldy + h * y_head + m] = from_f32<TY>(v);
     }
 }
 
@@ -512,10 +534,11 @@ constexpr int CONV_TILE = 16;  // tokens per CTA; at least CONV_MAX - 1, so a se
 
 // A thread owns one channel for CONV_TILE tokens.  The CTA of a sequence's first tile reads the carried inputs and is also
 // the one that replaces them (from the sequence's last rows), so no other CTA touches the state.
-// CM: the number of taps rounded up to an instantiated size.
+// CM: the number of taps rounded up to an instantiated size.  `bias` (or null) joins the sum, `in_bias` (or null) every input of
+// the sequence, which is then rounded to T, as the carried ones are.
 template <typename T, int CM>
-__global__ void __launch_bounds__(128) conv_silu_kernel(const T* __restrict__ x, long long ldx, const float* __restrict__ w, T* __restrict__ state, T* __restrict__ out, long long ldo, const int* __restrict__ q_indptr,
-                                                        const int* __restrict__ slots, int channels, int taps, long long slot_stride) {
+__global__ void __launch_bounds__(128) short_conv_kernel(const T* __restrict__ x, long long ldx, const float* __restrict__ w, const float* __restrict__ bias, const float* __restrict__ in_bias, T* __restrict__ state,
+                                                         T* __restrict__ out, long long ldo, const int* __restrict__ q_indptr, const int* __restrict__ slots, int channels, int taps, long long slot_stride, int silu) {
   PG_PDL_ENTRY();
   const int b = blockIdx.z, c = blockIdx.x * 128 + threadIdx.x;
   const int q0 = q_indptr[b], n = q_indptr[b + 1] - q0;
@@ -525,6 +548,8 @@ __global__ void __launch_bounds__(128) conv_silu_kernel(const T* __restrict__ x,
   T* st = state + slot * slot_stride + (long long)c * (taps - 1);
   const int back = taps - 1;
   const int n_here = min(CONV_TILE, n - s0);
+  const float cb = bias ? bias[c] : 0.f, ib = in_bias ? in_bias[c] : 0.f;
+  auto input = [&](T v) { return in_bias ? from_f32<T>(to_f32(v) + ib) : v; };
   T rows[CONV_TILE];  // all loads of the tile in flight together
 #pragma unroll
   for (int i = 0; i < CONV_TILE; ++i)
@@ -535,24 +560,24 @@ __global__ void __launch_bounds__(128) conv_silu_kernel(const T* __restrict__ x,
   for (int j = 0; j < CM; ++j) {
     const int tap = j - (CM - taps), at = s0 + j - (CM - 1);
     wt[j] = tap >= 0 ? w[(long long)c * taps + tap] : 0.f;
-    win[j] = tap >= 0 && j < CM - 1 ? (at < 0 ? to_f32(st[back + at]) : to_f32(x[(long long)(q0 + at) * ldx + c])) : 0.f;
+    win[j] = tap >= 0 && j < CM - 1 ? (at < 0 ? to_f32(st[back + at]) : to_f32(input(x[(long long)(q0 + at) * ldx + c]))) : 0.f;
   }
   T keep[CM];
   if (s0 == 0) {
 #pragma unroll
     for (int j = 0; j < CM - 1; ++j) {
       const int at = n - back + j;
-      if (j < back) keep[j] = at < 0 ? st[back + at] : x[(long long)(q0 + at) * ldx + c];
+      if (j < back) keep[j] = at < 0 ? st[back + at] : input(x[(long long)(q0 + at) * ldx + c]);
     }
   }
 #pragma unroll
   for (int i = 0; i < CONV_TILE; ++i) {
     if (i >= n_here) break;
-    win[CM - 1] = to_f32(rows[i]);
-    float a = 0.f;
+    win[CM - 1] = to_f32(input(rows[i]));
+    float a = cb;
 #pragma unroll
     for (int j = 0; j < CM; ++j) a = fmaf(win[j], wt[j], a);
-    out[(long long)(q0 + s0 + i) * ldo + c] = from_f32<T>(__fdividef(a, 1.f + __expf(-a)));
+    out[(long long)(q0 + s0 + i) * ldo + c] = from_f32<T>(silu ? __fdividef(a, 1.f + __expf(-a)) : a);
 #pragma unroll
     for (int j = 0; j < CM - 1; ++j) win[j] = win[j + 1];
   }
@@ -675,15 +700,15 @@ extern "C" int pg_add_layer_norm(const void* y, int y_f32, long long ldy, const 
   return PG_OK;
 }
 
-extern "C" int pg_gated_row_norm(const void* x, const void* gate, long long ldg, const void* w, void* y, int tokens, int heads, int dim, float eps, int silu, int w_heads, int is_f32,
-                                 cudaStream_t stream) {
+extern "C" int pg_gated_row_norm(const void* x, const void* gate, long long ldg, const void* w, void* y, int tokens, int heads, int dim, float eps, int silu, int w_heads, int gate_first,
+                                 int is_f32, cudaStream_t stream) {
   if (tokens == 0) return PG_OK;
   const long long rows = (long long)tokens * heads;
   const bool wide = dim > 512;
   const bool v8 = !is_f32 && dim % 8 == 0 && ldg % 8 == 0 && al(x, 16) && al(gate, 16) && al(w, 16) && al(y, 16);
   const bool half = v8 && dim <= 128;  // a half warp covers the row with one access per lane
   const dim3 grid((unsigned)(wide ? rows : half ? (rows + 15) / 16 : (rows + 7) / 8));
-#define PG_GRN(T, V, TPR) launch_pdl(gated_row_norm_kernel<T, V, TPR>, grid, dim3(256), (size_t)0, stream, (const T*)x, (const T*)gate, ldg, (const float*)w, (T*)y, rows, heads, dim, eps, silu, w_heads)
+#define PG_GRN(T, V, TPR) launch_pdl(gated_row_norm_kernel<T, V, TPR>, grid, dim3(256), (size_t)0, stream, (const T*)x, (const T*)gate, ldg, (const float*)w, (T*)y, rows, heads, dim, eps, silu, w_heads, gate_first)
   if (is_f32) {
     PG_CUDA(wide ? PG_GRN(float, 1, 256) : PG_GRN(float, 1, 32));
   } else {
@@ -702,6 +727,17 @@ extern "C" int pg_glu_rows_f32(const void* gu, void* out, int rows, int inter, l
   long long blocks = ((long long)rows * inter + 255) / 256;
   if (blocks > 148 * 16) blocks = 148 * 16;
   PG_CUDA(launch_pdl(glu_rows_kernel, dim3((unsigned)blocks), dim3(256), (size_t)0, stream, (const float*)gu, (float*)out, rows, inter, ldin, gelu));
+  PG_LAUNCH_CHECK();
+  return PG_OK;
+}
+
+// act: f32 softplus(p), 1/2 + softplus(q).
+extern "C" int pg_xielu_rows(const void* x, void* y, const void* act, long long n, int is_f32, cudaStream_t stream) {
+  if (n == 0) return PG_OK;
+  long long blocks = (n + 255) / 256;
+  if (blocks > 148 * 16) blocks = 148 * 16;
+  PG_CUDA(is_f32 ? launch_pdl(xielu_rows_kernel<float>, dim3((unsigned)blocks), dim3(256), (size_t)0, stream, (const float*)x, (float*)y, (const float*)act, n)
+                 : launch_pdl(xielu_rows_kernel<bf16>, dim3((unsigned)blocks), dim3(256), (size_t)0, stream, (const bf16*)x, (bf16*)y, (const float*)act, n));
   PG_LAUNCH_CHECK();
   return PG_OK;
 }
@@ -731,12 +767,13 @@ extern "C" int pg_gemm_simt(const void* x, const void* w, int x_f32, void* y, in
 }
 
 extern "C" int pg_head_gemm_simt(const void* x, long long ldx, long long x_head, const void* w, void* y, long long ldy, long long y_head, const void* gate, long long ldg, long long g_head, int heads,
-                                 int rows, int M, int K, int is_f32, cudaStream_t stream) {
+                                 int rows, int M, int K, int y_f32, int is_f32, cudaStream_t stream) {
   PG_REQUIRE(heads > 0 && rows > 0 && M > 0 && K > 0, "head_gemm_simt: empty problem");
   const dim3 grid((M + 63) / 64, (rows + 63) / 64, heads);
   PG_REQUIRE(grid.y <= 65535u && grid.z <= 65535u, "head_gemm_simt: %d rows of %d heads", rows, heads);
-#define PG_HG(T) launch_pdl(head_gemm_simt_kernel<T>, grid, dim3(256), (size_t)0, stream, (const T*)x, ldx, x_head, (const T*)w, (T*)y, ldy, y_head, (const T*)gate, ldg, g_head, rows, M, K)
-  PG_CUDA(is_f32 ? PG_HG(float) : PG_HG(bf16));
+#define PG_HG(T, TY) launch_pdl(head_gemm_simt_kernel<T, TY>, grid, dim3(256), (size_t)0, stream, (const T*)x, ldx, x_head, (const T*)w, (TY*)y, ldy, y_head, (const T*)gate, ldg, g_head, rows, M, K)
+  PG_REQUIRE(y_f32 || !is_f32, "head_gemm_simt: f32 operands give f32");
+  PG_CUDA(is_f32 ? PG_HG(float, float) : y_f32 ? PG_HG(bf16, float) : PG_HG(bf16, bf16));
 #undef PG_HG
   PG_LAUNCH_CHECK();
   return PG_OK;
@@ -755,13 +792,14 @@ extern "C" int pg_expert_gemm_simt(const void* x, long long ldx, const void* sor
   return PG_OK;
 }
 
-extern "C" int pg_conv_silu(const void* x, long long ldx, const void* w, void* state, void* out, long long ldo, const void* q_indptr, const void* slots, int num_seqs, int channels, int taps, long long slot_stride,
-                            int max_q_len, int is_f32, cudaStream_t stream) {
-  PG_REQUIRE(taps >= 1 && taps <= CONV_MAX, "conv_silu: %d taps (1..%d)", taps, CONV_MAX);
+// bias, in_bias: f32 [channels] or null; silu: the activation of the sum.
+extern "C" int pg_short_conv(const void* x, long long ldx, const void* w, const void* bias, const void* in_bias, void* state, void* out, long long ldo, const void* q_indptr, const void* slots, int num_seqs, int channels,
+                             int taps, long long slot_stride, int max_q_len, int silu, int is_f32, cudaStream_t stream) {
+  PG_REQUIRE(taps >= 1 && taps <= CONV_MAX, "short_conv: %d taps (1..%d)", taps, CONV_MAX);
   if (num_seqs == 0) return PG_OK;
   const dim3 grid((channels + 127) / 128, (max_q_len + CONV_TILE - 1) / CONV_TILE, num_seqs);
-  PG_REQUIRE(grid.y <= 65535u && grid.z <= 65535u, "conv_silu: %d sequences of %d rows", num_seqs, max_q_len);
-#define PG_CONV(T, CM) launch_pdl(conv_silu_kernel<T, CM>, grid, dim3(128), (size_t)0, stream, (const T*)x, ldx, (const float*)w, (T*)state, (T*)out, ldo, (const int*)q_indptr, (const int*)slots, channels, taps, slot_stride)
+  PG_REQUIRE(grid.y <= 65535u && grid.z <= 65535u, "short_conv: %d sequences of %d rows", num_seqs, max_q_len);
+#define PG_CONV(T, CM) launch_pdl(short_conv_kernel<T, CM>, grid, dim3(128), (size_t)0, stream, (const T*)x, ldx, (const float*)w, (const float*)bias, (const float*)in_bias, (T*)state, (T*)out, ldo, (const int*)q_indptr, (const int*)slots, channels, taps, slot_stride, silu)
 #define PG_CONVS(T) (taps <= 2 ? PG_CONV(T, 2) : taps <= 4 ? PG_CONV(T, 4) : taps <= 8 ? PG_CONV(T, 8) : PG_CONV(T, 16))
   PG_CUDA(is_f32 ? PG_CONVS(float) : PG_CONVS(bf16));
 #undef PG_CONVS

@@ -112,7 +112,7 @@ class SsdPart:
 class Feed:
     up: torch.Tensor
     down: torch.Tensor
-    act: torch.Tensor
+    act: torch.Tensor  # the activation's two constants as it uses them
 
 
 @dataclass
@@ -190,7 +190,8 @@ class NonetarModel(HybridLayers):
         if spec.ff:
             pad = pad8(spec.ff) - spec.ff  # zero rows: their activations are zero
             up, down = src.get(p + "mlp.up", dev, self.dtype), src.get(p + "mlp.down", dev, self.dtype)
-            L.ff = Feed(torch.nn.functional.pad(up, (0, 0, 0, pad)).contiguous(), torch.nn.functional.pad(down, (0, pad)).contiguous(), vec("mlp.act"))
+            L.ff = Feed(torch.nn.functional.pad(up, (0, 0, 0, pad)).contiguous(), torch.nn.functional.pad(down, (0, pad)).contiguous(),
+                        torch.nn.functional.softplus(vec("mlp.act")) + torch.tensor([0.0, 0.5], device=dev))
             L.norm2 = 1 + vec("norm2")
         return L
 

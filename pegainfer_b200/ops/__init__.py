@@ -137,7 +137,7 @@ def logprobs_topk(logits, picked, k):
 # Load-time and test helpers that are plain tensor arithmetic on whatever device their inputs
 # live on (quantisers, repackers, RoPE tables, the dense-attention oracle): these have no kernel.
 _HOST_UTILS = frozenset(
-    ("rope_tables", "pair_rope_tables", "temperature_table", "position_tables", "xielu", "dense_causal_attention", "filtered_probs", "dequant_int4_g32", "quant_int4_g32", "repack_int4_pairs", "unrepack_int4_pairs", "plain_int4", "dequant_fp8_block", "quant_fp8_block", "dequant_mxfp4", "quant_mxfp4")
+    ("rope_tables", "pair_rope_tables", "temperature_table", "position_tables", "dense_causal_attention", "filtered_probs", "dequant_int4_g32", "quant_int4_g32", "repack_int4_pairs", "unrepack_int4_pairs", "plain_int4", "dequant_fp8_block", "quant_fp8_block", "dequant_mxfp4", "quant_mxfp4")
 )
 
 

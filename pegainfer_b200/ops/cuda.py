@@ -15,7 +15,7 @@ from typing import Optional
 import torch
 
 from .. import _native
-from .reference import AttnMeta
+from .reference import POSITION_FINE, AttnMeta, StreamMix
 
 _c = ctypes
 _vp = ctypes.c_void_p
@@ -875,6 +875,36 @@ def embed_stream(ids, table, act_dtype):
     return x, xt
 
 
+def embed_positions(ids, table, tables, meta: AttnMeta):
+    """f32 rows of the table plus the sinusoids of their positions (``reference.embed_positions``)."""
+    coarse, fine = tables
+    ids = ids.to(torch.int32).contiguous()
+    t, width = ids.numel(), table.shape[1]
+    assert table.stride(1) == 1 and coarse.dtype == fine.dtype == torch.float32 and coarse.is_contiguous() and fine.is_contiguous() and coarse.shape[1:] == fine.shape[1:] == ((width + 1) // 2, 2) and fine.shape[0] == POSITION_FINE
+    x = torch.empty((t, width), dtype=torch.float32, device=table.device)
+    c = ctx(table.device)
+    _check(lib().pg_embed_positions(_ptr(table), _ci(_is_f32(table)), _ll(table.stride(0)), _ptr(coarse), _ci(coarse.shape[0]), _ptr(fine), _ptr(ids), _ptr(meta.positions), _ptr(x), _ci(t), _ci(width),
+                                    _ll(table.shape[0]), _ptr(c.status), _stream()), c)
+    return x
+
+
+def streams_norm(x, y, m: StreamMix, w, eps: float, act_dtype, shift=None, carried=None, meta: Optional[AttnMeta] = None, keep: bool = True):
+    """One pass between two sublayers over the copies of the stream: new copies, next input, its norm, token shift
+    (``reference.streams_norm``)."""
+    t, s_in, width = x.shape
+    s_out = m.out.shape[0]
+    assert x.dtype == w.dtype == torch.float32 and x.is_contiguous() and m.mix.shape == (s_in, s_out) and m.packed.numel() == s_in * s_out + s_out + s_in + 1 and w.numel() == width
+    assert y is None or (y.shape == (t, width) and y.stride(1) == 1)
+    assert shift is None or (shift.dtype == carried.dtype == torch.float32 and carried.is_contiguous() and carried[0].numel() == shift.numel() == width)
+    new = torch.empty((t, s_out, width), dtype=torch.float32, device=x.device) if keep and y is not None else None
+    h = torch.empty((t, width), dtype=act_dtype, device=x.device)
+    moved = shift is not None
+    _check(lib().pg_streams_norm(_ptr(x), _ci(s_in), _ptr(y), _ci(_is_f32(y) if y is not None else 0), _ll(y.stride(0) if y is not None else 0), _ptr(m.packed), _ptr(new), _ci(s_out), _ptr(w), _ptr(h),
+                                 _ci(int(act_dtype == torch.float32)), _ptr(shift), _ptr(carried if moved else None), _ptr(_unit_seq(meta, x.device) if moved else None),
+                                 _ptr(meta.q_indptr if moved else None), _ptr(meta.state_slots if moved else None), _ci(t), _ci(width), _cf(eps), _stream()), ctx(x.device))
+    return x if y is None else new, h
+
+
 def embed_pairs_norm(ids, table, pairs, scale: float, bigram, carried, w, eps: float, meta: AttnMeta, act_dtype):
     """Stream of scaled table rows plus token-pair rows, and its RMS norm (``reference.embed_pairs_norm``)."""
     ids = ids.to(torch.int32).contiguous()
@@ -925,14 +955,14 @@ def token_mix(h, mu, carried, meta: AttnMeta):
     return out
 
 
-def multi_dense(x, w):
-    """``y[t, i] = w[i] x[t, i]``: one batched launch, or the two-SM GEMM per matrix where it serves the problem."""
+def multi_dense(x, w, out_dtype=None):
+    """``y[t, i] = w[i] x[t, i]``: one batched launch, or the two-SM GEMM per matrix where it serves the problem (bf16 results)."""
     (t, n, k), m = x.shape, w.shape[1]
     assert w.shape == (n, m, k) and w.is_contiguous() and x.stride(2) == 1 and x.dtype == w.dtype
-    y = torch.empty((t, n, m), dtype=x.dtype, device=x.device)
+    y = torch.empty((t, n, m), dtype=out_dtype or x.dtype, device=x.device)
     if t == 0:
         return y
-    if not _is_f32(x) and k % 8 == 0 and x.stride(0) % 8 == 0 and x.stride(1) % 8 == 0 and not _BATCH_INVARIANT and m % 8 == 0 and lib().pg_gemm2sm_eligible(_ci(t), _ci(m), _ci(k)):
+    if not _is_f32(y) and k % 8 == 0 and x.stride(0) % 8 == 0 and x.stride(1) % 8 == 0 and not _BATCH_INVARIANT and m % 8 == 0 and lib().pg_gemm2sm_eligible(_ci(t), _ci(m), _ci(k)):
         for i in range(n):
             linear(x[:, i], w[i], out=y[:, i])
         return y
@@ -994,13 +1024,13 @@ def stream_layer_norm(x, w, eps: float, act_dtype):
     return _add_layer_norm(x, None, None, None, w, eps, act_dtype)
 
 
-def gated_row_norm(x, gate, w, eps: float, act: str = "sigmoid"):
+def gated_row_norm(x, gate, w, eps: float, act: str = "sigmoid", gate_first: bool = False):
     """``rms_norm(x) * w * act(gate)`` over the last axis of ``x`` [T, H, D]; ``gate`` [T, H * D], unit column stride; ``w`` [D]
-    or [H * D]; ``act``: sigmoid or silu."""
+    or [H * D]; ``act``: sigmoid or silu; ``gate_first``: ``rms_norm(x * act(gate)) * w``."""
     t, h, d = x.shape
     assert x.is_contiguous() and gate.shape == (t, h * d) and gate.stride(1) == 1 and gate.dtype == x.dtype and w.dtype == torch.float32 and w.numel() in (d, h * d) and act in ("sigmoid", "silu")
     y = torch.empty((t, h, d), dtype=x.dtype, device=x.device)
-    _check(lib().pg_gated_row_norm(_ptr(x), _ptr(gate), _ll(gate.stride(0)), _ptr(w), _ptr(y), _ci(t), _ci(h), _ci(d), _cf(eps), _ci(int(act == "silu")), _ci(int(w.numel() > d)), _ci(_is_f32(x)), _stream()),
+    _check(lib().pg_gated_row_norm(_ptr(x), _ptr(gate), _ll(gate.stride(0)), _ptr(w), _ptr(y), _ci(t), _ci(h), _ci(d), _cf(eps), _ci(int(act == "silu")), _ci(int(w.numel() > d)), _ci(int(gate_first)), _ci(_is_f32(x)), _stream()),
            ctx(x.device))
     return y
 
@@ -1044,6 +1074,24 @@ def dense_glu(x, gate_up, interleaved: bool = False, act: str = "silu"):
     return geglu(dense(x, gate_up), interleaved) if gelu else swiglu(dense(x, gate_up), interleaved)
 
 
+def dense_xielu(x, w, act):
+    """``xielu(x @ w.T)`` with the constants ``act`` f32 [2], in the GEMM's epilogue for bf16 rows that TMA can address."""
+    t, k = x.shape
+    m = w.shape[0]
+    assert x.stride(1) == 1 and w.stride(1) == 1 and x.dtype == w.dtype and act.dtype == torch.float32 and act.numel() == 2
+    c = ctx(x.device)
+    if not _is_f32(x) and k % 8 == 0 and x.stride(0) % 8 == 0 and x.data_ptr() % 16 == 0 and w.stride(0) % 8 == 0:
+        y = torch.empty((t, m), dtype=x.dtype, device=x.device)
+        GemmTrace.arm(f"xielu {t}x{m}x{k}")
+        _check(lib().pg_gemm_bf16_tn_xielu(_ptr(x), _ptr(w), _ptr(y), _ci(t), _ci(m), _ci(k), _ll(x.stride(0)), _ll(w.stride(0)), _ll(y.stride(0)), _ptr(act), _ptr(c.gemm_ws), _ll(c.gemm_ws.numel()),
+                                           _ptr(c.gemm_counters), _ll(c.gemm_counters.numel() * 4), _ptr(c.status), _ci(1 if _BATCH_INVARIANT else 0), _stream()), c)
+        return y
+    z = dense(x, w)
+    y = torch.empty_like(z)
+    _check(lib().pg_xielu_rows(_ptr(z), _ptr(y), _ptr(act), _ll(z.numel()), _ci(_is_f32(z)), _stream()), c)
+    return y
+
+
 def softcap_rows(logits, cap: float):
     """``cap * tanh(logits / cap)`` on f32 logits."""
     assert logits.dtype == torch.float32
@@ -1068,47 +1116,53 @@ def row_norm_rope_append(q, k, v, q_norm_w, k_norm_w, cos, sin, meta: AttnMeta, 
     return out
 
 
-def head_norm_append(q, k, v, q_norm_w, k_norm_w, temp, meta: AttnMeta, kv_layer, heads: int, kv_heads: int, dim: int, vdim: int, eps: float):
-    """Per-head query and key norms, query temperature and paged append (``reference.head_norm_append``)."""
+def head_norm_append(q, k, v, q_norm_w, k_norm_w, temp, meta: AttnMeta, kv_layer, heads: int, kv_heads: int, dim: int, vdim: int, eps: float, bias=None):
+    """Biases, per-head query and key norms, query temperature and paged append (``reference.head_norm_append``)."""
     t = q.shape[0]
     ld = _same_rows(q, k, v)
     assert q.stride(1) == k.stride(1) == v.stride(1) == 1 and q.dtype == k.dtype == v.dtype == kv_layer.dtype and q_norm_w.dtype == k_norm_w.dtype == torch.float32
     assert q.shape[1] == heads * dim and k.shape[1] == kv_heads * dim and v.shape[1] == kv_heads * vdim and kv_layer.is_contiguous() and kv_layer.shape[1] == meta.page_size * kv_heads * (dim + vdim)
     assert temp is None or (temp.dtype == torch.float32 and temp.is_contiguous())
+    assert q_norm_w.is_contiguous() and q_norm_w.numel() in (dim, heads * dim) and k_norm_w.numel() == dim
+    qb, kb, vb = bias or (None, None, None)
+    assert bias is None or (all(b.dtype == torch.float32 and b.is_contiguous() for b in bias) and (qb.numel(), kb.numel(), vb.numel()) == (heads * dim, kv_heads * dim, kv_heads * vdim))
     out = torch.empty((t, heads, dim), dtype=q.dtype, device=q.device)
     c = ctx(q.device)
-    _check(lib().pg_head_norm_append(_ptr(q), _ptr(k), _ptr(v), _ll(ld), _ptr(q_norm_w), _ptr(k_norm_w), _ptr(temp), _ci(temp.shape[0] if temp is not None else 0), _ptr(meta.positions),
+    _check(lib().pg_head_norm_append(_ptr(q), _ptr(k), _ptr(v), _ll(ld), _ptr(q_norm_w), _ci(int(q_norm_w.numel() > dim)), _ptr(k_norm_w), _ptr(qb), _ptr(kb), _ptr(vb), _ptr(temp), _ci(temp.shape[0] if temp is not None else 0), _ptr(meta.positions),
                                      _ptr(meta.slot_mapping), _ptr(out), _ptr(kv_layer), _ci(t), _ci(heads), _ci(kv_heads), _ci(dim), _ci(vdim), _ci(meta.page_size), _ll(kv_layer.shape[0]), _cf(eps),
                                      _ci(_is_f32(q)), _ptr(c.status), _stream()), c)
     return out
 
 
-def capped_attention(q, kv_layer, kv_heads: int, vdim: int, meta: AttnMeta, scale: float, softcap: float = 0.0, gate=None):
-    """Causal attention over the paged cache with its own value size, an optional soft cap on the scores and an optional
-    sigmoid gate per (token, head).  Head sizes that are multiples of 8 up to 256 run on tensor-core kernels (split-KV
+def capped_attention(q, kv_layer, kv_heads: int, vdim: int, meta: AttnMeta, scale: float, softcap: float = 0.0, gate=None, window: int = 0, slopes=None, out_scale: float = 1.0, out=None):
+    """Causal attention over the paged cache with its own value size, an optional soft cap on the scores, an optional
+    sigmoid gate per (token, head), a sliding window and a bias on the distance (``reference.capped_attention``).  Head sizes that are multiples of 8 up to 256 run on tensor-core kernels (split-KV
     decode, tiled prefill), others and f32 on the CUDA-core kernel."""
     t, hq, dim = q.shape
     f32 = _is_f32(q)
     assert q.is_contiguous() and kv_layer.is_contiguous() and kv_layer.dtype == q.dtype and (gate is None or (gate.dtype == q.dtype and gate.stride(1) == 1))
-    out = torch.empty((t, hq * vdim), dtype=q.dtype, device=q.device)
+    if out is None:
+        out = torch.empty((t, hq * vdim), dtype=q.dtype, device=q.device)
+    assert out.shape == (t, hq * vdim) and out.stride(1) == 1 and out.dtype == q.dtype and (slopes is None or (slopes.dtype == torch.float32 and slopes.numel() == hq))
     c = ctx(q.device)
     ps, pages, table = meta.page_size, kv_layer.shape[0], meta.block_table
+    extra = (_ci(window), _ptr(slopes), _cf(out_scale), _ll(out.stride(0) if t > 1 else max(out.stride(0), hq * vdim)))
     assert kv_layer.shape[1] == ps * kv_heads * (dim + vdim)
     gate_args = (_ptr(gate), _ll(gate.stride(0) if gate is not None else 0))
-    if f32 or dim % 8 or vdim % 8 or max(dim, vdim) > 256 or ps not in (16, 32, 64):
+    if f32 or dim % 8 or vdim % 8 or max(dim, vdim) > 256 or ps not in (16, 32, 64) or out.stride(0) % 2 or out.data_ptr() % 16:
         _check(lib().pg_attention_plain(_ptr(q), _ptr(kv_layer), _ptr(out), _ptr(meta.q_indptr), _ptr(meta.kv_lens), _ptr(table), _ci(table.stride(0)), _ci(t), _ci(meta.num_seqs), _ci(hq), _ci(kv_heads),
-                                        _ci(dim), _ci(vdim), _ci(ps), _ll(pages), _cf(scale), _cf(softcap), *gate_args, _ci(f32), _stream()), c)
+                                        _ci(dim), _ci(vdim), _ci(ps), _ll(pages), _cf(scale), _cf(softcap), *gate_args, *extra, _ci(f32), _stream()), c)
         return out
 
     def run(first: int, n: int, mode: int, splits: int = 1, q_tiles: int = 0):
         lse_off = n * hq * splits * vdim * 4
         rc = lib().pg_attention_capped(_ptr(q), _ptr(kv_layer), _ptr(out), _ptr(meta.q_indptr[first:]), _ptr(meta.kv_lens[first:]), _ptr(table[first:]), _ci(table.stride(0)), _ci(n), _ci(hq),
-                                       _ci(kv_heads), _ci(dim), _ci(vdim), _ci(ps), _ll(pages), _cf(scale), _cf(softcap), *gate_args, _ci(mode), _ci(splits), _ptr(c.attn_part),
+                                       _ci(kv_heads), _ci(dim), _ci(vdim), _ci(ps), _ll(pages), _cf(scale), _cf(softcap), *gate_args, *extra, _ci(mode), _ci(splits), _ptr(c.attn_part),
                                        _ptr(c.attn_part[lse_off:]), _ci(q_tiles), _ptr(c.status), _stream())
         _check(rc, c, 2 if splits > 1 else 1)
 
     def decode_rows(first: int, n: int, plan=None):
-        splits = plan if isinstance(plan, int) else plan_decode_splits(n, kv_heads * ((hq // kv_heads + 7) // 8), meta.max_kv_len, q.device)
+        splits = plan if isinstance(plan, int) else plan_decode_splits(n, kv_heads * ((hq // kv_heads + 7) // 8), min(meta.max_kv_len, window) if window else meta.max_kv_len, q.device)
         need = n * hq * splits * (vdim + 1) * 4
         if need > c.attn_part.numel():
             splits = max(1, c.attn_part.numel() // (n * hq * (vdim + 1) * 4))
@@ -1123,7 +1177,7 @@ def capped_attention(q, kv_layer, kv_heads: int, vdim: int, meta: AttnMeta, scal
         n_pf -= 1
     if meta.num_seqs - n_pf < (1 if _BATCH_INVARIANT else _MIXED_DECODE_MIN):
         n_pf = meta.num_seqs
-    if (n_pf > 0 and dim == vdim == 128 and _PREFILL_TC and not _BATCH_INVARIANT and max(qi[b + 1] - qi[b] for b in range(n_pf)) >= _PREFILL_TC_MIN_ROWS
+    if (n_pf > 0 and dim == vdim == 128 and not window and slopes is None and out_scale == 1.0 and out.is_contiguous() and _PREFILL_TC and not _BATCH_INVARIANT and max(qi[b + 1] - qi[b] for b in range(n_pf)) >= _PREFILL_TC_MIN_ROWS
             and (meta.h_kv_lens is None or max(meta.h_kv_lens[:n_pf]) >= _PREFILL_TC_MIN_KV)):
         PREFILL_TC_CALLS["hd128"] += 1
         tiles = _ci(sum((qi[b + 1] - qi[b] + 255) // 256 for b in range(n_pf)))
@@ -1142,12 +1196,18 @@ def capped_attention(q, kv_layer, kv_heads: int, vdim: int, meta: AttnMeta, scal
 
 def conv_silu(x, conv_w, conv_state, meta: AttnMeta):
     """Causal depthwise convolution of up to 16 taps + SiLU with carried inputs; ``conv_w`` f32 [C, taps]."""
+    return short_conv(x, conv_w, None, conv_state, meta)
+
+
+def short_conv(x, conv_w, bias, conv_state, meta: AttnMeta, act: str = "silu", in_bias=None):
+    """Causal depthwise convolution of up to 16 taps with carried inputs, biases and SiLU as asked (``reference.short_conv``)."""
     t, ch = x.shape
     taps = conv_w.shape[1]
     assert x.stride(1) == 1 and conv_w.is_contiguous() and conv_w.dtype == torch.float32 and conv_state.is_contiguous() and conv_state.dtype == x.dtype
     out = torch.empty((t, ch), dtype=x.dtype, device=x.device)
-    _check(lib().pg_conv_silu(_ptr(x), _ll(x.stride(0)), _ptr(conv_w), _ptr(conv_state), _ptr(out), _ll(out.stride(0)), _ptr(meta.q_indptr), _ptr(meta.state_slots), _ci(meta.num_seqs), _ci(ch), _ci(taps),
-                              _ll(conv_state.stride(0)), _ci(max(int(meta.max_q_len), 1)), _ci(_is_f32(x)), _stream()), ctx(x.device))
+    assert act in ("silu", "none") and all(b is None or (b.dtype == torch.float32 and b.is_contiguous() and b.numel() == ch) for b in (bias, in_bias))
+    _check(lib().pg_short_conv(_ptr(x), _ll(x.stride(0)), _ptr(conv_w), _ptr(bias), _ptr(in_bias), _ptr(conv_state), _ptr(out), _ll(out.stride(0)), _ptr(meta.q_indptr), _ptr(meta.state_slots),
+                               _ci(meta.num_seqs), _ci(ch), _ci(taps), _ll(conv_state.stride(0)), _ci(max(int(meta.max_q_len), 1)), _ci(int(act == "silu")), _ci(_is_f32(x)), _stream()), ctx(x.device))
     return out
 
 
@@ -1222,6 +1282,40 @@ def wkv_attention(r, k, v, f, w0, u, state, meta: AttnMeta, blocks: Optional[boo
         _check(lib().pg_wkv_block(*args, _ci(_WKV_BLOCK_MIN), _stream()), c)
     if not blocks or _has_short_rows(meta, _WKV_BLOCK_MIN):
         _check(lib().pg_wkv_recurrent(*args, _ci(int(meta.max_q_len)), _ci(_WKV_BLOCK_MIN if blocks else 0), _ci(f32), _stream()), c)
+    return out
+
+
+def ssd_attention(x, B, C, dt, dt_bias, a_log, D, state, meta: AttnMeta, chunked: Optional[bool] = None):
+    """State-space duality (``reference.ssd_attention``); ``x, B, C`` share a row stride.  Sequences of 32 tokens or more run on
+    the chunk-wise tensor-core kernel (bf16, sizes that are multiples of 8), shorter ones on the recurrence."""
+    t, h, dv = x.shape
+    g, n = B.shape[1:]
+    assert B.shape == C.shape and x.stride(2) == B.stride(2) == C.stride(2) == 1 and x.stride(1) == dv and B.stride(1) == C.stride(1) == n and dt.shape == (t, h) and dt.stride(1) == 1 and dt.dtype == x.dtype
+    assert state.is_contiguous() and state.shape[1:] == (h, n, dv) and all(z.dtype == torch.float32 and z.is_contiguous() for z in (state, dt_bias, a_log, D))
+    out = torch.empty((t, h, dv), dtype=x.dtype, device=x.device)
+    f32, ld, c = _is_f32(x), _same_rows(x, B, C), ctx(x.device)
+    args = (_ptr(C), _ptr(B), _ptr(x), _ll(ld), _ptr(dt), _ll(dt.stride(0)), _ptr(a_log), _ptr(dt_bias), _ptr(D), _ptr(state), _ptr(out), _ptr(meta.q_indptr), _ptr(meta.state_slots), _ci(meta.num_seqs),
+            _ci(h), _ci(g), _ci(n), _ci(dv))
+    aligned = n % 8 == 0 and dv % 8 == 0 and n <= 128 and ld % 8 == 0 and all(z.data_ptr() % 16 == 0 for z in (x, B, C))
+    chunked = (_LINEAR_CHUNKED if chunked is None else chunked) and int(meta.max_q_len) >= _GDN_CHUNK_MIN and not f32 and aligned
+    if chunked:
+        _check(lib().pg_ssd_chunked(*args, _ci(_GDN_CHUNK_MIN), _stream()), c)
+    if not chunked or _has_short_rows(meta, _GDN_CHUNK_MIN):
+        _check(lib().pg_ssd_recurrent(*args, _ci(int(meta.max_q_len)), _ci(_GDN_CHUNK_MIN if chunked else 0), _ci(f32), _stream()), c)
+    return out
+
+
+def gated_lru(gates, gate_bias, u, lam, y, y_bias, state, meta: AttnMeta, scale: float = 1.0, out=None):
+    """Real-gated linear recurrence per channel times its GELU branch (``reference.gated_lru``)."""
+    t, w = u.shape
+    blocks = gates.shape[1]
+    if out is None:
+        out = torch.empty((t, w), dtype=u.dtype, device=u.device)
+    assert gates.dtype == torch.float32 and gates.is_contiguous() and gates.shape == (t, blocks, 2 * (w // blocks)) and gate_bias.is_contiguous() and gate_bias.numel() == 2 * w
+    assert u.dtype == y.dtype == out.dtype and u.shape == y.shape == out.shape and u.stride(1) == y.stride(1) == out.stride(1) == 1 and lam.numel() == y_bias.numel() == w
+    assert state.is_contiguous() and state[0].numel() == w and gate_bias.dtype == lam.dtype == y_bias.dtype == state.dtype == torch.float32
+    _check(lib().pg_gated_lru(_ptr(gates), _ptr(gate_bias), _ptr(u), _ll(u.stride(0)), _ptr(lam), _ptr(y), _ll(y.stride(0)), _ptr(y_bias), _ptr(state), _ptr(out), _ll(out.stride(0)), _ptr(meta.q_indptr),
+                              _ptr(meta.state_slots), _ci(meta.num_seqs), _ci(w), _ci(blocks), _cf(scale), _ci(int(meta.max_q_len)), _ci(_is_f32(u)), _stream()), ctx(u.device))
     return out
 
 
@@ -1609,14 +1703,15 @@ def _head_gemm(x, x_tok: int, x_head: int, w, y, gate=None):
     rows, heads, m = y.shape
     k = w.shape[2]
     c = ctx(y.device)
-    args = (_ptr(x), _ll(x_tok), _ll(x_head), _ptr(w), _ptr(y), _ll(heads * m), _ll(m), _ptr(gate), _ll(gate.stride(0) if gate is not None else 0), _ll(m), _ci(heads), _ci(rows), _ci(m), _ci(k))
-    if y.dtype == torch.bfloat16 and k % 8 == 0 and x_tok % 8 == 0 and x_head % 8 == 0 and x.data_ptr() % 16 == 0 and heads <= 512:
+    front, rest = (_ptr(x), _ll(x_tok), _ll(x_head), _ptr(w), _ptr(y)), (_ll(heads * m), _ll(m), _ptr(gate), _ll(gate.stride(0) if gate is not None else 0), _ll(m), _ci(heads), _ci(rows), _ci(m), _ci(k))
+    y_f32 = _ci(int(y.dtype == torch.float32))
+    if w.dtype == torch.bfloat16 and k % 8 == 0 and x_tok % 8 == 0 and x_head % 8 == 0 and x.data_ptr() % 16 == 0 and heads <= 512:
         bn, tiles = _token_tile(heads * rows, heads), heads * ((m + 127) // 128)
         while bn > 16 and tiles * ((rows + bn - 1) // bn) < c.sms:  # narrower token tiles until every SM has one (a head's weights come from L2 again)
             bn //= 2
-        _check(lib().pg_head_gemm(*args, _ci(bn), _ptr(c.status), _stream()), c)
+        _check(lib().pg_head_gemm(*front, y_f32, *rest, _ci(bn), _ptr(c.status), _stream()), c)
     else:
-        _check(lib().pg_head_gemm_simt(*args, _ci(_is_f32(y)), _stream()), c)
+        _check(lib().pg_head_gemm_simt(*front, *rest, y_f32, _ci(_is_f32(w)), _stream()), c)
 
 
 def _latent_key_plan(meta: AttnMeta, n: int, window: int, device):

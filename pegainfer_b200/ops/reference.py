@@ -272,15 +272,11 @@ def dense_glu(x, gate_up, interleaved: bool = False, act: str = "silu"):
     return swiglu(y, interleaved)
 
 
-def xielu(z, p, q):
-    """``softplus(p) z^2 + z / 2`` above zero, ``(1/2 + softplus(q)) (e^z - 1 - z) + z / 2`` below, in f32."""
-    z = z.float()
-    return torch.where(z > 0, F.softplus(p.float()) * z * z, (0.5 + F.softplus(q.float())) * (torch.expm1(z.clamp(max=0)) - z)) + 0.5 * z
-
-
 def dense_xielu(x, w, act):
-    """``xielu(x @ w.T, *act)`` with ``act`` f32 [2]."""
-    return xielu(x.float() @ w.float().t(), act[0], act[1]).to(x.dtype)
+    """xIELU of ``z = x @ w.T`` in f32: ``act[0] z^2 + z / 2`` above zero, ``act[1] (e^z - 1 - z) + z / 2`` below; ``act`` f32 [2] holds
+    the layer's constants in the form softplus(p), 1/2 + softplus(q)."""
+    z = x.float() @ w.float().t()
+    return (torch.where(z > 0, act[0] * z * z, act[1] * (torch.expm1(z.clamp(max=0)) - z)) + 0.5 * z).to(x.dtype)
 
 
 def softcap_rows(logits, cap: float):
