@@ -94,9 +94,9 @@ int pg_prefill_attention_tc(const void* q, const void* kv_layer, void* out, cons
                             int num_seqs, int tokens, int hq, int hkv, int dim, int page_size, long long num_pages, float scale, int q_tiles, void* status,
                             cudaStream_t stream);
 void pg_prefill_attention_tc_variant(int v);
-int pg_prefill_attention_tc_capped(const void* q, const void* kv_layer, void* out, const void* q_indptr, const void* kv_lens, const void* table, int table_stride, int num_seqs, int tokens,
-                                   int hq, int hkv, int page_size, long long num_pages, float scale, float softcap, const void* gate, long long ld_gate, int q_tiles, void* status,
-                                   cudaStream_t stream);
+int pg_prefill_attention_tc_capped(const void* q, const void* kv_layer, void* out, const void* q_indptr, const void* kv_lens, const void* table, int table_stride, int num_seqs,
+                                   int tokens, int hq, int hkv, int page_size, long long num_pages, float scale, float softcap, const void* gate, long long ld_gate, int window,
+                                   const void* slopes, float out_scale, long long ld_out, int q_tiles, void* status, cudaStream_t stream);
 
 // ---- expanded-form latent prefill on tcgen05 (mla_prefill.cu) ------------------------------
 int pg_latent_gather(const void* latent_layer, int page_size, long long num_pages, int width, const void* table, int table_stride, const void* kv_indptr, const void* starts, int num_seqs, int total_kv,

@@ -43,10 +43,13 @@ struct TcAttnParams {
   int table_stride, num_seqs, hq, hkv, page_size;
   long long num_pages;
   float scale_log2;       // softmax scale * log2(e)
-  int window;             // head dim 256 only: a row sees its last `window` keys (0: all of them)
+  int window;             // head dim 256 and the biased form: a row sees its last `window` keys (0: all of them)
   float cap_in;           // capped form: softmax scale / cap, and scale_log2 holds cap * log2(e); 0: no cap
   const bf16* gate;       // capped form: [T, >= hq] rows of stride ld_gate whose sigmoid multiplies a head's output, or null
   long long ld_gate;
+  const float* slopes;    // biased form: [hq], a (capped) score loses slope * distance; or null
+  float out_scale;        // capped and biased form, on the output
+  long long ld_out;       // row stride of out
   int mn_lbo_first;       // descriptor variant of the MN-major operand (1: LBO = stride between 64-column blocks)
   uint32_t* status;
 };
@@ -67,8 +70,10 @@ __device__ __forceinline__ float2 tanh2_poly(float2 z) {
 }
 __device__ __forceinline__ float tanh_ex2(float z) { return 1.f - __fdividef(2.f, 1.f + ex2_approx(z * 2.8853900817779268f)); }
 
-// CAPPED: soft cap on the scores and a sigmoid gate per (token, head) on the output.
-template <bool CAPPED>
+// CAPPED: soft cap on the scores and a sigmoid gate per (token, head) on the output.  BIASED: and a sliding window (key tiles in
+// front of the first row's window are skipped; tile numbers below count from j0) and a bias that grows with the distance.
+enum { FORM_PLAIN = 0, FORM_CAPPED = 1, FORM_BIASED = 2 };
+template <int FORM>
 __global__ void __launch_bounds__(THREADS, 1) prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_kv, const TcAttnParams p) {
   extern __shared__ uint8_t smem_raw[];
   const uint32_t base = smem_u32(smem_raw);
@@ -77,6 +82,7 @@ __global__ void __launch_bounds__(THREADS, 1) prefill_attn_tc_kernel(const __gri
   uint8_t* k_tile = tiles + GROUPS * TILE_BYTES;      // 2 x 32 KB
   uint8_t* v_tile = k_tile + 2 * TILE_BYTES;          // 2 x 32 KB
   TcSmem* sh = reinterpret_cast<TcSmem*>(v_tile + 2 * TILE_BYTES);
+  constexpr bool CAPPED = FORM != FORM_PLAIN, BIASED = FORM == FORM_BIASED;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   // one-dimensional grid, query tile slowest: every head's late tiles (most keys) are handed out before any early
   // tile, so the long CTAs start first on all SMs and the short ones fill the tail
@@ -132,12 +138,13 @@ __global__ void __launch_bounds__(THREADS, 1) prefill_attn_tc_kernel(const __gri
   const int row_base = tile_in_seq * BQ2;
   const int rows_here = min(BQ2, q_len - row_base);
   const int pos_base = kv_len - q_len + row_base;  // position of the CTA's first row
+  const int j0 = BIASED && p.window > 0 ? max(0, pos_base - p.window + 1) / BKV : 0;
   // tiles of 128 keys each group needs: up to its last row's position
   int n_g[GROUPS];
 #pragma unroll
   for (int g = 0; g < GROUPS; ++g) {
     const int rows_of_g = min(128, rows_here - g * 128);
-    n_g[g] = (rows_of_g > 0 && kv_len > 0) ? min(pos_base + g * 128 + rows_of_g - 1, kv_len - 1) / BKV + 1 : 0;
+    n_g[g] = (rows_of_g > 0 && kv_len > 0) ? min(pos_base + g * 128 + rows_of_g - 1, kv_len - 1) / BKV + 1 - j0 : 0;
   }
   const int n_tiles = max(n_g[0], n_g[1]);
   const int* table_row = p.table + (long long)b * p.table_stride;
@@ -161,8 +168,8 @@ __global__ void __launch_bounds__(THREADS, 1) prefill_attn_tc_kernel(const __gri
       const int per_kv = 2 * ppt, slots = 4 * ppt;
       auto page_of = [&](int j, int slot) -> int {
         const int pg = (slot % per_kv) >> 1;
-        const int pages_live = min(ppt, (kv_len - j * BKV + p.page_size - 1) / p.page_size);
-        int page = (slot < slots && pg < pages_live) ? __ldg(table_row + j * ppt + pg) : 0;  // past the end: the padding page, keys masked
+        const int pages_live = min(ppt, (kv_len - (j0 + j) * BKV + p.page_size - 1) / p.page_size);
+        int page = (slot < slots && pg < pages_live) ? __ldg(table_row + (j0 + j) * ppt + pg) : 0;  // past the end: the padding page, keys masked
         if (page < 0 || page >= p.num_pages) {
           atomicCAS(p.status, PG_ST_OK, PG_ST_BOUNDS | (41u << 8));
           page = 0;
@@ -268,6 +275,8 @@ __global__ void __launch_bounds__(THREADS, 1) prefill_attn_tc_kernel(const __gri
     const uint32_t s_row = tmem + ((uint32_t)(wq * 32) << 16) + (uint32_t)(g * 128);
     const uint32_t o_row = s_row + 256u;
     float m = -INFINITY, l = 0.f;  // m: the maximum the exponentials refer to (may lag the true maximum by up to 2^8)
+    // bias per position in units of the raw (or capped) score, which scale_log2 turns into log2
+    const float slope = BIASED && p.slopes ? p.slopes[hq] * 1.4426950408889634f / p.scale_log2 : 0.f;
     bool ok = true;
     // One key tile of this group.  MASK (a tile that the causal edge or the end of the keys crosses) is a compile-time
     // property: the plain tiles, nearly all of them, carry no compare or select per element.
@@ -275,7 +284,9 @@ __global__ void __launch_bounds__(THREADS, 1) prefill_attn_tc_kernel(const __gri
       constexpr bool MASK = decltype(mask_tag)::value;
       if (!mbar_wait(&sh->s_full[g], (uint32_t)(j & 1), abort_flag)) return false;
       tc_fence_after();
-      const int limit = min(my_pos, kv_len - 1) - j * BKV;  // columns 0 .. limit are visible to this row
+      const int key0 = (j0 + j) * BKV;
+      const int limit = min(my_pos, kv_len - 1) - key0;                                      // columns lo + 1 .. limit are visible to this row
+      const int lo = BIASED && p.window > 0 ? my_pos - p.window - key0 : -1;
       // the whole row of S goes to registers in one round trip (four loads in flight, one wait): both the maximum
       // and the exponentials work from there, and S in tensor memory may be overwritten by P right away
       uint32_t v[BKV];
@@ -303,12 +314,21 @@ __global__ void __launch_bounds__(THREADS, 1) prefill_attn_tc_kernel(const __gri
           }
         }
       }
+      if constexpr (BIASED) {
+        const float2 away = make_float2((float)(key0 - my_pos), (float)(key0 - my_pos)), sl = make_float2(slope, slope);
+#pragma unroll
+        for (int i = 0; i < BKV; i += 2) {
+          const float2 t = __ffma2_rn(__fadd2_rn(make_float2((float)i, (float)(i + 1)), away), sl, make_float2(__uint_as_float(v[i]), __uint_as_float(v[i + 1])));
+          v[i] = __float_as_uint(t.x);
+          v[i + 1] = __float_as_uint(t.y);
+        }
+      }
       float mx_raw;
       if constexpr (MASK) {
         mx_raw = -INFINITY;
 #pragma unroll
         for (int i = 0; i < BKV; ++i)
-          if (i <= limit) mx_raw = fmaxf(mx_raw, __uint_as_float(v[i]));
+          if (i <= limit && (!BIASED || i > lo)) mx_raw = fmaxf(mx_raw, __uint_as_float(v[i]));
       } else {
         // three-input maximum, four chains instead of one long one
         float m0 = max3(__uint_as_float(v[0]), __uint_as_float(v[1]), __uint_as_float(v[2]));
@@ -371,10 +391,10 @@ __global__ void __launch_bounds__(THREADS, 1) prefill_attn_tc_kernel(const __gri
           float2 e = make_float2(ex2_approx(t2.x), ex2_approx(t2.y));
           float2 f = make_float2(ex2_approx(t3.x), ex2_approx(t3.y));
           if constexpr (MASK) {
-            if (c + i > limit) e.x = 0.f;
-            if (c + i + 1 > limit) e.y = 0.f;
-            if (c + i + 2 > limit) f.x = 0.f;
-            if (c + i + 3 > limit) f.y = 0.f;
+            if (c + i > limit || (BIASED && c + i <= lo)) e.x = 0.f;
+            if (c + i + 1 > limit || (BIASED && c + i + 1 <= lo)) e.y = 0.f;
+            if (c + i + 2 > limit || (BIASED && c + i + 2 <= lo)) f.x = 0.f;
+            if (c + i + 3 > limit || (BIASED && c + i + 3 <= lo)) f.y = 0.f;
           }
           sum2 = __fadd2_rn(sum2, e);
           sum3 = __fadd2_rn(sum3, f);
@@ -393,7 +413,8 @@ __global__ void __launch_bounds__(THREADS, 1) prefill_attn_tc_kernel(const __gri
       return true;
     };
     for (int j = 0; j < my_n && ok; ++j) {
-      const bool need_mask = j * BKV + BKV - 1 > min(pos0, kv_len - 1);
+      const int key0 = (j0 + j) * BKV;
+      const bool need_mask = key0 + BKV - 1 > min(pos0, kv_len - 1) || (BIASED && p.window > 0 && key0 <= pos0 + 127 - p.window);
       ok = need_mask ? tile(j, std::true_type{}) : tile(j, std::false_type{});
     }
     const int rows_g = min(128, rows_here - g * 128);
@@ -403,9 +424,10 @@ __global__ void __launch_bounds__(THREADS, 1) prefill_attn_tc_kernel(const __gri
     }
     float inv = (ok && l > 0.f) ? 1.f / l : 0.f;
     if constexpr (CAPPED) {
+      inv *= p.out_scale;
       if (p.gate && r < rows_g) inv /= 1.f + __expf(-__bfloat162float(p.gate[(long long)(q0 + row_base + g * 128 + r) * p.ld_gate + hq]));
     }
-    bf16* dst = p.out + ((long long)(q0 + row_base + g * 128 + r) * p.hq + hq) * D;
+    bf16* dst = p.out + (CAPPED ? (q0 + row_base + g * 128 + r) * p.ld_out + hq * D : ((long long)(q0 + row_base + g * 128 + r) * p.hq + hq) * D);
 #pragma unroll
     for (int c = 0; c < D; c += 32) {
       uint32_t w[32];
@@ -675,28 +697,30 @@ extern "C" void pg_prefill_attention_tc_variant(int v) { g_mn_variant = v; }
 // q [T, hq, d] bf16 (contiguous), kv_layer [pages, 2, page_size, hkv, d], out [T, hq * d], d = 128 or 256.  `q_tiles` = sum
 // over the sequences of ceil(query rows / 256) for d = 128 and of ceil(query rows / 128) for d = 256.
 static int prefill_tc_impl(const void* q, const void* kv_layer, void* out, const void* q_indptr, const void* kv_lens, const void* table, int table_stride, int num_seqs, int tokens, int hq,
-                           int hkv, int dim, int page_size, long long num_pages, float scale, int q_tiles, int window, bool capped, float softcap, const void* gate, long long ld_gate,
-                           void* status, cudaStream_t stream);
+                           int hkv, int dim, int page_size, long long num_pages, float scale, int q_tiles, int window, int form, float softcap, const void* gate, long long ld_gate,
+                           const void* slopes, float out_scale, long long ld_out, void* status, cudaStream_t stream);
 
 extern "C" int pg_prefill_attention_tc(const void* q, const void* kv_layer, void* out, const void* q_indptr, const void* kv_lens, const void* table, int table_stride,
                                        int num_seqs, int tokens, int hq, int hkv, int dim, int page_size, long long num_pages, float scale, int q_tiles, int window,
                                        void* status, cudaStream_t stream) {
-  return prefill_tc_impl(q, kv_layer, out, q_indptr, kv_lens, table, table_stride, num_seqs, tokens, hq, hkv, dim, page_size, num_pages, scale, q_tiles, window, false, 0.f, nullptr, 0, status,
-                         stream);
+  return prefill_tc_impl(q, kv_layer, out, q_indptr, kv_lens, table, table_stride, num_seqs, tokens, hq, hkv, dim, page_size, num_pages, scale, q_tiles, window, FORM_PLAIN, 0.f, nullptr, 0,
+                         nullptr, 1.f, (long long)hq * dim, status, stream);
 }
 
-// Head dim 128 with a soft cap on the scores (softcap > 0) and a sigmoid gate per (token, head) (gate: bf16 rows or null).
+// Head dim 128 with a soft cap on the scores (softcap > 0), a sigmoid gate per (token, head) (gate: bf16 rows or null), a sliding window
+// (> 0), a bias of slope * distance (slopes: f32 [hq] or null); output rows of stride ld_out, times out_scale.
 extern "C" int pg_prefill_attention_tc_capped(const void* q, const void* kv_layer, void* out, const void* q_indptr, const void* kv_lens, const void* table, int table_stride, int num_seqs,
-                                              int tokens, int hq, int hkv, int page_size, long long num_pages, float scale, float softcap, const void* gate, long long ld_gate, int q_tiles,
-                                              void* status, cudaStream_t stream) {
-  return prefill_tc_impl(q, kv_layer, out, q_indptr, kv_lens, table, table_stride, num_seqs, tokens, hq, hkv, D, page_size, num_pages, scale, q_tiles, 0, true, softcap, gate, ld_gate, status,
-                         stream);
+                                              int tokens, int hq, int hkv, int page_size, long long num_pages, float scale, float softcap, const void* gate, long long ld_gate, int window,
+                                              const void* slopes, float out_scale, long long ld_out, int q_tiles, void* status, cudaStream_t stream) {
+  PG_REQUIRE(window >= 0 && ld_out % 8 == 0 && ((uintptr_t)out & 15) == 0, "tcgen05 prefill attention: a window of %d keys, output rows of %lld that must start on 16 bytes", window, ld_out);
+  return prefill_tc_impl(q, kv_layer, out, q_indptr, kv_lens, table, table_stride, num_seqs, tokens, hq, hkv, D, page_size, num_pages, scale, q_tiles, window,
+                         window > 0 || slopes ? FORM_BIASED : FORM_CAPPED, softcap, gate, ld_gate, slopes, out_scale, ld_out, status, stream);
 }
 
 static int prefill_tc_impl(const void* q, const void* kv_layer, void* out, const void* q_indptr, const void* kv_lens, const void* table, int table_stride, int num_seqs, int tokens, int hq,
-                           int hkv, int dim, int page_size, long long num_pages, float scale, int q_tiles, int window, bool capped, float softcap, const void* gate, long long ld_gate,
-                           void* status, cudaStream_t stream) {
-  PG_REQUIRE(window == 0 || dim == D2, "tcgen05 prefill attention: a sliding window is built for head dim 256 only");
+                           int hkv, int dim, int page_size, long long num_pages, float scale, int q_tiles, int window, int form, float softcap, const void* gate, long long ld_gate,
+                           const void* slopes, float out_scale, long long ld_out, void* status, cudaStream_t stream) {
+  PG_REQUIRE(window == 0 || dim == D2 || form == FORM_BIASED, "tcgen05 prefill attention: a sliding window is built for head dim 256 and the biased form only");
   PG_REQUIRE(dim == D || dim == D2, "tcgen05 prefill attention is built for head dims 128 and 256 (got %d)", dim);
   const int key_tile = dim == D ? BKV : BKV2;
   PG_REQUIRE(page_size >= 8 && page_size <= key_tile && key_tile % page_size == 0, "page size %d does not tile %d keys", page_size, key_tile);
@@ -724,6 +748,9 @@ static int prefill_tc_impl(const void* q, const void* kv_layer, void* out, const
   p.gate = (const bf16*)gate;
   p.ld_gate = ld_gate;
   p.window = window;
+  p.slopes = (const float*)slopes;
+  p.out_scale = out_scale;
+  p.ld_out = ld_out;
   p.mn_lbo_first = g_mn_variant < 0 ? 1 : g_mn_variant;
   p.status = (uint32_t*)status;
   if (dim == D2) {
@@ -740,11 +767,12 @@ static int prefill_tc_impl(const void* q, const void* kv_layer, void* out, const
   const size_t smem = 1024 + (GROUPS + 4) * (size_t)TILE_BYTES + sizeof(TcSmem) + 64;
   static bool attr_done = false;
   if (!attr_done) {
-    PG_CUDA(cudaFuncSetAttribute(prefill_attn_tc_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-    PG_CUDA(cudaFuncSetAttribute(prefill_attn_tc_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    PG_CUDA(cudaFuncSetAttribute(prefill_attn_tc_kernel<FORM_PLAIN>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    PG_CUDA(cudaFuncSetAttribute(prefill_attn_tc_kernel<FORM_CAPPED>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    PG_CUDA(cudaFuncSetAttribute(prefill_attn_tc_kernel<FORM_BIASED>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     attr_done = true;
   }
-  PG_CUDA(launch_pdl(capped ? prefill_attn_tc_kernel<true> : prefill_attn_tc_kernel<false>, dim3((unsigned)q_tiles * (unsigned)hq), dim3(THREADS), smem, stream, tm_q, tm_kv, p));
+  PG_CUDA(launch_pdl(form == FORM_BIASED ? prefill_attn_tc_kernel<FORM_BIASED> : form == FORM_CAPPED ? prefill_attn_tc_kernel<FORM_CAPPED> : prefill_attn_tc_kernel<FORM_PLAIN>, dim3((unsigned)q_tiles * (unsigned)hq), dim3(THREADS), smem, stream, tm_q, tm_kv, p));
   PG_LAUNCH_CHECK();
   return PG_OK;
 }

@@ -1177,16 +1177,16 @@ def capped_attention(q, kv_layer, kv_heads: int, vdim: int, meta: AttnMeta, scal
         n_pf -= 1
     if meta.num_seqs - n_pf < (1 if _BATCH_INVARIANT else _MIXED_DECODE_MIN):
         n_pf = meta.num_seqs
-    if (n_pf > 0 and dim == vdim == 128 and not window and slopes is None and out_scale == 1.0 and out.is_contiguous() and _PREFILL_TC and not _BATCH_INVARIANT and max(qi[b + 1] - qi[b] for b in range(n_pf)) >= _PREFILL_TC_MIN_ROWS
+    if (n_pf > 0 and dim == vdim == 128 and out.stride(0) % 8 == 0 and _PREFILL_TC and not _BATCH_INVARIANT and max(qi[b + 1] - qi[b] for b in range(n_pf)) >= _PREFILL_TC_MIN_ROWS
             and (meta.h_kv_lens is None or max(meta.h_kv_lens[:n_pf]) >= _PREFILL_TC_MIN_KV)):
         PREFILL_TC_CALLS["hd128"] += 1
         tiles = _ci(sum((qi[b + 1] - qi[b] + 255) // 256 for b in range(n_pf)))
-        if softcap == 0.0 and gate is None:
+        if softcap == 0.0 and gate is None and not window and slopes is None and out_scale == 1.0 and out.is_contiguous():
             _check(lib().pg_prefill_attention_tc(_ptr(q), _ptr(kv_layer), _ptr(out), _ptr(meta.q_indptr), _ptr(meta.kv_lens), _ptr(table), _ci(table.stride(0)), _ci(n_pf), _ci(qi[n_pf]), _ci(hq), _ci(kv_heads),
                                                  _ci(dim), _ci(ps), _ll(pages), _cf(scale), tiles, _ci(0), _ptr(c.status), _stream()), c)
         else:
             _check(lib().pg_prefill_attention_tc_capped(_ptr(q), _ptr(kv_layer), _ptr(out), _ptr(meta.q_indptr), _ptr(meta.kv_lens), _ptr(table), _ci(table.stride(0)), _ci(n_pf), _ci(qi[n_pf]), _ci(hq),
-                                                  _ci(kv_heads), _ci(ps), _ll(pages), _cf(scale), _cf(softcap), *gate_args, tiles, _ptr(c.status), _stream()), c)
+                                                  _ci(kv_heads), _ci(ps), _ll(pages), _cf(scale), _cf(softcap), *gate_args, *extra, tiles, _ptr(c.status), _stream()), c)
     elif n_pf > 0:
         run(0, n_pf, 1, 1, sum((qi[b + 1] - qi[b] + 63) // 64 for b in range(n_pf)))
     if n_pf < meta.num_seqs:
