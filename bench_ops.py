@@ -6,7 +6,7 @@ distinct weight / KV buffers (larger than L2 in total, so every launch streams f
 HBM), replayed after warm-up and timed with CUDA events.  Fractions are against the
 measured peaks in MEASURED_PEAKS.json (copy bandwidth, cuBLAS bf16 throughput).
 
-    python bench_ops.py [--only gemm|attn|small|gdn|kda|nemipel|vekalorn|zeripel|moe|mla] [--iters 16] [--json out.json]
+    python bench_ops.py [--only gemm|attn|small|gdn|kda|nemipel|vekalorn|zeripel|nonetar|moe|mla] [--iters 16] [--json out.json]
     python bench_ops.py --single gemm:64x4096x4096      # one op, few launches (ncu target)
 
 Plays the role of the reference's kernel/op report binaries
@@ -337,6 +337,96 @@ def vekalorn_cases(iters):
         by = t * (qr + c + r) * 4
         pair(f"latent_rows {t} ({qr}, {c} + {r})", "rms_norm + mla_append", lambda i: K.latent_rows(z[i][:, :qr], z[i][:, qr:], qw, kw, cos, sin, meta, cache, c, 1e-5),
              lambda i: (K.rms_norm(z[i][:, :qr], qw16, 1e-5), K.mla_append(z[i][:, qr:], kw16, c16, s16, meta, old, c, 1e-5)), by, by, 0, 0, 4, iters)
+    return rows
+
+
+def nonetar_cases(iters):
+    """Kernels of the Nonetar line, each beside the like kernel of the closest line at the same size (indented rows): the copies'
+    row kernel beside the norms of one stream, windowed and biased attention beside the Nemipel line's capped one (over the
+    window's keys in decoding, over all keys with the FLOPs of all in prompts), the gated recurrence beside the convolution that
+    streams the same channels, state-space duality beside lightning attention of the same state."""
+    from pegainfer_b200.config import alibi_slopes
+    from pegainfer_b200.ops import cuda as K
+    from pegainfer_b200.ops.reference import StreamMix, position_tables
+
+    rows, page, hkv, d = [], 16, 8, 128
+    few = max(2, iters // 4)
+    bf = lambda *s: torch.randn(*s, device=DEV).bfloat16()
+    f32 = lambda *s: torch.randn(*s, device=DEV)
+
+    def pair(name, like, new, old, by, by_old, fl, fl_old, nvar, it):
+        rows.append((name, time_graph(new, nvar, it), by, fl))
+        rows.append(("  " + like, time_graph(old, nvar, it), by_old, fl_old))
+
+    def step(lens, ctx=None):
+        meta, pages = _meta_for(lens, ctx or lens, page)
+        meta.state_slots = torch.arange(len(lens), dtype=torch.int32, device=DEV)
+        return meta, pages
+
+    for hq, bs, ctx, window in ((32, 64, 1152, 2048), (32, 64, 4096, 1024), (32, 64, 4096, 4096), (40, 8, 16384, 4096), (32, 1, 8192, 2048)):
+        sl, n = torch.tensor(alibi_slopes(hq), device=DEV), min(ctx, window)
+        meta, pages = step([1] * bs, [ctx] * bs)
+        meta_old, pages_old = step([1] * bs, [n] * bs)
+        kv, old, q = [bf(pages, 2 * page * hkv * d) for _ in range(2)], [bf(pages_old, 2 * page * hkv * d) for _ in range(2)], bf(bs, hq, d)
+        by, fl = bs * n * 2 * hkv * d * 2, 4.0 * bs * n * hq * d
+        pair(f"capped_attention decode {hq}h {bs}x{ctx} window {window}, slopes", f"capped_attention {bs}x{n}", lambda i: K.capped_attention(q, kv[i], hkv, d, meta, d ** -0.5, 50.0, window=window, slopes=sl),
+             lambda i: K.capped_attention(q, old[i], hkv, d, meta_old, d ** -0.5, 50.0), by, by, fl, fl, 2, iters)
+    for hq, ns, ql, window in ((32, 1, 4096, 4096), (32, 1, 4096, 1024), (32, 8, 1024, 2048), (32, 1, 16384, 2048), (32, 1, 16384, 16384)):
+        sl, t = torch.tensor(alibi_slopes(hq), device=DEV), ns * ql
+        meta, pages = step([ql] * ns)
+        kv, q = bf(pages, 2 * page * hkv * d), bf(t, hq, d)
+        w = min(window, ql)
+        by = t * (2 * hq + 2 * hkv) * d * 2
+        pair(f"capped_attention prefill {hq}h {ns}x{ql} window {window}, slopes", "capped_attention, all keys", lambda i: K.capped_attention(q, kv, hkv, d, meta, d ** -0.5, 50.0, window=window, slopes=sl),
+             lambda i: K.capped_attention(q, kv, hkv, d, meta, d ** -0.5, 50.0), by, by, 4.0 * ns * hq * d * (w * ql - w * w / 2), 2.0 * ns * ql * ql * hq * d, 1, few)
+    for h, dv, n, g in ((128, 64, 128, 8),):
+        hl = h // 2
+        for name, lens in (("decode 64", [1] * 64), ("decode 8", [1] * 8), ("decode 1", [1]), ("prefill 1x4096", [4096]), ("prefill 8x1024", [1024] * 8), ("prefill 16x256", [256] * 16), ("prefill 64x16", [16] * 64)):
+            meta, _ = step(lens)
+            t, b = sum(lens), len(lens)
+            st, so = [torch.zeros(b, h, n, dv, device=DEV) for _ in range(3)], [torch.zeros(b, hl, 128, 128, device=DEV) for _ in range(3)]
+            c, dt, p, z = bf(t, h * dv + 2 * g * n), bf(t, h), f32(3, h), bf(t, 3 * hl * 128)
+            x, B, C = c[:, : h * dv].unflatten(1, (h, dv)), c[:, h * dv : h * dv + g * n].unflatten(1, (g, n)), c[:, h * dv + g * n :].unflatten(1, (g, n))
+            q, k, v = (z[:, j * hl * 128 : (j + 1) * hl * 128].view(t, hl, 128) for j in range(3))
+            dec = torch.full((hl,), 0.98, device=DEV)
+            sb, fl = b * h * n * dv * 8, 4.0 * t * h * n * dv
+            pair(f"ssd_attention {name}", "decay_attention", lambda i: K.ssd_attention(x, B, C, dt, p[0], p[1], p[2], st[i], meta), lambda i: K.decay_attention(q, k, v, dec, so[i], meta), sb + t * (2 * h * dv + 2 * g * n) * 2,
+                 sb + t * 4 * hl * 128 * 2, fl, fl, 3, few)
+    for name, lens in (("decode 64", [1] * 64), ("decode 1", [1]), ("prefill 1x4096", [4096]), ("prefill 8x1024", [1024] * 8), ("prefill 16x256", [256] * 16)):
+        meta, _ = step(lens)
+        t, b, w, blocks = sum(lens), len(lens), 4096, 16
+        g, u, y, o, p, st = f32(t, blocks, 512), [bf(t, w) for _ in range(3)], bf(t, w), bf(t, 2 * w), f32(4, 2 * w), torch.zeros(b, 1, 1, w, device=DEV)
+        cw, cb, cs = f32(w, 4), f32(2, w), torch.zeros(b, w, 3, device=DEV).bfloat16()
+        pair(f"gated_lru {name} {w}", "conv_silu", lambda i: K.gated_lru(g, p[0], u[i], p[1, :w], y, p[2, :w], st, meta, 0.5, o[:, w:]), lambda i: K.conv_silu(u[i], cw, cs, meta), t * w * 14 + b * w * 8, t * w * 4 + b * w * 12,
+             0, 0, 3, iters)
+        pair(f"short_conv biases {name} {w}", "conv_silu", lambda i: K.short_conv(u[i], cw, cb[0], cs, meta, "none", cb[1]), lambda i: K.conv_silu(u[i], cw, cs, meta), *[t * w * 4 + b * w * 12] * 2, 0, 0, 3, iters)
+        mats, big = [bf(blocks, 512, 256) * 0.05 for _ in range(3)], [bf(blocks * 512, 256) * 0.05 for _ in range(3)]
+        by, fl = t * w * 2 + t * w * 8 + blocks * 512 * 256 * 2, 2.0 * t * blocks * 512 * 256
+        pair(f"multi_dense gates f32 {name}", "multi_dense bf16", lambda i: K.multi_dense(u[i].view(t, blocks, 256), mats[i], torch.float32), lambda i: K.multi_dense(u[i].view(t, blocks, 256), mats[i]), by, by - t * w * 4, fl, fl, 3,
+             iters)
+    for t in (64, 4096):
+        w, s = 4096, 4
+        meta, pages = step([1] * 64 if t == 64 else [1024] * 4)
+        n = meta.num_seqs
+        m = StreamMix(f32(s, s), f32(s), f32(s))
+        x, y32, y16, one, w16 = [f32(t, s, w) for _ in range(2)], [f32(t, w) for _ in range(2)], [bf(t, w) for _ in range(2)], torch.ones(w, device=DEV), torch.ones(w, device=DEV).bfloat16()
+        xs, y, car, mu = [f32(t, w) for _ in range(2)], y32 if t == 64 else y16, torch.zeros(n, 1, 1, w, device=DEV), torch.rand(w, device=DEV)
+        yb = y[0].element_size()
+        pair(f"streams_norm {t}x{s}x{w}, shift", "residual_norm", lambda i: K.streams_norm(x[i], y[i], m, one, 1e-6, torch.bfloat16, shift=mu, carried=car, meta=meta), lambda i: K.residual_norm(y[i], xs[i], one, 1e-6, 0.5, torch.bfloat16),
+             t * w * (8 * s + 2 + yb), t * w * (10 + yb), 0, 0, 2, iters)
+        pair(f"streams_norm {t}x{s}x{w}", "post_norm", lambda i: K.streams_norm(x[i], y[i], m, one, 1e-6, torch.bfloat16), lambda i: K.post_norm(y[i], xs[i], one, 1e-6, 2.0, torch.bfloat16), t * w * (8 * s + 2 + yb), t * w * (10 + yb), 0, 0,
+             2, iters)
+        o, gt, wh = [bf(t, 8, 1024) for _ in range(3)], [bf(t, 8192) for _ in range(3)], torch.ones(8192, device=DEV)
+        pair(f"gated_row_norm gate first {t}x8x1024", "gated_row_norm", lambda i: K.gated_row_norm(o[i], gt[i], wh, 1e-6, "silu", gate_first=True), lambda i: K.gated_row_norm(o[i], gt[i], wh, 1e-6, "silu"), *[t * 8192 * 6] * 2, 0, 0, 3, iters)
+        table, tab, ids = bf(65536, w), position_tables(8192, w, DEV), torch.randint(0, 65536, (t,), dtype=torch.int32, device=DEV)
+        pair(f"embed_positions {t}x{w}", "embed_stream", lambda i: K.embed_positions(ids, table, tab, meta), lambda i: K.embed_stream(ids, table, torch.bfloat16), t * w * 6, t * w * 8, 0, 0, 1, iters)
+        z, kv, b = [bf(t, 48 * d) for _ in range(3)], bf(pages, 2 * page * 8 * d), [f32(k * d) for k in (32, 8, 8)]
+        cut = lambda r: (r[:, : 32 * d], r[:, 32 * d : 40 * d], r[:, 40 * d :])
+        pair(f"head_norm_append biases {t}", "head_norm_append", lambda i: K.head_norm_append(*cut(z[i]), b[0], b[1][:d], None, meta, kv, 32, 8, d, d, 1e-6, bias=b), lambda i: K.head_norm_append(*cut(z[i]), b[0][:d], b[1][:d], None, meta, kv, 32, 8, d, d, 1e-6),
+             *[t * 48 * d * 4] * 2, 0, 0, 3, iters)
+        up, act = [bf(18432, w) * 0.02 for _ in range(3)], torch.tensor([0.9, 1.1], device=DEV)
+        by, fl = 18432 * w * 2 + t * (w + 18432) * 2, 2.0 * t * w * 18432
+        pair(f"dense_xielu {t} x 18432 x {w}", "linear", lambda i: K.dense_xielu(y16[0], up[i], act), lambda i: K.linear(y16[0], up[i]), by, by, fl, fl, 3, few)
     return rows
 
 
@@ -830,6 +920,8 @@ def main():
             rows.extend(vekalorn_cases(args.iters))
         if args.only in (None, "zeripel"):
             rows.extend(zeripel_cases(args.iters))
+        if args.only in (None, "nonetar"):
+            rows.extend(nonetar_cases(args.iters))
         if args.only in (None, "moe"):
             rows.extend(moe_cases(args.iters))
         if args.only in (None, "mla"):

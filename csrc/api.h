@@ -272,7 +272,7 @@ int pg_expert_gemm_simt(const void* x, long long ldx, const void* sorted_src, in
 int pg_gated_row_norm(const void* x, const void* gate, long long ldg, const void* w, void* y, int tokens, int heads, int dim, float eps, int silu, int w_heads, int gate_first,
                       int is_f32, cudaStream_t stream);
 int pg_glu_rows_f32(const void* gu, void* out, int rows, int inter, long long ldin, int gelu, cudaStream_t stream);
-int pg_xielu_rows(const void* x, void* y, const void* act, long long n, int is_f32, cudaStream_t stream);
+int pg_xielu_rows(const void* x, void* y, const void* act, long long n, int y_f32, cudaStream_t stream);
 int pg_softcap_f32(const void* x, void* y, long long n, float cap, cudaStream_t stream);
 int pg_gemm_simt(const void* x, const void* w, int x_f32, void* y, int y_f32, int T, int M, int K, long long ldx, long long ldw, long long ldy, cudaStream_t stream);
 // causal depthwise convolution over ragged sequences with carried inputs; biases on the inputs and the sum, SiLU optional

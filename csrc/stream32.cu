@@ -394,11 +394,11 @@ __global__ void __launch_bounds__(256) gated_row_norm_kernel(const T* __restrict
   }
 }
 
-template <typename T>
-__global__ void xielu_rows_kernel(const T* __restrict__ x, T* __restrict__ y, const float* __restrict__ act, long long n) {
+template <typename TO>
+__global__ void xielu_rows_kernel(const float* __restrict__ x, TO* __restrict__ y, const float* __restrict__ act, long long n) {
   PG_PDL_ENTRY();
   const float a = act[0], b = act[1];
-  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x) y[i] = from_f32<T>(xielu(to_f32(x[i]), a, b));
+  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x) y[i] = from_f32<TO>(xielu(x[i], a, b));
 }
 
 __global__ void glu_rows_kernel(const float* __restrict__ gu, float* __restrict__ out, int rows, int inter, long long ldin, int gelu) {
@@ -731,13 +731,13 @@ extern "C" int pg_glu_rows_f32(const void* gu, void* out, int rows, int inter, l
   return PG_OK;
 }
 
-// act: f32 softplus(p), 1/2 + softplus(q).
-extern "C" int pg_xielu_rows(const void* x, void* y, const void* act, long long n, int is_f32, cudaStream_t stream) {
+// x f32, y f32 or bf16; act: f32 softplus(p), 1/2 + softplus(q).
+extern "C" int pg_xielu_rows(const void* x, void* y, const void* act, long long n, int y_f32, cudaStream_t stream) {
   if (n == 0) return PG_OK;
   long long blocks = (n + 255) / 256;
   if (blocks > 148 * 16) blocks = 148 * 16;
-  PG_CUDA(is_f32 ? launch_pdl(xielu_rows_kernel<float>, dim3((unsigned)blocks), dim3(256), (size_t)0, stream, (const float*)x, (float*)y, (const float*)act, n)
-                 : launch_pdl(xielu_rows_kernel<bf16>, dim3((unsigned)blocks), dim3(256), (size_t)0, stream, (const bf16*)x, (bf16*)y, (const float*)act, n));
+  PG_CUDA(y_f32 ? launch_pdl(xielu_rows_kernel<float>, dim3((unsigned)blocks), dim3(256), (size_t)0, stream, (const float*)x, (float*)y, (const float*)act, n)
+                : launch_pdl(xielu_rows_kernel<bf16>, dim3((unsigned)blocks), dim3(256), (size_t)0, stream, (const float*)x, (bf16*)y, (const float*)act, n));
   PG_LAUNCH_CHECK();
   return PG_OK;
 }

@@ -1086,9 +1086,9 @@ def dense_xielu(x, w, act):
         _check(lib().pg_gemm_bf16_tn_xielu(_ptr(x), _ptr(w), _ptr(y), _ci(t), _ci(m), _ci(k), _ll(x.stride(0)), _ll(w.stride(0)), _ll(y.stride(0)), _ptr(act), _ptr(c.gemm_ws), _ll(c.gemm_ws.numel()),
                                            _ptr(c.gemm_counters), _ll(c.gemm_counters.numel() * 4), _ptr(c.status), _ci(1 if _BATCH_INVARIANT else 0), _stream()), c)
         return y
-    z = dense(x, w)
-    y = torch.empty_like(z)
-    _check(lib().pg_xielu_rows(_ptr(z), _ptr(y), _ptr(act), _ll(z.numel()), _ci(_is_f32(z)), _stream()), c)
+    z = dense(x, w, torch.float32)  # odd sizes: the CUDA-core GEMM
+    y = torch.empty((t, m), dtype=x.dtype, device=x.device)
+    _check(lib().pg_xielu_rows(_ptr(z), _ptr(y), _ptr(act), _ll(z.numel()), _ci(_is_f32(y)), _stream()), c)
     return y
 
 

@@ -6,6 +6,9 @@
 * ``zeripel`` beside the Kimi-K3 line (a recurrence with a decay per key channel, latent attention and sigmoid-routed experts
   with a shared one): the same layer order, heads, latents and expert weights; its full-attention layers stand in for both
   kinds of Zeripel attention, and its routed experts work behind two further projections of the stream's width.
+* ``nonetar`` beside the Nemipel line (soft-capped attention and linear attention with one decay per head, f32 stream): the same
+  layer order, heads, state sizes and feed-forward weights.  A Nonetar attention layer also has a recurrent block of the
+  stream's width (three more square matrices and its gates), every layer four copies of the stream, its attention a window.
 
 Device time (CUDA events) of whole steps of the executor: prefill steps of the given batches, and replays of the decode graph
 at a batch and context.  Weights and state are larger than L2 at every size, so no flush is needed.
@@ -56,6 +59,16 @@ def _zeripel_configs(width, ff, heads, kv_heads, experts, top, expert_ff, shared
     return {"zeripel": a, "kimi_k3": b}
 
 
+def _nonetar_configs(width, ff, heads, kv_heads, window, ssd_heads, periods, vocab=32768):
+    from ..config import MixerSpec, LayerSpec, _nemipel, _nonetar, _nonetar_parallel, _nonetar_ssd
+
+    a = _nonetar(width, vocab, ff * 3 // 2, 4, _nonetar_parallel(heads, kv_heads, 128, 128, 128 ** -0.5, 50.0, window, width, width // 256, 4, (1.0, 0.5)), _nonetar_ssd(ssd_heads, 64, 128, 8, 8, 4), periods,
+                 max_position=16384)
+    b = _nemipel(width, vocab, ff, heads, kv_heads, 128, heads, 128, 128, periods, lightning_ff=ff, max_position=16384)
+    attn, lin = MixerSpec("attention", heads, 128, 128, kv_heads=kv_heads, scale=128 ** -0.5, softcap=50.0), MixerSpec("lightning", ssd_heads // 2, 128, 128, decay=(0.98,) * (ssd_heads // 2))
+    return {"nonetar": a, "nemipel": replace(b, layer_specs=tuple(LayerSpec(m, ff) for _ in range(periods) for m in (attn, attn, lin)))}
+
+
 LINES = {
     "nemipel": Comparison("qwen35", ("width", "ff", "heads", "kv_heads", "recurrent_heads"), (("2048", (2048, 6144, 16, 8, 16)), ("4096", (4096, 12288, 32, 8, 32)), ("5120", (5120, 17408, 40, 8, 40))),
                           ((1, 4096), (8, 1024)), ((64, 1024), (8, 1024), (1, 1024)), _nemipel_configs, (("layers", 12), ("head_dim", 128))),
@@ -67,6 +80,10 @@ LINES = {
                           (("2048", (2048, 8192, 16, 4, 64, 6, 1408, 2816, 3)), ("4096", (4096, 12288, 32, 8, 32, 4, 2048, 4096, 2)), ("7168", (7168, 18432, 64, 8, 16, 4, 2048, 2048, 2))),
                           ((1, 4096), (8, 1024)), ((64, 1024), (16, 8192), (8, 1024), (1, 1024)), _zeripel_configs,
                           (("kv_rank", 512), ("dim", 128), ("rot_dim", 64), ("layers_per_period", "latent, latent over the same cache, WKV, attention"))),
+    "nonetar": Comparison("nemipel", ("width", "ff", "heads", "kv_heads", "window", "ssd_heads", "periods"),
+                          (("2048", (2048, 6144, 16, 8, 1024, 64, 4)), ("4096", (4096, 12288, 32, 8, 2048, 128, 3)), ("5120", (5120, 16384, 40, 8, 4096, 160, 2))),
+                          ((1, 4096), (8, 1024), (1, 16384)), ((64, 1024), (16, 8192), (8, 1024), (1, 1024)), _nonetar_configs,
+                          (("dim", 128), ("streams", 4), ("layers_per_period", "2 attention (Nonetar: beside a recurrent block), 1 state-space / lightning"))),
 }
 
 
