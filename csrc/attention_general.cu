@@ -172,8 +172,10 @@ __global__ void __launch_bounds__(256) head_norm_append_kernel(const T* __restri
     auto get = [&](int i) {
       load_vec<V>(src + i * V, f);
       if (bias) {
+        float bf[V];
+        load_vec<V>(bias + i * V, bf);
 #pragma unroll
-        for (int j = 0; j < V; ++j) f[j] += bias[i * V + j];
+        for (int j = 0; j < V; ++j) f[j] += bf[j];
       }
     };
     for (int i = me; i < n; i += TPR) {
@@ -303,7 +305,8 @@ extern "C" int pg_head_norm_append(const void* q, const void* k, const void* v, 
                                    void* q_out, void* kv, int tokens, int hq, int hkv, int dim, int vdim, int page_size, long long num_pages, float eps, int is_f32, void* status, cudaStream_t stream) {
   PG_REQUIRE(hq >= 1 && hkv >= 1 && dim >= 1 && vdim >= 1 && (temp == nullptr || max_pos > 0), "head_norm_append: heads %d / %d of %d / %d columns", hq, hkv, dim, vdim);
   if (tokens == 0) return PG_OK;
-  const bool v8 = dim % 8 == 0 && vdim % 8 == 0 && ld % 8 == 0 && ((((uintptr_t)q | (uintptr_t)k | (uintptr_t)v | (uintptr_t)q_out | (uintptr_t)kv | (uintptr_t)q_w | (uintptr_t)k_w) & 15) == 0);
+  const uintptr_t all = (uintptr_t)q | (uintptr_t)k | (uintptr_t)v | (uintptr_t)q_out | (uintptr_t)kv | (uintptr_t)q_w | (uintptr_t)k_w | (uintptr_t)q_b | (uintptr_t)k_b | (uintptr_t)v_b;
+  const bool v8 = dim % 8 == 0 && vdim % 8 == 0 && ld % 8 == 0 && (all & 15) == 0;
 #define PG_HN(T, V, TPR)                                                                                                                                                                            \
   launch_pdl(head_norm_append_kernel<T, V, TPR>, dim3(tokens), dim3(256), (size_t)0, stream, (const T*)q, (const T*)k, (const T*)v, ld, (const float*)q_w, q_w_heads, (const float*)k_w, (const float*)q_b, (const float*)k_b, (const float*)v_b, (const float*)temp, max_pos, \
              (const int*)positions, (const int*)slots, (T*)q_out, (T*)kv, hq, hkv, dim, vdim, page_size, num_pages, eps, (uint32_t*)status)

@@ -82,8 +82,18 @@ __device__ __forceinline__ float glu_act(float z, bool gelu) {
 
 // xIELU with its learned constants in the form a = softplus(p), b = 1/2 + softplus(q).
 __device__ __forceinline__ float xielu(float z, float a, float b) {
+  // e^m - 1 - m: near zero the Taylor polynomial through m^9 (truncation 3e-8 relative at 1/2), else as it stands
   const float m = fminf(z, 0.f);
-  return (z > 0.f ? a * z * z : b * (expm1f(m) - m)) + 0.5f * z;
+  float s = 1.f / 362880.f;
+  s = fmaf(s, m, 1.f / 40320.f);
+  s = fmaf(s, m, 1.f / 5040.f);
+  s = fmaf(s, m, 1.f / 720.f);
+  s = fmaf(s, m, 1.f / 120.f);
+  s = fmaf(s, m, 1.f / 24.f);
+  s = fmaf(s, m, 1.f / 6.f);
+  s = fmaf(s, m, 0.5f);
+  const float e = m > -0.5f ? s * m * m : (__expf(m) - 1.f) - m;
+  return fmaf(z > 0.f ? a : b, z > 0.f ? z * z : e, 0.5f * z);
 }
 
 struct __align__(16) bf16x8 {

@@ -60,14 +60,14 @@ __global__ void __launch_bounds__(LW * 32) gated_lru_scan_kernel(const LruArgs<T
   float S = in ? p.state[(long long)slot * p.width + c] : 0.f;
   float r[LT], i[LT];
   T u[LT], y[LT];
-  auto load = [&](int t0) {
+  const float* gp = p.gates + g_at;
+  const T *up = p.u + cc, *yp = p.y + cc;
+  auto load = [&](int t0) {  // rows past the end: the last one once more, so that nothing is conditional and all loads are in flight
 #pragma unroll
     for (int j = 0; j < LT; ++j) {
-      const int t = t0 + warp * LT + j;
-      if (in && t < q1) {
-        r[j] = p.gates[t * g_ld + g_at], i[j] = p.gates[t * g_ld + g_at + p.part];
-        u[j] = p.u[t * p.ldu + c], y[j] = p.y[t * p.ldy + c];
-      }
+      const long long t = min(t0 + warp * LT + j, q1 - 1);
+      r[j] = gp[t * g_ld], i[j] = gp[t * g_ld + p.part];
+      u[j] = up[t * p.ldu], y[j] = yp[t * p.ldy];
     }
   };
   load(q0);
@@ -75,11 +75,9 @@ __global__ void __launch_bounds__(LW * 32) gated_lru_scan_kernel(const LruArgs<T
     float a[LT], b[LT], g[LT], A = 1.f, B = 0.f;
 #pragma unroll
     for (int j = 0; j < LT; ++j) {
-      a[j] = 1.f, b[j] = 0.f, g[j] = 0.f;  // rows past the end leave the state as it is
-      if (in && t0 + warp * LT + j < q1) {
-        gate_pair(r[j] + br, i[j] + bi, to_f32(u[j]), k8, a[j], b[j]);
-        g[j] = glu_act(to_f32(y[j]) + yb, true) * p.scale;
-      }
+      gate_pair(r[j] + br, i[j] + bi, to_f32(u[j]), k8, a[j], b[j]);
+      g[j] = glu_act(to_f32(y[j]) + yb, true) * p.scale;
+      if (t0 + warp * LT + j >= q1) a[j] = 1.f, b[j] = 0.f;  // rows past the end leave the state as it is
       A *= a[j];
       B = fmaf(a[j], B, b[j]);
     }
