@@ -80,10 +80,8 @@ __device__ __forceinline__ float glu_act(float z, bool gelu) {
   return z / (1.f + __expf(-t));
 }
 
-// xIELU with its learned constants in the form a = softplus(p), b = 1/2 + softplus(q).
-__device__ __forceinline__ float xielu(float z, float a, float b) {
-  // e^m - 1 - m: near zero the Taylor polynomial through m^9 (truncation 3e-8 relative at 1/2), else as it stands
-  const float m = fminf(z, 0.f);
+// e^m - 1 - m for m <= 0: near zero the Taylor polynomial through m^9 (truncation 3e-8 relative at 1/2), else as it stands.
+__device__ __forceinline__ float exp_tail(float m) {
   float s = 1.f / 362880.f;
   s = fmaf(s, m, 1.f / 40320.f);
   s = fmaf(s, m, 1.f / 5040.f);
@@ -92,7 +90,11 @@ __device__ __forceinline__ float xielu(float z, float a, float b) {
   s = fmaf(s, m, 1.f / 24.f);
   s = fmaf(s, m, 1.f / 6.f);
   s = fmaf(s, m, 0.5f);
-  const float e = m > -0.5f ? s * m * m : (__expf(m) - 1.f) - m;
+  return m > -0.5f ? s * m * m : (__expf(m) - 1.f) - m;
+}
+// xIELU with its learned constants in the form a = softplus(p), b = 1/2 + softplus(q).
+__device__ __forceinline__ float xielu(float z, float a, float b) {
+  const float e = exp_tail(fminf(z, 0.f));
   return fmaf(z > 0.f ? a : b, z > 0.f ? z * z : e, 0.5f * z);
 }
 

@@ -1,7 +1,8 @@
 // Gated linear recurrence per channel (the recurrent block of Griffin): with r and i the sigmoids of two block-diagonal
 // projections of u,
 //   log a = -8 r softplus(lam),   S <- a S + sqrt(1 - a^2) i u,   out = S * gelu_tanh(y + y_bias) * scale,
-// everything in 32 bits but u, y and out.  a and 1 - a^2 come from one expm1: a = 1 + e, 1 - a^2 = -e (2 + e).
+// everything in 32 bits but u, y and out.  a and 1 - a^2 come from e = exp(log a) - 1, formed without cancellation: a = 1 + e, 1 - a^2 =
+// -e (2 + e).
 //
 //  * gated_lru_scan: prompts.  A CTA owns 32 channels of a sequence; 16 warps take 8 tokens each of a tile of 128.  Every warp runs
 //    its tokens from zero and hands the product of its decays and its result to the others; the tile's carry is then walked over
@@ -41,7 +42,7 @@ __device__ __forceinline__ float sigmoidf(float x) { return __fdividef(1.f, 1.f 
 
 // decay and input of one token of a channel; k8 = -8 softplus(lam)
 __device__ __forceinline__ void gate_pair(float r, float i, float u, float k8, float& a, float& b) {
-  const float e = expm1f(k8 * sigmoidf(r));
+  const float la = k8 * sigmoidf(r), e = la + exp_tail(la);
   a = 1.f + e;
   b = sqrtf(-e * (2.f + e)) * sigmoidf(i) * u;
 }
@@ -60,14 +61,19 @@ __global__ void __launch_bounds__(LW * 32) gated_lru_scan_kernel(const LruArgs<T
   float S = in ? p.state[(long long)slot * p.width + c] : 0.f;
   float r[LT], i[LT];
   T u[LT], y[LT];
+  // byte strides in 32 bits: one widening multiply-add per address
+  const int ldg = (int)(g_ld * sizeof(float)), ldu = (int)(p.ldu * sizeof(T)), ldy = (int)(p.ldy * sizeof(T)), ldo = (int)(p.ldo * sizeof(T));
+  auto at = [](auto* base, int t, int ld) { return reinterpret_cast<decltype(base)>(reinterpret_cast<uintptr_t>(base) + (long long)t * ld); };
   const float* gp = p.gates + g_at;
   const T *up = p.u + cc, *yp = p.y + cc;
+  T* op = p.out + cc;
   auto load = [&](int t0) {  // rows past the end: the last one once more, so that nothing is conditional and all loads are in flight
 #pragma unroll
     for (int j = 0; j < LT; ++j) {
-      const long long t = min(t0 + warp * LT + j, q1 - 1);
-      r[j] = gp[t * g_ld], i[j] = gp[t * g_ld + p.part];
-      u[j] = up[t * p.ldu], y[j] = yp[t * p.ldy];
+      const int t = min(t0 + warp * LT + j, q1 - 1);
+      const float* g = at(gp, t, ldg);
+      r[j] = g[0], i[j] = g[p.part];
+      u[j] = *at(up, t, ldu), y[j] = *at(yp, t, ldy);
     }
   };
   load(q0);
@@ -94,7 +100,7 @@ __global__ void __launch_bounds__(LW * 32) gated_lru_scan_kernel(const LruArgs<T
     for (int j = 0; j < LT; ++j) {
       const int t = t0 + warp * LT + j;
       mine = fmaf(a[j], mine, b[j]);
-      if (in && t < q1) p.out[t * p.ldo + c] = from_f32<T>(mine * g[j]);
+      if (in && t < q1) *at(op, t, ldo) = from_f32<T>(mine * g[j]);
     }
   }
   if (in && warp == 0) p.state[(long long)slot * p.width + c] = S;
@@ -135,7 +141,7 @@ int run_lru(const LruArgs<T>& p, int num_seqs, int max_q_len, cudaStream_t strea
 extern "C" int pg_gated_lru(const void* gates, const void* gate_bias, const void* u, long long ldu, const void* lam, const void* y, long long ldy, const void* y_bias, void* state, void* out, long long ldo,
                             const void* q_indptr, const void* slots, int num_seqs, int width, int blocks, float scale, int max_q_len, int is_f32, cudaStream_t stream) {
   PG_REQUIRE(blocks >= 1 && width >= 1 && width % blocks == 0, "gated_lru: %d channels in %d blocks", width, blocks);
-  PG_REQUIRE(num_seqs <= 65535, "gated_lru: %d sequences", num_seqs);
+  PG_REQUIRE(num_seqs <= 65535 && width < (1 << 27) && ldu < (1ll << 28) && ldy < (1ll << 28) && ldo < (1ll << 28), "gated_lru: %d sequences, rows of %lld / %lld / %lld", num_seqs, ldu, ldy, ldo);
   if (num_seqs == 0) return PG_OK;
 #define PG_LRU(T)                                                                                                                                                                         \
   run_lru<T>(LruArgs<T>{(const float*)gates, (const float*)gate_bias, (const T*)u, ldu, (const float*)lam, (const T*)y, ldy, (const float*)y_bias, (float*)state, (T*)out, ldo, \
