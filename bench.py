@@ -51,7 +51,7 @@ def parse():
     ap.add_argument("--prefill-chunk", type=int, default=4096, help="token budget of one prefill step (max_prefill_tokens)")
     ap.add_argument("--profile-host", default=None, help="write a cProfile of the scheduler thread during the e2e phase to this path")
     ap.add_argument("--no-library-arm", action="store_true", help="skip the cuBLAS + NCCL arm that is timed after the main arm and reported as `library_arm`")
-    ap.add_argument("--line-speed", nargs="?", const="nemipel", choices=["nemipel", "vekalorn", "zeripel", "nonetar"], help="instead of the headline workload: prefill and decode throughput of a model line beside its closest neighbour (nemipel: the Qwen3.5 line, vekalorn: the DeepSeek-V2 line, zeripel: the Kimi-K3 line) at equal layer sizes, one JSON line per size")
+    ap.add_argument("--line-speed", nargs="?", const="nemipel", choices=["nemipel", "vekalorn", "zeripel", "nonetar"], help="instead of the headline workload: prefill and decode throughput of a model line beside its closest neighbour (nemipel: the Qwen3.5 line, vekalorn: the DeepSeek-V2 line, zeripel: the Kimi-K3 line, nonetar: the Nemipel line) at equal layer sizes, one JSON line per size")
     return ap.parse_args()
 
 
